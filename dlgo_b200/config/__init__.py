@@ -7,8 +7,9 @@ from .dedutar import DedutarConfig
 from .monolix import MonolixConfig
 from .bazurax import BazuraxConfig
 from .ragilorn import RagilornConfig
+from .zetavik import ZetavikConfig
 
 __all__ = [
-    "ArchitectureSpec", "BazuraxConfig", "ConfigError", "DedutarConfig", "LayerSpec", "LlamaConfig", "MonolixConfig", "PartSpec", "RagilornConfig", "RopeScaling", "RunEntry",
+    "ArchitectureSpec", "BazuraxConfig", "ConfigError", "DedutarConfig", "LayerSpec", "LlamaConfig", "MonolixConfig", "PartSpec", "RagilornConfig", "RopeScaling", "RunEntry", "ZetavikConfig",
     "config_class_for", "config_from_dict", "load_config", "register_architecture", "registered_architectures",
 ]

@@ -51,6 +51,7 @@ LIBRARIES: Dict[str, List[str]] = {
     "wholenorm_append": ["wholenorm_append.cu"],
     "conv_rope_append": ["conv_rope_append.cu"],
     "gated_residual": ["gated_residual.cu"],
+    "ssd": ["ssd.cu"],
 }
 _HEADERS = ["common.cuh", "attention_noalloc.h", "attention_combine.cuh", "attention_decode_tiles.cuh", "tcgen05.cuh",
             "async_copy.cuh"]

@@ -286,13 +286,59 @@ def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, w: Optional[torch.Tensor]
 
 
 # ------------------------------------------------------------- latent attention
+class LatentRope:
+    """The rotated part of latent attention's key rows and query heads: their last ``dims`` numbers turn by
+    ``float(position) * freq[i]`` (cosine and sine times ``amplitude``), number i paired with number i + dims / 2
+    (``halves``) or 2i with 2i + 1."""
+
+    __slots__ = ("freq", "amplitude", "dims", "halves")
+
+    def __init__(self, freq: torch.Tensor, amplitude: float, dims: int, halves: bool):
+        _need(freq, torch.float32, "freq")
+        if dims <= 0 or dims % 2 or freq.numel() != dims // 2:
+            raise KernelError("LatentRope: an even number of dims and a frequency per pair")
+        self.freq, self.amplitude, self.dims, self.halves = freq, float(amplitude), int(dims), bool(halves)
+
+
+def _rope_args(rope: Optional[LatentRope]) -> list:
+    if rope is None:
+        return [_p(0), _f(1.0), _i(0), _i(0)]
+    return [_ptr(rope.freq), _f(rope.amplitude), _i(rope.dims), _i(1 if rope.halves else 0)]
+
+
+def _gate_args(gate: Optional[torch.Tensor], T: int, num_heads: int) -> list:
+    """A head gate's logits: fp32 [T, heads] with any row stride, or None."""
+    if gate is None:
+        return [_p(0), _i(0)]
+    if gate.dtype != torch.float32 or tuple(gate.shape) != (T, num_heads) or gate.stride(1) != 1 or not gate.is_cuda:
+        raise KernelError("the head gate must be float32 [T, heads] on the GPU with unit inner stride")
+    return [_ptr(gate), _i(gate.stride(0))]
+
+
+def latent_queries(q: torch.Tensor, num_heads: int, q_head: int, d_out: int, rope: Optional[LatentRope],
+                   token_pos: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """Query heads [T, heads * q_head] (fp32) with their rotated part turned, as [T, heads * d_out] in ``out_dtype``
+    (numbers q_head .. d_out of every head are zero)."""
+    if q.dtype != torch.float32 or q.dim() != 2 or q.stride(1) != 1 or q.shape[1] < num_heads * q_head or d_out < q_head:
+        raise KernelError("latent_queries: q must be 2-D float32 with unit inner stride and hold every head")
+    _need(token_pos, torch.int32, "token_pos")
+    T = q.shape[0]
+    out = torch.empty((T, num_heads * d_out), dtype=out_dtype, device=q.device)
+    st = _lib("latent_attention").dlgo_latent_queries(_ptr(q), _i(q.stride(0)), _ptr(out), _i(dtype_code(out_dtype)),
+                                                      _ptr(token_pos), _i(T), _i(num_heads), _i(q_head), _i(d_out),
+                                                      *_rope_args(rope), _stream())
+    _check(st, "latent_queries")
+    return out
+
+
 def latent_norm_append(proj: torch.Tensor, kv_off: int, kv_rank: int, w_kv: torch.Tensor, q_off: int, q_rank: int,
                        w_q: Optional[torch.Tensor], eps: float, token_pos: torch.Tensor, token_seq: torch.Tensor,
                        seq_slot: torch.Tensor, page_table: torch.Tensor, pages: torch.Tensor,
-                       write_cache: bool = True) -> Optional[torch.Tensor]:
+                       write_cache: bool = True, rope: Optional[LatentRope] = None) -> Optional[torch.Tensor]:
     """RMS norms of the latents in fp32 ``proj`` [T, ld]: columns ``kv_off ...`` go (normed, times ``w_kv``) to
     the paged cache ``pages`` [n, 1, page, kv_rank] at each token's position; with ``q_rank`` > 0 columns
-    ``q_off ...`` come back normed (times ``w_q``) as [T, q_rank] in the cache's type."""
+    ``q_off ...`` come back normed (times ``w_q``) as [T, q_rank] in the cache's type.  ``rope``: the columns behind the
+    latent are one key part that turns with the position and is kept behind the latent in the same cache row."""
     if proj.dtype != torch.float32 or proj.dim() != 2 or proj.stride(1) != 1:
         raise KernelError("latent_norm_append: proj must be 2-D float32 with unit inner stride")
     _need(w_kv, torch.float32, "w_kv")
@@ -300,8 +346,9 @@ def latent_norm_append(proj: torch.Tensor, kv_off: int, kv_rank: int, w_kv: torc
     for n, t in (("token_pos", token_pos), ("token_seq", token_seq), ("seq_slot", seq_slot), ("page_table", page_table)):
         _need(t, torch.int32, n)
     T = proj.shape[0]
-    if pages.shape[-1] != kv_rank or w_kv.numel() != kv_rank:
-        raise KernelError("latent_norm_append: the cache's rows and the norm weight must have kv_rank elements")
+    if pages.shape[-1] != kv_rank + (rope.dims if rope is not None else 0) or w_kv.numel() != kv_rank:
+        raise KernelError("latent_norm_append: the norm weight must have kv_rank elements, the cache's rows those and the "
+                          "rotated part")
     cq = None
     if q_rank > 0:
         _need(w_q, torch.float32, "w_q")
@@ -309,46 +356,22 @@ def latent_norm_append(proj: torch.Tensor, kv_off: int, kv_rank: int, w_kv: torc
     st = _lib("latent_attention").dlgo_latent_norm_append(
         _ptr(proj), _i(proj.stride(0)), _i(T), _i(kv_off), _i(kv_rank), _ptr(w_kv), _i(q_off), _i(q_rank), _ptr(w_q),
         _ptr(cq), _f(eps), _ptr(token_pos), _ptr(token_seq), _ptr(seq_slot), _ptr(page_table), _i(page_table.shape[1]),
-        _ptr(pages), _i(dtype_code(pages.dtype)), _i(pages.shape[-2]), _i(1 if write_cache else 0), _stream())
+        _ptr(pages), _i(dtype_code(pages.dtype)), _i(pages.shape[-2]), _i(1 if write_cache else 0), *_rope_args(rope),
+        _stream())
     _check(st, "latent_norm_append")
     return cq
-
-
-def latent_rope_append(proj: torch.Tensor, kv_off: int, kv_rank: int, w_kv: torch.Tensor, q_off: int, num_heads: int,
-                       q_head: int, rope: int, freq: torch.Tensor, amplitude: float, eps: float,
-                       token_pos: torch.Tensor, token_seq: torch.Tensor, seq_slot: torch.Tensor,
-                       page_table: torch.Tensor, pages: torch.Tensor, write_cache: bool = True) -> None:
-    """Latents with a rotated key part, from fp32 ``proj`` [T, ld]: columns ``kv_off ...`` hold ``kv_rank`` numbers
-    that are RMS-normed (times ``w_kv``) and ``rope`` numbers that turn with the position in neighbouring pairs
-    (angle ``float(pos) * freq[i]``, cosine and sine times ``amplitude``); both go to the token's row of the paged
-    cache ``pages`` [n, 1, page, kv_rank + rope].  The queries at ``q_off`` ([heads, q_head] per token) turn IN
-    PLACE in the last ``rope`` numbers of every head."""
-    if proj.dtype != torch.float32 or proj.dim() != 2 or proj.stride(1) != 1:
-        raise KernelError("latent_rope_append: proj must be 2-D float32 with unit inner stride")
-    _need(w_kv, torch.float32, "w_kv")
-    _need(freq, torch.float32, "freq")
-    _need(pages, None, "pages")
-    for n, t in (("token_pos", token_pos), ("token_seq", token_seq), ("seq_slot", seq_slot), ("page_table", page_table)):
-        _need(t, torch.int32, n)
-    if pages.shape[-1] != kv_rank + rope or w_kv.numel() != kv_rank or freq.numel() != rope // 2:
-        raise KernelError("latent_rope_append: cache rows hold kv_rank + rope numbers; rope / 2 frequencies")
-    if q_off + num_heads * q_head > proj.shape[1] or kv_off + kv_rank + rope > proj.shape[1]:
-        raise KernelError("latent_rope_append: the columns named lie outside proj")
-    st = _lib("latent_attention").dlgo_latent_rope_append(
-        _ptr(proj), _i(proj.stride(0)), _i(proj.shape[0]), _i(kv_off), _i(kv_rank), _ptr(w_kv), _i(q_off),
-        _i(num_heads), _i(q_head), _i(rope), _ptr(freq), _f(amplitude), _f(eps), _ptr(token_pos), _ptr(token_seq),
-        _ptr(seq_slot), _ptr(page_table), _i(page_table.shape[1]), _ptr(pages), _i(dtype_code(pages.dtype)),
-        _i(pages.shape[-2]), _i(1 if write_cache else 0), _stream())
-    _check(st, "latent_rope_append")
 
 
 def latent_attention(q: torch.Tensor, w_k: torch.Tensor, w_v: torch.Tensor, sink: Optional[torch.Tensor],
                      pages: torch.Tensor, page_table: torch.Tensor, seq_slot: torch.Tensor, token_seq: torch.Tensor,
                      token_pos: torch.Tensor, num_heads: int, qk_dim: int, v_dim: int, scale: float,
-                     window: int = 0) -> torch.Tensor:
+                     window: int = 0, rope: Optional[LatentRope] = None,
+                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of packed tokens over cached latents ``pages`` [n, 1, page, rank]: per head
     ``softmax((Wk^T q) . c * scale) c`` carried out through ``Wv``; ``q`` [T, >= H*qk_dim] (fp32 or the cache's
-    type), ``w_k`` [H*qk_dim, rank], ``w_v`` [H*v_dim, rank] in the cache's type.  Returns [T, H*v_dim]."""
+    type), ``w_k`` [H*qk_dim, rank], ``w_v`` [H*v_dim, rank] in the cache's type.  ``rope``: the end of every query head
+    turns with the token's position first; ``gate`` (fp32 [T, H]): a head's output is multiplied by sigmoid(gate).
+    Returns [T, H*v_dim]."""
     _need(pages, None, "pages")
     _need(w_k, pages.dtype, "w_k")
     _need(w_v, pages.dtype, "w_v")
@@ -366,7 +389,8 @@ def latent_attention(q: torch.Tensor, w_k: torch.Tensor, w_v: torch.Tensor, sink
         _ptr(q), _i(1 if q.dtype == torch.float32 else 0), _i(q.stride(0)), _ptr(w_k), _ptr(w_v), _ptr(sink),
         _ptr(pages), _i(dtype_code(pages.dtype)), _ptr(page_table), _i(page_table.shape[1]), _i(pages.shape[-2]),
         _ptr(seq_slot), _ptr(token_seq), _ptr(token_pos), _ptr(out), _i(out.stride(0)), _i(T), _i(num_heads),
-        _i(qk_dim), _i(v_dim), _i(rank), _f(scale), _i(window), _stream())
+        _i(qk_dim), _i(v_dim), _i(rank), _f(scale), _i(window), *_rope_args(rope), *_gate_args(gate, T, num_heads),
+        _stream())
     _check(st, "latent_attention")
     return out
 
@@ -380,8 +404,8 @@ def latent_attention_few_takes(dtype: torch.dtype, rank: int) -> bool:
 def latent_attention_few(q: torch.Tensor, w_k: torch.Tensor, w_v: torch.Tensor, sink: Optional[torch.Tensor],
                          pages: torch.Tensor, page_table: torch.Tensor, seq_slot: torch.Tensor,
                          token_seq: torch.Tensor, token_pos: torch.Tensor, num_heads: int, qk_dim: int, v_dim: int,
-                         scale: float, window: int, n_slices: int, q_lat: torch.Tensor,
-                         parts: torch.Tensor) -> torch.Tensor:
+                         scale: float, window: int, n_slices: int, q_lat: torch.Tensor, parts: torch.Tensor,
+                         rope: Optional[LatentRope] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """:func:`latent_attention` for steps of few tokens, as three launches that each fill the GPU: the queries
     into latent space (``q_lat`` [T, H, rank] fp32 scratch), the softmax over every token's visible latents cut
     into ``n_slices`` slices (``parts`` [T, H, n_slices, rank + 2] fp32 scratch), and the slices' meeting, the
@@ -406,7 +430,8 @@ def latent_attention_few(q: torch.Tensor, w_k: torch.Tensor, w_v: torch.Tensor, 
         _ptr(q), _i(1 if q.dtype == torch.float32 else 0), _i(q.stride(0)), _ptr(w_k), _ptr(w_v), _ptr(sink),
         _ptr(pages), _i(dtype_code(pages.dtype)), _ptr(page_table), _i(page_table.shape[1]), _i(pages.shape[-2]),
         _ptr(seq_slot), _ptr(token_seq), _ptr(token_pos), _ptr(out), _i(out.stride(0)), _i(T), _i(num_heads),
-        _i(qk_dim), _i(v_dim), _i(rank), _f(scale), _i(window), _i(n_slices), _ptr(q_lat), _ptr(parts), _stream())
+        _i(qk_dim), _i(v_dim), _i(rank), _f(scale), _i(window), _i(n_slices), _ptr(q_lat), _ptr(parts),
+        *_rope_args(rope), *_gate_args(gate, T, num_heads), _stream())
     _check(st, "latent_attention_few", 3)
     return out
 
@@ -421,8 +446,8 @@ def latent_attention_tiles_takes(dtype: torch.dtype, num_heads: int, rank: int) 
 def latent_attention_tiles(q: torch.Tensor, w_k: torch.Tensor, w_v: torch.Tensor, sink: Optional[torch.Tensor],
                            pages: torch.Tensor, page_table: torch.Tensor, seq_slot: torch.Tensor,
                            token_seq: torch.Tensor, token_pos: torch.Tensor, num_heads: int, qk_dim: int, v_dim: int,
-                           scale: float, window: int, n_slices: int, q_lat: torch.Tensor,
-                           parts: torch.Tensor) -> torch.Tensor:
+                           scale: float, window: int, n_slices: int, q_lat: torch.Tensor, parts: torch.Tensor,
+                           rope: Optional[LatentRope] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """:func:`latent_attention_few` with every latent row read once per token instead of once per head: four
     launches (queries into latent space; tiles of 32 keys in shared memory serving all heads, a block per token and
     slice of the keys; the slices' meeting; out through ``w_v``).  Same arguments and scratch."""
@@ -446,7 +471,8 @@ def latent_attention_tiles(q: torch.Tensor, w_k: torch.Tensor, w_v: torch.Tensor
         _ptr(q), _i(1 if q.dtype == torch.float32 else 0), _i(q.stride(0)), _ptr(w_k), _ptr(w_v), _ptr(sink),
         _ptr(pages), _i(dtype_code(pages.dtype)), _ptr(page_table), _i(page_table.shape[1]), _i(pages.shape[-2]),
         _ptr(seq_slot), _ptr(token_seq), _ptr(token_pos), _ptr(out), _i(out.stride(0)), _i(T), _i(num_heads),
-        _i(qk_dim), _i(v_dim), _i(rank), _f(scale), _i(window), _i(n_slices), _ptr(q_lat), _ptr(parts), _stream())
+        _i(qk_dim), _i(v_dim), _i(rank), _f(scale), _i(window), _i(n_slices), _ptr(q_lat), _ptr(parts),
+        *_rope_args(rope), *_gate_args(gate, T, num_heads), _stream())
     _check(st, "latent_attention_tiles", 4)
     return out
 
@@ -575,6 +601,153 @@ def rotate_scale(proj: torch.Tensor, q_off: int, k_off: int, freq: Optional[torc
                                              _ptr(freq if rot else None), _i(rot), _ptr(token_pos), _i(proj.shape[0]),
                                              _i(num_heads), _i(qk_dim), _f(k_scale), _stream())
     _check(st, "rotate_scale")
+
+
+# ----------------------------------------------------------- state-space mixing
+class SsdShape:
+    """Sizes of a state-space mixer: heads, groups of heads that share B and C, state rows N, value columns P, taps of
+    its convolution over time."""
+
+    __slots__ = ("heads", "groups", "state", "v_dim", "taps")
+
+    def __init__(self, heads: int, groups: int, state: int, v_dim: int, taps: int):
+        self.heads, self.groups, self.state, self.v_dim, self.taps = heads, groups, state, v_dim, taps
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.v_dim
+
+    @property
+    def channels(self) -> int:
+        """Channels that pass the convolution: x, B and C."""
+        return self.inner + 2 * self.groups * self.state
+
+    @property
+    def columns(self) -> int:
+        """Columns of the projection: z, x, B, C, dt."""
+        return self.inner + self.channels + self.heads
+
+    def state_floats(self) -> int:
+        """Numbers of one sequence's state row: the state, then the convolution's last inputs (to whole 16 bytes)."""
+        n = self.heads * self.state * self.v_dim + (self.taps - 1) * self.channels
+        return n + -n % 4
+
+    def args(self) -> list:
+        return [_i(self.heads), _i(self.groups), _i(self.state), _i(self.v_dim), _i(self.taps)]
+
+
+SSD_MAX_STATE = 512
+
+
+def _ssd_check(what: str, s: SsdShape, proj: Optional[torch.Tensor], state: torch.Tensor) -> None:
+    if s.state > SSD_MAX_STATE:
+        raise KernelError(f"{what}: at most {SSD_MAX_STATE} state rows, got {s.state}")
+    if proj is not None and (proj.dtype != torch.float32 or proj.dim() != 2 or proj.stride(1) != 1 or
+                             proj.shape[1] < s.columns):
+        raise KernelError(f"{what}: proj must be 2-D float32 with unit inner stride and {s.columns} columns")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < s.state_floats() or \
+            not state.is_cuda:
+        raise KernelError(f"{what}: state must be [slots, >= {s.state_floats()}] float32 on the GPU")
+
+
+def ssd_conv(proj: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+             tiles: torch.Tensor, n_tiles: int, token_seq: torch.Tensor, seq_slot: torch.Tensor, state: torch.Tensor,
+             shape: SsdShape) -> tuple:
+    """Causal convolution over time, bias and silu of the columns x | B | C of ``proj`` (fp32 [T, >= columns]), reaching
+    back into the state rows for a sequence's earlier inputs; and per head d = softplus(dt + dt_bias) and
+    f = exp(-exp(a_log) d).  ``tiles`` [n_tiles, 3] cut the step's tokens into runs of one sequence.  Returns
+    (x | B | C [T, channels], [T, heads, 2]), fp32."""
+    _ssd_check("ssd_conv", shape, proj, state)
+    for n, t, k in (("taps", taps, shape.channels * shape.taps), ("bias", bias, shape.channels),
+                    ("dt_bias", dt_bias, shape.heads), ("a_log", a_log, shape.heads)):
+        _need(t, torch.float32, n)
+        if t.numel() != k:
+            raise KernelError(f"ssd_conv: {n} must have {k} numbers, has {t.numel()}")
+    for n, t in (("tiles", tiles), ("token_seq", token_seq), ("seq_slot", seq_slot)):
+        _need(t, torch.int32, n)
+    T = proj.shape[0]
+    xbc = torch.empty((T, shape.channels + -shape.channels % 4), dtype=torch.float32, device=proj.device)
+    steps = torch.empty((T, shape.heads, 2), dtype=torch.float32, device=proj.device)
+    st = _lib("ssd").dlgo_ssd_conv(_ptr(proj), _i(proj.stride(0)), _ptr(taps), _ptr(bias), _ptr(dt_bias), _ptr(a_log),
+                                   _ptr(tiles), _i(n_tiles), _ptr(token_seq), _ptr(seq_slot), _ptr(state),
+                                   _ll(state.stride(0)), _ptr(xbc), _i(xbc.stride(0)), _ptr(steps), *shape.args(),
+                                   _stream())
+    _check(st, "ssd_conv")
+    return xbc, steps
+
+
+def ssd_scratch_floats(n_tiles: int, shape: SsdShape) -> int:
+    return n_tiles * shape.heads * (shape.state * shape.v_dim + 1)
+
+
+def ssd_segments(xbc: torch.Tensor, steps: torch.Tensor, D: torch.Tensor, tiles: torch.Tensor, n_tiles: int, direct: bool,
+                 seq_slot: torch.Tensor, state: torch.Tensor, scratch: Optional[torch.Tensor],
+                 shape: SsdShape) -> torch.Tensor:
+    """The recurrence over the step's tokens from :func:`ssd_conv`'s results: S <- f S + d B x^T, y = S^T C + D x, every
+    sequence from (and back into) its state row.  ``tiles`` cut a sequence's tokens into consecutive segments that run
+    side by side; ``direct``: one segment per sequence; else ``scratch`` holds :func:`ssd_scratch_floats`.
+    Returns fp32 [T, heads * v_dim]."""
+    _ssd_check("ssd_segments", shape, None, state)
+    _need(D, torch.float32, "D")
+    _need(xbc, torch.float32, "xbc")
+    _need(steps, torch.float32, "steps")
+    _need(tiles, torch.int32, "tiles")
+    _need(seq_slot, torch.int32, "seq_slot")
+    T = xbc.shape[0]
+    if D.numel() != shape.heads or xbc.shape[1] < shape.channels or tuple(steps.shape) != (T, shape.heads, 2):
+        raise KernelError("ssd_segments: shapes do not fit")
+    if not direct:
+        need = ssd_scratch_floats(n_tiles, shape)
+        if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
+            raise KernelError(f"ssd_segments: {n_tiles} segments need {need} floats of scratch")
+    out = torch.empty((T, shape.inner), dtype=torch.float32, device=xbc.device)
+    st = _lib("ssd").dlgo_ssd_segments(_ptr(xbc), _i(xbc.stride(0)), _ptr(steps), _ptr(D), _ptr(tiles), _i(n_tiles),
+                                       _i(1 if direct else 0), _ptr(seq_slot), _ptr(state), _ll(state.stride(0)),
+                                       _ptr(scratch), _ptr(out), _i(out.stride(0)), *shape.args(), _stream())
+    _check(st, "ssd_segments", 1 if direct else 3)
+    return out
+
+
+def ssd_step(proj: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+             D: torch.Tensor, seq_slot: torch.Tensor, state: torch.Tensor, shape: SsdShape) -> torch.Tensor:
+    """:func:`ssd_conv` and :func:`ssd_segments` in one launch for steps of one token per sequence (row t of ``proj``
+    belongs to sequence t)."""
+    _ssd_check("ssd_step", shape, proj, state)
+    for n, t, k in (("taps", taps, shape.channels * shape.taps), ("bias", bias, shape.channels), ("D", D, shape.heads),
+                    ("dt_bias", dt_bias, shape.heads), ("a_log", a_log, shape.heads)):
+        _need(t, torch.float32, n)
+        if t.numel() != k:
+            raise KernelError(f"ssd_step: {n} must have {k} numbers, has {t.numel()}")
+    _need(seq_slot, torch.int32, "seq_slot")
+    T = proj.shape[0]
+    out = torch.empty((T, shape.inner), dtype=torch.float32, device=proj.device)
+    st = _lib("ssd").dlgo_ssd_step(_ptr(proj), _i(proj.stride(0)), _ptr(taps), _ptr(bias), _ptr(dt_bias), _ptr(a_log),
+                                   _ptr(D), _ptr(seq_slot), _ptr(state), _ll(state.stride(0)), _ptr(out),
+                                   _i(out.stride(0)), _i(T), *shape.args(), _stream())
+    _check(st, "ssd_step")
+    return out
+
+
+def ssd_gate_norm(y: torch.Tensor, proj: torch.Tensor, w: torch.Tensor, norm_groups: int, eps: float,
+                  out_dtype: torch.dtype, token_seq: torch.Tensor, seq_slot: torch.Tensor, state: torch.Tensor,
+                  shape: SsdShape) -> torch.Tensor:
+    """``rms(y * silu(z)) * w`` with the root mean square taken over each of ``norm_groups`` equal parts of a row (z: the
+    first columns of ``proj``); the token that ends a sequence's part of the step moves the convolution's last inputs
+    into the state row.  Returns [T, heads * v_dim] in ``out_dtype``."""
+    _ssd_check("ssd_gate_norm", shape, proj, state)
+    _need(w, torch.float32, "w")
+    _need(y, torch.float32, "y")
+    _need(token_seq, torch.int32, "token_seq")
+    _need(seq_slot, torch.int32, "seq_slot")
+    T = proj.shape[0]
+    if tuple(y.shape) != (T, shape.inner) or w.numel() != shape.inner or norm_groups <= 0 or shape.inner % norm_groups:
+        raise KernelError("ssd_gate_norm: shapes do not fit")
+    out = torch.empty((T, shape.inner), dtype=out_dtype, device=proj.device)
+    st = _lib("ssd").dlgo_ssd_gate_norm(_ptr(y), _i(y.stride(0)), _ptr(proj), _i(proj.stride(0)), _ptr(w), _ptr(out),
+                                        _i(dtype_code(out_dtype)), _i(norm_groups), _f(eps), _ptr(token_seq), _i(T),
+                                        _ptr(seq_slot), _ptr(state), _ll(state.stride(0)), *shape.args(), _stream())
+    _check(st, "ssd_gate_norm")
+    return out
 
 
 # ------------------------------------------------------------------ time mixing
@@ -857,16 +1030,16 @@ def scale_softcap(logits: torch.Tensor, scale: float, cap: float) -> torch.Tenso
     return logits
 
 
-def scale_heads(a: torch.Tensor, gate: torch.Tensor, head_dim: int) -> torch.Tensor:
-    """``a[t, h, :] *= gate[t, h]`` in place for ``a`` [T, H * head_dim] (float32 or bfloat16) and fp32 ``gate`` [T, H]."""
+def scale_heads(a: torch.Tensor, gate: torch.Tensor, head_dim: int, sigmoid: bool = False) -> torch.Tensor:
+    """``a[t, h, :] *= gate[t, h]`` in place for ``a`` [T, H * head_dim] (float32 or bfloat16) and fp32 ``gate`` [T, H]
+    (any row stride); ``sigmoid``: the factor is sigmoid(gate)."""
     _need(a, None, "a")
-    _need(gate, torch.float32, "gate")
     T, n = a.shape
     H = gate.shape[1]
-    if n != H * head_dim or gate.shape[0] != T:
+    if n != H * head_dim:
         raise KernelError("scale_heads: a must be [T, H * head_dim] and gate [T, H]")
-    st = _lib("wholenorm_append").dlgo_scale_heads(_ptr(a), _ptr(gate), _i(dtype_code(a.dtype)), _i(T), _i(H),
-                                                   _i(head_dim), _stream())
+    st = _lib("wholenorm_append").dlgo_scale_heads(_ptr(a), *_gate_args(gate, T, H), _i(dtype_code(a.dtype)), _i(T), _i(H),
+                                                   _i(head_dim), _i(1 if sigmoid else 0), _stream())
     _check(st, "scale_heads")
     return a
 
@@ -1005,9 +1178,10 @@ MOE_FEW_ROWS, MOE_TILE_ROWS, MOE_TC_ROWS, MOE_TC_PAIR_ROWS = 8, 64, 128, 256    
 
 def moe_router(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], n_outputs: int,
                has_gate: bool, top: int, groups: int, keep: int, sigmoid_scores: bool = False,
-               renormalize: bool = False, plan: Optional[tuple] = None, logit_bias: Optional[torch.Tensor] = None):
+               renormalize: bool = False, plan: Optional[tuple] = None, logit_bias: Optional[torch.Tensor] = None,
+               weight_scale: float = 1.0):
     """Router of a mixture of experts for ``h`` [T, d]: returns (chosen outputs [T, top] int32, their weights
-    [T, top] fp32, gate [T] fp32 or None, plan).  ``w_router`` is fp32 [n_outputs (+ 1 gate row), d].
+    [T, top] fp32, times ``weight_scale``; gate [T] fp32 or None, plan).  ``w_router`` is fp32 [n_outputs (+ 1 gate row), d].
     ``plan`` = (experts that hold tensors, rows per tile): the :class:`MoEPlan` of :func:`moe_plan` is made as well,
     in the choice's own launch where the step has few tokens, else by a launch of its own; without it None."""
     _need(w_router, torch.float32, "w_router")
@@ -1034,7 +1208,7 @@ def moe_router(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[tor
     st = _lib("moe").dlgo_moe_router(
         _ptr(h), _i(dtype_code(h.dtype)), _i(h.stride(0)), _ptr(w_router), _ptr(correction), _ptr(logit_bias), _ptr(z), _ptr(idx),
         _ptr(wt), _ptr(gate), _i(T), _i(d), _i(n_outputs), _i(1 if has_gate else 0), _i(top), _i(groups), _i(keep),
-        _i(1 if sigmoid_scores else 0), _i(1 if renormalize else 0), _i(plan[0] if p is not None else 0),
+        _i(1 if sigmoid_scores else 0), _i(1 if renormalize else 0), _f(weight_scale), _i(plan[0] if p is not None else 0),
         _i(plan[1] if p is not None else 0), _ptr(p.offsets if p is not None else None),
         _ptr(p.sorted_pair if p is not None else None), _ptr(p.tile_expert if p is not None else None),
         _ptr(p.tile_row0 if p is not None else None), _ptr(p.n_tiles if p is not None else None),

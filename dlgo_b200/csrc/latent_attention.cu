@@ -6,10 +6,12 @@
 // and neither keys nor values are ever materialised: the query is carried into the latent space once, the
 // softmax runs over the latents themselves, and the weighted latent is carried out through Wv at the end.
 // Causal; `window` > 0 keeps keys with 0 <= i - j < window; `sink` (one number per head) adds exp(sink) to the
-// softmax's denominator and nothing else.  No positions are encoded.
+// softmax's denominator and nothing else.  Positions enter, if at all, through a rotated part: a cache row then ends
+// in one rotated key part shared by all heads, and every query head ends in a part that turns with the query's own
+// position (LatentRope).  `gate` (one logit per token and head): a head's output is multiplied by sigmoid(gate).
 //
-// latent_norm_append: the RMS norms of the down-projections (fp32), the kv latent appended to the paged
-// cache, the query latent (if the queries go through one) handed on in the activation type.
+// latent_norm_append: the RMS norms of the down-projections (fp32), the kv latent (and the shared key part, turned)
+// appended to the paged cache, the query latent (if the queries go through one) handed on in the activation type.
 // latent_attention:   one block per (token, head), all arithmetic in fp32; T is the type of the cache, the
 //                     weights and the output.  Keys are spread over the block's warps in a fixed pattern, so a
 //                     token's result does not depend on what else is in the batch.
@@ -17,13 +19,34 @@
 
 namespace dlgo {
 
+// The rotated part of a key row or a query head: its last `dims` numbers turn by the angle float(position) * freq[i],
+// formed, like its cosine and sine (times `amplitude`), in fp32.  `halves`: number i is paired with number i + dims/2,
+// else neighbours are paired (2i, 2i + 1).  dims 0: nothing turns.
+struct LatentRope {
+  const float* freq;
+  float amplitude;
+  int dims, halves;
+};
+
+// the pair i of the `dims` numbers at src, turned: its places within the part are left in a and b
+__device__ __forceinline__ float2 turned_pair(const float* src, int i, int pos, const LatentRope& rp, int& a, int& b) {
+  a = rp.halves ? i : 2 * i;
+  b = rp.halves ? i + rp.dims / 2 : 2 * i + 1;
+  float sn, cs;
+  sincosf((float)pos * rp.freq[i], &sn, &cs);
+  sn *= rp.amplitude;
+  cs *= rp.amplitude;
+  const float u = src[a], v = src[b];
+  return make_float2(u * cs - v * sn, v * cs + u * sn);
+}
+
 template <typename T>
-__global__ void latent_norm_append_kernel(const float* __restrict__ proj, int ld, int kv_off, int kv_rank,
+__global__ void latent_norm_append_kernel(const float* proj, int ld, int kv_off, int kv_rank,
                                           const float* __restrict__ w_kv, int q_off, int q_rank,
-                                          const float* __restrict__ w_q, T* __restrict__ cq, float eps,
+                                          const float* __restrict__ w_q, T* cq, float eps,
                                           const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                                           const int* __restrict__ seq_slot, const int* __restrict__ page_table,
-                                          int max_pages, T* __restrict__ pages, int page_size, int write_cache) {
+                                          int max_pages, T* pages, int page_size, int write_cache, LatentRope rope) {
   pdl_launch_dependents();
   __shared__ float scratch[32];
   __shared__ float scale_s;
@@ -31,14 +54,14 @@ __global__ void latent_norm_append_kernel(const float* __restrict__ proj, int ld
   const bool is_q = blockIdx.y == 1;
   const int n = is_q ? q_rank : kv_rank;
   const float* w = is_q ? w_q : w_kv;
+  const int pos = token_pos[t];
   T* dst = nullptr;
   if (is_q) {
     dst = cq + (size_t)t * q_rank;
   } else if (write_cache) {
-    const int pos = token_pos[t];
     const int slot = seq_slot[token_seq[t]];
     const int page = page_table[(size_t)slot * max_pages + pos / page_size];
-    if (page >= 0) dst = pages + ((size_t)page * page_size + pos % page_size) * kv_rank;
+    if (page >= 0) dst = pages + ((size_t)page * page_size + pos % page_size) * (kv_rank + rope.dims);
   }
   pdl_wait();
   if (dst == nullptr) return;
@@ -50,68 +73,44 @@ __global__ void latent_norm_append_kernel(const float* __restrict__ proj, int ld
   __syncthreads();
   const float sc = scale_s;
   for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = from_float<T>(x[i] * sc * w[i]);
+  if (is_q) return;
+  for (int i = threadIdx.x; i < rope.dims / 2; i += blockDim.x) {
+    int a, b;
+    const float2 v = turned_pair(x + kv_rank, i, pos, rope, a, b);
+    dst[kv_rank + a] = from_float<T>(v.x);
+    dst[kv_rank + b] = from_float<T>(v.y);
+  }
 }
 
-// The same for latents that carry a rotated key part: the down-projection has kv_rank + rope numbers; the first
-// kv_rank are normed (times w_kv) as above, the last `rope` are one key part shared by all heads, which turns with
-// the position (entries 2i and 2i + 1 by the angle pos * freq[i], cosine and sine times `amplitude`) and is kept
-// behind the latent in the same cache row ([.., page, kv_rank + rope]).  Queries q [T, H, dq] (fp32, inside
-// proj at q_off) turn in place in their last `rope` numbers of every head.  blockIdx.y: 0 the cache row, 1 the
-// queries.  Angles are float(pos) * freq in fp32.
+// Query heads made ready for the prompt kernels: q [T, H * dq] fp32 rows (ldq apart), every head's last rope.dims numbers
+// turned, into out [T, H, d_out] in the run's type (numbers dq .. d_out of a head are zero).  A warp per (token, head).
+constexpr int LQ_WARPS = 4;
 template <typename T>
-__global__ void latent_rope_append_kernel(float* proj, int ld, int kv_off, int kv_rank, const float* __restrict__ w_kv,
-                                          int q_off, int H, int dq, int rope, const float* __restrict__ freq,
-                                          float amplitude, float eps, const int* __restrict__ token_pos,
-                                          const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
-                                          const int* __restrict__ page_table, int max_pages, T* pages, int page_size,
-                                          int write_cache) {
+__global__ void __launch_bounds__(LQ_WARPS * 32)
+latent_queries_kernel(const float* q, int ldq, T* out, const int* __restrict__ token_pos, int n_tokens, int H, int dq,
+                      int d_out, LatentRope rope) {
   pdl_launch_dependents();
-  __shared__ float scratch[32];
-  __shared__ float scale_s;
-  const int t = blockIdx.x;
-  const int pos = token_pos[t];
-  const int half = rope / 2;
-  if (blockIdx.y == 1) {
-    pdl_wait();
-    float* q = proj + (size_t)t * ld + q_off;
-    for (int idx = threadIdx.x; idx < H * half; idx += blockDim.x) {
-      const int h = idx / half, i = idx - h * half;
-      float* pair = q + (size_t)h * dq + (dq - rope) + 2 * i;
-      float sn, cs;
-      sincosf((float)pos * freq[i], &sn, &cs);
-      sn *= amplitude;
-      cs *= amplitude;
-      const float u = pair[0], v = pair[1];
-      pair[0] = u * cs - v * sn;
-      pair[1] = v * cs + u * sn;
-    }
-    return;
-  }
-  T* dst = nullptr;
-  if (write_cache) {
-    const int slot = seq_slot[token_seq[t]];
-    const int page = page_table[(size_t)slot * max_pages + pos / page_size];
-    if (page >= 0) dst = pages + ((size_t)page * page_size + pos % page_size) * (kv_rank + rope);
-  }
+  const int lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * LQ_WARPS + (threadIdx.x >> 5);
   pdl_wait();
-  if (dst == nullptr) return;
-  const float* x = proj + (size_t)t * ld + kv_off;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
-  ss = block_sum(ss, scratch);
-  if (threadIdx.x == 0) scale_s = 1.0f / sqrtf(ss / (float)kv_rank + eps);
-  __syncthreads();
-  const float sc = scale_s;
-  for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) dst[i] = from_float<T>(x[i] * sc * w_kv[i]);
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    float sn, cs;
-    sincosf((float)pos * freq[i], &sn, &cs);
-    sn *= amplitude;
-    cs *= amplitude;
-    const float u = x[kv_rank + 2 * i], v = x[kv_rank + 2 * i + 1];
-    dst[kv_rank + 2 * i] = from_float<T>(u * cs - v * sn);
-    dst[kv_rank + 2 * i + 1] = from_float<T>(v * cs + u * sn);
+  if (item >= (long long)n_tokens * H) return;
+  const int t = (int)(item / H), h = (int)(item - (long long)t * H);
+  const float* src = q + (size_t)t * ldq + (size_t)h * dq;
+  T* dst = out + (size_t)item * d_out;
+  const int plain = dq - rope.dims;
+  for (int i = lane; i < plain; i += 32) dst[i] = from_float<T>(src[i]);
+  for (int i = dq + lane; i < d_out; i += 32) dst[i] = from_float<T>(0.f);
+  const int pos = token_pos[t];
+  for (int i = lane; i < rope.dims / 2; i += 32) {
+    int a, b;
+    const float2 v = turned_pair(src + plain, i, pos, rope, a, b);
+    dst[plain + a] = from_float<T>(v.x);
+    dst[plain + b] = from_float<T>(v.y);
   }
+}
+
+__device__ __forceinline__ float head_gate(const float* gate, int ldg, int t, int h) {
+  return gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h]));
 }
 
 // Latents of the pages a prompt step attends, gathered into rows [n_tmp * page_size, rank] (row = temporary page
@@ -120,9 +119,9 @@ __global__ void latent_rope_append_kernel(float* proj, int ld, int kv_off, int k
 constexpr int GATHER_PARTS = 8;     // blocks that share a page
 
 template <typename T>
-__global__ void latent_gather_kernel(const T* __restrict__ pages, const int* __restrict__ page_table, int max_pages,
+__global__ void latent_gather_kernel(const T* pages, const int* __restrict__ page_table, int max_pages,
                                      int page_size, const int* __restrict__ tmp_pages,
-                                     const int* __restrict__ seq_slot, T* __restrict__ out, int rank) {
+                                     const int* __restrict__ seq_slot, T* out, int rank) {
   pdl_launch_dependents();
   const int tp = blockIdx.x;
   const int seq = tmp_pages[tp * 3], lp = tmp_pages[tp * 3 + 1], valid = tmp_pages[tp * 3 + 2];
@@ -137,7 +136,7 @@ __global__ void latent_gather_kernel(const T* __restrict__ pages, const int* __r
   if ((rank % V) == 0 && (per % V) == 0 && ((uintptr_t)pages & 15) == 0 && ((uintptr_t)out & 15) == 0) {
     // written rows end at a multiple of `rank`, so a 16-byte piece is wholly written or wholly not
     for (int i = lo + threadIdx.x * V; i < hi; i += blockDim.x * V)
-      *reinterpret_cast<uint4*>(dst + i) = i < n_valid ? __ldg(reinterpret_cast<const uint4*>(src + i))
+      *reinterpret_cast<uint4*>(dst + i) = i < n_valid ? *reinterpret_cast<const uint4*>(src + i)
                                                         : make_uint4(0u, 0u, 0u, 0u);
     return;
   }
@@ -161,12 +160,12 @@ constexpr int LA_WARPS = 8;
 // NP: pairs of latent dimensions a lane holds (rank <= 64 * NP, rank even)
 template <typename T, int NP>
 __global__ void __launch_bounds__(LA_WARPS * 32)
-latent_attention_kernel(const void* __restrict__ q, int q_is_f32, int ldq, const T* __restrict__ w_k,
-                        const T* __restrict__ w_v, const float* __restrict__ sink, const T* __restrict__ pages,
+latent_attention_kernel(const void* q, int q_is_f32, int ldq, const T* __restrict__ w_k,
+                        const T* __restrict__ w_v, const float* __restrict__ sink, const T* pages,
                         const int* __restrict__ page_table, int max_pages, int page_size,
                         const int* __restrict__ seq_slot, const int* __restrict__ token_seq,
-                        const int* __restrict__ token_pos, T* __restrict__ out, int ldo, int dk, int dv, int rank,
-                        float scale, int window) {
+                        const int* __restrict__ token_pos, T* out, int ldo, int dk, int dv, int rank,
+                        float scale, int window, LatentRope rope, const float* gate, int ldg) {
   pdl_launch_dependents();
   extern __shared__ float smem[];
   float* s_q = smem;                         // [dk] the head's query
@@ -185,6 +184,15 @@ latent_attention_kernel(const void* __restrict__ q, int q_is_f32, int ldq, const
     s_q[i] = q_is_f32 ? reinterpret_cast<const float*>(q)[(size_t)t * ldq + h * dk + i]
                       : to_float(reinterpret_cast<const __nv_bfloat16*>(q)[(size_t)t * ldq + h * dk + i]);
   __syncthreads();
+  if (rope.dims > 0) {                       // a thread turns its own pairs in place
+    for (int i = threadIdx.x; i < rope.dims / 2; i += blockDim.x) {
+      int a, b;
+      const float2 v = turned_pair(s_q + dk - rope.dims, i, pos, rope, a, b);
+      s_q[dk - rope.dims + a] = v.x;
+      s_q[dk - rope.dims + b] = v.y;
+    }
+    __syncthreads();
+  }
   // the query in latent space: (Wk_h)^T q
   const T* wk = w_k + (size_t)h * dk * rank;
   for (int r = threadIdx.x; r < rank; r += blockDim.x) {
@@ -254,6 +262,7 @@ latent_attention_kernel(const void* __restrict__ q, int q_is_f32, int ldq, const
   __syncthreads();
   // out through Wv_h: a warp per output column
   const T* wv = w_v + (size_t)h * dv * rank;
+  const float hg = head_gate(gate, ldg, t, h);
   for (int e = warp; e < dv; e += LA_WARPS) {
     const T* row = wv + (size_t)e * rank;
     float a = 0.f;
@@ -263,7 +272,7 @@ latent_attention_kernel(const void* __restrict__ q, int q_is_f32, int ldq, const
       if (r + 1 < rank) a = fmaf(wv2.y, s_lat[r + 1], a);
     }
     a = warp_sum(a);
-    if (lane == 0) out[(size_t)t * ldo + h * dv + e] = from_float<T>(a);
+    if (lane == 0) out[(size_t)t * ldo + h * dv + e] = from_float<T>(a * hg);
   }
 }
 
@@ -281,8 +290,8 @@ constexpr int AB_COLS = 32;     // latent columns of a block (a lane each); its 
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_absorb_kernel(const void* __restrict__ q, int q_is_f32, int ldq, const T* __restrict__ w_k,
-                     float* __restrict__ q_lat, int n_tokens, int H, int dk, int rank) {
+latent_absorb_kernel(const void* q, int q_is_f32, int ldq, const T* __restrict__ w_k, float* q_lat, int n_tokens, int H,
+                     int dk, int rank, const int* __restrict__ token_pos, LatentRope rope) {
   pdl_launch_dependents();
   extern __shared__ float s_q[];                                // [AB_TOKENS][dk], then [4][AB_TOKENS][AB_COLS]
   float* s_part = s_q + AB_TOKENS * dk;
@@ -304,6 +313,18 @@ latent_absorb_kernel(const void* __restrict__ q, int q_is_f32, int ldq, const T*
                       : to_float(reinterpret_cast<const __nv_bfloat16*>(q)[(size_t)t * ldq + c]);
   }
   __syncthreads();
+  if (rope.dims > 0) {                                          // a thread turns its own pairs in place
+    const int half = rope.dims / 2;
+    for (int i = threadIdx.x; i < nt * half; i += 128) {
+      const int t = i / half;
+      float* part = s_q + (size_t)t * dk + dk - rope.dims;
+      int a, b;
+      const float2 v = turned_pair(part, i - t * half, token_pos[t0 + t], rope, a, b);
+      part[a] = v.x;
+      part[b] = v.y;
+    }
+    __syncthreads();
+  }
   for (int ib = i0; ib < i1; ib += 16) {
     float w[16];
 #pragma unroll
@@ -371,9 +392,9 @@ template <> struct Vec16<__nv_bfloat16> {
 // fetched together before any of them is used.
 template <typename T, int CH>
 __global__ void __launch_bounds__(LP_WARPS * 32)
-latent_partial_kernel(const float* __restrict__ q_lat, const T* __restrict__ pages, const int* __restrict__ page_table,
+latent_partial_kernel(const float* q_lat, const T* pages, const int* __restrict__ page_table,
                       int max_pages, int page_size, const int* __restrict__ seq_slot,
-                      const int* __restrict__ token_seq, const int* __restrict__ token_pos, float* __restrict__ parts,
+                      const int* __restrict__ token_seq, const int* __restrict__ token_pos, float* parts,
                       int H, int rank, int n_slices, float scale, int window) {
   constexpr int V = Vec16<T>::V;
   pdl_launch_dependents();
@@ -499,8 +520,8 @@ constexpr int LO_TOKENS = 8;    // tokens whose weighted latents sit in shared m
 
 template <typename T, int CH>
 __global__ void __launch_bounds__(LO_COLS * 32)
-latent_out_kernel(const float* __restrict__ parts, const T* __restrict__ w_v, const float* __restrict__ sink,
-                  T* __restrict__ out, int ldo, int n_tokens, int H, int dv, int rank, int n_slices) {
+latent_out_kernel(const float* parts, const T* __restrict__ w_v, const float* __restrict__ sink, T* out, int ldo,
+                  int n_tokens, int H, int dv, int rank, int n_slices, const float* gate, int ldg) {
   constexpr int V = Vec16<T>::V;
   pdl_launch_dependents();
   extern __shared__ float s_lat[];                              // [LO_TOKENS][rank]
@@ -558,7 +579,7 @@ latent_out_kernel(const float* __restrict__ parts, const T* __restrict__ w_v, co
           }
         }
         a = warp_sum(a);
-        if (lane == 0) out[(size_t)(t0 + tt) * ldo + h * dv + e] = from_float<T>(a);
+        if (lane == 0) out[(size_t)(t0 + tt) * ldo + h * dv + e] = from_float<T>(a * head_gate(gate, ldg, t0 + tt, h));
       }
     }
   }
@@ -569,13 +590,15 @@ static int launch_latent_few(const void* q, int q_is_f32, int ldq, const void* w
                              const void* pages, const int* page_table, int max_pages, int page_size,
                              const int* seq_slot, const int* token_seq, const int* token_pos, void* out, int ldo,
                              int n_tokens, int H, int dk, int dv, int rank, float scale, int window, int n_slices,
-                             float* q_lat, float* parts, cudaStream_t stream) {
+                             float* q_lat, float* parts, LatentRope rope,
+                             const float* gate, int ldg, cudaStream_t stream) {
   const size_t smem_a = (size_t)(AB_TOKENS * dk + 4 * AB_TOKENS * AB_COLS) * sizeof(float);
   const size_t smem_p = (size_t)LP_WARPS * rank * sizeof(float);
   const size_t smem_o = (size_t)LO_TOKENS * rank * sizeof(float);
   if (smem_a > 48 * 1024 || smem_p > 48 * 1024 || smem_o > 48 * 1024) return DLGO_ERR_SIZE;
   launch_kernel(latent_absorb_kernel<T>, dim3(H, (rank + AB_COLS - 1) / AB_COLS, (n_tokens + AB_TOKENS - 1) / AB_TOKENS), dim3(128),
-                smem_a, stream, q, q_is_f32, ldq, (const T*)w_k, q_lat, n_tokens, H, dk, rank);
+                smem_a, stream, q, q_is_f32, ldq, (const T*)w_k, q_lat, n_tokens, H, dk, rank,
+                token_pos, rope);
   int st = launch_status();
   if (st != DLGO_OK) return st;
   launch_kernel(latent_partial_kernel<T, CH>, dim3(n_tokens, H, n_slices), dim3(LP_WARPS * 32), smem_p, stream, q_lat,
@@ -584,7 +607,7 @@ static int launch_latent_few(const void* q, int q_is_f32, int ldq, const void* w
   st = launch_status();
   if (st != DLGO_OK) return st;
   launch_kernel(latent_out_kernel<T, CH>, dim3(H, (dv + LO_COLS - 1) / LO_COLS), dim3(LO_COLS * 32), smem_o, stream,
-                parts, (const T*)w_v, sink, (T*)out, ldo, n_tokens, H, dv, rank, n_slices);
+                parts, (const T*)w_v, sink, (T*)out, ldo, n_tokens, H, dv, rank, n_slices, gate, ldg);
   return launch_status();
 }
 
@@ -793,7 +816,7 @@ constexpr int LPJ_TOKENS = 8;   // tokens of a block of `project`
 template <typename T, int RC>
 __global__ void __launch_bounds__(256)
 latent_project_kernel(const float* lat, const T* __restrict__ w_v, T* out, int ldo, int n_tokens, int H, int dv,
-                      int rank) {
+                      int rank, const float* gate, int ldg) {
   constexpr int TG = RC <= 20 ? 4 : 2;
   pdl_launch_dependents();
   const int h = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -830,8 +853,9 @@ latent_project_kernel(const float* lat, const T* __restrict__ w_v, T* out, int l
       a0 = warp_sum(a0);
       a1 = warp_sum(a1);
       if (lane == 0 && tb + g < t_end) {
-        out[(size_t)(tb + g) * ldo + h * dv + e0] = from_float<T>(a0);
-        if (e0 + 1 < dv) out[(size_t)(tb + g) * ldo + h * dv + e0 + 1] = from_float<T>(a1);
+        const float hg = head_gate(gate, ldg, tb + g, h);
+        out[(size_t)(tb + g) * ldo + h * dv + e0] = from_float<T>(a0 * hg);
+        if (e0 + 1 < dv) out[(size_t)(tb + g) * ldo + h * dv + e0 + 1] = from_float<T>(a1 * hg);
       }
     }
   }
@@ -895,11 +919,13 @@ static int launch_latent_tiles(const void* q, int q_is_f32, int ldq, const void*
                                const void* pages, const int* page_table, int max_pages, int page_size,
                                const int* seq_slot, const int* token_seq, const int* token_pos, void* out, int ldo,
                                int n_tokens, int H, int dk, int dv, int rank, float scale, int window, int n_slices,
-                               float* q_lat, float* parts, cudaStream_t stream) {
+                               float* q_lat, float* parts, LatentRope rope,
+                             const float* gate, int ldg, cudaStream_t stream) {
   const size_t smem_a = (size_t)(AB_TOKENS * dk + 4 * AB_TOKENS * AB_COLS) * sizeof(float);
   if (smem_a > 48 * 1024) return DLGO_ERR_SIZE;
   launch_kernel(latent_absorb_kernel<T>, dim3(H, (rank + AB_COLS - 1) / AB_COLS, (n_tokens + AB_TOKENS - 1) / AB_TOKENS),
-                dim3(128), smem_a, stream, q, q_is_f32, ldq, (const T*)w_k, q_lat, n_tokens, H, dk, rank);
+                dim3(128), smem_a, stream, q, q_is_f32, ldq, (const T*)w_k, q_lat, n_tokens, H, dk, rank,
+                token_pos, rope);
   int st = launch_status();
   if (st != DLGO_OK) return st;
 #define LT_ARGS q_lat, pages, page_table, max_pages, page_size, seq_slot, token_seq, token_pos, parts, n_tokens, H, rank, \
@@ -918,10 +944,10 @@ static int launch_latent_tiles(const void* q, int q_is_f32, int ldq, const void*
   st = launch_status();
   if (st != DLGO_OK) return st;
   const dim3 grid(H, (dv + LPJ_COLS - 1) / LPJ_COLS, (n_tokens + LPJ_TOKENS - 1) / LPJ_TOKENS);
-  if (rc == 4) launch_kernel(latent_project_kernel<T, 4>, grid, dim3(256), 0, stream, q_lat, (const T*)w_v, (T*)out, ldo, n_tokens, H, dv, rank);
-  else if (rc == 8) launch_kernel(latent_project_kernel<T, 8>, grid, dim3(256), 0, stream, q_lat, (const T*)w_v, (T*)out, ldo, n_tokens, H, dv, rank);
-  else if (rc == 20) launch_kernel(latent_project_kernel<T, 20>, grid, dim3(256), 0, stream, q_lat, (const T*)w_v, (T*)out, ldo, n_tokens, H, dv, rank);
-  else launch_kernel(latent_project_kernel<T, 32>, grid, dim3(256), 0, stream, q_lat, (const T*)w_v, (T*)out, ldo, n_tokens, H, dv, rank);
+  if (rc == 4) launch_kernel(latent_project_kernel<T, 4>, grid, dim3(256), 0, stream, q_lat, (const T*)w_v, (T*)out, ldo, n_tokens, H, dv, rank, gate, ldg);
+  else if (rc == 8) launch_kernel(latent_project_kernel<T, 8>, grid, dim3(256), 0, stream, q_lat, (const T*)w_v, (T*)out, ldo, n_tokens, H, dv, rank, gate, ldg);
+  else if (rc == 20) launch_kernel(latent_project_kernel<T, 20>, grid, dim3(256), 0, stream, q_lat, (const T*)w_v, (T*)out, ldo, n_tokens, H, dv, rank, gate, ldg);
+  else launch_kernel(latent_project_kernel<T, 32>, grid, dim3(256), 0, stream, q_lat, (const T*)w_v, (T*)out, ldo, n_tokens, H, dv, rank, gate, ldg);
   return launch_status();
 }
 
@@ -929,14 +955,15 @@ template <typename T, int NP>
 static int launch_latent(const void* q, int q_is_f32, int ldq, const void* w_k, const void* w_v, const float* sink,
                          const void* pages, const int* page_table, int max_pages, int page_size, const int* seq_slot,
                          const int* token_seq, const int* token_pos, void* out, int ldo, int T_tokens, int H, int dk,
-                         int dv, int rank, float scale, int window, cudaStream_t stream) {
+                         int dv, int rank, float scale, int window, LatentRope rope,
+                             const float* gate, int ldg, cudaStream_t stream) {
   const size_t smem = (size_t)(dk + rank + LA_WARPS * rank) * sizeof(float);
   if (smem > 200 * 1024) return DLGO_ERR_SIZE;
   if (smem > 48 * 1024)
     cudaFuncSetAttribute(latent_attention_kernel<T, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   launch_kernel(latent_attention_kernel<T, NP>, dim3(T_tokens, H), dim3(LA_WARPS * 32), smem, stream, q, q_is_f32, ldq,
                 (const T*)w_k, (const T*)w_v, sink, (const T*)pages, page_table, max_pages, page_size, seq_slot,
-                token_seq, token_pos, (T*)out, ldo, dk, dv, rank, scale, window);
+                token_seq, token_pos, (T*)out, ldo, dk, dv, rank, scale, window, rope, gate, ldg);
   return launch_status();
 }
 
@@ -944,47 +971,51 @@ static int launch_latent(const void* q, int q_is_f32, int ldq, const void* w_k, 
 
 using namespace dlgo;
 
+// rope_dims numbers of a part of `whole` turn: an even number of them, with a frequency per pair
+static bool rope_ok(const float* freq, int rope_dims, int whole) {
+  return rope_dims >= 0 && rope_dims % 2 == 0 && rope_dims <= whole && (rope_dims == 0 || freq != nullptr);
+}
+
+// q [T, ldq] fp32 (H heads of dq numbers), out [T, H, d_out] in `dtype`: see latent_queries_kernel
+DLGO_EXPORT int dlgo_latent_queries(const float* q, int ldq, void* out, int dtype, const int* token_pos, int T, int H, int dq,
+                                    int d_out, const float* freq, float amplitude, int rope_dims, int halves,
+                                    cudaStream_t stream) {
+  if (T <= 0) return DLGO_OK;
+  if (H <= 0 || dq <= 0 || d_out < dq || !rope_ok(freq, rope_dims, dq)) return DLGO_ERR_SIZE;
+  const long long blocks = ((long long)T * H + LQ_WARPS - 1) / LQ_WARPS;
+  if (blocks > 0x7fffffffLL) return DLGO_ERR_SIZE;
+  const LatentRope rope{freq, amplitude, rope_dims, halves};
+  if (dtype == DLGO_F32)
+    launch_kernel(latent_queries_kernel<float>, dim3((unsigned)blocks), dim3(LQ_WARPS * 32), 0, stream, q, ldq, (float*)out,
+                  token_pos, T, H, dq, d_out, rope);
+  else if (dtype == DLGO_BF16)
+    launch_kernel(latent_queries_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(LQ_WARPS * 32), 0, stream, q, ldq,
+                  (__nv_bfloat16*)out, token_pos, T, H, dq, d_out, rope);
+  else
+    return DLGO_ERR_DTYPE;
+  return launch_status();
+}
+
 DLGO_EXPORT int dlgo_latent_norm_append(const float* proj, int ld, int T_tokens, int kv_off, int kv_rank,
                                         const float* w_kv, int q_off, int q_rank, const float* w_q, void* cq,
                                         float eps, const int* token_pos, const int* token_seq, const int* seq_slot,
                                         const int* page_table, int max_pages, void* pages, int dtype, int page_size,
-                                        int write_cache, cudaStream_t stream) {
+                                        int write_cache, const float* freq, float amplitude, int rope_dims, int halves,
+                                        cudaStream_t stream) {
   if (T_tokens <= 0) return DLGO_OK;
-  if (kv_rank <= 0 || q_rank < 0 || page_size <= 0) return DLGO_ERR_SIZE;
+  if (kv_rank <= 0 || q_rank < 0 || page_size <= 0 || !rope_ok(freq, rope_dims, rope_dims)) return DLGO_ERR_SIZE;
+  const LatentRope rope{freq, amplitude, rope_dims, halves};
   const dim3 grid(T_tokens, q_rank > 0 ? 2 : 1);
   const int n = kv_rank > q_rank ? kv_rank : q_rank;
   const int threads = n >= 1024 ? 256 : 128;
   if (dtype == DLGO_F32)
     launch_kernel(latent_norm_append_kernel<float>, grid, dim3(threads), 0, stream, proj, ld, kv_off, kv_rank, w_kv,
                   q_off, q_rank, w_q, (float*)cq, eps, token_pos, token_seq, seq_slot, page_table, max_pages,
-                  (float*)pages, page_size, write_cache);
+                  (float*)pages, page_size, write_cache, rope);
   else if (dtype == DLGO_BF16)
     launch_kernel(latent_norm_append_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, proj, ld, kv_off, kv_rank,
                   w_kv, q_off, q_rank, w_q, (__nv_bfloat16*)cq, eps, token_pos, token_seq, seq_slot, page_table,
-                  max_pages, (__nv_bfloat16*)pages, page_size, write_cache);
-  else
-    return DLGO_ERR_DTYPE;
-  return launch_status();
-}
-
-DLGO_EXPORT int dlgo_latent_rope_append(float* proj, int ld, int T_tokens, int kv_off, int kv_rank, const float* w_kv,
-                                        int q_off, int H, int dq, int rope, const float* freq, float amplitude,
-                                        float eps, const int* token_pos, const int* token_seq, const int* seq_slot,
-                                        const int* page_table, int max_pages, void* pages, int dtype, int page_size,
-                                        int write_cache, cudaStream_t stream) {
-  if (T_tokens <= 0) return DLGO_OK;
-  if (kv_rank <= 0 || page_size <= 0 || rope <= 0 || (rope & 1) || rope > dq || H <= 0 || freq == nullptr)
-    return DLGO_ERR_SIZE;
-  const dim3 grid(T_tokens, 2);
-  const int threads = kv_rank >= 1024 ? 256 : 128;
-  if (dtype == DLGO_F32)
-    launch_kernel(latent_rope_append_kernel<float>, grid, dim3(threads), 0, stream, proj, ld, kv_off, kv_rank, w_kv,
-                  q_off, H, dq, rope, freq, amplitude, eps, token_pos, token_seq, seq_slot, page_table, max_pages,
-                  (float*)pages, page_size, write_cache);
-  else if (dtype == DLGO_BF16)
-    launch_kernel(latent_rope_append_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, proj, ld, kv_off, kv_rank,
-                  w_kv, q_off, H, dq, rope, freq, amplitude, eps, token_pos, token_seq, seq_slot, page_table, max_pages,
-                  (__nv_bfloat16*)pages, page_size, write_cache);
+                  max_pages, (__nv_bfloat16*)pages, page_size, write_cache, rope);
   else
     return DLGO_ERR_DTYPE;
   return launch_status();
@@ -1007,13 +1038,14 @@ DLGO_EXPORT int dlgo_latent_gather(const void* pages, int dtype, const int* page
 }
 
 #define LATENT_ARGS q, q_is_f32, ldq, w_k, w_v, sink, pages, page_table, max_pages, page_size, seq_slot, token_seq, \
-                    token_pos, out, ldo, T_tokens, H, dk, dv, rank, scale, window, stream
+                    token_pos, out, ldo, T_tokens, H, dk, dv, rank, scale, window, rope, gate, ldg, stream
 
 template <typename T>
 static int latent_by_rank(const void* q, int q_is_f32, int ldq, const void* w_k, const void* w_v, const float* sink,
                           const void* pages, const int* page_table, int max_pages, int page_size, const int* seq_slot,
                           const int* token_seq, const int* token_pos, void* out, int ldo, int T_tokens, int H, int dk,
-                          int dv, int rank, float scale, int window, cudaStream_t stream) {
+                          int dv, int rank, float scale, int window, LatentRope rope,
+                             const float* gate, int ldg, cudaStream_t stream) {
   if (rank <= 64) return launch_latent<T, 1>(LATENT_ARGS);
   if (rank <= 128) return launch_latent<T, 2>(LATENT_ARGS);
   if (rank <= 256) return launch_latent<T, 4>(LATENT_ARGS);
@@ -1023,14 +1055,15 @@ static int latent_by_rank(const void* q, int q_is_f32, int ldq, const void* w_k,
 }
 
 #define FEW_ARGS q, q_is_f32, ldq, w_k, w_v, sink, pages, page_table, max_pages, page_size, seq_slot, token_seq, \
-                 token_pos, out, ldo, T_tokens, H, dk, dv, rank, scale, window, n_slices, q_lat, parts, stream
+                 token_pos, out, ldo, T_tokens, H, dk, dv, rank, scale, window, n_slices, q_lat, parts, rope, gate, ldg, stream
 
 template <typename T>
 static int latent_few_by_rank(const void* q, int q_is_f32, int ldq, const void* w_k, const void* w_v,
                               const float* sink, const void* pages, const int* page_table, int max_pages,
                               int page_size, const int* seq_slot, const int* token_seq, const int* token_pos,
                               void* out, int ldo, int T_tokens, int H, int dk, int dv, int rank, float scale,
-                              int window, int n_slices, float* q_lat, float* parts, cudaStream_t stream) {
+                              int window, int n_slices, float* q_lat, float* parts, LatentRope rope,
+                             const float* gate, int ldg, cudaStream_t stream) {
   constexpr int V = 16 / (int)sizeof(T);
   if (rank % V) return DLGO_ERR_SIZE;                           // rows are read 16 bytes at a time
   const int lanes = (rank + V - 1) / V;                         // 16-byte pieces of a row
@@ -1054,11 +1087,14 @@ DLGO_EXPORT int dlgo_latent_attention_few(const void* q, int q_is_f32, int ldq, 
                                           int max_pages, int page_size, const int* seq_slot, const int* token_seq,
                                           const int* token_pos, void* out, int ldo, int T_tokens, int H, int dk,
                                           int dv, int rank, float scale, int window, int n_slices, float* q_lat,
-                                          float* parts, cudaStream_t stream) {
+                                          float* parts, const float* freq, float amplitude, int rope_dims,
+                                          int halves, const float* gate, int ldg, cudaStream_t stream) {
   if (T_tokens <= 0) return DLGO_OK;
   if (H <= 0 || dk <= 0 || dv <= 0 || rank <= 0 || page_size <= 0 || window < 0 || n_slices < 1 ||
       n_slices > 32 || H > 65535)      // (a lane per slice where the slices meet)
     return DLGO_ERR_SIZE;
+  if (!rope_ok(freq, rope_dims, dk)) return DLGO_ERR_SIZE;
+  const LatentRope rope{freq, amplitude, rope_dims, halves};
   if (((uintptr_t)pages & 15) || ((uintptr_t)w_v & 15)) return DLGO_ERR_ALIGN;
   if (dtype == DLGO_F32) return latent_few_by_rank<float>(FEW_ARGS);
   if (dtype == DLGO_BF16) {
@@ -1078,14 +1114,17 @@ DLGO_EXPORT int dlgo_latent_attention_tiles(const void* q, int q_is_f32, int ldq
                                             int max_pages, int page_size, const int* seq_slot, const int* token_seq,
                                             const int* token_pos, void* out, int ldo, int T_tokens, int H, int dk,
                                             int dv, int rank, float scale, int window, int n_slices, float* q_lat,
-                                            float* parts, cudaStream_t stream) {
+                                            float* parts, const float* freq, float amplitude, int rope_dims,
+                                          int halves, const float* gate, int ldg, cudaStream_t stream) {
   if (T_tokens <= 0) return DLGO_OK;
   if (H <= 0 || dk <= 0 || dv <= 0 || rank <= 0 || page_size <= 0 || window < 0 || n_slices < 1 || n_slices > 32 ||
       H > 65535 || !dlgo_latent_attention_tiles_takes(dtype, H, rank))
     return DLGO_ERR_SIZE;
+  if (!rope_ok(freq, rope_dims, dk)) return DLGO_ERR_SIZE;
+  const LatentRope rope{freq, amplitude, rope_dims, halves};
   if (((uintptr_t)pages & 15) || ((uintptr_t)q_lat & 15)) return DLGO_ERR_ALIGN;
 #define TILES_ARGS q, q_is_f32, ldq, w_k, w_v, sink, pages, page_table, max_pages, page_size, seq_slot, token_seq, \
-                   token_pos, out, ldo, T_tokens, H, dk, dv, rank, scale, window, n_slices, q_lat, parts, stream
+                   token_pos, out, ldo, T_tokens, H, dk, dv, rank, scale, window, n_slices, q_lat, parts, rope, gate, ldg, stream
   if (dtype == DLGO_F32) return launch_latent_tiles<float>(TILES_ARGS);
   return launch_latent_tiles<__nv_bfloat16>(TILES_ARGS);
 #undef TILES_ARGS
@@ -1097,9 +1136,12 @@ DLGO_EXPORT int dlgo_latent_attention(const void* q, int q_is_f32, int ldq, cons
                                       const float* sink, const void* pages, int dtype, const int* page_table,
                                       int max_pages, int page_size, const int* seq_slot, const int* token_seq,
                                       const int* token_pos, void* out, int ldo, int T_tokens, int H, int dk, int dv,
-                                      int rank, float scale, int window, cudaStream_t stream) {
+                                      int rank, float scale, int window, const float* freq, float amplitude, int rope_dims,
+                                      int halves, const float* gate, int ldg, cudaStream_t stream) {
   if (T_tokens <= 0) return DLGO_OK;
   if (H <= 0 || dk <= 0 || dv <= 0 || rank <= 0 || page_size <= 0 || window < 0) return DLGO_ERR_SIZE;
+  if (!rope_ok(freq, rope_dims, dk)) return DLGO_ERR_SIZE;
+  const LatentRope rope{freq, amplitude, rope_dims, halves};
   if (((uintptr_t)pages & 7) || ((uintptr_t)w_v & 7)) return DLGO_ERR_ALIGN;
   if (dtype == DLGO_F32) return latent_by_rank<float>(LATENT_ARGS);
   if (dtype == DLGO_BF16) {

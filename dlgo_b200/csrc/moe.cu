@@ -4,7 +4,7 @@
 //                  router outputs, choice scores c = s + correction, group-limited choice of `top` outputs
 //                  (outputs form `groups` equal groups of neighbours; a group's score is its largest choice
 //                  score; only outputs of the `keep` best groups can be chosen, the others count as minus
-//                  infinity), weights = the chosen outputs' s (optionally renormalised).  A bias on the logits
+//                  infinity), weights = the chosen outputs' s (optionally renormalised) times a constant.  A bias on the logits
 //                  (`zbias`, one number per output) is part of z: it moves scores and weights alike.  A further row of Wr
 //                  (`has_gate`) gives a per-token gate sigmoid(w_g . h) for a shared expert.
 // 2. moe_plan:     (token, choice) pairs sorted by expert: offsets per expert, the sorted pair list, and a list
@@ -77,7 +77,7 @@ template <> struct Quad<__nv_bfloat16> {
 
 template <typename T, int TOK, bool VEC>
 __global__ void __launch_bounds__(RL_WARPS * 32)
-moe_logits_kernel(const T* __restrict__ h, int ldh, const float* __restrict__ Wr, float* __restrict__ z, int tokens,
+moe_logits_kernel(const T* h, int ldh, const float* __restrict__ Wr, float* z, int tokens,
                   int d, int rows) {
   __shared__ float part[RL_WARPS][RL_OB * TOK];
   pdl_launch_dependents();
@@ -147,10 +147,10 @@ moe_logits_kernel(const T* __restrict__ h, int ldh, const float* __restrict__ Wr
 constexpr int RC_WARPS = 4;
 
 // One token's choice by one warp; zt / ct / gt are the warp's scratch rows (rows, n and groups floats).
-__device__ __forceinline__ void choose_token(const float* __restrict__ zg, const float* __restrict__ corr,
-                                             const float* __restrict__ zbias, int* __restrict__ idx, float* __restrict__ wt, float* __restrict__ gate,
+__device__ __forceinline__ void choose_token(const float* zg, const float* __restrict__ corr,
+                                             const float* __restrict__ zbias, int* idx, float* wt, float* gate,
                                              int t, int n, int has_gate, int top, int groups, int keep,
-                                             int sigmoid_scores, int renormalize, float* zt, float* ct, float* gt,
+                                             int sigmoid_scores, int renormalize, float wscale, float* zt, float* ct, float* gt,
                                              int lane) {
   const int rows = n + (has_gate ? 1 : 0);
   for (int j = lane; j < rows; j += 32) zt[j] = zg[(size_t)t * rows + j] + (zbias != nullptr && j < n ? zbias[j] : 0.f);
@@ -208,7 +208,7 @@ __device__ __forceinline__ void choose_token(const float* __restrict__ zg, const
     __syncwarp();
     if (lane == 0) {
       idx[(size_t)t * top + r] = at;
-      wt[(size_t)t * top + r] = wv;
+      wt[(size_t)t * top + r] = wv * wscale;
       ct[at] = -CUDART_INF_F;
     }
     __syncwarp();
@@ -218,10 +218,10 @@ __device__ __forceinline__ void choose_token(const float* __restrict__ zg, const
 }
 
 __global__ void __launch_bounds__(RC_WARPS * 32)
-moe_choose_kernel(const float* __restrict__ zg, const float* __restrict__ corr, const float* __restrict__ zbias,
-                  int* __restrict__ idx,
-                  float* __restrict__ wt, float* __restrict__ gate, int tokens, int n, int has_gate, int top, int groups,
-                  int keep, int sigmoid_scores, int renormalize) {
+moe_choose_kernel(const float* zg, const float* __restrict__ corr, const float* __restrict__ zbias,
+                  int* idx,
+                  float* wt, float* gate, int tokens, int n, int has_gate, int top, int groups,
+                  int keep, int sigmoid_scores, int renormalize, float wscale) {
   extern __shared__ float rt_smem[];
   pdl_launch_dependents();
   const int rows = n + (has_gate ? 1 : 0);
@@ -230,7 +230,7 @@ moe_choose_kernel(const float* __restrict__ zg, const float* __restrict__ corr, 
   const int t = blockIdx.x * RC_WARPS + warp;
   pdl_wait();
   if (t >= tokens) return;
-  choose_token(zg, corr, zbias, idx, wt, gate, t, n, has_gate, top, groups, keep, sigmoid_scores, renormalize, zt, zt + rows,
+  choose_token(zg, corr, zbias, idx, wt, gate, t, n, has_gate, top, groups, keep, sigmoid_scores, renormalize, wscale, zt, zt + rows,
                zt + rows + n, lane);
 }
 
@@ -238,10 +238,10 @@ moe_choose_kernel(const float* __restrict__ zg, const float* __restrict__ corr, 
 constexpr int PLAN_THREADS = 1024;
 
 // The whole block; count / cursor are n_experts ints of shared memory each, count zeroed (and a barrier passed).
-__device__ __forceinline__ void plan_block(const int* __restrict__ idx, int pairs, int n_experts, int tile_rows,
-                                           int* __restrict__ offsets, int* __restrict__ sorted_pair,
-                                           int* __restrict__ tile_expert, int* __restrict__ tile_row0,
-                                           int* __restrict__ n_tiles, int max_tiles, int* count, int* cursor) {
+__device__ __forceinline__ void plan_block(const int* idx, int pairs, int n_experts, int tile_rows,
+                                           int* offsets, int* sorted_pair,
+                                           int* tile_expert, int* tile_row0,
+                                           int* n_tiles, int max_tiles, int* count, int* cursor) {
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
     const int e = idx[i];
     if (e >= 0 && e < n_experts) atomicAdd(&count[e], 1);
@@ -272,9 +272,9 @@ __device__ __forceinline__ void plan_block(const int* __restrict__ idx, int pair
 }
 
 __global__ void __launch_bounds__(PLAN_THREADS)
-moe_plan_kernel(const int* __restrict__ idx, int pairs, int n_experts, int tile_rows, int* __restrict__ offsets,
-                int* __restrict__ sorted_pair, int* __restrict__ tile_expert, int* __restrict__ tile_row0,
-                int* __restrict__ n_tiles, int max_tiles) {
+moe_plan_kernel(const int* idx, int pairs, int n_experts, int tile_rows, int* offsets,
+                int* sorted_pair, int* tile_expert, int* tile_row0,
+                int* n_tiles, int max_tiles) {
   extern __shared__ int pl_smem[];
   int* count = pl_smem;                  // [n_experts]
   int* cursor = count + n_experts;       // [n_experts]
@@ -288,12 +288,12 @@ moe_plan_kernel(const int* __restrict__ idx, int pairs, int n_experts, int tile_
 
 // Choice and plan of a step of few tokens in one launch: one block, a warp per token in turn, then the plan.
 __global__ void __launch_bounds__(PLAN_THREADS)
-moe_choose_plan_kernel(const float* __restrict__ zg, const float* __restrict__ corr,
-                       const float* __restrict__ zbias, int* __restrict__ idx,
-                       float* __restrict__ wt, float* __restrict__ gate, int tokens, int n, int has_gate, int top,
-                       int groups, int keep, int sigmoid_scores, int renormalize, int n_experts, int tile_rows,
-                       int* __restrict__ offsets, int* __restrict__ sorted_pair, int* __restrict__ tile_expert,
-                       int* __restrict__ tile_row0, int* __restrict__ n_tiles, int max_tiles) {
+moe_choose_plan_kernel(const float* zg, const float* __restrict__ corr,
+                       const float* __restrict__ zbias, int* idx,
+                       float* wt, float* gate, int tokens, int n, int has_gate, int top,
+                       int groups, int keep, int sigmoid_scores, int renormalize, float wscale, int n_experts, int tile_rows,
+                       int* offsets, int* sorted_pair, int* tile_expert,
+                       int* tile_row0, int* n_tiles, int max_tiles) {
   extern __shared__ float rt_smem[];
   pdl_launch_dependents();
   const int rows = n + (has_gate ? 1 : 0);
@@ -304,7 +304,7 @@ moe_choose_plan_kernel(const float* __restrict__ zg, const float* __restrict__ c
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) count[e] = 0;
   pdl_wait();
   for (int t = warp; t < tokens; t += n_warps) {
-    choose_token(zg, corr, zbias, idx, wt, gate, t, n, has_gate, top, groups, keep, sigmoid_scores, renormalize, zt, zt + rows,
+    choose_token(zg, corr, zbias, idx, wt, gate, t, n, has_gate, top, groups, keep, sigmoid_scores, renormalize, wscale, zt, zt + rows,
                  zt + rows + n, lane);
     __syncwarp();
   }
@@ -496,9 +496,9 @@ moe_gemm_tiles_kernel(GroupedArgs g) {
 // experts' results (fp32 or the run's type).
 template <typename T, typename P, bool VEC>
 __global__ void __launch_bounds__(256)
-moe_combine_kernel(float* __restrict__ y, const P* __restrict__ pair_out, const T* __restrict__ h, int ldh,
-                   const int* __restrict__ idx, const float* __restrict__ wt, const float* __restrict__ shared,
-                   const float* __restrict__ gate, int tokens, int d, int top, int n_experts) {
+moe_combine_kernel(float* y, const P* pair_out, const T* h, int ldh,
+                   const int* idx, const float* wt, const float* shared,
+                   const float* gate, int tokens, int d, int top, int n_experts) {
   pdl_launch_dependents();
   constexpr int W = VEC ? 4 : 1;
   const int per_row = (d + W - 1) / W;
@@ -597,7 +597,7 @@ static void launch_logits(const void* h, int ldh, const float* Wr, float* z, int
 DLGO_EXPORT int dlgo_moe_router(const void* h, int dtype, int ldh, const float* Wr, const float* corr,
                                 const float* zbias, float* z, int* idx,
                                 float* wt, float* gate, int tokens, int d, int n, int has_gate, int top, int groups,
-                                int keep, int sigmoid_scores, int renormalize, int plan_experts, int tile_rows,
+                                int keep, int sigmoid_scores, int renormalize, float wscale, int plan_experts, int tile_rows,
                                 int* offsets, int* sorted_pair, int* tile_expert, int* tile_row0, int* n_tiles,
                                 int max_tiles, int* fused, cudaStream_t stream) {
   if (fused != nullptr) *fused = 0;
@@ -618,14 +618,15 @@ DLGO_EXPORT int dlgo_moe_router(const void* h, int dtype, int ldh, const float* 
     const int pairs = tokens * top;
     if (both <= 48 * 1024 && tile_rows > 0 && max_tiles >= (pairs + tile_rows - 1) / tile_rows + plan_experts) {
       launch_kernel(moe_choose_plan_kernel, dim3(1), dim3(warps * 32), both, stream, (const float*)z, corr, zbias, idx, wt, gate,
-                    tokens, n, has_gate, top, groups, keep, sigmoid_scores, renormalize, plan_experts, tile_rows, offsets,
+                    tokens, n, has_gate, top, groups, keep, sigmoid_scores, renormalize, wscale, plan_experts, tile_rows, offsets,
                     sorted_pair, tile_expert, tile_row0, n_tiles, max_tiles);
       *fused = 1;
       return launch_status();
     }
   }
   launch_kernel(moe_choose_kernel, dim3((tokens + RC_WARPS - 1) / RC_WARPS), dim3(RC_WARPS * 32), smem, stream,
-                (const float*)z, corr, zbias, idx, wt, gate, tokens, n, has_gate, top, groups, keep, sigmoid_scores, renormalize);
+                (const float*)z, corr, zbias, idx, wt, gate, tokens, n, has_gate, top, groups, keep, sigmoid_scores, renormalize,
+                wscale);
   return launch_status();
 }
 

@@ -437,9 +437,9 @@ moe_gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
 // Rows of the step's tokens in sorted pair order: dst[r] = src[pair(r) / div] for the r < offsets[experts] rows
 // that belong to an expert (16 bytes per thread and step).
 __global__ void __launch_bounds__(256)
-moe_gather_rows_kernel(const uint4* __restrict__ src, long long src_ld16, uint4* __restrict__ dst, int row16,
-                       const int* __restrict__ sorted_pair, const int* __restrict__ total, int div, int max_rows,
-                       const float* __restrict__ pair_scale) {
+moe_gather_rows_kernel(const uint4* src, long long src_ld16, uint4* dst, int row16,
+                       const int* sorted_pair, const int* total, int div, int max_rows,
+                       const float* pair_scale) {
   pdl_launch_dependents();
   pdl_wait();
   const int n = min(*total, max_rows);

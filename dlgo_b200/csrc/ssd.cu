@@ -1,0 +1,652 @@
+// State-space mixing with a scalar decay per head and token (the recurrence of Mamba-2), its short convolution and its
+// gated group norm.
+//
+// One projection row per token holds [z: H P | x: H P | B: G N | C: G N | dt: H] (fp32).  With a the silu:
+//   conv:   (x | B | C)_t <- a(bias + sum_j taps[:, j] u_(t - n + 1 + j))   per channel, u = 0 before a sequence's start
+//   step:   d_t = softplus(dt_t + dt_bias),  f_t = exp(-exp(A_log) d_t)     per head
+//   state:  S_t = f_t S_(t-1) + d_t B_t x_t^T                               S [N, P] per head, fp32, zero at the start
+//   out:    y_t = S_t^T C_t + D x_t                                         head h reads B and C of group h / (H / G)
+//   norm:   u = y * a(z);  each of `groups` equal parts of u divided by its root mean square, then times w
+// A sequence's state row is [H N P numbers of S | (n - 1) inputs of the convolution, oldest first], fp32, `state_ld`
+// floats apart, and is carried from step to step.
+//
+// ssd_conv       prompts: convolution and silu of every channel, d and f of every head, for all tokens of the step
+// ssd_segments   prompts: a sequence's tokens are cut into segments that run side by side
+//                  LOCAL   every segment but a sequence's last runs from a zero state: its end state L_j, and the
+//                          product F_j of its decays
+//                  carry   starts[j] = F_(j-1) starts[j-1] + L_(j-1) from the stored state, element by element
+//                  FULL    every segment walks its tokens from its start; the last one stores the sequence's new state
+//                with one segment per sequence FULL runs alone from the stored state
+// ssd_step       decoding: convolution, step, state and output of one token per sequence in one launch
+// ssd_gate_norm  gate and norm; the token that ends a sequence's part of the step also moves the convolution's inputs
+//                into the state row (every reader of the old ones ran in an earlier launch)
+//
+// The state kernels share one layout: a thread holds 16 rows x 4 columns of a head's state in registers.  RS
+// neighbouring lanes share four columns; lane r of them holds rows 4 (i RS + r) .. + 3 for i = 0 .. 3 (so that their
+// 16-byte reads of B and C fall side by side), and their parts of y meet by shuffles.  N up to 512;
+// rows beyond N and columns beyond P are computed on zeros and not stored.  Everything is fp32 in every precision.
+#include "common.cuh"
+#include "async_copy.cuh"
+
+namespace dlgo {
+
+__device__ __forceinline__ float ssd_silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float ssd_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
+// where a sequence's inputs of earlier steps lie: entry j of taps - 1, oldest first
+struct SsdShape {
+  int H, G, N, P, taps;
+  __host__ __device__ int inner() const { return H * P; }
+  __host__ __device__ int channels() const { return H * P + 2 * G * N; }
+  __host__ __device__ long long conv_off() const { return (long long)H * N * P; }
+};
+
+// The input of channel c at packed token `tok` of sequence `seq` (tok may lie before the sequence's first token of
+// this step; `first` is that token): a projected number, or one kept from an earlier step.
+__device__ __forceinline__ float conv_input(const float* xbc, int ld, int tok, int first, int c, const float* kept,
+                                            int taps, int channels) {
+  if (tok >= first) return xbc[(size_t)tok * ld + c];
+  return kept[(size_t)(taps - 1 + tok - first) * channels + c];
+}
+
+// ------------------------------------------------------------------------------- convolution (prompts)
+constexpr int SC_THREADS = 128;
+
+// A thread owns W neighbouring channels and walks its tile's tokens with the taps' reach in registers (TAPS > 0) or
+// reads every tap from memory (TAPS 0: any number of taps).
+template <int TAPS, int W>
+__global__ void __launch_bounds__(SC_THREADS)
+ssd_conv_kernel(const float* proj, int ld, const float* __restrict__ w_taps, const float* __restrict__ w_bias,
+                const float* __restrict__ dt_bias, const float* __restrict__ a_log, const int* __restrict__ tiles,
+                const int* __restrict__ token_seq, const int* __restrict__ seq_slot, const float* state,
+                long long state_ld, float* out, int ldo, float* steps, SsdShape s) {
+  pdl_launch_dependents();
+  const int tile = blockIdx.x;
+  const int seq = tiles[tile * 3 + 0], t0 = tiles[tile * 3 + 1], count = tiles[tile * 3 + 2];
+  const int C = s.channels(), n_taps = TAPS > 0 ? TAPS : s.taps;
+  if (blockIdx.y == gridDim.y - 1) {               // the heads' steps and decays
+    pdl_wait();
+    const float* dt = proj + s.inner() + C;
+    for (int i = threadIdx.x; i < count * s.H; i += SC_THREADS) {
+      const int t = t0 + i / s.H, h = i % s.H;
+      const float d = ssd_softplus(dt[(size_t)t * ld + h] + dt_bias[h]);
+      steps[((size_t)t * s.H + h) * 2] = d;
+      steps[((size_t)t * s.H + h) * 2 + 1] = expf(-expf(a_log[h]) * d);
+    }
+    return;
+  }
+  const int c = (blockIdx.y * SC_THREADS + threadIdx.x) * W;
+  if (c >= C) return;
+  int first = t0;                                  // the sequence's first token of this step, if within the taps' reach
+  while (first > 0 && first > t0 - n_taps + 1 && token_seq[first - 1] == seq) --first;
+  const float* kept = state + (size_t)seq_slot[seq] * state_ld + s.conv_off();
+  const float* xbc = proj + s.inner();
+  float bias[W];
+#pragma unroll
+  for (int k = 0; k < W; ++k) bias[k] = w_bias[c + k];
+  if (TAPS > 0) {
+    constexpr int R = TAPS > 0 ? TAPS : 1;
+    float tap[R][W], u[R][W];
+#pragma unroll
+    for (int j = 0; j < R; ++j)
+#pragma unroll
+      for (int k = 0; k < W; ++k) tap[j][k] = w_taps[(size_t)(c + k) * R + j];
+    pdl_wait();
+#pragma unroll
+    for (int j = 0; j < R - 1; ++j) {
+#pragma unroll
+      for (int k = 0; k < W; ++k) u[j][k] = conv_input(xbc, ld, t0 - R + 1 + j, first, c + k, kept, R, C);
+    }
+    for (int tb = 0; tb < count; tb += 4) {
+      float in[4][W];                              // four tokens' fetches in flight
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float* src = xbc + (size_t)(t0 + min(tb + q, count - 1)) * ld + c;
+        if (W == 4) {
+          const float4 v = *reinterpret_cast<const float4*>(src);
+          in[q][0] = v.x; in[q][1 % W] = v.y; in[q][2 % W] = v.z; in[q][3 % W] = v.w;
+        } else {
+          in[q][0] = src[0];
+        }
+      }
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        if (tb + q >= count) break;
+        float y[W];
+#pragma unroll
+        for (int k = 0; k < W; ++k) {
+          u[R - 1][k] = in[q][k];
+          float a = bias[k];
+#pragma unroll
+          for (int j = 0; j < R; ++j) a = fmaf(tap[j][k], u[j][k], a);
+          y[k] = ssd_silu(a);
+#pragma unroll
+          for (int j = 0; j < R - 1; ++j) u[j][k] = u[j + 1][k];
+        }
+        float* dst = out + (size_t)(t0 + tb + q) * ldo + c;
+        if (W == 4) *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1 % W], y[2 % W], y[3 % W]);
+        else dst[0] = y[0];
+      }
+    }
+    return;
+  }
+  pdl_wait();
+  for (int t = t0; t < t0 + count; ++t) {
+#pragma unroll
+    for (int k = 0; k < W; ++k) {
+      float a = bias[k];
+      for (int j = 0; j < n_taps; ++j)
+        a = fmaf(w_taps[(size_t)(c + k) * n_taps + j], conv_input(xbc, ld, t - n_taps + 1 + j, first, c + k, kept, n_taps, C), a);
+      out[(size_t)t * ldo + c + k] = ssd_silu(a);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------- the state in registers
+// y[k] of the RS lanes that share four columns brought together: afterwards lane r < min(RS, 4) holds the sum of
+// columns (4 / min(RS, 4)) * r .. in y[0 ..].
+template <int RS>
+__device__ __forceinline__ void ssd_meet(float (&y)[4], int r) {
+  if (RS >= 4) {             // lanes 2 apart trade halves, neighbours trade one of two, then the lanes 4, 8, .. apart add up
+    const bool hi2 = (r & 2) != 0, hi1 = (r & 1) != 0;
+    const float a0 = hi2 ? y[0] : y[2], a1 = hi2 ? y[1] : y[3];
+    const float b0 = __shfl_xor_sync(0xffffffffu, a0, 2), b1 = __shfl_xor_sync(0xffffffffu, a1, 2);
+    const float k0 = (hi2 ? y[2] : y[0]) + b0, k1 = (hi2 ? y[3] : y[1]) + b1;
+    const float b = __shfl_xor_sync(0xffffffffu, hi1 ? k0 : k1, 1);
+    y[0] = (hi1 ? k1 : k0) + b;
+#pragma unroll
+    for (int o = 4; o < RS; o <<= 1) y[0] += __shfl_xor_sync(0xffffffffu, y[0], o);
+  } else if (RS == 2) {
+    const bool hi = (r & 1) != 0;
+    const float a0 = hi ? y[0] : y[2], a1 = hi ? y[1] : y[3];
+    const float b0 = __shfl_xor_sync(0xffffffffu, a0, 1), b1 = __shfl_xor_sync(0xffffffffu, a1, 1);
+    y[0] = (hi ? y[2] : y[0]) + b0;
+    y[1] = (hi ? y[3] : y[1]) + b1;
+  }
+}
+
+// rows of one thread's share of a head's state, and where they lie
+template <int RS>
+__device__ __forceinline__ int ssd_row(int i, int r) { return 4 * (i * RS + r); }
+
+template <int RS>
+__device__ __forceinline__ void ssd_load_state(float (&S)[16][4], const float* st, int N, int P, int e, int r, bool vec) {
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const int n = ssd_row<RS>(i, r) + q;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (n < N && e < P) {
+        const float* p = st + (size_t)n * P + e;
+        if (vec) {
+          v = *reinterpret_cast<const float4*>(p);
+        } else {
+          v.x = p[0];
+          if (e + 1 < P) v.y = p[1];
+          if (e + 2 < P) v.z = p[2];
+          if (e + 3 < P) v.w = p[3];
+        }
+      }
+      S[i * 4 + q][0] = v.x; S[i * 4 + q][1] = v.y; S[i * 4 + q][2] = v.z; S[i * 4 + q][3] = v.w;
+    }
+}
+
+template <int RS>
+__device__ __forceinline__ void ssd_store_state(const float (&S)[16][4], float* st, int N, int P, int e, int r, bool vec) {
+  if (e >= P) return;
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const int n = ssd_row<RS>(i, r) + q;
+      if (n >= N) continue;
+      float* p = st + (size_t)n * P + e;
+      const float* v = S[i * 4 + q];
+      if (vec) {
+        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+      } else {
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (e + k < P) p[k] = v[k];
+      }
+    }
+}
+
+// one token: S <- f S + B v^T (v = d x), and with OUT the thread's part of S^T C
+template <int RS, bool OUT>
+__device__ __forceinline__ void ssd_token(float (&S)[16][4], const float* B, const float* C, float f, float4 v, int r,
+                                          float (&y)[4]) {
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float4 b4 = *reinterpret_cast<const float4*>(B + ssd_row<RS>(i, r));
+    const float b[4] = {b4.x, b4.y, b4.z, b4.w};
+    float c[4] = {0.f, 0.f, 0.f, 0.f};
+    if (OUT) {
+      const float4 c4 = *reinterpret_cast<const float4*>(C + ssd_row<RS>(i, r));
+      c[0] = c4.x; c[1] = c4.y; c[2] = c4.z; c[3] = c4.w;
+    }
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      float* s = S[i * 4 + q];
+      s[0] = fmaf(f, s[0], b[q] * v.x);
+      s[1] = fmaf(f, s[1], b[q] * v.y);
+      s[2] = fmaf(f, s[2], b[q] * v.z);
+      s[3] = fmaf(f, s[3], b[q] * v.w);
+      if (OUT) {
+        y[0] = fmaf(s[0], c[q], y[0]);
+        y[1] = fmaf(s[1], c[q], y[1]);
+        y[2] = fmaf(s[2], c[q], y[2]);
+        y[3] = fmaf(s[3], c[q], y[3]);
+      }
+    }
+  }
+}
+
+// y of a token written by the lanes that hold the sums; `x` are the token's value columns from e on (D x joins here)
+template <int RS>
+__device__ __forceinline__ void ssd_write(const float (&y)[4], const float* x, float D, float* out, int e, int P, int r) {
+  constexpr int L = RS < 4 ? RS : 4, K = 4 / L;                    // lanes that write, columns of each
+  if (r >= L) return;
+#pragma unroll
+  for (int k = 0; k < K; ++k) {
+    const int c = r * K + k;
+    if (e + c < P) out[e + c] = fmaf(D, x[c], y[k]);
+  }
+}
+
+enum { SSD_LOCAL = 0, SSD_FULL = 1 };
+
+template <int RS> struct SsdTile {
+  static constexpr int NPAD = 16 * RS;                             // rows, padded
+  static constexpr int COLS = RS <= 8 ? 512 / RS : 64;             // columns of a block
+  static constexpr int CH = RS <= 8 ? 8 : 4;                       // tokens fetched together
+  static constexpr int ROW = 2 * NPAD + COLS + 4;                  // B | C | x | d, f
+};
+
+// tokens arrive in chunks through a ring of two shared-memory buffers, one chunk ahead of the products
+template <int RS, int MODE>
+__global__ void __launch_bounds__(RS <= 8 ? 128 : 16 * RS)
+ssd_segments_kernel(const float* xbc, int ld, const float* steps, const float* __restrict__ D,
+                    const int* __restrict__ tiles, int n_tiles, const int* __restrict__ seq_slot, float* state,
+                    long long state_ld, float* seg, float* seg_decay, float* out, int ldo, SsdShape s, int direct,
+                    int vec) {
+  using TL = SsdTile<RS>;
+  constexpr int CH = TL::CH, ROW = TL::ROW, NPAD = TL::NPAD;
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float ring[];                    // [2][CH][ROW]
+  const int tile = blockIdx.x, h = blockIdx.y;
+  const int seq = tiles[tile * 3 + 0], t0 = tiles[tile * 3 + 1], count = tiles[tile * 3 + 2];
+  const bool last = tile + 1 == n_tiles || tiles[(tile + 1) * 3] != seq;
+  if (MODE == SSD_LOCAL && last) return;                           // nobody starts from its end
+  const int N = s.N, P = s.P, g = h / (s.H / s.G);
+  const int r = threadIdx.x % RS, cl = (threadIdx.x / RS) * 4;     // this thread's row group and first column of the block
+  const int e0 = blockIdx.z * TL::COLS, e = e0 + cl;
+  const int nx = min(TL::COLS, P - e0);
+  float* st = state + (size_t)seq_slot[seq] * state_ld + (size_t)h * N * P;
+  float* sg = seg == nullptr ? nullptr : seg + ((size_t)tile * s.H + h) * N * P;
+  const float Dh = D[h];
+  for (int i = threadIdx.x; i < 2 * CH * ROW; i += blockDim.x) ring[i] = 0.f;      // (rows beyond N stay zero)
+  __syncthreads();
+  pdl_wait();
+  const int b_off = s.inner() + g * N, c_off = b_off + s.G * N, x_off = h * P + e0;
+  auto load_chunk = [&](int c, float* buf) {
+    const int tok0 = t0 + c * CH, nt = min(CH, count - c * CH);
+    const int unit = vec ? 4 : 1, nb = N / unit, per = 2 * nb + (nx + unit - 1) / unit;
+    for (int i = threadIdx.x; i < nt * per; i += blockDim.x) {
+      const int t = i / per, p = i - t * per;
+      const float* row = xbc + (size_t)(tok0 + t) * ld;
+      float* dst = buf + t * ROW;
+      const float* src;
+      if (p < nb) { src = row + b_off + p * unit; dst += p * unit; }
+      else if (p < 2 * nb) { src = row + c_off + (p - nb) * unit; dst += NPAD + (p - nb) * unit; }
+      else { src = row + x_off + (p - 2 * nb) * unit; dst += 2 * NPAD + (p - 2 * nb) * unit; }
+      if (vec) copy16_async(dst, src);
+      else copy4_async(dst, src);
+    }
+    for (int i = threadIdx.x; i < nt * 2; i += blockDim.x)
+      copy4_async(buf + (i >> 1) * ROW + 2 * NPAD + TL::COLS + (i & 1), steps + ((size_t)(tok0 + (i >> 1)) * s.H + h) * 2 + (i & 1));
+    copies_commit();
+  };
+  const int n_chunks = (count + CH - 1) / CH;
+  load_chunk(0, ring);
+  float S[16][4];
+  if (MODE == SSD_LOCAL) {
+#pragma unroll
+    for (int i = 0; i < 16; ++i)
+#pragma unroll
+      for (int k = 0; k < 4; ++k) S[i][k] = 0.f;
+  } else {
+    ssd_load_state<RS>(S, direct ? st : sg, N, P, e, r, vec);
+  }
+  float prod = 1.f;
+  for (int c = 0; c < n_chunks; ++c) {
+    float* buf = ring + (c & 1) * CH * ROW;
+    if (c + 1 < n_chunks) {
+      load_chunk(c + 1, ring + ((c + 1) & 1) * CH * ROW);          // (its last readers passed the barrier that ended chunk c - 1)
+      copies_wait<1>();
+    } else {
+      copies_wait<0>();
+    }
+    __syncthreads();
+    const int nt = min(CH, count - c * CH);
+    for (int t = 0; t < nt; ++t) {
+      const float* cur = buf + t * ROW;
+      const float d = cur[2 * NPAD + TL::COLS], f = cur[2 * NPAD + TL::COLS + 1];
+      float4 v = *reinterpret_cast<const float4*>(cur + 2 * NPAD + cl);
+      v.x *= d; v.y *= d; v.z *= d; v.w *= d;
+      float y[4] = {0.f, 0.f, 0.f, 0.f};
+      ssd_token<RS, MODE == SSD_FULL>(S, cur, cur + NPAD, f, v, r, y);
+      if (MODE == SSD_LOCAL) {
+        prod *= f;
+      } else {
+        ssd_meet<RS>(y, r);
+        ssd_write<RS>(y, cur + 2 * NPAD + cl, Dh, out + (size_t)(t0 + c * CH + t) * ldo + (size_t)h * P, e, P, r);
+      }
+    }
+    __syncthreads();                                               // the buffer is free for the chunk after next
+  }
+  if (MODE == SSD_LOCAL) {
+    ssd_store_state<RS>(S, sg, N, P, e, r, vec);
+    if (threadIdx.x == 0 && blockIdx.z == 0) seg_decay[(size_t)tile * s.H + h] = prod;
+  } else if (last) {
+    ssd_store_state<RS>(S, st, N, P, e, r, vec);
+  }
+}
+
+// seg[j] <- the state segment j starts from.  A block row per first segment of a sequence, a thread per W neighbouring
+// elements of the state; the ends of up to eight segments are fetched together.
+template <int W>
+__global__ void __launch_bounds__(256)
+ssd_carry_kernel(const int* __restrict__ tiles, int n_tiles, const int* __restrict__ seq_slot, const float* state,
+                 long long state_ld, float* seg, const float* seg_decay, SsdShape s) {
+  pdl_launch_dependents();
+  const int j0 = blockIdx.y;
+  const int seq = tiles[j0 * 3];
+  if (j0 > 0 && tiles[(j0 - 1) * 3] == seq) return;
+  const long long per_head = (long long)s.N * s.P, total = per_head * s.H;
+  const long long i = ((long long)blockIdx.x * 256 + threadIdx.x) * W;
+  if (i >= total) return;
+  const int h = (int)(i / per_head);                               // (W = 4 only where a head's numbers are a multiple of 4)
+  pdl_wait();
+  float S[W];
+  const float* st = state + (size_t)seq_slot[seq] * state_ld + i;
+#pragma unroll
+  for (int k = 0; k < W; ++k) S[k] = st[k];
+  for (int jb = j0; jb < n_tiles && tiles[jb * 3] == seq; jb += 8) {
+    float L[8][W], F[8];
+    int n = 0;
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      const int j = jb + u;
+      const bool in = j < n_tiles && tiles[j * 3] == seq;
+      n += in;
+      const bool more = in && j + 1 < n_tiles && tiles[(j + 1) * 3] == seq;   // (a sequence's last segment left no end)
+      F[u] = more ? seg_decay[(size_t)j * s.H + h] : 0.f;
+      if (W == 4) {
+        const float4 v = more ? *reinterpret_cast<const float4*>(seg + (size_t)j * total + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        L[u][0] = v.x; L[u][1 % W] = v.y; L[u][2 % W] = v.z; L[u][3 % W] = v.w;
+      } else {
+        L[u][0] = more ? seg[(size_t)j * total + i] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      if (u < n) {
+        float* dst = seg + (size_t)(jb + u) * total + i;
+        if (W == 4) *reinterpret_cast<float4*>(dst) = make_float4(S[0], S[1 % W], S[2 % W], S[3 % W]);
+        else dst[0] = S[0];
+#pragma unroll
+        for (int k = 0; k < W; ++k) S[k] = fmaf(F[u], S[k], L[u][k]);
+      }
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------- one token per sequence
+template <int RS>
+__global__ void __launch_bounds__(RS <= 8 ? 128 : 16 * RS)
+ssd_step_kernel(const float* proj, int ld, const float* __restrict__ w_taps, const float* __restrict__ w_bias,
+                const float* __restrict__ dt_bias, const float* __restrict__ a_log, const float* __restrict__ D,
+                const int* __restrict__ seq_slot, float* state, long long state_ld, float* out, int ldo, SsdShape s,
+                int vec) {
+  using TL = SsdTile<RS>;
+  constexpr int NPAD = TL::NPAD;
+  pdl_launch_dependents();
+  __shared__ __align__(16) float row[2 * NPAD + TL::COLS];         // B | C | x
+  const int t = blockIdx.x, h = blockIdx.y;
+  const int N = s.N, P = s.P, g = h / (s.H / s.G), C = s.channels();
+  const int r = threadIdx.x % RS, cl = (threadIdx.x / RS) * 4;
+  const int e0 = blockIdx.z * TL::COLS, e = e0 + cl;
+  const int nx = min(TL::COLS, P - e0);
+  float* srow = state + (size_t)seq_slot[t] * state_ld;
+  float* st = srow + (size_t)h * N * P;
+  const float* kept = srow + s.conv_off();
+  const float Dh = D[h], rate = expf(a_log[h]), db = dt_bias[h];
+  for (int i = threadIdx.x; i < 2 * NPAD + TL::COLS; i += blockDim.x) row[i] = 0.f;
+  __syncthreads();
+  pdl_wait();
+  float S[16][4];
+  ssd_load_state<RS>(S, st, N, P, e, r, vec);                      // in flight while the convolution is formed
+  const float* pr = proj + (size_t)t * ld + s.inner();
+  const int b_off = s.inner() + g * N, c_off = b_off + s.G * N, x_off = h * P + e0;
+  for (int i = threadIdx.x; i < 2 * N + nx; i += blockDim.x) {
+    int c, dst;
+    if (i < N) { c = b_off + i; dst = i; }
+    else if (i < 2 * N) { c = c_off + i - N; dst = NPAD + i - N; }
+    else { c = x_off + i - 2 * N; dst = 2 * NPAD + i - 2 * N; }
+    const float now = pr[c];
+    float a = w_bias[c];
+    for (int j = 0; j < s.taps - 1; ++j) a = fmaf(w_taps[(size_t)c * s.taps + j], kept[(size_t)j * C + c], a);
+    row[dst] = ssd_silu(fmaf(w_taps[(size_t)c * s.taps + s.taps - 1], now, a));
+  }
+  const float d = ssd_softplus(pr[C + h] + db), f = expf(-rate * d);
+  __syncthreads();
+  float4 v = *reinterpret_cast<const float4*>(row + 2 * NPAD + cl);
+  v.x *= d; v.y *= d; v.z *= d; v.w *= d;
+  float y[4] = {0.f, 0.f, 0.f, 0.f};
+  ssd_token<RS, true>(S, row, row + NPAD, f, v, r, y);
+  ssd_store_state<RS>(S, st, N, P, e, r, vec);
+  ssd_meet<RS>(y, r);
+  ssd_write<RS>(y, row + 2 * NPAD + cl, Dh, out + (size_t)t * ldo + (size_t)h * P, e, P, r);
+}
+
+// ------------------------------------------------------------------------------- gate and norm
+// A block per (token, part).  `stash`: the part's gated numbers stay in shared memory between the passes.
+template <typename TO>
+__global__ void __launch_bounds__(512)
+ssd_gate_norm_kernel(const float* y, int ldy, const float* proj, int ld, const float* __restrict__ w, TO* out, int groups,
+                     float eps, const int* __restrict__ token_seq, int T, const int* __restrict__ seq_slot, float* state,
+                     long long state_ld, SsdShape s, int stash) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float u_s[];
+  __shared__ float red[32];
+  const int t = blockIdx.x, part = blockIdx.y, n = s.inner() / groups;
+  const int seq = token_seq[t];
+  const bool ends = t + 1 == T || token_seq[t + 1] != seq;
+  pdl_wait();
+  const float* yr = y + (size_t)t * ldy + (size_t)part * n;
+  const float* zr = proj + (size_t)t * ld + (size_t)part * n;
+  float ss = 0.f;
+  const bool four = n % 4 == 0 && ldy % 4 == 0 && ld % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)proj & 15) == 0;
+  if (stash && four) {
+    for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
+      const float4 a = *reinterpret_cast<const float4*>(yr + i), z = *reinterpret_cast<const float4*>(zr + i);
+      const float4 u = make_float4(a.x * ssd_silu(z.x), a.y * ssd_silu(z.y), a.z * ssd_silu(z.z), a.w * ssd_silu(z.w));
+      ss += (u.x * u.x + u.y * u.y) + (u.z * u.z + u.w * u.w);
+      *reinterpret_cast<float4*>(u_s + i) = u;
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+      const float u = yr[i] * ssd_silu(zr[i]);
+      ss = fmaf(u, u, ss);
+      if (stash) u_s[i] = u;
+    }
+  }
+  const float sc = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
+  TO* dst = out + (size_t)t * s.inner() + (size_t)part * n;
+  const float* wp = w + (size_t)part * n;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const float u = stash ? u_s[i] : yr[i] * ssd_silu(zr[i]);      // (block_sum's barriers lie between u_s's writes and reads)
+    dst[i] = from_float<TO>(u * sc * wp[i]);
+  }
+  // the convolution's inputs that the sequence's next tokens reach back to
+  const int keep = s.taps - 1;
+  if (!ends || keep == 0) return;
+  const int C = s.channels();
+  int here = 1;                                    // tokens of this step that the new row can take
+  while (here < keep && t - here >= 0 && token_seq[t - here] == seq) ++here;
+  const int old = keep - min(here, keep);          // entries that stay from the old row
+  const bool all = here >= keep;
+  float* kept = state + (size_t)seq_slot[seq] * state_ld + s.conv_off();
+  const float* xbc = proj + s.inner();
+  for (int c = part * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
+    for (int j = 0; j < keep; ++j) {
+      // entry j is the input `keep - 1 - j` tokens back; ascending j: an old entry is read before it is overwritten
+      const int back = keep - 1 - j;
+      kept[(size_t)j * C + c] = (all || j >= old) ? xbc[(size_t)(t - back) * ld + c] : kept[(size_t)(j + here) * C + c];
+    }
+  }
+}
+
+static bool ssd_shape_ok(const SsdShape& s) {
+  return s.H > 0 && s.G > 0 && s.H % s.G == 0 && s.N > 0 && s.N <= 512 && s.P > 0 && s.taps > 0 && s.H <= 65535;
+}
+static int ssd_row_split(int N) {
+  int rs = 1;
+  while (rs * 16 < N) rs *= 2;
+  return rs;
+}
+template <int RS> static dim3 ssd_block(int P) {
+  const int cols = P < SsdTile<RS>::COLS ? P : SsdTile<RS>::COLS;
+  const int threads = RS * ((cols + 3) / 4);
+  return dim3((threads + 31) / 32 * 32);
+}
+template <int RS> static int ssd_col_blocks(int P) { return (P + SsdTile<RS>::COLS - 1) / SsdTile<RS>::COLS; }
+
+template <int RS>
+static int launch_ssd_segments(const float* xbc, int ld, const float* steps, const float* D, const int* tiles, int n_tiles,
+                               int direct, const int* seq_slot, float* state, long long state_ld, float* scratch,
+                               float* out, int ldo, SsdShape s, int vec, cudaStream_t stream) {
+  using TL = SsdTile<RS>;
+  const dim3 grid(n_tiles, s.H, ssd_col_blocks<RS>(s.P)), block = ssd_block<RS>(s.P);
+  const size_t smem = sizeof(float) * 2 * TL::CH * TL::ROW;
+  float* seg = direct ? nullptr : scratch;
+  float* dec = direct ? nullptr : scratch + (size_t)n_tiles * s.H * s.N * s.P;
+  if (!direct) {
+    launch_kernel(ssd_segments_kernel<RS, SSD_LOCAL>, grid, block, smem, stream, xbc, ld, steps, D, tiles, n_tiles,
+                  seq_slot, state, state_ld, seg, dec, out, ldo, s, direct, vec);
+    int st = launch_status();
+    if (st != DLGO_OK) return st;
+    const long long total = (long long)s.H * s.N * s.P;
+    const bool four = vec && ((long long)s.N * s.P) % 4 == 0;
+    const long long items = four ? total / 4 : total;
+    const dim3 cgrid((unsigned)((items + 255) / 256), n_tiles);
+    if (four) launch_kernel(ssd_carry_kernel<4>, cgrid, dim3(256), 0, stream, tiles, n_tiles, seq_slot, state, state_ld, seg, dec, s);
+    else launch_kernel(ssd_carry_kernel<1>, cgrid, dim3(256), 0, stream, tiles, n_tiles, seq_slot, state, state_ld, seg, dec, s);
+    st = launch_status();
+    if (st != DLGO_OK) return st;
+  }
+  launch_kernel(ssd_segments_kernel<RS, SSD_FULL>, grid, block, smem, stream, xbc, ld, steps, D, tiles, n_tiles, seq_slot,
+                state, state_ld, seg, dec, out, ldo, s, direct, vec);
+  return launch_status();
+}
+
+}  // namespace dlgo
+
+using namespace dlgo;
+
+// proj [T, ld] fp32 with the columns [z | x | B | C | dt]; w_taps [C, taps], w_bias [C], dt_bias, a_log [H] fp32;
+// tiles [n_tiles, 3] (sequence, first packed token, count); out [T, ldo >= C] fp32: x | B | C;
+// steps [T, H, 2] fp32: d and f
+DLGO_EXPORT int dlgo_ssd_conv(const float* proj, int ld, const float* w_taps, const float* w_bias, const float* dt_bias,
+                              const float* a_log, const int* tiles, int n_tiles, const int* token_seq,
+                              const int* seq_slot, const float* state, long long state_ld, float* out, int ldo,
+                              float* steps, int H, int G, int N, int P, int taps, cudaStream_t stream) {
+  if (n_tiles <= 0) return DLGO_OK;
+  const SsdShape s{H, G, N, P, taps};
+  if (!ssd_shape_ok(s)) return DLGO_ERR_SIZE;
+  const int C = s.channels();
+  const bool four = taps <= 4 && C % 4 == 0 && s.inner() % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 &&
+                    ((uintptr_t)proj & 15) == 0 && ((uintptr_t)out & 15) == 0;
+  const int w = four ? 4 : 1;
+  const dim3 grid(n_tiles, (C + SC_THREADS * w - 1) / (SC_THREADS * w) + 1), block(SC_THREADS);
+#define CONV_ARGS grid, block, 0, stream, proj, ld, w_taps, w_bias, dt_bias, a_log, tiles, token_seq, seq_slot, state, \
+                  state_ld, out, ldo, steps, s
+  if (four && taps == 4) launch_kernel(ssd_conv_kernel<4, 4>, CONV_ARGS);
+  else if (four && taps == 3) launch_kernel(ssd_conv_kernel<3, 4>, CONV_ARGS);
+  else if (four && taps == 2) launch_kernel(ssd_conv_kernel<2, 4>, CONV_ARGS);
+  else if (four && taps == 1) launch_kernel(ssd_conv_kernel<1, 4>, CONV_ARGS);
+  else launch_kernel(ssd_conv_kernel<0, 1>, CONV_ARGS);
+#undef CONV_ARGS
+  return launch_status();
+}
+
+// xbc [T, ld] fp32 (x | B | C) and steps of dlgo_ssd_conv; D [H] fp32; tiles [n_tiles, 3], a sequence's segments side by
+// side in token order; out [T, ldo >= H P] fp32.  `direct`: one segment per sequence; else scratch holds
+// n_tiles * H * (N P + 1) floats.
+DLGO_EXPORT int dlgo_ssd_segments(const float* xbc, int ld, const float* steps, const float* D, const int* tiles,
+                                  int n_tiles, int direct, const int* seq_slot, float* state, long long state_ld,
+                                  float* scratch, float* out, int ldo, int H, int G, int N, int P, int taps,
+                                  cudaStream_t stream) {
+  if (n_tiles <= 0) return DLGO_OK;
+  const SsdShape s{H, G, N, P, taps};
+  if (!ssd_shape_ok(s) || n_tiles > 65535 || (!direct && scratch == nullptr)) return DLGO_ERR_SIZE;
+  const int vec = ((N | P | ld) & 3) == 0 && (state_ld & 3) == 0 && ((uintptr_t)xbc & 15) == 0 &&
+                  ((uintptr_t)state & 15) == 0 && ((uintptr_t)scratch & 15) == 0;
+#define SSD_ARGS xbc, ld, steps, D, tiles, n_tiles, direct, seq_slot, state, state_ld, scratch, out, ldo, s, vec, stream
+  switch (ssd_row_split(N)) {
+    case 1: return launch_ssd_segments<1>(SSD_ARGS);
+    case 2: return launch_ssd_segments<2>(SSD_ARGS);
+    case 4: return launch_ssd_segments<4>(SSD_ARGS);
+    case 8: return launch_ssd_segments<8>(SSD_ARGS);
+    case 16: return launch_ssd_segments<16>(SSD_ARGS);
+    default: return launch_ssd_segments<32>(SSD_ARGS);
+  }
+#undef SSD_ARGS
+}
+
+// One token per sequence (token t belongs to sequence t of the step).
+DLGO_EXPORT int dlgo_ssd_step(const float* proj, int ld, const float* w_taps, const float* w_bias, const float* dt_bias,
+                              const float* a_log, const float* D, const int* seq_slot, float* state, long long state_ld,
+                              float* out, int ldo, int T, int H, int G, int N, int P, int taps, cudaStream_t stream) {
+  if (T <= 0) return DLGO_OK;
+  const SsdShape s{H, G, N, P, taps};
+  if (!ssd_shape_ok(s)) return DLGO_ERR_SIZE;
+  const int vec = ((N | P) & 3) == 0 && (state_ld & 3) == 0 && ((uintptr_t)state & 15) == 0;
+#define STEP_LAUNCH(RS) \
+  launch_kernel(ssd_step_kernel<RS>, dim3(T, H, ssd_col_blocks<RS>(P)), ssd_block<RS>(P), 0, stream, proj, ld, w_taps, w_bias, \
+                dt_bias, a_log, D, seq_slot, state, state_ld, out, ldo, s, vec)
+  switch (ssd_row_split(N)) {
+    case 1: STEP_LAUNCH(1); break;
+    case 2: STEP_LAUNCH(2); break;
+    case 4: STEP_LAUNCH(4); break;
+    case 8: STEP_LAUNCH(8); break;
+    case 16: STEP_LAUNCH(16); break;
+    default: STEP_LAUNCH(32); break;
+  }
+#undef STEP_LAUNCH
+  return launch_status();
+}
+
+// y [T, ldy] fp32, proj as above (its z columns gate), w [H P] fp32, out [T, H P] in `dtype`; `groups` divides H P
+DLGO_EXPORT int dlgo_ssd_gate_norm(const float* y, int ldy, const float* proj, int ld, const float* w, void* out, int dtype,
+                                   int groups, float eps, const int* token_seq, int T, const int* seq_slot, float* state,
+                                   long long state_ld, int H, int G, int N, int P, int taps, cudaStream_t stream) {
+  if (T <= 0) return DLGO_OK;
+  const SsdShape s{H, G, N, P, taps};
+  if (!ssd_shape_ok(s) || groups <= 0 || s.inner() % groups || groups > 65535) return DLGO_ERR_SIZE;
+  const int n = s.inner() / groups;
+  const int stash = n * sizeof(float) <= 40 * 1024;
+  const size_t smem = stash ? n * sizeof(float) : 0;
+  const int threads = n >= 2048 ? 512 : (n >= 512 ? 256 : (n >= 128 ? 128 : 64));
+  if (dtype == DLGO_F32)
+    launch_kernel(ssd_gate_norm_kernel<float>, dim3(T, groups), dim3(threads), smem, stream, y, ldy, proj, ld, w, (float*)out,
+                  groups, eps, token_seq, T, seq_slot, state, state_ld, s, stash);
+  else if (dtype == DLGO_BF16)
+    launch_kernel(ssd_gate_norm_kernel<__nv_bfloat16>, dim3(T, groups), dim3(threads), smem, stream, y, ldy, proj, ld, w,
+                  (__nv_bfloat16*)out, groups, eps, token_seq, T, seq_slot, state, state_ld, s, stash);
+  else
+    return DLGO_ERR_DTYPE;
+  return launch_status();
+}

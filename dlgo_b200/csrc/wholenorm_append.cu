@@ -81,14 +81,41 @@ wholenorm_append_kernel(float* proj, int ld, const float* __restrict__ w_q, cons
   }
 }
 
-// a[t, h, :] *= gate[t, h]   (a in the run's type, heads of hd numbers; the product is formed in fp32)
-template <typename T>
+// a[t, h, :] *= gate[t, h], or sigmoid(gate[t, h])   (a in the run's type, heads of hd numbers; the product is formed in
+// fp32).  W neighbouring numbers of a head per thread and trip.
+template <typename T, int W>
 __global__ void __launch_bounds__(256)
-scale_heads_kernel(T* a, const float* gate, long long total, int hd) {
+scale_heads_kernel(T* a, const float* gate, int ldg, long long total, int H, int hd, int sigmoid) {
   pdl_launch_dependents();
   pdl_wait();
-  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x)
-    a[i] = from_float<T>(to_float(a[i]) * gate[i / hd]);
+  for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * W; i < total;
+       i += (long long)gridDim.x * blockDim.x * W) {
+    const long long th = i / hd;
+    const int t = (int)(th / H), h = (int)(th - (long long)t * H);
+    const float z = gate[(size_t)t * ldg + h];
+    const float f = sigmoid ? 1.0f / (1.0f + expf(-z)) : z;
+    if (W * sizeof(T) == 16) {
+      __align__(16) T v[W];
+      *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(a + i);
+#pragma unroll
+      for (int k = 0; k < W; ++k) v[k] = from_float<T>(to_float(v[k]) * f);
+      *reinterpret_cast<uint4*>(a + i) = *reinterpret_cast<const uint4*>(v);
+    } else {
+      a[i] = from_float<T>(to_float(a[i]) * f);
+    }
+  }
+}
+
+template <typename T>
+int launch_scale_heads(T* a, const float* gate, int ldg, int n_tokens, int H, int hd, int sigmoid, cudaStream_t stream) {
+  constexpr int V = 16 / (int)sizeof(T);
+  const long long total = (long long)n_tokens * H * hd;
+  const bool vec = hd % V == 0 && ((uintptr_t)a & 15) == 0;
+  const long long want = (total / (vec ? V : 1) + 255) / 256;
+  const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
+  if (vec) launch_kernel(scale_heads_kernel<T, V>, dim3(blocks), dim3(256), 0, stream, a, gate, ldg, total, H, hd, sigmoid);
+  else launch_kernel(scale_heads_kernel<T, 1>, dim3(blocks), dim3(256), 0, stream, a, gate, ldg, total, H, hd, sigmoid);
+  return launch_status();
 }
 
 template <typename T>
@@ -127,21 +154,15 @@ DLGO_EXPORT int dlgo_wholenorm_append(float* proj, int ld, const float* w_q, con
   return DLGO_ERR_DTYPE;
 }
 
-// a [T, H * hd] in `dtype` (contiguous), gate [T, H] fp32
-DLGO_EXPORT int dlgo_scale_heads(void* a, const float* gate, int dtype, int T, int H, int hd, cudaStream_t stream) {
+// a [T, H * hd] in `dtype` (contiguous), gate [T, ldg >= H] fp32
+DLGO_EXPORT int dlgo_scale_heads(void* a, const float* gate, int ldg, int dtype, int T, int H, int hd, int sigmoid,
+                                 cudaStream_t stream) {
   if (T <= 0) return DLGO_OK;
-  if (H <= 0 || hd <= 0) return DLGO_ERR_SIZE;
-  const long long total = (long long)T * H * hd;
-  const long long want = (total + 255) / 256;
-  const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
-  if (dtype == DLGO_F32)
-    dlgo::launch_kernel(dlgo::scale_heads_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)a, gate, total, hd);
-  else if (dtype == DLGO_BF16)
-    dlgo::launch_kernel(dlgo::scale_heads_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (__nv_bfloat16*)a,
-                        gate, total, hd);
-  else
-    return DLGO_ERR_DTYPE;
-  return dlgo::launch_status();
+  if (H <= 0 || hd <= 0 || ldg < H) return DLGO_ERR_SIZE;
+  if (dtype == DLGO_F32) return dlgo::launch_scale_heads<float>((float*)a, gate, ldg, T, H, hd, sigmoid, stream);
+  if (dtype == DLGO_BF16)
+    return dlgo::launch_scale_heads<__nv_bfloat16>((__nv_bfloat16*)a, gate, ldg, T, H, hd, sigmoid, stream);
+  return DLGO_ERR_DTYPE;
 }
 
 // The error word (1: a position had no page), cleared by the read.

@@ -47,6 +47,27 @@ class PreNormBlock(Block):
         self.ffn.forward(x, residual, ctx)
 
 
+class ParallelPreNormBlock(Block):
+    """Mixer and feed-forward side by side: ``x <- x + (mixer(n) + ffn(n))`` with ONE ``n = norm(x)`` that both read
+    (a layer without a feed-forward: ``x + mixer(n)``).  Both add straight into the fp32 residual stream, which neither
+    reads."""
+
+    handles_pending = True   # reads the residual only through norm_of
+
+    def __init__(self, mixer: Any, ffn: Any, norms: Mapping[str, Any], connections: Any = None):
+        super().__init__(mixer, ffn, norms, connections)
+        if mixer is None or "mixer_norm" not in self.norms:
+            raise ValueError("a parallel pre-norm block needs a mixer and the norm 'mixer_norm'")
+        self.mixer_norm = self.norms["mixer_norm"]
+
+    def forward(self, residual: torch.Tensor, ctx: Any, cache: Any, state: Optional[torch.Tensor],
+                positions: Mapping[str, PositionEncoding]) -> None:
+        n = norm_of(self.mixer_norm, residual, ctx)
+        self.mixer.forward(n, residual, ctx, cache, state, positions)
+        if self.ffn is not None:
+            self.ffn.forward(n, residual, ctx)
+
+
 class HyperConnection(Part):
     """How one sublayer sits on ``streams`` residual streams x_1 .. x_s: it reads ``u = sum_r read[r] x_r`` and
     its result y returns as ``x_q <- sum_r mix[r, q] x_r + write[q] * y`` for every q at once (``mix`` is
@@ -388,6 +409,7 @@ class GatedPreNormBlock(Block):
 
 
 BLOCKS.register("prenorm", PreNormBlock)
+BLOCKS.register("parallel_prenorm", ParallelPreNormBlock)
 BLOCKS.register("gated_prenorm", GatedPreNormBlock)
 BLOCKS.register("result_norm", ResultNormBlock)
 BLOCKS.register("hyper_prenorm", HyperPreNormBlock)

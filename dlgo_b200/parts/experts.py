@@ -6,11 +6,13 @@
     c = s + correction               choice scores (``correction``: a stored per-output bias used for choosing only)
     outputs form ``group_count`` equal groups of neighbours; a group's score is its largest c; only outputs of
     the ``group_keep`` best groups can be chosen (the others count as minus infinity); the ``top`` largest c win
-    y = sum over the chosen e of s_e * expert_e(h)            (``renormalize``: s_e / sum of the chosen s)
+    y = sum over the chosen e of s_e * expert_e(h)            (``renormalize``: s_e / sum of the chosen s;
+                                                              ``weight_scale``: s_e times a constant)
     expert_e(h) = Wdown_e act(Wup_e h)                        for e < num_experts
                   (``gated``: Wdown_e (silu(Wgate_e h) * (Wup_e h)), a third matrix per expert)
     expert_e(h) = h                                           for the ``identity_experts`` outputs after them
-    y += gate * shared(h),  gate = sigmoid(w_g . h) per token (``shared_size``, ``shared_gate``)
+    y += gate * shared(h),  gate = sigmoid(w_g . h) per token (``shared_size``, ``shared_gate``; without the gate 1);
+                                                              the shared expert has the experts' form (``gated`` or not)
     ``weight_on`` = "input": y = sum over the chosen e of expert_e(s_e * h) instead (the weight multiplies what the
     expert reads, which differs from the above as soon as an expert is not linear)
 
@@ -30,7 +32,8 @@ import torch
 
 from ..csrc import kernels as K
 from .base import FeedForward, ParamSpec
-from .linear import STORE_F32, Linear
+from .feedforward import SwiGLU
+from .linear import ADD_F32, STORE_F32, Linear
 from .registry import FEED_FORWARDS
 
 _ACTS = {"none": K.ACT_NONE, "relu2": K.ACT_RELU2, "silu": K.ACT_SILU, "gelu_tanh": K.ACT_GELU_TANH}
@@ -53,17 +56,18 @@ class RoutedExperts(FeedForward):
                  renormalize: bool = False, correction: bool = False, activation: str = "relu2",
                  shared_size: Optional[int] = None, shared_gate: bool = False,
                  names: Optional[Mapping[str, str]] = None, logit_bias: bool = False, gated: bool = False,
-                 weight_on: str = "output"):
+                 weight_on: str = "output", weight_scale: float = 1.0):
         super().__init__(hidden_size=hidden_size, intermediate_size=intermediate_size, num_experts=num_experts, top=top,
                          identity_experts=identity_experts, group_count=group_count, group_keep=group_keep,
                          score=score, renormalize=renormalize, correction=correction, activation=activation,
                          shared_size=shared_size, shared_gate=shared_gate, names=names, logit_bias=logit_bias,
-                         gated=gated, weight_on=weight_on)
+                         gated=gated, weight_on=weight_on, weight_scale=weight_scale)
         if weight_on not in ("output", "input"):
             raise ValueError(f"weight_on must be 'output' or 'input', got {weight_on!r}")
         if weight_on == "input" and identity_experts:
             raise ValueError("identity experts take their weight on the output")
         self.weight_on_input = weight_on == "input"
+        self.weight_scale = float(weight_scale)
         self.logit_bias = bool(logit_bias)
         self.gated = bool(gated)
         if self.gated and activation != "silu":
@@ -91,7 +95,7 @@ class RoutedExperts(FeedForward):
         self.shared_gate = bool(shared_gate) and self.shared_size is not None
         self.names = {"router": "router.weight", "correction": "router.bias", "logit_bias": "router.logit_bias",
                       "gate": "gate_proj.weight", "expert": "experts.{}.",
-                      "up": "up_proj.weight", "down": "down_proj.weight", "shared_up": "shared.up_proj.weight",
+                      "up": "up_proj.weight", "down": "down_proj.weight", "shared_gate_proj": "shared.gate_proj.weight", "shared_up": "shared.up_proj.weight",
                       "shared_down": "shared.down_proj.weight", "shared_gate": "shared.gate.weight"}
         self.names.update(names or {})
         self.w_router: Optional[torch.Tensor] = None        # fp32 [outputs (+ gate row), hidden]
@@ -101,6 +105,11 @@ class RoutedExperts(FeedForward):
         self.w_down: Optional[torch.Tensor] = None          # [experts, hidden, ff]
         self.shared_up: Optional[Linear] = None
         self.shared_down: Optional[Linear] = None
+        # a gated shared expert is a gated feed-forward of its own that every token passes
+        self.shared: Optional[SwiGLU] = None
+        if self.gated and self.shared_size is not None:
+            self.shared = SwiGLU(self.hidden_size, self.shared_size, names={
+                "gate": self.names["shared_gate_proj"], "up": self.names["shared_up"], "down": self.names["shared_down"]})
         self.on_tensor_cores = False
 
     def param_specs(self) -> Dict[str, ParamSpec]:
@@ -117,6 +126,8 @@ class RoutedExperts(FeedForward):
             specs[p + n["up"]] = ParamSpec((f, d))
             specs[p + n["down"]] = ParamSpec((d, f))
         if self.shared_size is not None:
+            if self.gated:
+                specs[n["shared_gate_proj"]] = ParamSpec((self.shared_size, d))
             specs[n["shared_up"]] = ParamSpec((self.shared_size, d))
             specs[n["shared_down"]] = ParamSpec((d, self.shared_size))
             if self.shared_gate:
@@ -153,7 +164,9 @@ class RoutedExperts(FeedForward):
             self.on_tensor_cores = (_TENSOR_CORES and
                                     K.moe_gemm_tc_takes(self.w_up.dtype, self.w_up.shape[1], self.hidden_size) and
                                     K.moe_gemm_tc_takes(self.w_down.dtype, self.hidden_size, self.intermediate_size))
-        if self.shared_size is not None:
+        if self.shared is not None:
+            self.shared.load(get, runtime)
+        elif self.shared_size is not None:
             self.shared_up = Linear(get(n["shared_up"]), runtime)
             self.shared_down = Linear(get(n["shared_down"]), runtime)
 
@@ -168,7 +181,8 @@ class RoutedExperts(FeedForward):
                      (K.MOE_FEW_ROWS if few else K.MOE_TILE_ROWS))
         idx, wt, gate, plan = K.moe_router(x, self.w_router, self.b_choice, self.n_outputs, self.shared_gate, self.top,
                                            self.group_count, self.group_keep, self.sigmoid_scores, self.renormalize,
-                                           plan=(self.num_experts, tile_rows), logit_bias=self.b_logit)
+                                           plan=(self.num_experts, tile_rows), logit_bias=self.b_logit,
+                                           weight_scale=self.weight_scale)
         pair_out = None
         src, div, scale = x, self.top, None
         if self.weight_on_input:
@@ -201,7 +215,13 @@ class RoutedExperts(FeedForward):
                     hidden = K.swiglu(hidden, block=self.gate_block)
                 K.moe_gemm(plan, hidden, self.w_down, pair_out, None, True, K.ACT_NONE)    # rows scattered by pair
         shared = None
-        if self.shared_size is not None:
+        if self.shared is not None:
+            h = self.shared.hidden(x)
+            if self.shared_gate:
+                shared = self.shared.w_down(h, STORE_F32)
+            else:
+                self.shared.w_down(h, ADD_F32, residual)        # no factor: it adds itself
+        elif self.shared_size is not None:
             shared = self.shared_down(self.shared_up.bias_act(x, None, self.act), STORE_F32)
         K.moe_combine(residual, pair_out, x, idx, wt, self.num_experts, shared, gate)
 

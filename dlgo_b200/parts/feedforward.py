@@ -53,11 +53,12 @@ class SwiGLU(FeedForward):
             self.w_gate_up = Linear(torch.cat([gate, up], dim=0), runtime)
         self.w_down = Linear(get(self.names["down"]), runtime)
 
+    def hidden(self, x: Any) -> torch.Tensor:
+        """``silu(Wg . x) * (Wu . x)``: what the down projection reads."""
+        return self.w_gate_up(x) if self.fused else K.swiglu(self.w_gate_up(x, STORE))
+
     def forward(self, x: Any, residual: torch.Tensor, ctx: Any) -> None:
-        if self.fused:
-            h = self.w_gate_up(x)
-        else:
-            h = K.swiglu(self.w_gate_up(x, STORE))
+        h = self.hidden(x)
         parts = self.w_down.partials(h, for_residual=True) if ctx is not None and hasattr(ctx, "defer") else None
         if parts is not None:
             ctx.defer(residual, parts)      # the next norm adds the slices to the residual

@@ -155,19 +155,23 @@ def test_latents_with_a_rotated_key_part(H, dk, r, R, act_dtype):
     table = i32([[3, 1], [0, 2]])
     seq = [0, 0, 0, 0, 1, 1, 1, 1, 1]
     dev = proj.to(DEV)
-    K.latent_rope_append(dev, n_q, R, w.to(DEV), 0, H, dk + r, r, torch.tensor(freq, dtype=torch.float32, device=DEV), amp,
-                         eps, i32(pos), i32(seq), i32([0, 1]), table, pages.view(4, PS, R + r))
+    rope = K.LatentRope(torch.tensor(freq, dtype=torch.float32, device=DEV), amp, r, halves=False)
+    assert K.latent_norm_append(dev, n_q, R, w.to(DEV), 0, 0, None, eps, i32(pos), i32(seq), i32([0, 1]), table,
+                                pages.view(4, PS, R + r), rope=rope) is None
     tol = dict(rtol=2e-2, atol=2e-2) if act_dtype == torch.bfloat16 else dict(rtol=1e-5, atol=1e-5)
-    got_q = dev[:, :n_q].cpu().view(T, H, dk + r)
+    assert torch.equal(dev.cpu(), proj)                                                    # nothing is rewritten
+    wide = dk + r + 6
+    got_q = K.latent_queries(dev[:, :n_q], H, dk + r, wide, rope, i32(pos), act_dtype).cpu().view(T, H, wide)
+    assert not got_q[..., dk + r:].any()
+    got_q = got_q[..., :dk + r]
     for t in range(T):
         q = proj[t, :n_q].view(1, H, dk + r).double()
         want = torch.cat([q[..., :dk], P.rotate_pairs(q[..., dk:].contiguous(), rotd, first=pos[t])], -1)
-        assert torch.allclose(got_q[t].double(), want[0], rtol=1e-5, atol=1e-5)          # queries stay fp32, in place
+        assert torch.allclose(got_q[t].double(), want[0], **tol)
         c = P.rms_norm(proj[t, n_q:n_q + R].double(), w.double(), eps)
         kr = P.rotate_pairs(proj[t, n_q + R:n_q + R + r].view(1, 1, r).double(), rotd, first=pos[t])[0, 0]
         row = pages[int(table[seq[t]][pos[t] // PS]), 0, pos[t] % PS].float().cpu().double()
         assert torch.allclose(row, torch.cat([c, kr]), **tol), t
-    assert torch.equal(dev[:, n_q:].cpu(), proj[:, n_q:])                                   # nothing else is rewritten
 
 
 @pytest.mark.parametrize("act_dtype", [torch.float32, torch.bfloat16])
