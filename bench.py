@@ -460,8 +460,44 @@ def ragilorn_pair(size):
     return rag, llama
 
 
-def dedutar_compare(size, batch, steps, warmup, prefill_tokens, profile, design="dedutar"):
-    """Prefill and decode throughput of both models, and (with `profile`) the time per kernel entry point of
+# --only zetavik: the Zetavik design beside its closest relatives and Llama at equal layer sizes (random weights)
+ZETAVIK_SIZES = {
+    # width; heads, value columns, state rows, groups and norm groups of the state-space layers; heads, unrotated and
+    # rotated query sizes, value size and the two latents of the latent-attention layer; heads and head size of the linear
+    # attention; dense feed-forward; experts, groups, kept, chosen, expert and shared widths
+    "small": dict(width=1024, sheads=32, sv=64, state=128, sgroups=4, lheads=16, ldim=32, lrot=32, lv=64, qrank=384, rank=256,
+                  heads=16, dim=64, ff=4224, experts=16, groups=4, keep=2, top=2, eff=896, shared=1024, vocab=32000),
+    "1b": dict(width=2048, sheads=64, sv=64, state=128, sgroups=8, lheads=16, ldim=64, lrot=64, lv=128, qrank=768, rank=512,
+               heads=16, dim=128, ff=8448, experts=32, groups=8, keep=4, top=4, eff=1024, shared=1536, vocab=32000),
+    "3b": dict(width=3072, sheads=96, sv=64, state=128, sgroups=8, lheads=24, ldim=64, lrot=64, lv=128, qrank=1536, rank=512,
+               heads=24, dim=128, ff=12288, experts=32, groups=8, keep=4, top=4, eff=1536, shared=2048, vocab=32000),
+}
+
+
+def zetavik_set(size):
+    """[(name, config.json)]: Zetavik with four layers (linear attention and a dense feed-forward; state-space mixing
+    and experts; latent attention and experts; state-space mixing and a dense feed-forward; a token's chosen and shared
+    experts spend the dense one's FLOPs), and the models closest to it at the same width and feed-forward FLOPs: Bazurax
+    (recurrences, gated experts), Ragilorn (latent attention with a rotated part, gated experts) and Llama."""
+    z = ZETAVIK_SIZES[size]
+    H = z["heads"]
+    lin = {"heads": H, "dim": z["dim"], "vdim": z["dim"], "decay": [1.0 - 2.0 ** -(3 + 5 * i / H) for i in range(H)]}
+    ssm = {"heads": z["sheads"], "vdim": z["sv"], "state": z["state"], "groups": z["sgroups"], "conv": 4,
+           "norm_groups": z["sgroups"]}
+    lat = {"heads": z["lheads"], "dim": z["ldim"], "rot_dim": z["lrot"], "vdim": z["lv"], "q_rank": z["qrank"],
+           "kv_rank": z["rank"], "scale": (z["ldim"] + z["lrot"]) ** -0.5, "rot": {"base": 1e6, "dims": z["lrot"]}}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["eff"]}, "shared": {"ff": z["shared"]},
+           "router": {"experts": z["experts"], "top": z["top"], "scale": 2.5, "groups": {"count": z["groups"], "keep": z["keep"]}}}
+    zet = {"architecture": "Zetavik", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+           "layers": [{"type": "lightning", "mixer": lin, "mlp": dense}, {"type": "mamba2", "mixer": ssm, "mlp": moe},
+                      {"type": "latent_attention", "mixer": lat, "mlp": moe}, {"type": "mamba2", "mixer": ssm, "mlp": dense}]}
+    baz, llama = bazurax_pair(size)
+    return [("zetavik", zet), ("bazurax", baz), ("ragilorn", ragilorn_pair(size)[0]), ("llama", llama)]
+
+
+def dedutar_compare(size, batch, steps, warmup, prefill_tokens, profile, design="dedutar", only_models=()):
+    """Prefill and decode throughput of the models (``only_models``: of these), and (with `profile`) the time per kernel entry point of
     one prompt step and of decode steps launched one by one."""
     import torch
     import dlgo_b200
@@ -470,8 +506,14 @@ def dedutar_compare(size, batch, steps, warmup, prefill_tokens, profile, design=
     from dlgo_b200.weights import write_random_model
     out = {"only": design, "size": size, "batch": batch, "prefill_tokens": prefill_tokens, "dtype": "bf16",
            "data": "synthetic", "models": {}}
-    pair = {"monolix": monolix_pair, "dedutar": dedutar_pair, "bazurax": bazurax_pair, "ragilorn": ragilorn_pair}[design](size)
-    for name, cfg in zip((design, "llama"), pair):
+    if design == "zetavik":
+        models = zetavik_set(size)
+    else:
+        pair = {"monolix": monolix_pair, "dedutar": dedutar_pair, "bazurax": bazurax_pair, "ragilorn": ragilorn_pair}[design]
+        models = list(zip((design, "llama"), pair(size)))
+    for name, cfg in models:
+        if only_models and name not in only_models:
+            continue
         tmp = tempfile.mkdtemp(prefix=f"bench_{name}_")
         try:
             write_random_model(config_from_dict(cfg), 2, tmp, device="cuda")
@@ -567,10 +609,13 @@ def main() -> int:
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="--only prefill: tokens of the prompt")
     ap.add_argument("--prefill-batch", type=int, default=0,
                     help="--only prefill: a packed batch of that many prompts with lengths from --prompt-range")
-    ap.add_argument("--only", choices=["decode", "prefill", "phases", "sampled", "dedutar", "monolix", "bazurax", "ragilorn"],
+    ap.add_argument("--only", choices=["decode", "prefill", "phases", "sampled", "dedutar", "monolix", "bazurax", "ragilorn", "zetavik"],
                     help="run one small workload (for profiling) and stop; phases: see phase_stamps(); dedutar, "
-                         "monolix, bazurax, ragilorn: prefill and decode of that design beside Llama at equal layer sizes")
+                         "monolix, bazurax, ragilorn, zetavik: prefill and decode of that design beside Llama (zetavik: and its "
+                         "closest relatives) at equal layer sizes")
     ap.add_argument("--bazurax-size", default="1b", choices=sorted(BAZURAX_SIZES), help="--only bazurax: layer sizes")
+    ap.add_argument("--zetavik-size", default="1b", choices=sorted(ZETAVIK_SIZES), help="--only zetavik: layer sizes")
+    ap.add_argument("--models", default="", help="--only zetavik: names of the models to run (default: all of the set)")
     ap.add_argument("--ragilorn-size", default="1b", choices=sorted(RAGILORN_SIZES), help="--only ragilorn: layer sizes")
     ap.add_argument("--monolix-size", default="1b", choices=sorted(MONOLIX_SIZES), help="--only monolix: layer sizes")
     ap.add_argument("--dedutar-size", default="1b", choices=sorted(DEDUTAR_SIZES), help="--only dedutar: layer sizes")
@@ -601,6 +646,10 @@ def main() -> int:
     if a.only == "ragilorn":
         print(json.dumps(dedutar_compare(a.ragilorn_size, a.batch, a.steps, warmup, a.prefill_tokens, a.kernels,
                                          design="ragilorn")))
+        return 0
+    if a.only == "zetavik":
+        print(json.dumps(dedutar_compare(a.zetavik_size, a.batch, a.steps, warmup, a.prefill_tokens, a.kernels,
+                                         design="zetavik", only_models=tuple(n for n in a.models.split(",") if n))))
         return 0
     if a.only == "bazurax":
         print(json.dumps(dedutar_compare(a.bazurax_size, a.batch, a.steps, warmup, a.prefill_tokens, a.kernels,

@@ -52,9 +52,10 @@ LIBRARIES: Dict[str, List[str]] = {
     "conv_rope_append": ["conv_rope_append.cu"],
     "gated_residual": ["gated_residual.cu"],
     "ssd": ["ssd.cu"],
+    "ssd_tc": ["ssd_tc.cu"],
 }
 _HEADERS = ["common.cuh", "attention_noalloc.h", "attention_combine.cuh", "attention_decode_tiles.cuh", "tcgen05.cuh",
-            "async_copy.cuh"]
+            "async_copy.cuh", "ssd.cuh"]
 
 ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 BASE_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-shared", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden"]

@@ -652,11 +652,11 @@ def _ssd_check(what: str, s: SsdShape, proj: Optional[torch.Tensor], state: torc
 
 def ssd_conv(proj: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
              tiles: torch.Tensor, n_tiles: int, token_seq: torch.Tensor, seq_slot: torch.Tensor, state: torch.Tensor,
-             shape: SsdShape) -> tuple:
+             shape: SsdShape, out_dtype: torch.dtype = torch.float32, log_decay: bool = False) -> tuple:
     """Causal convolution over time, bias and silu of the columns x | B | C of ``proj`` (fp32 [T, >= columns]), reaching
     back into the state rows for a sequence's earlier inputs; and per head d = softplus(dt + dt_bias) and
     f = exp(-exp(a_log) d).  ``tiles`` [n_tiles, 3] cut the step's tokens into runs of one sequence.  Returns
-    (x | B | C [T, channels], [T, heads, 2]), fp32."""
+    (x | B | C [T, >= channels] in ``out_dtype``, (d, f) [T, heads, 2] fp32; ``log_decay``: f's logarithm instead)."""
     _ssd_check("ssd_conv", shape, proj, state)
     for n, t, k in (("taps", taps, shape.channels * shape.taps), ("bias", bias, shape.channels),
                     ("dt_bias", dt_bias, shape.heads), ("a_log", a_log, shape.heads)):
@@ -666,12 +666,12 @@ def ssd_conv(proj: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor, dt_bias
     for n, t in (("tiles", tiles), ("token_seq", token_seq), ("seq_slot", seq_slot)):
         _need(t, torch.int32, n)
     T = proj.shape[0]
-    xbc = torch.empty((T, shape.channels + -shape.channels % 4), dtype=torch.float32, device=proj.device)
+    xbc = torch.empty((T, shape.channels + -shape.channels % 8), dtype=out_dtype, device=proj.device)
     steps = torch.empty((T, shape.heads, 2), dtype=torch.float32, device=proj.device)
     st = _lib("ssd").dlgo_ssd_conv(_ptr(proj), _i(proj.stride(0)), _ptr(taps), _ptr(bias), _ptr(dt_bias), _ptr(a_log),
                                    _ptr(tiles), _i(n_tiles), _ptr(token_seq), _ptr(seq_slot), _ptr(state),
-                                   _ll(state.stride(0)), _ptr(xbc), _i(xbc.stride(0)), _ptr(steps), *shape.args(),
-                                   _stream())
+                                   _ll(state.stride(0)), _ptr(xbc), _i(dtype_code(out_dtype)), _i(xbc.stride(0)),
+                                   _ptr(steps), _i(1 if log_decay else 0), *shape.args(), _stream())
     _check(st, "ssd_conv")
     return xbc, steps
 
@@ -705,6 +705,49 @@ def ssd_segments(xbc: torch.Tensor, steps: torch.Tensor, D: torch.Tensor, tiles:
                                        _i(1 if direct else 0), _ptr(seq_slot), _ptr(state), _ll(state.stride(0)),
                                        _ptr(scratch), _ptr(out), _i(out.stride(0)), *shape.args(), _stream())
     _check(st, "ssd_segments", 1 if direct else 3)
+    return out
+
+
+def ssd_chunks_takes(dtype: torch.dtype, state_rows: int, v_dim: int) -> bool:
+    """Whether the tensor-core recurrence takes these sizes (bfloat16 runs)."""
+    return dtype == torch.bfloat16 and bool(_lib("ssd_tc").dlgo_ssd_chunks_takes(_i(state_rows), _i(v_dim)))
+
+
+def ssd_chunks(xbc: torch.Tensor, x_col: int, b_col: int, c_col: int, steps: Optional[torch.Tensor],
+               log_decay: Optional[torch.Tensor], D: Optional[torch.Tensor], tiles: torch.Tensor, n_tiles: int,
+               direct: bool, seq_slot: torch.Tensor, state: torch.Tensor, scratch: Optional[torch.Tensor],
+               heads: int, groups: int, state_rows: int, v_dim: int) -> torch.Tensor:
+    """:func:`ssd_segments` for prompts in bfloat16, on the tensor cores: x, B and C are the bfloat16 columns ``x_col``
+    (heads of v_dim), ``b_col`` and ``c_col`` (groups of state_rows) of ``xbc`` [T, ld].  ``steps`` [T, heads, 2] fp32
+    holds d and the logarithm of f; without it d = 1 and ``log_decay`` [heads] is the logarithm.  A slot's state is the
+    first heads * state_rows * v_dim numbers of its row of ``state`` (fp32)."""
+    if xbc.dtype != torch.bfloat16 or xbc.dim() != 2 or xbc.stride(1) != 1 or not xbc.is_cuda:
+        raise KernelError("ssd_chunks: xbc must be 2-D bfloat16 on the GPU with unit inner stride")
+    T, width = xbc.shape
+    if x_col + heads * v_dim > width or max(b_col, c_col) + groups * state_rows > width or min(x_col, b_col, c_col) < 0:
+        raise KernelError("ssd_chunks: the columns named lie outside xbc")
+    floats = heads * state_rows * v_dim
+    if state.dtype != torch.float32 or state.numel() // state.shape[0] < floats or not state[0].is_contiguous():
+        raise KernelError(f"ssd_chunks: state rows must hold {floats} float32 numbers")
+    for n, t in (("tiles", tiles), ("seq_slot", seq_slot)):
+        _need(t, torch.int32, n)
+    if (steps is None) == (log_decay is None):
+        raise KernelError("ssd_chunks: either steps or log_decay")
+    for n, t, k in (("steps", steps, T * heads * 2), ("log_decay", log_decay, heads), ("D", D, heads)):
+        if t is not None:
+            _need(t, torch.float32, n)
+            if t.numel() != k:
+                raise KernelError(f"ssd_chunks: {n} must have {k} numbers, has {t.numel()}")
+    if not direct:
+        need = n_tiles * heads * (state_rows * v_dim + 1)
+        if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
+            raise KernelError(f"ssd_chunks: {n_tiles} segments need {need} floats of scratch")
+    out = torch.empty((T, heads * v_dim), dtype=torch.float32, device=xbc.device)
+    st = _lib("ssd_tc").dlgo_ssd_chunks(
+        _ptr(xbc), _i(xbc.stride(0)), _i(x_col), _i(b_col), _i(c_col), _ptr(steps), _ptr(log_decay), _ptr(D), _ptr(tiles),
+        _i(n_tiles), _i(1 if direct else 0), _ptr(seq_slot), _ptr(state), _ll(state.stride(0)), _ptr(scratch), _ptr(out),
+        _i(out.stride(0)), _i(heads), _i(groups), _i(state_rows), _i(v_dim), _stream())
+    _check(st, "ssd_chunks", 1 if direct else 3)
     return out
 
 

@@ -25,21 +25,13 @@
 // neighbouring lanes share four columns; lane r of them holds rows 4 (i RS + r) .. + 3 for i = 0 .. 3 (so that their
 // 16-byte reads of B and C fall side by side), and their parts of y meet by shuffles.  N up to 512;
 // rows beyond N and columns beyond P are computed on zeros and not stored.  Everything is fp32 in every precision.
-#include "common.cuh"
+#include "ssd.cuh"
 #include "async_copy.cuh"
 
 namespace dlgo {
 
 __device__ __forceinline__ float ssd_silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float ssd_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-
-// where a sequence's inputs of earlier steps lie: entry j of taps - 1, oldest first
-struct SsdShape {
-  int H, G, N, P, taps;
-  __host__ __device__ int inner() const { return H * P; }
-  __host__ __device__ int channels() const { return H * P + 2 * G * N; }
-  __host__ __device__ long long conv_off() const { return (long long)H * N * P; }
-};
 
 // The input of channel c at packed token `tok` of sequence `seq` (tok may lie before the sequence's first token of
 // this step; `first` is that token): a projected number, or one kept from an earlier step.
@@ -52,14 +44,20 @@ __device__ __forceinline__ float conv_input(const float* xbc, int ld, int tok, i
 // ------------------------------------------------------------------------------- convolution (prompts)
 constexpr int SC_THREADS = 128;
 
+__device__ __forceinline__ void conv_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void conv_store4(__nv_bfloat16* p, float4 v) {
+  __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+  *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(h);
+}
+
 // A thread owns W neighbouring channels and walks its tile's tokens with the taps' reach in registers (TAPS > 0) or
 // reads every tap from memory (TAPS 0: any number of taps).
-template <int TAPS, int W>
+template <typename TO, int TAPS, int W>
 __global__ void __launch_bounds__(SC_THREADS)
 ssd_conv_kernel(const float* proj, int ld, const float* __restrict__ w_taps, const float* __restrict__ w_bias,
                 const float* __restrict__ dt_bias, const float* __restrict__ a_log, const int* __restrict__ tiles,
                 const int* __restrict__ token_seq, const int* __restrict__ seq_slot, const float* state,
-                long long state_ld, float* out, int ldo, float* steps, SsdShape s) {
+                long long state_ld, TO* out, int ldo, float* steps, int log_decay, SsdShape s) {
   pdl_launch_dependents();
   const int tile = blockIdx.x;
   const int seq = tiles[tile * 3 + 0], t0 = tiles[tile * 3 + 1], count = tiles[tile * 3 + 2];
@@ -71,7 +69,8 @@ ssd_conv_kernel(const float* proj, int ld, const float* __restrict__ w_taps, con
       const int t = t0 + i / s.H, h = i % s.H;
       const float d = ssd_softplus(dt[(size_t)t * ld + h] + dt_bias[h]);
       steps[((size_t)t * s.H + h) * 2] = d;
-      steps[((size_t)t * s.H + h) * 2 + 1] = expf(-expf(a_log[h]) * d);
+      const float lf = -expf(a_log[h]) * d;
+      steps[((size_t)t * s.H + h) * 2 + 1] = log_decay ? lf : expf(lf);
     }
     return;
   }
@@ -123,9 +122,9 @@ ssd_conv_kernel(const float* proj, int ld, const float* __restrict__ w_taps, con
 #pragma unroll
           for (int j = 0; j < R - 1; ++j) u[j][k] = u[j + 1][k];
         }
-        float* dst = out + (size_t)(t0 + tb + q) * ldo + c;
-        if (W == 4) *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1 % W], y[2 % W], y[3 % W]);
-        else dst[0] = y[0];
+        TO* dst = out + (size_t)(t0 + tb + q) * ldo + c;
+        if (W == 4) conv_store4(dst, make_float4(y[0], y[1 % W], y[2 % W], y[3 % W]));
+        else dst[0] = from_float<TO>(y[0]);
       }
     }
     return;
@@ -137,7 +136,7 @@ ssd_conv_kernel(const float* proj, int ld, const float* __restrict__ w_taps, con
       float a = bias[k];
       for (int j = 0; j < n_taps; ++j)
         a = fmaf(w_taps[(size_t)(c + k) * n_taps + j], conv_input(xbc, ld, t - n_taps + 1 + j, first, c + k, kept, n_taps, C), a);
-      out[(size_t)t * ldo + c + k] = ssd_silu(a);
+      out[(size_t)t * ldo + c + k] = from_float<TO>(ssd_silu(a));
     }
   }
 }
@@ -165,80 +164,103 @@ __device__ __forceinline__ void ssd_meet(float (&y)[4], int r) {
   }
 }
 
-// rows of one thread's share of a head's state, and where they lie
+// Two fp32 numbers in a 64-bit register: one instruction multiplies or multiplies-and-adds both (each rounded like its
+// scalar form).
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+  f32x2 v;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(lo), "f"(hi));
+  return v;
+}
+__device__ __forceinline__ float2 unpack2(f32x2 v) {
+  float2 o;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(o.x), "=f"(o.y) : "l"(v));
+  return o;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+
+// one thread's share of a head's state: S[j][k] holds rows ssd_row(j / 2, r) + 2 (j % 2) and the next, column k
 template <int RS>
 __device__ __forceinline__ int ssd_row(int i, int r) { return 4 * (i * RS + r); }
 
-template <int RS>
-__device__ __forceinline__ void ssd_load_state(float (&S)[16][4], const float* st, int N, int P, int e, int r, bool vec) {
-#pragma unroll
-  for (int i = 0; i < 4; ++i)
-#pragma unroll
-    for (int q = 0; q < 4; ++q) {
-      const int n = ssd_row<RS>(i, r) + q;
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (n < N && e < P) {
-        const float* p = st + (size_t)n * P + e;
-        if (vec) {
-          v = *reinterpret_cast<const float4*>(p);
-        } else {
-          v.x = p[0];
-          if (e + 1 < P) v.y = p[1];
-          if (e + 2 < P) v.z = p[2];
-          if (e + 3 < P) v.w = p[3];
-        }
-      }
-      S[i * 4 + q][0] = v.x; S[i * 4 + q][1] = v.y; S[i * 4 + q][2] = v.z; S[i * 4 + q][3] = v.w;
-    }
+__device__ __forceinline__ float4 ssd_load4(const float* p, int left, bool vec) {
+  if (vec) return *reinterpret_cast<const float4*>(p);
+  return make_float4(p[0], left > 1 ? p[1] : 0.f, left > 2 ? p[2] : 0.f, left > 3 ? p[3] : 0.f);
+}
+__device__ __forceinline__ void ssd_store4(float* p, float4 v, int left, bool vec) {
+  if (vec) {
+    *reinterpret_cast<float4*>(p) = v;
+    return;
+  }
+  p[0] = v.x;
+  if (left > 1) p[1] = v.y;
+  if (left > 2) p[2] = v.z;
+  if (left > 3) p[3] = v.w;
 }
 
 template <int RS>
-__device__ __forceinline__ void ssd_store_state(const float (&S)[16][4], float* st, int N, int P, int e, int r, bool vec) {
+__device__ __forceinline__ void ssd_load_state(f32x2 (&S)[8][4], const float* st, int N, int P, int e, int r, bool vec) {
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int n = ssd_row<RS>(j / 2, r) + 2 * (j % 2);
+    const float* p = st + (size_t)n * P + e;
+    const float4 a = (n < N && e < P) ? ssd_load4(p, P - e, vec) : zero;
+    const float4 b = (n + 1 < N && e < P) ? ssd_load4(p + P, P - e, vec) : zero;
+    S[j][0] = pack2(a.x, b.x); S[j][1] = pack2(a.y, b.y); S[j][2] = pack2(a.z, b.z); S[j][3] = pack2(a.w, b.w);
+  }
+}
+
+template <int RS>
+__device__ __forceinline__ void ssd_store_state(const f32x2 (&S)[8][4], float* st, int N, int P, int e, int r, bool vec) {
   if (e >= P) return;
 #pragma unroll
-  for (int i = 0; i < 4; ++i)
-#pragma unroll
-    for (int q = 0; q < 4; ++q) {
-      const int n = ssd_row<RS>(i, r) + q;
-      if (n >= N) continue;
-      float* p = st + (size_t)n * P + e;
-      const float* v = S[i * 4 + q];
-      if (vec) {
-        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-      } else {
-#pragma unroll
-        for (int k = 0; k < 4; ++k)
-          if (e + k < P) p[k] = v[k];
-      }
-    }
+  for (int j = 0; j < 8; ++j) {
+    const int n = ssd_row<RS>(j / 2, r) + 2 * (j % 2);
+    float* p = st + (size_t)n * P + e;
+    const float2 x = unpack2(S[j][0]), y = unpack2(S[j][1]), z = unpack2(S[j][2]), w = unpack2(S[j][3]);
+    if (n < N) ssd_store4(p, make_float4(x.x, y.x, z.x, w.x), P - e, vec);
+    if (n + 1 < N) ssd_store4(p + P, make_float4(x.y, y.y, z.y, w.y), P - e, vec);
+  }
 }
 
 // one token: S <- f S + B v^T (v = d x), and with OUT the thread's part of S^T C
 template <int RS, bool OUT>
-__device__ __forceinline__ void ssd_token(float (&S)[16][4], const float* B, const float* C, float f, float4 v, int r,
+__device__ __forceinline__ void ssd_token(f32x2 (&S)[8][4], const float* B, const float* C, float f, float4 v, int r,
                                           float (&y)[4]) {
+  const f32x2 ff = pack2(f, f);
+  const f32x2 vv[4] = {pack2(v.x, v.x), pack2(v.y, v.y), pack2(v.z, v.z), pack2(v.w, v.w)};
+  f32x2 acc[4] = {0ull, 0ull, 0ull, 0ull};                         // (two zeros)
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
-    const float4 b4 = *reinterpret_cast<const float4*>(B + ssd_row<RS>(i, r));
-    const float b[4] = {b4.x, b4.y, b4.z, b4.w};
-    float c[4] = {0.f, 0.f, 0.f, 0.f};
-    if (OUT) {
-      const float4 c4 = *reinterpret_cast<const float4*>(C + ssd_row<RS>(i, r));
-      c[0] = c4.x; c[1] = c4.y; c[2] = c4.z; c[3] = c4.w;
+    const ulonglong2 b = *reinterpret_cast<const ulonglong2*>(B + ssd_row<RS>(i, r));
+    ulonglong2 c = make_ulonglong2(0ull, 0ull);
+    if (OUT) c = *reinterpret_cast<const ulonglong2*>(C + ssd_row<RS>(i, r));
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      S[2 * i][k] = fma2(ff, S[2 * i][k], mul2(b.x, vv[k]));
+      if (OUT) acc[k] = fma2(S[2 * i][k], c.x, acc[k]);
     }
 #pragma unroll
-    for (int q = 0; q < 4; ++q) {
-      float* s = S[i * 4 + q];
-      s[0] = fmaf(f, s[0], b[q] * v.x);
-      s[1] = fmaf(f, s[1], b[q] * v.y);
-      s[2] = fmaf(f, s[2], b[q] * v.z);
-      s[3] = fmaf(f, s[3], b[q] * v.w);
-      if (OUT) {
-        y[0] = fmaf(s[0], c[q], y[0]);
-        y[1] = fmaf(s[1], c[q], y[1]);
-        y[2] = fmaf(s[2], c[q], y[2]);
-        y[3] = fmaf(s[3], c[q], y[3]);
-      }
+    for (int k = 0; k < 4; ++k) {
+      S[2 * i + 1][k] = fma2(ff, S[2 * i + 1][k], mul2(b.y, vv[k]));
+      if (OUT) acc[k] = fma2(S[2 * i + 1][k], c.y, acc[k]);
+    }
+  }
+  if (OUT) {
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 a = unpack2(acc[k]);
+      y[k] = a.x + a.y;
     }
   }
 }
@@ -310,12 +332,12 @@ ssd_segments_kernel(const float* xbc, int ld, const float* steps, const float* _
   };
   const int n_chunks = (count + CH - 1) / CH;
   load_chunk(0, ring);
-  float S[16][4];
+  f32x2 S[8][4];
   if (MODE == SSD_LOCAL) {
 #pragma unroll
-    for (int i = 0; i < 16; ++i)
+    for (int j = 0; j < 8; ++j)
 #pragma unroll
-      for (int k = 0; k < 4; ++k) S[i][k] = 0.f;
+      for (int k = 0; k < 4; ++k) S[j][k] = 0ull;
   } else {
     ssd_load_state<RS>(S, direct ? st : sg, N, P, e, r, vec);
   }
@@ -354,55 +376,6 @@ ssd_segments_kernel(const float* xbc, int ld, const float* steps, const float* _
   }
 }
 
-// seg[j] <- the state segment j starts from.  A block row per first segment of a sequence, a thread per W neighbouring
-// elements of the state; the ends of up to eight segments are fetched together.
-template <int W>
-__global__ void __launch_bounds__(256)
-ssd_carry_kernel(const int* __restrict__ tiles, int n_tiles, const int* __restrict__ seq_slot, const float* state,
-                 long long state_ld, float* seg, const float* seg_decay, SsdShape s) {
-  pdl_launch_dependents();
-  const int j0 = blockIdx.y;
-  const int seq = tiles[j0 * 3];
-  if (j0 > 0 && tiles[(j0 - 1) * 3] == seq) return;
-  const long long per_head = (long long)s.N * s.P, total = per_head * s.H;
-  const long long i = ((long long)blockIdx.x * 256 + threadIdx.x) * W;
-  if (i >= total) return;
-  const int h = (int)(i / per_head);                               // (W = 4 only where a head's numbers are a multiple of 4)
-  pdl_wait();
-  float S[W];
-  const float* st = state + (size_t)seq_slot[seq] * state_ld + i;
-#pragma unroll
-  for (int k = 0; k < W; ++k) S[k] = st[k];
-  for (int jb = j0; jb < n_tiles && tiles[jb * 3] == seq; jb += 8) {
-    float L[8][W], F[8];
-    int n = 0;
-#pragma unroll
-    for (int u = 0; u < 8; ++u) {
-      const int j = jb + u;
-      const bool in = j < n_tiles && tiles[j * 3] == seq;
-      n += in;
-      const bool more = in && j + 1 < n_tiles && tiles[(j + 1) * 3] == seq;   // (a sequence's last segment left no end)
-      F[u] = more ? seg_decay[(size_t)j * s.H + h] : 0.f;
-      if (W == 4) {
-        const float4 v = more ? *reinterpret_cast<const float4*>(seg + (size_t)j * total + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-        L[u][0] = v.x; L[u][1 % W] = v.y; L[u][2 % W] = v.z; L[u][3 % W] = v.w;
-      } else {
-        L[u][0] = more ? seg[(size_t)j * total + i] : 0.f;
-      }
-    }
-#pragma unroll
-    for (int u = 0; u < 8; ++u) {
-      if (u < n) {
-        float* dst = seg + (size_t)(jb + u) * total + i;
-        if (W == 4) *reinterpret_cast<float4*>(dst) = make_float4(S[0], S[1 % W], S[2 % W], S[3 % W]);
-        else dst[0] = S[0];
-#pragma unroll
-        for (int k = 0; k < W; ++k) S[k] = fmaf(F[u], S[k], L[u][k]);
-      }
-    }
-  }
-}
-
 // ------------------------------------------------------------------------------- one token per sequence
 template <int RS>
 __global__ void __launch_bounds__(RS <= 8 ? 128 : 16 * RS)
@@ -426,7 +399,7 @@ ssd_step_kernel(const float* proj, int ld, const float* __restrict__ w_taps, con
   for (int i = threadIdx.x; i < 2 * NPAD + TL::COLS; i += blockDim.x) row[i] = 0.f;
   __syncthreads();
   pdl_wait();
-  float S[16][4];
+  f32x2 S[8][4];
   ssd_load_state<RS>(S, st, N, P, e, r, vec);                      // in flight while the convolution is formed
   const float* pr = proj + (size_t)t * ld + s.inner();
   const int b_off = s.inner() + g * N, c_off = b_off + s.G * N, x_off = h * P + e0;
@@ -452,7 +425,77 @@ ssd_step_kernel(const float* proj, int ld, const float* __restrict__ w_taps, con
 }
 
 // ------------------------------------------------------------------------------- gate and norm
-// A block per (token, part).  `stash`: the part's gated numbers stay in shared memory between the passes.
+// The convolution's inputs that a sequence's next tokens reach back to, moved into the state row by the token t that ends
+// its part of the step; this thread takes channels c0, c0 + stride, ...
+__device__ __forceinline__ void keep_conv_inputs(const float* proj, int ld, int t, int seq, const int* token_seq, float* row,
+                                                 const SsdShape& s, int c0, int stride) {
+  const int keep = s.taps - 1;
+  if (keep == 0) return;
+  const int C = s.channels();
+  int here = 1;                                    // tokens of this step that the new row can take
+  while (here < keep && t - here >= 0 && token_seq[t - here] == seq) ++here;
+  const int old = keep - min(here, keep);          // entries that stay from the old row
+  float* kept = row + s.conv_off();
+  const float* xbc = proj + s.inner();
+  for (int c = c0; c < C; c += stride)
+    for (int j = 0; j < keep; ++j) {
+      // entry j is the input `keep - 1 - j` tokens back; ascending j: an old entry is read before it is overwritten
+      const int back = keep - 1 - j;
+      kept[(size_t)j * C + c] = j >= old ? xbc[(size_t)(t - back) * ld + c] : kept[(size_t)(j + here) * C + c];
+    }
+}
+
+// A warp per (token, part) with the part's gated numbers in registers: parts of up to 128 NV numbers, a multiple of 4.
+constexpr int GN_WARPS = 4;
+template <typename TO, int NV>
+__global__ void __launch_bounds__(GN_WARPS * 32)
+ssd_gate_norm_warp_kernel(const float* y, int ldy, const float* proj, int ld, const float* __restrict__ w, TO* out, int groups,
+                          float eps, const int* __restrict__ token_seq, int T, const int* __restrict__ seq_slot, float* state,
+                          long long state_ld, SsdShape s) {
+  pdl_launch_dependents();
+  const int lane = threadIdx.x & 31, n = s.inner() / groups;
+  const long long item = (long long)blockIdx.x * GN_WARPS + (threadIdx.x >> 5);
+  if (item >= (long long)T * groups) return;
+  const int t = (int)(item / groups), part = (int)(item - (long long)t * groups);
+  const int seq = token_seq[t];
+  const bool ends = t + 1 == T || token_seq[t + 1] != seq;
+  float4 wv[NV], u[NV], z[NV];
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (v * 32 + lane) * 4;
+    if (i < n) wv[v] = *reinterpret_cast<const float4*>(w + (size_t)part * n + i);
+  }
+  pdl_wait();
+  const float* yr = y + (size_t)t * ldy + (size_t)part * n;
+  const float* zr = proj + (size_t)t * ld + (size_t)part * n;
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (v * 32 + lane) * 4;
+    if (i < n) {
+      u[v] = *reinterpret_cast<const float4*>(yr + i);
+      z[v] = *reinterpret_cast<const float4*>(zr + i);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < NV; ++v)
+    if ((v * 32 + lane) * 4 < n) {
+      u[v].x *= ssd_silu(z[v].x); u[v].y *= ssd_silu(z[v].y); u[v].z *= ssd_silu(z[v].z); u[v].w *= ssd_silu(z[v].w);
+      ss += (u[v].x * u[v].x + u[v].y * u[v].y) + (u[v].z * u[v].z + u[v].w * u[v].w);
+    }
+  const float sc = 1.0f / sqrtf(warp_sum(ss) / (float)n + eps);
+  TO* dst = out + (size_t)t * s.inner() + (size_t)part * n;
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (v * 32 + lane) * 4;
+    if (i < n)
+      conv_store4(dst + i, make_float4(u[v].x * sc * wv[v].x, u[v].y * sc * wv[v].y, u[v].z * sc * wv[v].z, u[v].w * sc * wv[v].w));
+  }
+  if (ends)
+    keep_conv_inputs(proj, ld, t, seq, token_seq, state + (size_t)seq_slot[seq] * state_ld, s, part * 32 + lane, groups * 32);
+}
+
+// A block per (token, part), parts of any size.  `stash`: the part's gated numbers stay in shared memory between the passes.
 template <typename TO>
 __global__ void __launch_bounds__(512)
 ssd_gate_norm_kernel(const float* y, int ldy, const float* proj, int ld, const float* __restrict__ w, TO* out, int groups,
@@ -490,23 +533,33 @@ ssd_gate_norm_kernel(const float* y, int ldy, const float* proj, int ld, const f
     const float u = stash ? u_s[i] : yr[i] * ssd_silu(zr[i]);      // (block_sum's barriers lie between u_s's writes and reads)
     dst[i] = from_float<TO>(u * sc * wp[i]);
   }
-  // the convolution's inputs that the sequence's next tokens reach back to
-  const int keep = s.taps - 1;
-  if (!ends || keep == 0) return;
-  const int C = s.channels();
-  int here = 1;                                    // tokens of this step that the new row can take
-  while (here < keep && t - here >= 0 && token_seq[t - here] == seq) ++here;
-  const int old = keep - min(here, keep);          // entries that stay from the old row
-  const bool all = here >= keep;
-  float* kept = state + (size_t)seq_slot[seq] * state_ld + s.conv_off();
-  const float* xbc = proj + s.inner();
-  for (int c = part * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
-    for (int j = 0; j < keep; ++j) {
-      // entry j is the input `keep - 1 - j` tokens back; ascending j: an old entry is read before it is overwritten
-      const int back = keep - 1 - j;
-      kept[(size_t)j * C + c] = (all || j >= old) ? xbc[(size_t)(t - back) * ld + c] : kept[(size_t)(j + here) * C + c];
-    }
+  if (ends)
+    keep_conv_inputs(proj, ld, t, seq, token_seq, state + (size_t)seq_slot[seq] * state_ld, s,
+                     part * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
+}
+
+template <typename TO>
+static int launch_ssd_gate_norm(const float* y, int ldy, const float* proj, int ld, const float* w, TO* out, int groups,
+                                float eps, const int* token_seq, int T, const int* seq_slot, float* state,
+                                long long state_ld, const SsdShape& s, cudaStream_t stream) {
+  const int n = s.inner() / groups;
+  const bool four = n % 4 == 0 && ldy % 4 == 0 && ld % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)proj & 15) == 0 &&
+                    ((uintptr_t)w & 15) == 0 && ((uintptr_t)out & 15) == 0;
+  if (four && n <= 1024) {
+    const dim3 grid((unsigned)(((long long)T * groups + GN_WARPS - 1) / GN_WARPS)), block(GN_WARPS * 32);
+#define GN_ARGS grid, block, 0, stream, y, ldy, proj, ld, w, out, groups, eps, token_seq, T, seq_slot, state, state_ld, s
+    if (n <= 128) launch_kernel(ssd_gate_norm_warp_kernel<TO, 1>, GN_ARGS);
+    else if (n <= 256) launch_kernel(ssd_gate_norm_warp_kernel<TO, 2>, GN_ARGS);
+    else if (n <= 512) launch_kernel(ssd_gate_norm_warp_kernel<TO, 4>, GN_ARGS);
+    else launch_kernel(ssd_gate_norm_warp_kernel<TO, 8>, GN_ARGS);
+#undef GN_ARGS
+    return launch_status();
   }
+  const int stash = n * sizeof(float) <= 40 * 1024;
+  const int threads = n >= 2048 ? 512 : (n >= 512 ? 256 : (n >= 128 ? 128 : 64));
+  launch_kernel(ssd_gate_norm_kernel<TO>, dim3(T, groups), dim3(threads), stash ? n * sizeof(float) : 0, stream, y, ldy, proj,
+                ld, w, out, groups, eps, token_seq, T, seq_slot, state, state_ld, s, stash);
+  return launch_status();
 }
 
 static bool ssd_shape_ok(const SsdShape& s) {
@@ -538,13 +591,7 @@ static int launch_ssd_segments(const float* xbc, int ld, const float* steps, con
                   seq_slot, state, state_ld, seg, dec, out, ldo, s, direct, vec);
     int st = launch_status();
     if (st != DLGO_OK) return st;
-    const long long total = (long long)s.H * s.N * s.P;
-    const bool four = vec && ((long long)s.N * s.P) % 4 == 0;
-    const long long items = four ? total / 4 : total;
-    const dim3 cgrid((unsigned)((items + 255) / 256), n_tiles);
-    if (four) launch_kernel(ssd_carry_kernel<4>, cgrid, dim3(256), 0, stream, tiles, n_tiles, seq_slot, state, state_ld, seg, dec, s);
-    else launch_kernel(ssd_carry_kernel<1>, cgrid, dim3(256), 0, stream, tiles, n_tiles, seq_slot, state, state_ld, seg, dec, s);
-    st = launch_status();
+    st = launch_ssd_carry(tiles, n_tiles, seq_slot, state, state_ld, seg, dec, s, stream);
     if (st != DLGO_OK) return st;
   }
   launch_kernel(ssd_segments_kernel<RS, SSD_FULL>, grid, block, smem, stream, xbc, ld, steps, D, tiles, n_tiles, seq_slot,
@@ -556,30 +603,43 @@ static int launch_ssd_segments(const float* xbc, int ld, const float* steps, con
 
 using namespace dlgo;
 
-// proj [T, ld] fp32 with the columns [z | x | B | C | dt]; w_taps [C, taps], w_bias [C], dt_bias, a_log [H] fp32;
-// tiles [n_tiles, 3] (sequence, first packed token, count); out [T, ldo >= C] fp32: x | B | C;
-// steps [T, H, 2] fp32: d and f
-DLGO_EXPORT int dlgo_ssd_conv(const float* proj, int ld, const float* w_taps, const float* w_bias, const float* dt_bias,
-                              const float* a_log, const int* tiles, int n_tiles, const int* token_seq,
-                              const int* seq_slot, const float* state, long long state_ld, float* out, int ldo,
-                              float* steps, int H, int G, int N, int P, int taps, cudaStream_t stream) {
-  if (n_tiles <= 0) return DLGO_OK;
-  const SsdShape s{H, G, N, P, taps};
-  if (!ssd_shape_ok(s)) return DLGO_ERR_SIZE;
+template <typename TO>
+static int launch_ssd_conv(const float* proj, int ld, const float* w_taps, const float* w_bias, const float* dt_bias,
+                           const float* a_log, const int* tiles, int n_tiles, const int* token_seq, const int* seq_slot,
+                           const float* state, long long state_ld, TO* out, int ldo, float* steps, int log_decay,
+                           const SsdShape& s, cudaStream_t stream) {
   const int C = s.channels();
-  const bool four = taps <= 4 && C % 4 == 0 && s.inner() % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 &&
+  const bool four = s.taps <= 4 && C % 4 == 0 && s.inner() % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 &&
                     ((uintptr_t)proj & 15) == 0 && ((uintptr_t)out & 15) == 0;
   const int w = four ? 4 : 1;
   const dim3 grid(n_tiles, (C + SC_THREADS * w - 1) / (SC_THREADS * w) + 1), block(SC_THREADS);
 #define CONV_ARGS grid, block, 0, stream, proj, ld, w_taps, w_bias, dt_bias, a_log, tiles, token_seq, seq_slot, state, \
-                  state_ld, out, ldo, steps, s
-  if (four && taps == 4) launch_kernel(ssd_conv_kernel<4, 4>, CONV_ARGS);
-  else if (four && taps == 3) launch_kernel(ssd_conv_kernel<3, 4>, CONV_ARGS);
-  else if (four && taps == 2) launch_kernel(ssd_conv_kernel<2, 4>, CONV_ARGS);
-  else if (four && taps == 1) launch_kernel(ssd_conv_kernel<1, 4>, CONV_ARGS);
-  else launch_kernel(ssd_conv_kernel<0, 1>, CONV_ARGS);
+                  state_ld, out, ldo, steps, log_decay, s
+  if (four && s.taps == 4) launch_kernel(ssd_conv_kernel<TO, 4, 4>, CONV_ARGS);
+  else if (four && s.taps == 3) launch_kernel(ssd_conv_kernel<TO, 3, 4>, CONV_ARGS);
+  else if (four && s.taps == 2) launch_kernel(ssd_conv_kernel<TO, 2, 4>, CONV_ARGS);
+  else if (four && s.taps == 1) launch_kernel(ssd_conv_kernel<TO, 1, 4>, CONV_ARGS);
+  else launch_kernel(ssd_conv_kernel<TO, 0, 1>, CONV_ARGS);
 #undef CONV_ARGS
   return launch_status();
+}
+
+// proj [T, ld] fp32 with the columns [z | x | B | C | dt]; w_taps [C, taps], w_bias [C], dt_bias, a_log [H] fp32;
+// tiles [n_tiles, 3] (sequence, first packed token, count); out [T, ldo >= C] in `dtype`: x | B | C; steps [T, H, 2] fp32:
+// d and f, or with `log_decay` d and the logarithm of f
+DLGO_EXPORT int dlgo_ssd_conv(const float* proj, int ld, const float* w_taps, const float* w_bias, const float* dt_bias,
+                              const float* a_log, const int* tiles, int n_tiles, const int* token_seq,
+                              const int* seq_slot, const float* state, long long state_ld, void* out, int dtype, int ldo,
+                              float* steps, int log_decay, int H, int G, int N, int P, int taps, cudaStream_t stream) {
+  if (n_tiles <= 0) return DLGO_OK;
+  const SsdShape s{H, G, N, P, taps};
+  if (!ssd_shape_ok(s)) return DLGO_ERR_SIZE;
+#define CONV_ARGS(T) proj, ld, w_taps, w_bias, dt_bias, a_log, tiles, n_tiles, token_seq, seq_slot, state, state_ld, (T*)out, ldo, \
+                     steps, log_decay, s, stream
+  if (dtype == DLGO_F32) return launch_ssd_conv<float>(CONV_ARGS(float));
+  if (dtype == DLGO_BF16) return launch_ssd_conv<__nv_bfloat16>(CONV_ARGS(__nv_bfloat16));
+#undef CONV_ARGS
+  return DLGO_ERR_DTYPE;
 }
 
 // xbc [T, ld] fp32 (x | B | C) and steps of dlgo_ssd_conv; D [H] fp32; tiles [n_tiles, 3], a sequence's segments side by
@@ -636,17 +696,9 @@ DLGO_EXPORT int dlgo_ssd_gate_norm(const float* y, int ldy, const float* proj, i
   if (T <= 0) return DLGO_OK;
   const SsdShape s{H, G, N, P, taps};
   if (!ssd_shape_ok(s) || groups <= 0 || s.inner() % groups || groups > 65535) return DLGO_ERR_SIZE;
-  const int n = s.inner() / groups;
-  const int stash = n * sizeof(float) <= 40 * 1024;
-  const size_t smem = stash ? n * sizeof(float) : 0;
-  const int threads = n >= 2048 ? 512 : (n >= 512 ? 256 : (n >= 128 ? 128 : 64));
-  if (dtype == DLGO_F32)
-    launch_kernel(ssd_gate_norm_kernel<float>, dim3(T, groups), dim3(threads), smem, stream, y, ldy, proj, ld, w, (float*)out,
-                  groups, eps, token_seq, T, seq_slot, state, state_ld, s, stash);
-  else if (dtype == DLGO_BF16)
-    launch_kernel(ssd_gate_norm_kernel<__nv_bfloat16>, dim3(T, groups), dim3(threads), smem, stream, y, ldy, proj, ld, w,
-                  (__nv_bfloat16*)out, groups, eps, token_seq, T, seq_slot, state, state_ld, s, stash);
-  else
-    return DLGO_ERR_DTYPE;
-  return launch_status();
+#define GN_ARGS(T_) y, ldy, proj, ld, w, (T_*)out, groups, eps, token_seq, T, seq_slot, state, state_ld, s, stream
+  if (dtype == DLGO_F32) return launch_ssd_gate_norm<float>(GN_ARGS(float));
+  if (dtype == DLGO_BF16) return launch_ssd_gate_norm<__nv_bfloat16>(GN_ARGS(__nv_bfloat16));
+#undef GN_ARGS
+  return DLGO_ERR_DTYPE;
 }

@@ -7,7 +7,8 @@ by ``Wo``.  The state [heads, qk_dim, v_dim] is fp32, zero at a sequence's start
 sequence's slot of the state area from step to step; no position is cached.
 
 q, k, v and the gate come from one contraction with an fp32 result; silu, decay, state, norm and gate are
-computed in fp32 in every precision.
+computed in fp32 in every precision.  A bfloat16 run's prompts take q, k and v as bfloat16 behind their silu (formed in
+the contraction's epilogue) and run the recurrence's products on the tensor cores, where its kernels take the sizes.
 
 :class:`Retention` is the same recurrence with other surroundings: ``q = Wq h`` and ``k = Wk h`` without an
 activation but with rotary positions (and a constant factor on k), ``v = Wv h``; every head's output is divided by
@@ -23,6 +24,7 @@ from ..csrc import kernels as K
 from .base import Mixer, ParamSpec, PositionEncoding, StateNeed
 from .linear import ADD_F32, STORE_F32, Linear, stack_rows
 from .registry import MIXERS
+from .state_space import TC_MIN_TOKENS, TC_SEGMENT
 
 _NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "gate": "g_proj.weight",
           "out": "o_proj.weight", "norm": "norm.weight"}
@@ -65,12 +67,35 @@ class LightningAttention(Mixer):
         self.wo = Linear(get(n["out"]), runtime)
         self.norm = get(n["norm"]).to(torch.float32).contiguous()
         self.decay = torch.tensor(self.decay_values, dtype=torch.float64).to(torch.float32).to(runtime.device)
+        # prompts on the tensor cores: q | k | v and the gate as contractions of their own over the same rows
+        H, n_qkv = self.n_heads, self.n_heads * (2 * self.qk_dim + self.v_dim)
+        self.w_qkv = self.w_gate = self.log_decay = None
+        if min(self.decay_values) > 0 and n_qkv % 8 == 0 and K.ssd_chunks_takes(runtime.dtype, self.qk_dim, self.v_dim):
+            self.w_qkv = Linear(self.w_in.weight[:n_qkv], runtime)
+            self.w_gate = Linear(self.w_in.weight[n_qkv:], runtime)
+            self.log_decay = torch.log(torch.tensor(self.decay_values, dtype=torch.float64)).to(torch.float32).to(runtime.device)
+
+    def _prompt_tc(self, x: torch.Tensor, ctx: Any, state: torch.Tensor) -> tuple:
+        """(outputs [T, H dv] fp32, gate logits) of a prompt step, the recurrence's products on the tensor cores."""
+        H, dk, dv = self.n_heads, self.qk_dim, self.v_dim
+        qkv = self.w_qkv.bias_act(x, None, K.ACT_SILU)
+        tiles, n_tiles, _ = ctx.tiles(TC_SEGMENT)
+        direct = n_tiles == ctx.n_seqs
+        scratch = None if direct else ctx.scratch("lightning_segments", n_tiles * H * (dk * dv + 1))
+        o = K.ssd_chunks(qkv, 2 * H * dk, H * dk, 0, None, self.log_decay, None, tiles, n_tiles, direct, ctx.seq_slot,
+                         state.view(state.shape[0], -1), scratch, H, H, dk, dv)
+        return o, self.w_gate(x, STORE_F32)
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: Any, cache: Any,
                 state: Optional[torch.Tensor], positions: Mapping[str, PositionEncoding]) -> None:
         if state is None:
             raise RuntimeError("lightning attention needs its state")
         H, dk, dv = self.n_heads, self.qk_dim, self.v_dim
+        if self.w_qkv is not None and not ctx.decode and 0 < TC_MIN_TOKENS <= ctx.n_tokens:
+            o, gate = self._prompt_tc(x, ctx, state)
+            a = K.gated_rmsnorm(o, gate, self.norm, self.eps, self.wo.weight.dtype)
+            self.wo(a, ADD_F32, residual)
+            return
         proj = self.w_in(x, STORE_F32)                      # [T, 2 H dk + 2 H dv] fp32
         if K.lightning_segments_takes(dk):
             # the state's columns in registers; a prompt's segments side by side

@@ -11,7 +11,8 @@ With h the mixer's input, one projection gives [z | x | B | C | dt] (``heads * v
 
 The state of a sequence is S for every head followed by the last ``conv_taps - 1`` inputs of the convolution, fp32, zero
 when the slot is taken; no position is cached.  The projection's result and everything up to the norm are fp32 in every
-precision.
+precision, but that a bfloat16 run's prompts take x, B and C as bfloat16 behind their silu and run the recurrence's
+products on the tensor cores.
 """
 from __future__ import annotations
 
@@ -28,6 +29,8 @@ from .registry import MIXERS
 _NAMES = {"in": "in_proj.weight", "conv": "conv.weight", "conv_bias": "conv.bias", "dt_bias": "dt_bias", "decay": "A_log",
           "skip": "D", "norm": "norm.weight", "out": "out_proj.weight"}
 SEGMENT = int(os.environ.get("DLGO_SSD_SEGMENT", 128))   # tokens of a segment where a prompt's segments run side by side
+TC_SEGMENT = int(os.environ.get("DLGO_SSD_TC_SEGMENT", 256))   # ... on the tensor cores (a multiple of 64)
+TC_MIN_TOKENS = int(os.environ.get("DLGO_SSD_TC_MIN_TOKENS", 64))   # prompt steps that run there (0: never)
 CONV_TILE = 16                                           # tokens of a block of the convolution
 
 
@@ -84,13 +87,20 @@ class StateSpaceMixer(Mixer):
         if ctx.decode:
             y = K.ssd_step(proj, self.taps, self.conv_bias, self.dt_bias, self.a_log, self.skip, ctx.seq_slot, state, s)
         else:
+            on_tc = 0 < TC_MIN_TOKENS <= ctx.n_tokens and K.ssd_chunks_takes(self.wo.weight.dtype, s.state, s.v_dim)
             tiles, n_tiles, _ = ctx.tiles(CONV_TILE)
             xbc, steps = K.ssd_conv(proj, self.taps, self.conv_bias, self.dt_bias, self.a_log, tiles, n_tiles,
-                                    ctx.token_seq, ctx.seq_slot, state, s)
-            tiles, n_tiles, _ = ctx.tiles(SEGMENT)
+                                    ctx.token_seq, ctx.seq_slot, state, s,
+                                    out_dtype=torch.bfloat16 if on_tc else torch.float32, log_decay=on_tc)
+            tiles, n_tiles, _ = ctx.tiles(TC_SEGMENT if on_tc else SEGMENT)
             direct = n_tiles == ctx.n_seqs
             scratch = None if direct else ctx.scratch("ssd_segments", K.ssd_scratch_floats(n_tiles, s))
-            y = K.ssd_segments(xbc, steps, self.skip, tiles, n_tiles, direct, ctx.seq_slot, state, scratch, s)
+            if on_tc:
+                bc = s.groups * s.state
+                y = K.ssd_chunks(xbc, 0, s.inner, s.inner + bc, steps, None, self.skip, tiles, n_tiles, direct, ctx.seq_slot,
+                                 state, scratch, s.heads, s.groups, s.state, s.v_dim)
+            else:
+                y = K.ssd_segments(xbc, steps, self.skip, tiles, n_tiles, direct, ctx.seq_slot, state, scratch, s)
         a = K.ssd_gate_norm(y, proj, self.norm, self.norm_groups, self.eps, self.wo.weight.dtype, ctx.token_seq,
                             ctx.seq_slot, state, s)
         self.wo(a, ADD_F32, residual)

@@ -609,3 +609,69 @@ def test_trace_replay_command(dirs, tmp_path):
     want = {0: torch.stack([ra[0], ra[27]]), 1: torch.stack([ra[28], rb[70]]), 2: rb[71:72], 3: rb[72:73]}
     for i, ref in want.items():
         assert_rows(outs[i], ref, "float32", f"step {i}")
+
+
+# ------------------------------------------------- the recurrence's products on the tensor cores (bfloat16 prompts)
+@pytest.mark.parametrize("segment", [64, 256])
+@pytest.mark.parametrize("fixed", [False, True], ids=["step per token", "fixed decay"])
+@pytest.mark.parametrize("H, G, N, P_", [(4, 2, 32, 48), (2, 1, 128, 64), (3, 3, 64, 72), (1, 1, 8, 8), (6, 2, 24, 136), (2, 2, 104, 16)])
+def test_recurrence_on_tensor_cores(H, G, N, P_, fixed, segment):
+    """Three sequences over two steps (a prompt, then a portion that continues it): outputs and the states left behind,
+    against the recurrence on the same bfloat16 inputs, at the precision of two bfloat16 terms."""
+    from dlgo_b200.csrc import kernels as K
+    assert K.ssd_chunks_takes(torch.bfloat16, N, P_) and not K.ssd_chunks_takes(torch.float32, N, P_)
+    if fixed:
+        G = H
+    g = torch.Generator().manual_seed(H * N + P_)
+    lens = [[300, 65], [1, 64], [130, 3]]
+    pad, width = 8, H * P_ + 2 * G * N + 16
+    x0, b0, c0 = pad, pad + H * P_, pad + H * P_ + G * N
+    rows = [torch.randn(sum(l), width, generator=g).to(torch.bfloat16) for l in lens]
+    D = None if fixed else torch.randn(H, generator=g)
+    decay = torch.tensor([0.999, 0.5, 0.97, 1.0, 0.9, 0.01][:H])
+    steps = [torch.stack([torch.rand(sum(l), H, generator=g) + 0.01, -torch.rand(sum(l), H, generator=g) ** 8 * 30], -1) for l in lens]
+    refs = []
+    for q in range(3):
+        r, T = rows[q].double(), rows[q].shape[0]
+        x, B, C = r[:, x0:b0].view(T, H, P_), r[:, b0:c0].view(T, G, N), r[:, c0:c0 + G * N].view(T, G, N)
+        if fixed:
+            S, y = torch.zeros(H, N, P_, dtype=torch.float64), torch.zeros(T, H, P_, dtype=torch.float64)
+            y = P.decayed_linear_attention(C, B, x, decay.double())
+            for t in range(T):
+                S = decay.double()[:, None, None] * S + B[t][:, :, None] * x[t][:, None, :]
+        else:
+            S, y = torch.zeros(H, N, P_, dtype=torch.float64), torch.zeros(T, H, P_, dtype=torch.float64)
+            d, f = steps[q][..., 0].double(), torch.exp(steps[q][..., 1].double())
+            per = H // G
+            for t in range(T):
+                Bt, Ct = B[t].repeat_interleave(per, 0), C[t].repeat_interleave(per, 0)
+                S = f[t][:, None, None] * S + (d[t][:, None] * Bt)[:, :, None] * x[t][:, None, :]
+                y[t] = torch.einsum("hnp,hn->hp", S, Ct) + D.double()[:, None] * x[t]
+        refs.append((y.reshape(T, H * P_), S))
+    state = torch.full((4, H * N * P_ + 4), float("nan"), device=DEV)
+    slots = [3, 0, 2]
+    state[slots] = 0.0
+    done = [0, 0, 0]
+    for step in range(2):
+        ns = [l[step] for l in lens]
+        cat = torch.cat([rows[q][done[q]:done[q] + ns[q]] for q in range(3)]).to(DEV)
+        st = torch.cat([steps[q][done[q]:done[q] + ns[q]] for q in range(3)]).to(DEV).contiguous()
+        tiles, off = [], 0
+        for q in range(3):
+            tiles += [[q, off + b, min(segment, ns[q] - b)] for b in range(0, ns[q], segment)]
+            off += ns[q]
+        direct = len(tiles) == 3
+        scratch = None if direct else torch.full((len(tiles) * H * (N * P_ + 1),), float("nan"), device=DEV)
+        y = K.ssd_chunks(cat, x0, b0, c0, None if fixed else st, torch.log(decay).to(DEV) if fixed else None,
+                         None if fixed else D.to(DEV), i32(tiles), len(tiles), direct, i32(slots), state, scratch, H, G, N, P_)
+        y, at = y.cpu().double(), 0
+        for q in range(3):
+            want = refs[q][0][done[q]:done[q] + ns[q]]
+            err = (y[at:at + ns[q]] - want).abs().max() / want.abs().max()
+            assert float(err) < 1e-4, (step, q, float(err))
+            at += ns[q]
+            done[q] += ns[q]
+    for q in range(3):
+        got = state[slots[q]][:H * N * P_].view(H, N, P_).cpu().double()
+        assert float((got - refs[q][1]).abs().max() / refs[q][1].abs().max()) < 1e-4
+    assert torch.isnan(state[1]).all()
