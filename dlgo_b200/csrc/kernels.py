@@ -772,23 +772,24 @@ def ssd_step(proj: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor, dt_bias
 
 
 def ssd_gate_norm(y: torch.Tensor, proj: torch.Tensor, w: torch.Tensor, norm_groups: int, eps: float,
-                  out_dtype: torch.dtype, token_seq: torch.Tensor, seq_slot: torch.Tensor, state: torch.Tensor,
+                  out_dtype: torch.dtype, seqs: torch.Tensor, n_seqs: int, seq_slot: torch.Tensor, state: torch.Tensor,
                   shape: SsdShape) -> torch.Tensor:
     """``rms(y * silu(z)) * w`` with the root mean square taken over each of ``norm_groups`` equal parts of a row (z: the
-    first columns of ``proj``); the token that ends a sequence's part of the step moves the convolution's last inputs
-    into the state row.  Returns [T, heads * v_dim] in ``out_dtype``."""
+    first columns of ``proj``); every sequence of the step (``seqs`` [n_seqs, 3]: sequence, first packed token, count)
+    gets the convolution's last inputs moved into its state row.  Returns [T, heads * v_dim] in ``out_dtype``."""
     _ssd_check("ssd_gate_norm", shape, proj, state)
     _need(w, torch.float32, "w")
     _need(y, torch.float32, "y")
-    _need(token_seq, torch.int32, "token_seq")
+    _need(seqs, torch.int32, "seqs")
     _need(seq_slot, torch.int32, "seq_slot")
     T = proj.shape[0]
-    if tuple(y.shape) != (T, shape.inner) or w.numel() != shape.inner or norm_groups <= 0 or shape.inner % norm_groups:
+    if tuple(y.shape) != (T, shape.inner) or w.numel() != shape.inner or norm_groups <= 0 or shape.inner % norm_groups or \
+            seqs.numel() < 3 * n_seqs:
         raise KernelError("ssd_gate_norm: shapes do not fit")
     out = torch.empty((T, shape.inner), dtype=out_dtype, device=proj.device)
     st = _lib("ssd").dlgo_ssd_gate_norm(_ptr(y), _i(y.stride(0)), _ptr(proj), _i(proj.stride(0)), _ptr(w), _ptr(out),
-                                        _i(dtype_code(out_dtype)), _i(norm_groups), _f(eps), _ptr(token_seq), _i(T),
-                                        _ptr(seq_slot), _ptr(state), _ll(state.stride(0)), *shape.args(), _stream())
+                                        _i(dtype_code(out_dtype)), _i(norm_groups), _f(eps), _ptr(seqs), _i(n_seqs),
+                                        _i(T), _ptr(seq_slot), _ptr(state), _ll(state.stride(0)), *shape.args(), _stream())
     _check(st, "ssd_gate_norm")
     return out
 

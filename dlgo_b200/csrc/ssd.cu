@@ -18,8 +18,8 @@
 //                  FULL    every segment walks its tokens from its start; the last one stores the sequence's new state
 //                with one segment per sequence FULL runs alone from the stored state
 // ssd_step       decoding: convolution, step, state and output of one token per sequence in one launch
-// ssd_gate_norm  gate and norm; the token that ends a sequence's part of the step also moves the convolution's inputs
-//                into the state row (every reader of the old ones ran in an earlier launch)
+// ssd_gate_norm  gate and norm; blocks of the same launch move the convolution's inputs into the state rows (every
+//                reader of the old ones ran in an earlier launch)
 //
 // The state kernels share one layout: a thread holds 16 rows x 4 columns of a head's state in registers.  RS
 // neighbouring lanes share four columns; lane r of them holds rows 4 (i RS + r) .. + 3 for i = 0 .. 3 (so that their
@@ -84,22 +84,28 @@ ssd_conv_kernel(const float* proj, int ld, const float* __restrict__ w_taps, con
 #pragma unroll
   for (int k = 0; k < W; ++k) bias[k] = w_bias[c + k];
   if (TAPS > 0) {
-    constexpr int R = TAPS > 0 ? TAPS : 1;
+    constexpr int R = TAPS > 0 ? TAPS : 1, FLY = 8;
     float tap[R][W], u[R][W];
 #pragma unroll
-    for (int j = 0; j < R; ++j)
+    for (int k = 0; k < W; ++k) {
+      if (R == 4 && W == 4) {                      // (four taps of a channel: 16 bytes)
+        const float4 v = *reinterpret_cast<const float4*>(w_taps + (size_t)(c + k) * 4);
+        tap[0][k] = v.x; tap[1 % R][k] = v.y; tap[2 % R][k] = v.z; tap[3 % R][k] = v.w;
+      } else {
 #pragma unroll
-      for (int k = 0; k < W; ++k) tap[j][k] = w_taps[(size_t)(c + k) * R + j];
+        for (int j = 0; j < R; ++j) tap[j][k] = w_taps[(size_t)(c + k) * R + j];
+      }
+    }
     pdl_wait();
 #pragma unroll
     for (int j = 0; j < R - 1; ++j) {
 #pragma unroll
       for (int k = 0; k < W; ++k) u[j][k] = conv_input(xbc, ld, t0 - R + 1 + j, first, c + k, kept, R, C);
     }
-    for (int tb = 0; tb < count; tb += 4) {
-      float in[4][W];                              // four tokens' fetches in flight
+    for (int tb = 0; tb < count; tb += FLY) {
+      float in[FLY][W];                            // several tokens' fetches in flight
 #pragma unroll
-      for (int q = 0; q < 4; ++q) {
+      for (int q = 0; q < FLY; ++q) {
         const float* src = xbc + (size_t)(t0 + min(tb + q, count - 1)) * ld + c;
         if (W == 4) {
           const float4 v = *reinterpret_cast<const float4*>(src);
@@ -109,7 +115,7 @@ ssd_conv_kernel(const float* proj, int ld, const float* __restrict__ w_taps, con
         }
       }
 #pragma unroll
-      for (int q = 0; q < 4; ++q) {
+      for (int q = 0; q < FLY; ++q) {
         if (tb + q >= count) break;
         float y[W];
 #pragma unroll
@@ -378,7 +384,7 @@ ssd_segments_kernel(const float* xbc, int ld, const float* steps, const float* _
 
 // ------------------------------------------------------------------------------- one token per sequence
 template <int RS>
-__global__ void __launch_bounds__(RS <= 8 ? 128 : 16 * RS)
+__global__ void __launch_bounds__(RS <= 8 ? 128 : 16 * RS, RS <= 8 ? 4 : (RS == 16 ? 2 : 1))
 ssd_step_kernel(const float* proj, int ld, const float* __restrict__ w_taps, const float* __restrict__ w_bias,
                 const float* __restrict__ dt_bias, const float* __restrict__ a_log, const float* __restrict__ D,
                 const int* __restrict__ seq_slot, float* state, long long state_ld, float* out, int ldo, SsdShape s,
@@ -425,24 +431,30 @@ ssd_step_kernel(const float* proj, int ld, const float* __restrict__ w_taps, con
 }
 
 // ------------------------------------------------------------------------------- gate and norm
-// The convolution's inputs that a sequence's next tokens reach back to, moved into the state row by the token t that ends
-// its part of the step; this thread takes channels c0, c0 + stride, ...
-__device__ __forceinline__ void keep_conv_inputs(const float* proj, int ld, int t, int seq, const int* token_seq, float* row,
-                                                 const SsdShape& s, int c0, int stride) {
-  const int keep = s.taps - 1;
-  if (keep == 0) return;
-  const int C = s.channels();
-  int here = 1;                                    // tokens of this step that the new row can take
-  while (here < keep && t - here >= 0 && token_seq[t - here] == seq) ++here;
-  const int old = keep - min(here, keep);          // entries that stay from the old row
-  float* kept = row + s.conv_off();
-  const float* xbc = proj + s.inner();
-  for (int c = c0; c < C; c += stride)
-    for (int j = 0; j < keep; ++j) {
-      // entry j is the input `keep - 1 - j` tokens back; ascending j: an old entry is read before it is overwritten
-      const int back = keep - 1 - j;
-      kept[(size_t)j * C + c] = j >= old ? xbc[(size_t)(t - back) * ld + c] : kept[(size_t)(j + here) * C + c];
+// The convolution's inputs that a sequence's next tokens reach back to, moved into its state row: blocks behind those of
+// the norm, a thread per (sequence, channel).  `seqs` [.., 3]: (sequence, first packed token, count) of the step.
+constexpr int KEEP_REGS = 8;
+__device__ __forceinline__ void keep_conv_inputs(const float* proj, int ld, const int* seqs, const int* seq_slot,
+                                                 float* state, long long state_ld, const SsdShape& s, int block) {
+  const int C = s.channels(), per_seq = (C + blockDim.x - 1) / blockDim.x, keep = s.taps - 1;
+  const int q = block / per_seq, c = (block - q * per_seq) * blockDim.x + threadIdx.x;
+  if (c >= C) return;
+  const int seq = seqs[q * 3], end = seqs[q * 3 + 1] + seqs[q * 3 + 2];
+  const int here = min(seqs[q * 3 + 2], keep);     // tokens of this step that the new row takes
+  float* kept = state + (size_t)seq_slot[seq] * state_ld + s.conv_off() + c;
+  const float* xbc = proj + s.inner() + c;
+  // entry j is the input `keep - j` tokens before the sequence's next one; entries that stay move down by `here`
+  for (int jb = 0; jb < keep; jb += KEEP_REGS) {   // (ascending: an old entry is read before it is overwritten)
+    float v[KEEP_REGS];
+#pragma unroll
+    for (int u = 0; u < KEEP_REGS; ++u) {
+      const int j = jb + u;
+      if (j < keep) v[u] = j >= keep - here ? xbc[(size_t)(end - keep + j) * ld] : kept[(size_t)(j + here) * C];
     }
+#pragma unroll
+    for (int u = 0; u < KEEP_REGS; ++u)
+      if (jb + u < keep) kept[(size_t)(jb + u) * C] = v[u];
+  }
 }
 
 // A warp per (token, part) with the part's gated numbers in registers: parts of up to 128 NV numbers, a multiple of 4.
@@ -450,15 +462,18 @@ constexpr int GN_WARPS = 4;
 template <typename TO, int NV>
 __global__ void __launch_bounds__(GN_WARPS * 32)
 ssd_gate_norm_warp_kernel(const float* y, int ldy, const float* proj, int ld, const float* __restrict__ w, TO* out, int groups,
-                          float eps, const int* __restrict__ token_seq, int T, const int* __restrict__ seq_slot, float* state,
-                          long long state_ld, SsdShape s) {
+                          float eps, const int* __restrict__ seqs, int T, int norm_blocks, const int* __restrict__ seq_slot,
+                          float* state, long long state_ld, SsdShape s) {
   pdl_launch_dependents();
+  if ((int)blockIdx.x >= norm_blocks) {
+    pdl_wait();
+    keep_conv_inputs(proj, ld, seqs, seq_slot, state, state_ld, s, blockIdx.x - norm_blocks);
+    return;
+  }
   const int lane = threadIdx.x & 31, n = s.inner() / groups;
   const long long item = (long long)blockIdx.x * GN_WARPS + (threadIdx.x >> 5);
   if (item >= (long long)T * groups) return;
   const int t = (int)(item / groups), part = (int)(item - (long long)t * groups);
-  const int seq = token_seq[t];
-  const bool ends = t + 1 == T || token_seq[t + 1] != seq;
   float4 wv[NV], u[NV], z[NV];
 #pragma unroll
   for (int v = 0; v < NV; ++v) {
@@ -491,23 +506,23 @@ ssd_gate_norm_warp_kernel(const float* y, int ldy, const float* proj, int ld, co
     if (i < n)
       conv_store4(dst + i, make_float4(u[v].x * sc * wv[v].x, u[v].y * sc * wv[v].y, u[v].z * sc * wv[v].z, u[v].w * sc * wv[v].w));
   }
-  if (ends)
-    keep_conv_inputs(proj, ld, t, seq, token_seq, state + (size_t)seq_slot[seq] * state_ld, s, part * 32 + lane, groups * 32);
 }
 
 // A block per (token, part), parts of any size.  `stash`: the part's gated numbers stay in shared memory between the passes.
 template <typename TO>
 __global__ void __launch_bounds__(512)
 ssd_gate_norm_kernel(const float* y, int ldy, const float* proj, int ld, const float* __restrict__ w, TO* out, int groups,
-                     float eps, const int* __restrict__ token_seq, int T, const int* __restrict__ seq_slot, float* state,
+                     float eps, const int* __restrict__ seqs, int norm_blocks, const int* __restrict__ seq_slot, float* state,
                      long long state_ld, SsdShape s, int stash) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float u_s[];
   __shared__ float red[32];
-  const int t = blockIdx.x, part = blockIdx.y, n = s.inner() / groups;
-  const int seq = token_seq[t];
-  const bool ends = t + 1 == T || token_seq[t + 1] != seq;
   pdl_wait();
+  if ((int)blockIdx.x >= norm_blocks) {
+    keep_conv_inputs(proj, ld, seqs, seq_slot, state, state_ld, s, blockIdx.x - norm_blocks);
+    return;
+  }
+  const int t = blockIdx.x / groups, part = blockIdx.x - t * groups, n = s.inner() / groups;
   const float* yr = y + (size_t)t * ldy + (size_t)part * n;
   const float* zr = proj + (size_t)t * ld + (size_t)part * n;
   float ss = 0.f;
@@ -533,21 +548,21 @@ ssd_gate_norm_kernel(const float* y, int ldy, const float* proj, int ld, const f
     const float u = stash ? u_s[i] : yr[i] * ssd_silu(zr[i]);      // (block_sum's barriers lie between u_s's writes and reads)
     dst[i] = from_float<TO>(u * sc * wp[i]);
   }
-  if (ends)
-    keep_conv_inputs(proj, ld, t, seq, token_seq, state + (size_t)seq_slot[seq] * state_ld, s,
-                     part * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
 }
 
 template <typename TO>
 static int launch_ssd_gate_norm(const float* y, int ldy, const float* proj, int ld, const float* w, TO* out, int groups,
-                                float eps, const int* token_seq, int T, const int* seq_slot, float* state,
+                                float eps, const int* seqs, int n_seqs, int T, const int* seq_slot, float* state,
                                 long long state_ld, const SsdShape& s, cudaStream_t stream) {
   const int n = s.inner() / groups;
+  auto movers = [&](int threads) { return s.taps > 1 ? (long long)n_seqs * ((s.channels() + threads - 1) / threads) : 0; };
   const bool four = n % 4 == 0 && ldy % 4 == 0 && ld % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)proj & 15) == 0 &&
                     ((uintptr_t)w & 15) == 0 && ((uintptr_t)out & 15) == 0;
   if (four && n <= 1024) {
-    const dim3 grid((unsigned)(((long long)T * groups + GN_WARPS - 1) / GN_WARPS)), block(GN_WARPS * 32);
-#define GN_ARGS grid, block, 0, stream, y, ldy, proj, ld, w, out, groups, eps, token_seq, T, seq_slot, state, state_ld, s
+    const long long norm_blocks = ((long long)T * groups + GN_WARPS - 1) / GN_WARPS, all = norm_blocks + movers(GN_WARPS * 32);
+    if (all > 0x7fffffffLL) return DLGO_ERR_SIZE;
+    const dim3 grid((unsigned)all), block(GN_WARPS * 32);
+#define GN_ARGS grid, block, 0, stream, y, ldy, proj, ld, w, out, groups, eps, seqs, T, (int)norm_blocks, seq_slot, state, state_ld, s
     if (n <= 128) launch_kernel(ssd_gate_norm_warp_kernel<TO, 1>, GN_ARGS);
     else if (n <= 256) launch_kernel(ssd_gate_norm_warp_kernel<TO, 2>, GN_ARGS);
     else if (n <= 512) launch_kernel(ssd_gate_norm_warp_kernel<TO, 4>, GN_ARGS);
@@ -557,8 +572,10 @@ static int launch_ssd_gate_norm(const float* y, int ldy, const float* proj, int 
   }
   const int stash = n * sizeof(float) <= 40 * 1024;
   const int threads = n >= 2048 ? 512 : (n >= 512 ? 256 : (n >= 128 ? 128 : 64));
-  launch_kernel(ssd_gate_norm_kernel<TO>, dim3(T, groups), dim3(threads), stash ? n * sizeof(float) : 0, stream, y, ldy, proj,
-                ld, w, out, groups, eps, token_seq, T, seq_slot, state, state_ld, s, stash);
+  const long long norm_blocks = (long long)T * groups, all = norm_blocks + movers(threads);
+  if (all > 0x7fffffffLL) return DLGO_ERR_SIZE;
+  launch_kernel(ssd_gate_norm_kernel<TO>, dim3((unsigned)all), dim3(threads), stash ? n * sizeof(float) : 0, stream, y, ldy,
+                proj, ld, w, out, groups, eps, seqs, (int)norm_blocks, seq_slot, state, state_ld, s, stash);
   return launch_status();
 }
 
@@ -610,7 +627,7 @@ static int launch_ssd_conv(const float* proj, int ld, const float* w_taps, const
                            const SsdShape& s, cudaStream_t stream) {
   const int C = s.channels();
   const bool four = s.taps <= 4 && C % 4 == 0 && s.inner() % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 &&
-                    ((uintptr_t)proj & 15) == 0 && ((uintptr_t)out & 15) == 0;
+                    ((uintptr_t)proj & 15) == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)w_taps & 15) == 0;
   const int w = four ? 4 : 1;
   const dim3 grid(n_tiles, (C + SC_THREADS * w - 1) / (SC_THREADS * w) + 1), block(SC_THREADS);
 #define CONV_ARGS grid, block, 0, stream, proj, ld, w_taps, w_bias, dt_bias, a_log, tiles, token_seq, seq_slot, state, \
@@ -689,14 +706,15 @@ DLGO_EXPORT int dlgo_ssd_step(const float* proj, int ld, const float* w_taps, co
   return launch_status();
 }
 
-// y [T, ldy] fp32, proj as above (its z columns gate), w [H P] fp32, out [T, H P] in `dtype`; `groups` divides H P
+// y [T, ldy] fp32, proj as above (its z columns gate), w [H P] fp32, out [T, H P] in `dtype`; `groups` divides H P;
+// seqs [n_seqs, 3] (sequence, first packed token, count): every sequence of the step
 DLGO_EXPORT int dlgo_ssd_gate_norm(const float* y, int ldy, const float* proj, int ld, const float* w, void* out, int dtype,
-                                   int groups, float eps, const int* token_seq, int T, const int* seq_slot, float* state,
-                                   long long state_ld, int H, int G, int N, int P, int taps, cudaStream_t stream) {
+                                   int groups, float eps, const int* seqs, int n_seqs, int T, const int* seq_slot,
+                                   float* state, long long state_ld, int H, int G, int N, int P, int taps, cudaStream_t stream) {
   if (T <= 0) return DLGO_OK;
   const SsdShape s{H, G, N, P, taps};
   if (!ssd_shape_ok(s) || groups <= 0 || s.inner() % groups || groups > 65535) return DLGO_ERR_SIZE;
-#define GN_ARGS(T_) y, ldy, proj, ld, w, (T_*)out, groups, eps, token_seq, T, seq_slot, state, state_ld, s, stream
+#define GN_ARGS(T_) y, ldy, proj, ld, w, (T_*)out, groups, eps, seqs, n_seqs, T, seq_slot, state, state_ld, s, stream
   if (dtype == DLGO_F32) return launch_ssd_gate_norm<float>(GN_ARGS(float));
   if (dtype == DLGO_BF16) return launch_ssd_gate_norm<__nv_bfloat16>(GN_ARGS(__nv_bfloat16));
 #undef GN_ARGS

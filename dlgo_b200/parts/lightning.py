@@ -24,7 +24,7 @@ from ..csrc import kernels as K
 from .base import Mixer, ParamSpec, PositionEncoding, StateNeed
 from .linear import ADD_F32, STORE_F32, Linear, stack_rows
 from .registry import MIXERS
-from .state_space import TC_MIN_TOKENS, TC_SEGMENT
+from .state_space import TC_MIN_TOKENS, tc_segment
 
 _NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "gate": "g_proj.weight",
           "out": "o_proj.weight", "norm": "norm.weight"}
@@ -79,7 +79,7 @@ class LightningAttention(Mixer):
         """(outputs [T, H dv] fp32, gate logits) of a prompt step, the recurrence's products on the tensor cores."""
         H, dk, dv = self.n_heads, self.qk_dim, self.v_dim
         qkv = self.w_qkv.bias_act(x, None, K.ACT_SILU)
-        tiles, n_tiles, _ = ctx.tiles(TC_SEGMENT)
+        tiles, n_tiles, _ = ctx.tiles(tc_segment(ctx.n_tokens, H, dv))
         direct = n_tiles == ctx.n_seqs
         scratch = None if direct else ctx.scratch("lightning_segments", n_tiles * H * (dk * dv + 1))
         o = K.ssd_chunks(qkv, 2 * H * dk, H * dk, 0, None, self.log_decay, None, tiles, n_tiles, direct, ctx.seq_slot,

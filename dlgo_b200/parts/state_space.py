@@ -29,9 +29,19 @@ from .registry import MIXERS
 _NAMES = {"in": "in_proj.weight", "conv": "conv.weight", "conv_bias": "conv.bias", "dt_bias": "dt_bias", "decay": "A_log",
           "skip": "D", "norm": "norm.weight", "out": "out_proj.weight"}
 SEGMENT = int(os.environ.get("DLGO_SSD_SEGMENT", 128))   # tokens of a segment where a prompt's segments run side by side
-TC_SEGMENT = int(os.environ.get("DLGO_SSD_TC_SEGMENT", 256))   # ... on the tensor cores (a multiple of 64)
+TC_SEGMENT = int(os.environ.get("DLGO_SSD_TC_SEGMENT", 0))   # ... on the tensor cores (0: see tc_segment)
+TC_BLOCKS = 400                                          # blocks the tensor-core recurrence is cut into (a few per SM)
 TC_MIN_TOKENS = int(os.environ.get("DLGO_SSD_TC_MIN_TOKENS", 64))   # prompt steps that run there (0: never)
 CONV_TILE = 16                                           # tokens of a block of the convolution
+_WHOLE_SEQUENCE = 1 << 30
+
+
+def tc_segment(tokens: int, heads: int, v_dim: int) -> int:
+    """Tokens of a segment on the tensor cores: as long as still makes enough blocks for the GPU, whole chunks of 64."""
+    if TC_SEGMENT > 0:
+        return TC_SEGMENT
+    want = tokens * heads * -(-v_dim // 64) // TC_BLOCKS
+    return min(1024, max(64, want // 64 * 64))
 
 
 class StateSpaceMixer(Mixer):
@@ -92,7 +102,7 @@ class StateSpaceMixer(Mixer):
             xbc, steps = K.ssd_conv(proj, self.taps, self.conv_bias, self.dt_bias, self.a_log, tiles, n_tiles,
                                     ctx.token_seq, ctx.seq_slot, state, s,
                                     out_dtype=torch.bfloat16 if on_tc else torch.float32, log_decay=on_tc)
-            tiles, n_tiles, _ = ctx.tiles(TC_SEGMENT if on_tc else SEGMENT)
+            tiles, n_tiles, _ = ctx.tiles(tc_segment(ctx.n_tokens, s.heads, s.v_dim) if on_tc else SEGMENT)
             direct = n_tiles == ctx.n_seqs
             scratch = None if direct else ctx.scratch("ssd_segments", K.ssd_scratch_floats(n_tiles, s))
             if on_tc:
@@ -101,7 +111,8 @@ class StateSpaceMixer(Mixer):
                                  state, scratch, s.heads, s.groups, s.state, s.v_dim)
             else:
                 y = K.ssd_segments(xbc, steps, self.skip, tiles, n_tiles, direct, ctx.seq_slot, state, scratch, s)
-        a = K.ssd_gate_norm(y, proj, self.norm, self.norm_groups, self.eps, self.wo.weight.dtype, ctx.token_seq,
+        seqs, n_seqs, _ = ctx.tiles(1 if ctx.decode else _WHOLE_SEQUENCE)
+        a = K.ssd_gate_norm(y, proj, self.norm, self.norm_groups, self.eps, self.wo.weight.dtype, seqs, n_seqs,
                             ctx.seq_slot, state, s)
         self.wo(a, ADD_F32, residual)
 

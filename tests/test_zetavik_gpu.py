@@ -134,7 +134,8 @@ def test_state_space_kernels(H, G, N, P_, taps, segment):
             direct = n == 2
             scratch = None if direct else torch.full((K.ssd_scratch_floats(n, s),), float("nan"), device=DEV)
             y = K.ssd_segments(xbc, steps, dev[4], tl, n, direct, i32(slots), state, scratch, s)
-        a = K.ssd_gate_norm(y, rows, dev[5], groups, eps, torch.float32, seq, i32(slots), state, s).cpu().double()
+        a = K.ssd_gate_norm(y, rows, dev[5], groups, eps, torch.float32, i32([[0, 0, ns[0]], [1, ns[0], ns[1]]]), 2, i32(slots),
+                            state, s).cpu().double()
         y = y.cpu().double()
         at = 0
         for q in range(2):
@@ -161,7 +162,8 @@ def test_gate_then_group_norm(n, groups, act_dtype):
     s = K.SsdShape(1, 1, 4, n, 1)
     y, proj, w = torch.randn(7, n, generator=g), torch.randn(7, s.columns, generator=g), 1 + 0.3 * torch.randn(n, generator=g)
     state = torch.zeros(2, s.state_floats(), device=DEV)
-    got = K.ssd_gate_norm(y.to(DEV), proj.to(DEV), w.to(DEV), groups, 0.03, act_dtype, i32([0] * 4 + [1] * 3), i32([1, 0]), state, s)
+    got = K.ssd_gate_norm(y.to(DEV), proj.to(DEV), w.to(DEV), groups, 0.03, act_dtype, i32([[0, 0, 4], [1, 4, 3]]), 2,
+                          i32([1, 0]), state, s)
     want = P.gate_then_group_norm(y.double(), proj[:, :n].double(), w.double(), groups, 0.03)
     tol = 1e-2 if act_dtype == torch.bfloat16 else 1e-5
     assert torch.allclose(got.cpu().double(), want, rtol=tol, atol=tol) and not state.any()
