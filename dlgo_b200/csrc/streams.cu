@@ -228,6 +228,51 @@ __global__ void gated_rmsnorm_kernel(const float* o, int ldo, const float* g, in
     out[(size_t)t * n + i] = from_float<TO>(orow[i] * sc * (w != nullptr ? w[i] : 1.0f) * gate_of(grow[i], gate_act));
 }
 
+// The same for rows of a multiple of four numbers that a block holds in registers (16-byte accesses, one pass).
+template <typename TO, int THREADS, int NV>
+__global__ void __launch_bounds__(THREADS)
+gated_rmsnorm_vec_kernel(const float* o, int ldo, const float* g, int ldg, const float* __restrict__ w, TO* out, int n,
+                         float eps, int gate_act, float c) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  float4 wv[NV], u[NV], z[NV];
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (v * THREADS + threadIdx.x) * 4;
+    wv[v] = (w != nullptr && i < n) ? *reinterpret_cast<const float4*>(w + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+  }
+  pdl_wait();
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (v * THREADS + threadIdx.x) * 4;
+    u[v] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < n) {
+      u[v] = *reinterpret_cast<const float4*>(o + (size_t)t * ldo + i);
+      z[v] = *reinterpret_cast<const float4*>(g + (size_t)t * ldg + i);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < NV; ++v) ss += (u[v].x * u[v].x + u[v].y * u[v].y) + (u[v].z * u[v].z + u[v].w * u[v].w);
+  const float sc = c / sqrtf(block_sum(ss, red) / (float)n + eps);
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (v * THREADS + threadIdx.x) * 4;
+    if (i < n) {
+      TO* dst = out + (size_t)t * n + i;
+      const float r[4] = {u[v].x * sc * wv[v].x * gate_of(z[v].x, gate_act), u[v].y * sc * wv[v].y * gate_of(z[v].y, gate_act),
+                          u[v].z * sc * wv[v].z * gate_of(z[v].z, gate_act), u[v].w * sc * wv[v].w * gate_of(z[v].w, gate_act)};
+      if (sizeof(TO) == 4) {
+        *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
+      } else {
+        __nv_bfloat162 h[2] = {__floats2bfloat162_rn(r[0], r[1]), __floats2bfloat162_rn(r[2], r[3])};
+        *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<uint2*>(h);
+      }
+    }
+  }
+}
+
 // The same with the mean taken over each group of `group` neighbours (a head) on its own: a warp per (token, group).
 constexpr int GG_WARPS = 4;
 template <typename TO>
@@ -310,6 +355,21 @@ DLGO_EXPORT int dlgo_gated_rmsnorm(const float* o, int ldo, const float* g, int 
     else
       launch_kernel(gated_groupnorm_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(GG_WARPS * 32), 0, stream, o, ldo,
                     g, ldg, w, (__nv_bfloat16*)out, T, n, group, eps, gate_act, c);
+    return launch_status();
+  }
+  if (n % 4 == 0 && n <= 4096 && ldo % 4 == 0 && ldg % 4 == 0 && ((uintptr_t)o & 15) == 0 && ((uintptr_t)g & 15) == 0 &&
+      ((uintptr_t)w & 15) == 0 && ((uintptr_t)out & 15) == 0) {
+#define GR_ARGS(TO) dim3(T), block, 0, stream, o, ldo, g, ldg, w, (TO*)out, n, eps, gate_act, c
+    if (n <= 1024) {
+      const dim3 block(128);
+      if (out_dtype == DLGO_F32) launch_kernel(gated_rmsnorm_vec_kernel<float, 128, 2>, GR_ARGS(float));
+      else launch_kernel(gated_rmsnorm_vec_kernel<__nv_bfloat16, 128, 2>, GR_ARGS(__nv_bfloat16));
+    } else {
+      const dim3 block(256);
+      if (out_dtype == DLGO_F32) launch_kernel(gated_rmsnorm_vec_kernel<float, 256, 4>, GR_ARGS(float));
+      else launch_kernel(gated_rmsnorm_vec_kernel<__nv_bfloat16, 256, 4>, GR_ARGS(__nv_bfloat16));
+    }
+#undef GR_ARGS
     return launch_status();
   }
   const int threads = n >= 2048 ? 512 : (n >= 512 ? 256 : 128);

@@ -69,29 +69,29 @@ class LightningAttention(Mixer):
         self.decay = torch.tensor(self.decay_values, dtype=torch.float64).to(torch.float32).to(runtime.device)
         # prompts on the tensor cores: q | k | v and the gate as contractions of their own over the same rows
         H, n_qkv = self.n_heads, self.n_heads * (2 * self.qk_dim + self.v_dim)
-        self.w_qkv = self.w_gate = self.log_decay = None
+        self.prompt_views = self.log_decay = None
         if min(self.decay_values) > 0 and n_qkv % 8 == 0 and K.ssd_chunks_takes(runtime.dtype, self.qk_dim, self.v_dim):
-            self.w_qkv = Linear(self.w_in.weight[:n_qkv], runtime)
-            self.w_gate = Linear(self.w_in.weight[n_qkv:], runtime)
+            self.prompt_views = (Linear(self.w_in.weight[:n_qkv], runtime), Linear(self.w_in.weight[n_qkv:], runtime))
             self.log_decay = torch.log(torch.tensor(self.decay_values, dtype=torch.float64)).to(torch.float32).to(runtime.device)
 
     def _prompt_tc(self, x: torch.Tensor, ctx: Any, state: torch.Tensor) -> tuple:
         """(outputs [T, H dv] fp32, gate logits) of a prompt step, the recurrence's products on the tensor cores."""
         H, dk, dv = self.n_heads, self.qk_dim, self.v_dim
-        qkv = self.w_qkv.bias_act(x, None, K.ACT_SILU)
+        w_qkv, w_gate = self.prompt_views
+        qkv = w_qkv.bias_act(x, None, K.ACT_SILU)
         tiles, n_tiles, _ = ctx.tiles(tc_segment(ctx.n_tokens, H, dv))
         direct = n_tiles == ctx.n_seqs
         scratch = None if direct else ctx.scratch("lightning_segments", n_tiles * H * (dk * dv + 1))
         o = K.ssd_chunks(qkv, 2 * H * dk, H * dk, 0, None, self.log_decay, None, tiles, n_tiles, direct, ctx.seq_slot,
                          state.view(state.shape[0], -1), scratch, H, H, dk, dv)
-        return o, self.w_gate(x, STORE_F32)
+        return o, w_gate(x, STORE_F32)
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: Any, cache: Any,
                 state: Optional[torch.Tensor], positions: Mapping[str, PositionEncoding]) -> None:
         if state is None:
             raise RuntimeError("lightning attention needs its state")
         H, dk, dv = self.n_heads, self.qk_dim, self.v_dim
-        if self.w_qkv is not None and not ctx.decode and 0 < TC_MIN_TOKENS <= ctx.n_tokens:
+        if self.prompt_views is not None and not ctx.decode and 0 < TC_MIN_TOKENS <= ctx.n_tokens:
             o, gate = self._prompt_tc(x, ctx, state)
             a = K.gated_rmsnorm(o, gate, self.norm, self.eps, self.wo.weight.dtype)
             self.wo(a, ADD_F32, residual)

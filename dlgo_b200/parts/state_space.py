@@ -30,18 +30,19 @@ _NAMES = {"in": "in_proj.weight", "conv": "conv.weight", "conv_bias": "conv.bias
           "skip": "D", "norm": "norm.weight", "out": "out_proj.weight"}
 SEGMENT = int(os.environ.get("DLGO_SSD_SEGMENT", 128))   # tokens of a segment where a prompt's segments run side by side
 TC_SEGMENT = int(os.environ.get("DLGO_SSD_TC_SEGMENT", 0))   # ... on the tensor cores (0: see tc_segment)
-TC_BLOCKS = 400                                          # blocks the tensor-core recurrence is cut into (a few per SM)
+TC_BLOCKS = 444                                          # blocks of the tensor-core recurrence on the GPU at once: three per SM
 TC_MIN_TOKENS = int(os.environ.get("DLGO_SSD_TC_MIN_TOKENS", 64))   # prompt steps that run there (0: never)
 CONV_TILE = 16                                           # tokens of a block of the convolution
 _WHOLE_SEQUENCE = 1 << 30
 
 
 def tc_segment(tokens: int, heads: int, v_dim: int) -> int:
-    """Tokens of a segment on the tensor cores: as long as still makes enough blocks for the GPU, whole chunks of 64."""
+    """Tokens of a segment on the tensor cores: whole chunks of 64, as many segments as run at the same time (one more
+    would be a second wave of blocks)."""
     if TC_SEGMENT > 0:
         return TC_SEGMENT
-    want = tokens * heads * -(-v_dim // 64) // TC_BLOCKS
-    return min(1024, max(64, want // 64 * 64))
+    segments = max(1, TC_BLOCKS // (heads * -(-v_dim // 64)))
+    return -(-tokens // (64 * segments)) * 64
 
 
 class StateSpaceMixer(Mixer):
