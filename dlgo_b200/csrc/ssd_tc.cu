@@ -22,7 +22,7 @@ namespace dlgo {
 constexpr int TC_TOKENS = 64, TC_COLS = 64, TC_PAD = 8;      // tokens of a chunk, columns of a block, elements between rows
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
-  asm volatile(
+  asm(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
@@ -79,7 +79,7 @@ template <int NT> struct SsdChunk {
 };
 
 template <int NT, int MODE>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, NT <= 4 ? 4 : 3)
 ssd_chunks_kernel(SsdChunkArgs a) {
   using SC = SsdChunk<NT>;
   constexpr int LDN = SC::LDN, LDX = SC::LDX, LDM = SC::LDM;
@@ -188,14 +188,18 @@ ssd_chunks_kernel(SsdChunkArgs a) {
         const int i0 = mt * 16 + r;
         const float li0 = ls[i0], li1 = ls[i0 + 8];
         for (int jt = 0; jt <= mt; ++jt) {
-          float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+          float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}}, odd[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
-          for (int kt = 0; kt < NT; ++kt) {
+          for (int kt = 0; kt < NT; ++kt) {        // (sums over even and odd steps: four chains of products in flight)
             unsigned bb[4];
             ldsm4(bb, Bs + (jt * 16 + nrow) * LDN + kt * 16 + ncol);
-            mma_bf16(acc[0], ca[kt], bb[0], bb[1]);
-            mma_bf16(acc[1], ca[kt], bb[2], bb[3]);
+            mma_bf16(kt & 1 ? odd[0] : acc[0], ca[kt], bb[0], bb[1]);
+            mma_bf16(kt & 1 ? odd[1] : acc[1], ca[kt], bb[2], bb[3]);
           }
+#pragma unroll
+          for (int q = 0; q < 2; ++q)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) acc[q][k] += odd[q][k];
 #pragma unroll
           for (int q = 0; q < 2; ++q) {
             const int j = jt * 16 + q * 8 + c2;
@@ -230,17 +234,17 @@ ssd_chunks_kernel(SsdChunkArgs a) {
         for (int q = 0; q < 2; ++q)
 #pragma unroll
           for (int k = 0; k < 2; ++k) split2(S[2 * kt + k][2 * q], S[2 * kt + k][2 * q + 1], sh[q][k], sl[q][k]);
+        unsigned ca[4][4];                                         // (rows beyond the chunk's tokens are zeros)
 #pragma unroll
-        for (int mt = 0; mt < 4; ++mt) {
-          if (mt * 16 >= nt) break;
-          unsigned ca[4];
-          ldsm4(ca, Cs + (mt * 16 + mrow) * LDN + kt * 16 + mcol);
+        for (int mt = 0; mt < 4; ++mt) ldsm4(ca[mt], Cs + (mt * 16 + mrow) * LDN + kt * 16 + mcol);
 #pragma unroll
-          for (int q = 0; q < 2; ++q) {
-            mma_bf16(y[mt][q], ca, sh[q][0], sh[q][1]);
-            mma_bf16(y[mt][q], ca, sl[q][0], sl[q][1]);
-          }
-        }
+        for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+          for (int q = 0; q < 2; ++q) mma_bf16(y[mt][q], ca[mt], sh[q][0], sh[q][1]);
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+          for (int q = 0; q < 2; ++q) mma_bf16(y[mt][q], ca[mt], sl[q][0], sl[q][1]);
       }
 #pragma unroll
       for (int mt = 0; mt < 4; ++mt) {
@@ -258,16 +262,15 @@ ssd_chunks_kernel(SsdChunkArgs a) {
         unsigned xb[4];                                            // columns 0-7: rows 0-7, 8-15; columns 8-15: the same
         ldsm4_t(xb, Xs + (kt * 16 + mrow) * LDX + warp * 16 + mcol);
 #pragma unroll
-        for (int mt = kt; mt < 4; ++mt) {
-          if (mt * 16 >= nt) break;
-          unsigned m[4];
-          ldsm4(m, Mh + (mt * 16 + mrow) * LDM + kt * 16 + mcol);
-          mma_bf16(y[mt][0], m, xb[0], xb[1]);
-          mma_bf16(y[mt][1], m, xb[2], xb[3]);
-          ldsm4(m, Ml + (mt * 16 + mrow) * LDM + kt * 16 + mcol);
-          mma_bf16(y[mt][0], m, xb[0], xb[1]);
-          mma_bf16(y[mt][1], m, xb[2], xb[3]);
-        }
+        for (int term = 0; term < 2; ++term)
+#pragma unroll
+          for (int mt = kt; mt < 4; ++mt) {
+            if (mt * 16 >= nt) break;
+            unsigned m[4];
+            ldsm4(m, (term ? Ml : Mh) + (mt * 16 + mrow) * LDM + kt * 16 + mcol);
+            mma_bf16(y[mt][0], m, xb[0], xb[1]);
+            mma_bf16(y[mt][1], m, xb[2], xb[3]);
+          }
       }
 #pragma unroll
       for (int mt = 0; mt < 4; ++mt)
@@ -305,14 +308,22 @@ ssd_chunks_kernel(SsdChunkArgs a) {
         const float2 w = q < 2 ? w0 : w1;
         split2(v.x * w.x, v.y * w.y, xh[q], xl[q]);
       }
+      constexpr int TB = NT < 4 ? NT : 4;                          // tiles of B in flight
 #pragma unroll
-      for (int t = 0; t < NT; ++t) {
-        unsigned bb[4];                                            // rows (tokens) 0-7, 8-15 of columns 0-7, then of 8-15
-        ldsm4_t(bb, Bs + (kt * 16 + mrow) * LDN + t * 16 + mcol);
-        mma_bf16(S[2 * t], xh, bb[0], bb[1]);
-        mma_bf16(S[2 * t + 1], xh, bb[2], bb[3]);
-        mma_bf16(S[2 * t], xl, bb[0], bb[1]);
-        mma_bf16(S[2 * t + 1], xl, bb[2], bb[3]);
+      for (int tb = 0; tb < NT; tb += TB) {
+        unsigned bb[TB][4];                                        // rows (tokens) 0-7, 8-15 of columns 0-7, then of 8-15
+#pragma unroll
+        for (int t = 0; t < TB; ++t) ldsm4_t(bb[t], Bs + (kt * 16 + mrow) * LDN + (tb + t) * 16 + mcol);
+#pragma unroll
+        for (int t = 0; t < TB; ++t) {
+          mma_bf16(S[2 * (tb + t)], xh, bb[t][0], bb[t][1]);
+          mma_bf16(S[2 * (tb + t) + 1], xh, bb[t][2], bb[t][3]);
+        }
+#pragma unroll
+        for (int t = 0; t < TB; ++t) {
+          mma_bf16(S[2 * (tb + t)], xl, bb[t][0], bb[t][1]);
+          mma_bf16(S[2 * (tb + t) + 1], xl, bb[t][2], bb[t][3]);
+        }
       }
     }
   }
