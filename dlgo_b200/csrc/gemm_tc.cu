@@ -104,7 +104,7 @@ __device__ __forceinline__ float silu_mul(float g, float u) {
 
 template <int ACT> __device__ __forceinline__ float act_value(float z) {
   if (ACT == TC_ACT_RELU2) { const float r = fmaxf(z, 0.f); return r * r; }
-  if (ACT == TC_ACT_SILU) return z / (1.0f + __expf(-z));
+  if (ACT == TC_ACT_SILU) return silu_mul(z, 1.0f);      // (results here are rounded to bfloat16 too)
   if (ACT == TC_ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
   return z;
 }
