@@ -8,8 +8,9 @@ from .monolix import MonolixConfig
 from .bazurax import BazuraxConfig
 from .ragilorn import RagilornConfig
 from .zetavik import ZetavikConfig
+from .bonusun import BonusunConfig
 
 __all__ = [
-    "ArchitectureSpec", "BazuraxConfig", "ConfigError", "DedutarConfig", "LayerSpec", "LlamaConfig", "MonolixConfig", "PartSpec", "RagilornConfig", "RopeScaling", "RunEntry", "ZetavikConfig",
+    "ArchitectureSpec", "BazuraxConfig", "BonusunConfig", "ConfigError", "DedutarConfig", "LayerSpec", "LlamaConfig", "MonolixConfig", "PartSpec", "RagilornConfig", "RopeScaling", "RunEntry", "ZetavikConfig",
     "config_class_for", "config_from_dict", "load_config", "register_architecture", "registered_architectures",
 ]

@@ -41,6 +41,7 @@ struct AttnParams {
   float* part_ml;   // [T, Hq, n_splits, 2]
   int Hq, Hkv, hd, page_size, n_splits, gchunk, n_gchunks, rows_max, window;
   float scale;
+  const float* sink;  // [Hq] fp32 or null: see join_sink
 };
 
 template <typename T> struct Vec;
@@ -201,7 +202,9 @@ __global__ void __launch_bounds__(ATT_THREADS) attention_kernel(AttnParams p) {
       const int head = kvh * G + g0 + g;
       const size_t token = tok0 + tq;
       if (p.n_splits == 1) {
-        ((T*)p.out)[token * p.ldo + (size_t)head * hd + d] = from_float<T>(acc[i] / l_s[r]);
+        float a = acc[i], l = l_s[r];
+        join_sink(a, l, m_s[r], p.sink, head);
+        ((T*)p.out)[token * p.ldo + (size_t)head * hd + d] = from_float<T>(a / l);
       } else {
         const size_t o = (token * p.Hq + head) * p.n_splits + split;
         p.part_acc[o * hd + d] = acc[i];
@@ -231,7 +234,7 @@ int launch_attention(const AttnParams& p, int n_tiles, int T_tokens, cudaStream_
   dim3 cgrid(T_tokens, p.Hq);
   const int threads = p.hd >= 128 ? 128 : (p.hd >= 64 ? 64 : 32);
   launch_kernel(attention_combine_kernel<T>, dim3(cgrid), dim3(threads), 0, stream, p.part_acc, p.part_ml, (T*)p.out, p.ldo, p.Hq, p.hd,
-                                                             p.n_splits);
+                                                             p.n_splits, p.sink);
   return launch_status();
 }
 
@@ -248,12 +251,12 @@ DLGO_EXPORT long long dlgo_attention_scratch_floats(int T, int Hq, int hd, int n
 
 // q[T, .] with row stride ldq (head h at column h*hd); pages [n_pages, Hkv, page_size, hd];
 // tiles[n_tiles][3]; rows_max = (largest token count of a tile) * gchunk;
-// out[T, Hq*hd] with row stride ldo.  `scratch` as sized above.
+// out[T, Hq*hd] with row stride ldo.  `scratch` as sized above.  `sink` [Hq] fp32 or null: joins the denominator.
 DLGO_EXPORT int dlgo_attention(const void* q, int dtype, int T, int ldq, const void* kpages, const void* vpages,
                                const int* page_table, int max_pages, const int* tiles, int n_tiles,
                                int tile_tokens_max, const int* seq_slot, const int* token_pos, void* out, int ldo,
                                float* scratch, int Hq, int Hkv, int hd, int page_size, int n_splits, int gchunk,
-                               int window, float scale, cudaStream_t stream) {
+                               int window, float scale, const float* sink, cudaStream_t stream) {
   if (T <= 0 || n_tiles <= 0) return DLGO_OK;
   if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || hd <= 0 || page_size <= 0 || page_size % 32 || n_splits <= 0 ||
       gchunk <= 0 || tile_tokens_max <= 0)
@@ -269,7 +272,7 @@ DLGO_EXPORT int dlgo_attention(const void* q, int dtype, int T, int ldq, const v
   p.Hq = Hq; p.Hkv = Hkv; p.hd = hd; p.page_size = page_size; p.n_splits = n_splits; p.gchunk = gchunk;
   p.n_gchunks = (G + gchunk - 1) / gchunk;
   p.rows_max = tile_tokens_max * gchunk;
-  p.window = window; p.scale = scale;
+  p.window = window; p.scale = scale; p.sink = sink;
   if ((long long)p.rows_max * hd > (long long)ATT_THREADS * ATT_MAX_ACC) return DLGO_ERR_SIZE;
   if (n_splits > 1 && scratch == nullptr) return DLGO_ERR_SIZE;
   if ((long long)Hkv * p.n_gchunks > 65535 || n_splits > 65535) return DLGO_ERR_SIZE;
@@ -328,5 +331,5 @@ DLGO_EXPORT int dlgo_attention_noalloc(const void* q, int dtype, int T, int ldq,
   }
   return dlgo_attention(q, dtype, T, ldq, kpages, vpages, page_table, max_pages, tiles, n_tiles, tile_tokens_max,
                         seq_slot, token_pos, out, ldo, scratch, Hq, Hkv, hd, page_size, n_splits, gchunk, window,
-                        scale, stream);
+                        scale, nullptr, stream);
 }

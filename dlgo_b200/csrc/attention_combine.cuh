@@ -6,10 +6,21 @@
 
 namespace dlgo {
 
-// out[token, head, :] = sum_s w_s acc_s / sum_s w_s l_s with w_s = exp(m_s - max m)
+// A sink is a number per head whose exponential joins the softmax's denominator once; it has no key and no value.
+// (a, l): a weighted sum and its denominator, both relative to the maximum m; afterwards relative to the larger of
+// m and the sink, with the sink in l.  `sink` null: no sink.
+__device__ __forceinline__ void join_sink(float& a, float& l, float m, const float* __restrict__ sink, int head) {
+  if (sink == nullptr) return;
+  const float s = sink[head], top = fmaxf(m, s), c = expf(m - top);
+  a *= c;
+  l = fmaf(l, c, expf(s - top));
+}
+
+// out[token, head, :] = sum_s w_s acc_s / (sum_s w_s l_s + the sink's share) with w_s = exp(m_s - max m)
 template <typename T>
 __global__ void attention_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
-                                         T* __restrict__ out, int ldo, int Hq, int hd, int n_splits) {
+                                         T* __restrict__ out, int ldo, int Hq, int hd, int n_splits,
+                                         const float* __restrict__ sink) {
   pdl_launch_dependents();
   pdl_wait();
   const int token = blockIdx.x, head = blockIdx.y;
@@ -27,7 +38,9 @@ __global__ void attention_combine_kernel(const float* __restrict__ part_acc, con
       const float ms = part_ml[(o + s) * 2];
       if (ms != -INFINITY) a = fmaf(expf(ms - m), part_acc[(o + s) * hd + d], a);
     }
-    out[(size_t)token * ldo + (size_t)head * hd + d] = from_float<T>(a / denom);
+    float l = denom;
+    join_sink(a, l, m, sink, head);
+    out[(size_t)token * ldo + (size_t)head * hd + d] = from_float<T>(a / l);
   }
 }
 

@@ -42,6 +42,7 @@ struct DecParams {
   int cluster;           // 1: the slices of a (sequence, kv head) form one thread-block cluster and combine
                          // through distributed shared memory; no scratch, no counters
   float scale;
+  const float* sink;     // [Hq] fp32 or null: see join_sink
 };
 
 template <typename T> struct Ld16;
@@ -292,6 +293,7 @@ __global__ void __launch_bounds__(DEC_THREADS, 4) attention_decode_kernel(DecPar
     }
     const int head = kvh * G + g0 + g;
     if (p.n_splits == 1) {
+      join_sink(a, ll, mm, p.sink, head);
       ((T*)p.out)[(size_t)b * p.ldo + (size_t)head * HD + d] = from_float<T>(a / ll);
     } else if (p.cluster) {
       cl_acc[g][d] = a;
@@ -346,6 +348,7 @@ __global__ void __launch_bounds__(DEC_THREADS, 4) attention_decode_kernel(DecPar
           a = fmaf(c, as[r], a);
           ll = fmaf(c, ls[r], ll);
         }
+        join_sink(a, ll, mm, p.sink, kvh * G + g0 + g);
         ((T*)p.out)[(size_t)b * p.ldo + (size_t)(kvh * G + g0 + g) * HD + d] = from_float<T>(a / ll);
       }
     }
@@ -394,7 +397,9 @@ __global__ void __launch_bounds__(DEC_THREADS, 4) attention_decode_kernel(DecPar
         w_s[g * NS + sp] = c;
         ll = fmaf(c, l_sm[g * NS + sp], ll);
       }
-      w_s[GC * NS + g] = 1.0f / ll;
+      float one = 1.0f;
+      join_sink(one, ll, mm, p.sink, kvh * G + g0 + g);
+      w_s[GC * NS + g] = one / ll;
     }
     __syncthreads();
   }
@@ -424,7 +429,9 @@ __global__ void __launch_bounds__(DEC_THREADS, 4) attention_decode_kernel(DecPar
         a = fmaf(c, __ldcg(&p.part_acc[(o + sp) * HD + d]), a);
         ll = fmaf(c, __ldcg(&p.part_ml[(o + sp) * 2 + 1]), ll);
       }
-      inv = 1.0f / ll;
+      float one = 1.0f;
+      join_sink(one, ll, mm, p.sink, head);
+      inv = one / ll;
     }
     ((T*)p.out)[(size_t)b * p.ldo + (size_t)head * HD + d] = from_float<T>(a * inv);
   }
@@ -444,7 +451,7 @@ int launch_decode(const DecParams& p, int B, cudaStream_t stream) {
   dim3 cgrid(B, p.Hq);
   const int threads = HD >= 128 ? 128 : (HD >= 64 ? 64 : 32);
   launch_kernel(attention_combine_kernel<T>, dim3(cgrid), dim3(threads), 0, stream, p.part_acc, p.part_ml, (T*)p.out, p.ldo, p.Hq, HD,
-                                                             p.n_splits);
+                                                             p.n_splits, p.sink);
   return launch_status();
 }
 
@@ -490,7 +497,7 @@ DLGO_EXPORT int dlgo_attention_decode(const void* q, int dtype, int B, int ldq, 
                                       const void* vpages, const int* page_table, int max_pages,
                                       const int* seq_slot, const int* token_pos, void* out, int ldo, float* scratch,
                                       int* counters, int Hq, int Hkv, int hd, int page_size, int n_splits,
-                                      int window, float scale, cudaStream_t stream) {
+                                      int window, float scale, const float* sink, cudaStream_t stream) {
   if (B <= 0) return DLGO_OK;
   if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || n_splits <= 0 || n_splits > 65535) return DLGO_ERR_SIZE;
   if (dtype != DLGO_F32 && dtype != DLGO_BF16) return DLGO_ERR_DTYPE;
@@ -507,7 +514,7 @@ DLGO_EXPORT int dlgo_attention_decode(const void* q, int dtype, int B, int ldq, 
   p.counters = counters;
   p.Hq = Hq; p.Hkv = Hkv; p.page_size = page_size; p.n_splits = n_splits;
   p.n_gchunks = (G + DEC_GMAX - 1) / DEC_GMAX;
-  p.window = window; p.scale = scale;
+  p.window = window; p.scale = scale; p.sink = sink;
   if ((long long)Hkv * p.n_gchunks > 65535) return DLGO_ERR_SIZE;
   return decode_common(p, dtype, B, hd, stream);
 }

@@ -61,12 +61,13 @@ struct DecMmaParams {
                          // cluster's first block) clears this (sequence, kv head)'s columns once all have read them
   float* part_acc;       // more than 8 slices: [B, Hq, n_splits, HD] and [B, Hq, n_splits, 2] scratch,
   float* part_ml;        // combined by a second kernel; else null (slices of a cluster combine on chip)
+  const float* sink;     // [Hq] fp32 or null: see join_sink
 };
 
 // NJ: 8-key n-tiles per warp iteration (2 or 4).  Heads of 128: two blocks per SM (255 registers a thread, nothing
 // spilled); at three (170 registers) the tile's 128 registers of keys and values spill, and a decode step at the
 // layer sizes of Llama 3.2 3B measured 2.12 ms against 2.06 ms at batch 8.
-template <int HD, int NJ>
+template <int HD, int NJ, bool SPLIT>
 __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 4 : 2) attention_decode_mma_kernel(DecMmaParams p) {
   using T = __nv_bfloat16;
   constexpr int TK = 8 * NJ;     // keys per warp iteration
@@ -227,7 +228,7 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 4 : 2) attention_decode
   for (int nt = 0; nt < NT; ++nt) o[nt][0] = o[nt][1] = 0.f;
   float m = -INFINITY, l = 0.f;   // of head r (l: this lane's share, summed over the quad at the end)
 
-  decode_attend_tiles<HD, NJ>(p.kpages, p.vpages, p.page_table + (size_t)slot * p.max_pages, p.Hkv, kvh, PS, pg_b,
+  decode_attend_tiles<HD, NJ, SPLIT>(p.kpages, p.vpages, p.page_table + (size_t)slot * p.max_pages, p.Hkv, kvh, PS, pg_b,
                               n_tiles, t_begin, t_end, p.scale, warp, DM_WARPS, lane, qa, o, m, l);
   if (threadIdx.x == 0) TSTAMP(3);
 
@@ -264,6 +265,7 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 4 : 2) attention_decode
       }
     }
     if (p.n_splits == 1) {
+      join_sink(a, ll, mm, p.sink, kvh * G + g0 + g);
       p.out[(size_t)b * p.ldo + (size_t)(kvh * G + g0 + g) * HD + d] = __float2bfloat16_rn(a / ll);
     } else if (p.part_acc != nullptr) {
       const size_t o = ((size_t)b * p.Hq + (kvh * G + g0 + g)) * p.n_splits + split;
@@ -335,6 +337,7 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 4 : 2) attention_decode
       a = fmaf(ck, as[k], a);
       ll = fmaf(ck, ls[k], ll);
     }
+    join_sink(a, ll, mm, p.sink, kvh * G + g0 + g);
     p.out[(size_t)b * p.ldo + (size_t)(kvh * G + g0 + g) * HD + d] = __float2bfloat16_rn(a / ll);
   }
   if (threadIdx.x == 0) TSTAMP(6);
@@ -342,19 +345,19 @@ __global__ void __launch_bounds__(DM_THREADS, HD <= 64 ? 4 : 2) attention_decode
   if (threadIdx.x == 0) TSTAMP(7);
 }
 
-template <int HD, int NJ>
+template <int HD, int NJ, bool SPLIT>
 int launch_decode_mma(const DecMmaParams& p, int B, cudaStream_t stream) {
   dim3 grid(B, p.Hkv * p.n_gchunks, p.n_splits);
   if (p.n_splits > 1 && p.part_acc == nullptr) {
-    launch_kernel_cluster(attention_decode_mma_kernel<HD, NJ>, grid, dim3(DM_THREADS), 0, stream,
+    launch_kernel_cluster(attention_decode_mma_kernel<HD, NJ, SPLIT>, grid, dim3(DM_THREADS), 0, stream,
                           dim3(1, 1, p.n_splits), p);
     return launch_status();
   }
-  launch_kernel(attention_decode_mma_kernel<HD, NJ>, grid, dim3(DM_THREADS), 0, stream, p);
+  launch_kernel(attention_decode_mma_kernel<HD, NJ, SPLIT>, grid, dim3(DM_THREADS), 0, stream, p);
   int st = launch_status();
   if (st != DLGO_OK || p.n_splits == 1) return st;
   launch_kernel(attention_combine_kernel<__nv_bfloat16>, dim3(B, p.Hq), dim3(HD >= 128 ? 128 : 64), 0, stream,
-                (const float*)p.part_acc, (const float*)p.part_ml, p.out, p.ldo, p.Hq, HD, p.n_splits);
+                (const float*)p.part_acc, (const float*)p.part_ml, p.out, p.ldo, p.Hq, HD, p.n_splits, p.sink);
   return launch_status();
 }
 
@@ -374,14 +377,15 @@ DLGO_EXPORT int dlgo_attention_decode_mma_takes(int hd, int page_size, int n_spl
 // Or, with `parts` ([S][B][ldq] fp32, slice stride part_stride floats: the unsummed K-slices of the q | k | v
 // projection) and cos/sin tables [positions][hd / 2]: q is null, the kernel sums, rotates (whole head,
 // pairs (i, i + hd/2)) and, with write_cache, appends the token's key and value itself.
-// keys_per_tile: 16 or 32 keys per warp iteration.
+// keys_per_tile: 16 or 32 keys per warp iteration.  `sink` [Hq] fp32 or null: joins the denominator.  `split`:
+// probabilities meet the values as two bfloat16 terms (16 bits of mantissa).
 DLGO_EXPORT int dlgo_attention_decode_mma(const void* q, int B, int ldq, const void* kpages, const void* vpages,
                                           const int* page_table, int max_pages, const int* seq_slot,
                                           const int* token_pos, void* out, int ldo, int Hq, int Hkv, int hd,
                                           int page_size, int n_splits, int window, float scale, int keys_per_tile,
                                           float* scratch, const float* parts, int S, long long part_stride,
                                           const float* cos_t, const float* sin_t, int write_cache, int clear_parts,
-                                          cudaStream_t stream) {
+                                          const float* sink, int split, cudaStream_t stream) {
   if (B <= 0) return DLGO_OK;
   if (Hq <= 0 || Hkv <= 0 || Hq % Hkv) return DLGO_ERR_SIZE;
   if (!dlgo_attention_decode_mma_takes(hd, page_size, n_splits)) return DLGO_ERR_SIZE;
@@ -410,11 +414,14 @@ DLGO_EXPORT int dlgo_attention_decode_mma(const void* q, int B, int ldq, const v
   p.parts = parts; p.S = S; p.part_stride = (size_t)part_stride; p.cos_t = cos_t; p.sin_t = sin_t;
   p.write_cache = write_cache;
   p.clear_parts = clear_parts;
+  p.sink = sink;
   p.part_acc = n_splits > 8 ? scratch : nullptr;
   p.part_ml = n_splits > 8 ? scratch + (size_t)B * Hq * n_splits * hd : nullptr;
   if ((long long)Hkv * p.n_gchunks > 65535) return DLGO_ERR_SIZE;
-  if (hd == 64) return keys_per_tile == 16 ? launch_decode_mma<64, 2>(p, B, stream) : launch_decode_mma<64, 4>(p, B, stream);
-  return keys_per_tile == 16 ? launch_decode_mma<128, 2>(p, B, stream) : launch_decode_mma<128, 4>(p, B, stream);
+#define DM_LAUNCH(HD, NJ) (split ? launch_decode_mma<HD, NJ, true>(p, B, stream) : launch_decode_mma<HD, NJ, false>(p, B, stream))
+  if (hd == 64) return keys_per_tile == 16 ? DM_LAUNCH(64, 2) : DM_LAUNCH(64, 4);
+  return keys_per_tile == 16 ? DM_LAUNCH(128, 2) : DM_LAUNCH(128, 4);
+#undef DM_LAUNCH
 }
 
 DLGO_TIMES_EXPORT

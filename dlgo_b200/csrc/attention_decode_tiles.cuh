@@ -18,6 +18,18 @@ __device__ __forceinline__ void mma_rows8(float& d0, float& d1, uint32_t a0, uin
       : "+f"(d0), "+f"(d1), "=f"(x2), "=f"(x3)
       : "r"(a0), "r"(0u), "r"(a2), "r"(0u), "r"(b0), "r"(b1), "f"(0.f));
 }
+// the same with rows 8-15 of A holding a second term of rows 0-7: both terms' products are added up
+__device__ __forceinline__ void mma_rows8_two(float& d0, float& d1, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
+                                              uint32_t b0, uint32_t b1) {
+  float x2, x3;
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+      "{%0, %1, %10, %10};"
+      : "+f"(d0), "+f"(d1), "=f"(x2), "=f"(x3)
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1), "f"(0.f));
+  d0 += x2;
+  d1 += x3;
+}
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<const uint32_t*>(&h);
@@ -35,8 +47,10 @@ __device__ __forceinline__ float fast_exp(float x) {
 // [(pg_b + i / tiles_per_page) * PS + (i % tiles_per_page) * TK, + TK) of the sequence whose page numbers are
 // `page_row[]`), keys t in [t_begin, t_end) only.  Lane (r = lane / 4, c = lane % 4): `qa` holds head r's
 // query fragments; `o` receives its output (MMA column nt * 8 + 2c + e is dimension (2c + e) * HD/8 + nt),
-// `m` its running maximum and `l` this lane's share of the sum (to be added over the quad).
-template <int HD, int NJ>
+// `m` its running maximum and `l` this lane's share of the sum (to be added over the quad).  SPLIT: a probability meets
+// the values as the sum of two bfloat16 numbers (its rounding, and the rounding of what that left over), the second
+// in the rows of the MMA tile that are otherwise zero.
+template <int HD, int NJ, bool SPLIT = false>
 __device__ __forceinline__ void decode_attend_tiles(const __nv_bfloat16* kpages, const __nv_bfloat16* vpages,
                                                     const int* __restrict__ page_row, int Hkv, int kvh, int PS,
                                                     int pg_b, int n_tiles, int t_begin, int t_end, float scale,
@@ -125,12 +139,25 @@ __device__ __forceinline__ void decode_attend_tiles(const __nv_bfloat16* kpages,
     for (int ks = 0; ks < NJ / 2; ++ks) {
       const uint32_t a0 = pack_bf16(s[2 * ks][0], s[2 * ks][1]);
       const uint32_t a2 = pack_bf16(s[2 * ks + 1][0], s[2 * ks + 1][1]);
+      uint32_t a1 = 0u, a3 = 0u;
+      if (SPLIT) {
+        const float2 f0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a0));
+        const float2 f2 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a2));
+        a1 = pack_bf16(s[2 * ks][0] - f0.x, s[2 * ks][1] - f0.y);
+        a3 = pack_bf16(s[2 * ks + 1][0] - f2.x, s[2 * ks + 1][1] - f2.y);
+      }
 #pragma unroll
       for (int w = 0; w < NT / 2; ++w) {          // 32-bit word w of the lane's piece holds n-tiles 2w and 2w + 1
         const uint32_t wa = word_of(vu[ks][0][w >> 2], w & 3), wb = word_of(vu[ks][1][w >> 2], w & 3);
         const uint32_t wc = word_of(vu[ks][2][w >> 2], w & 3), wd = word_of(vu[ks][3][w >> 2], w & 3);
-        mma_rows8(o[2 * w][0], o[2 * w][1], a0, a2, __byte_perm(wa, wb, 0x5410), __byte_perm(wc, wd, 0x5410));
-        mma_rows8(o[2 * w + 1][0], o[2 * w + 1][1], a0, a2, __byte_perm(wa, wb, 0x7632), __byte_perm(wc, wd, 0x7632));
+        if (SPLIT) {
+          mma_rows8_two(o[2 * w][0], o[2 * w][1], a0, a1, a2, a3, __byte_perm(wa, wb, 0x5410), __byte_perm(wc, wd, 0x5410));
+          mma_rows8_two(o[2 * w + 1][0], o[2 * w + 1][1], a0, a1, a2, a3, __byte_perm(wa, wb, 0x7632),
+                        __byte_perm(wc, wd, 0x7632));
+        } else {
+          mma_rows8(o[2 * w][0], o[2 * w][1], a0, a2, __byte_perm(wa, wb, 0x5410), __byte_perm(wc, wd, 0x5410));
+          mma_rows8(o[2 * w + 1][0], o[2 * w + 1][1], a0, a2, __byte_perm(wa, wb, 0x7632), __byte_perm(wc, wd, 0x7632));
+        }
       }
     }
   }

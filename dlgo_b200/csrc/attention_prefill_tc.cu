@@ -490,11 +490,13 @@ DLGO_EXPORT int dlgo_attention_prefill_tc_takes(int dtype, int hd, int page_size
 }
 
 // q[T, .] bf16 with row stride ldq (head h at column h*hd); pages [n_pages, Hkv, 64, hd] bf16;
-// tiles[n_tiles][3] of at most 128 tokens each; out[T, Hq*hd] bf16 with row stride ldo.
+// tiles[n_tiles][3] of at most 128 tokens each; out[T, Hq*hd] bf16 with row stride ldo.  `sink` [Hq] fp32 or null: its
+// exponential joins the denominator.  `split`: probabilities enter P V as two bfloat16 terms.
 DLGO_EXPORT int dlgo_attention_prefill_tc(const void* q, int T, int ldq, const void* kpages, const void* vpages,
                                           int n_pages, const int* page_table, int max_pages, const int* tiles,
                                           int n_tiles, const int* seq_slot, const int* token_pos, void* out, int ldo,
-                                          int Hq, int Hkv, int hd, int window, float scale, cudaStream_t stream) {
+                                          int Hq, int Hkv, int hd, int window, float scale, const float* sink, int split,
+                                          cudaStream_t stream) {
   if (T <= 0 || n_tiles <= 0) return DLGO_OK;
   if (n_tiles > 65535) return DLGO_ERR_SIZE;   // tiles are the grid's second dimension
   if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || !(hd == 64 || hd == 128) || Hq > 65535) return DLGO_ERR_SIZE;
@@ -510,10 +512,10 @@ DLGO_EXPORT int dlgo_attention_prefill_tc(const void* q, int T, int ldq, const v
   p.tiles = tiles; p.seq_slot = seq_slot; p.token_pos = token_pos; p.page_table = page_table; p.max_pages = max_pages;
   p.out = (__nv_bfloat16*)out; p.ldo = ldo; p.Hq = Hq; p.Hkv = Hkv; p.window = window;
   p.scale_log2e = scale * 1.4426950408889634f;
-  p.sink = nullptr;
+  p.sink = sink;
   p.kv_rows = 0;
-  if (hd == 64) return launch_pf<64>(mq, mk, mv, p, n_tiles, stream);
-  return launch_pf<128>(mq, mk, mv, p, n_tiles, stream);
+  if (hd == 64) return split ? launch_pf<64, true>(mq, mk, mv, p, n_tiles, stream) : launch_pf<64>(mq, mk, mv, p, n_tiles, stream);
+  return split ? launch_pf<128, true>(mq, mk, mv, p, n_tiles, stream) : launch_pf<128>(mq, mk, mv, p, n_tiles, stream);
 }
 
 // The same attention over keys and values that were made for the step and lie as rows of tokens:

@@ -53,9 +53,11 @@ LIBRARIES: Dict[str, List[str]] = {
     "gated_residual": ["gated_residual.cu"],
     "ssd": ["ssd.cu"],
     "ssd_tc": ["ssd_tc.cu"],
+    "mlstm": ["mlstm.cu"],
+    "rglru": ["rglru.cu"],
 }
 _HEADERS = ["common.cuh", "attention_noalloc.h", "attention_combine.cuh", "attention_decode_tiles.cuh", "tcgen05.cuh",
-            "async_copy.cuh", "ssd.cuh"]
+            "async_copy.cuh", "ssd.cuh", "ssd_state.cuh"]
 
 ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 BASE_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-shared", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden"]

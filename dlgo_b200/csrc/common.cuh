@@ -170,6 +170,17 @@ __device__ unsigned long long g_times[1024 * 8];
 #define DLGO_TIMES_EXPORT
 #endif
 
+// How a gate value g and an up value u make one number of a gated feed-forward's hidden row:
+//   limit <= 0:  silu(g) * u
+//   limit > 0:   g' = min(g, limit), u' = clamp(u, -limit, limit):  g' sigmoid(alpha g') (u' + offset)
+struct GluForm {
+  float limit, alpha, offset;
+};
+__device__ __forceinline__ void glu_clamp(const GluForm& f, float& g, float& u) {
+  g = fminf(g, f.limit);
+  u = fminf(fmaxf(u, -f.limit), f.limit) + f.offset;
+}
+
 // Which keys t <= pos a query at position pos sees, as ONE integer `span` that every attention kernel takes where
 // it takes a window: span > 0 is a sliding window (keys t > pos - span), span < 0 cuts the sequence into chunks of
 // -span positions counted from position 0 (keys of the query's own chunk only), 0 is every key.  The first visible

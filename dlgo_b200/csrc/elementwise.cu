@@ -296,11 +296,11 @@ __global__ void add_rmsnorm_cluster_kernel(float* __restrict__ x, const float* _
   if (live) store4<TO>(out + (size_t)r * d + i, v.x * sc * w0.x, v.y * sc * w0.y, v.z * sc * w0.z, v.w * sc * w0.w);
 }
 
-// ------------------------------------------------------------------- SwiGLU
+// ------------------------------------------------------------------- SwiGLU (and its clamped form: GluForm)
 // in: [T, 2F]: blocks of `block` gate columns, each followed by its `block` up columns (block = F: the gate in
 // columns [0, F) and the up projection in [F, 2F)).
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ in, T* __restrict__ out, int F, int block, size_t total) {
+__global__ void swiglu_kernel(const T* in, T* out, int F, int block, size_t total, GluForm form) {
   pdl_launch_dependents();
   pdl_wait();
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -310,7 +310,12 @@ __global__ void swiglu_kernel(const T* __restrict__ in, T* __restrict__ out, int
   const size_t at = t * 2 * F + (size_t)(c / block) * 2 * block + c % block;
   float g = to_float(in[at]);
   float u = to_float(in[at + block]);
-  float h = g / (1.0f + expf(-g)) * u;
+  float alpha = 1.0f;
+  if (form.limit > 0.f) {
+    glu_clamp(form, g, u);
+    alpha = form.alpha;
+  }
+  float h = g / (1.0f + expf(-alpha * g)) * u;
   out[i] = from_float<T>(h);
 }
 
@@ -368,7 +373,7 @@ DLGO_EXPORT int dlgo_rmsnorm(const float* x, const float* w, void* out, int out_
 }
 
 // in[T, 2F], out[T, F], same element type
-static int launch_swiglu(const void* in, void* out, int dtype, int T, int F, int block, cudaStream_t stream) {
+static int launch_swiglu(const void* in, void* out, int dtype, int T, int F, int block, GluForm form, cudaStream_t stream) {
   if (T <= 0) return DLGO_OK;
   if (F <= 0 || block <= 0 || F % block != 0) return DLGO_ERR_SIZE;
   const size_t total = (size_t)T * F;
@@ -376,22 +381,29 @@ static int launch_swiglu(const void* in, void* out, int dtype, int T, int F, int
   const unsigned blocks = (unsigned)((total + threads - 1) / threads);
   if (dtype == DLGO_F32)
     launch_kernel(swiglu_kernel<float>, dim3(blocks), dim3(threads), 0, stream, (const float*)in, (float*)out, F, block,
-                  total);
+                  total, form);
   else if (dtype == DLGO_BF16)
     launch_kernel(swiglu_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream, (const __nv_bfloat16*)in,
-                  (__nv_bfloat16*)out, F, block, total);
+                  (__nv_bfloat16*)out, F, block, total, form);
   else
     return DLGO_ERR_DTYPE;
   return launch_status();
 }
 
 DLGO_EXPORT int dlgo_swiglu(const void* in, void* out, int dtype, int T, int F, cudaStream_t stream) {
-  return launch_swiglu(in, out, dtype, T, F, F, stream);
+  return launch_swiglu(in, out, dtype, T, F, F, GluForm{0.f, 1.f, 0.f}, stream);
 }
 
 // gate and up columns in blocks of `block` (a divisor of F)
 DLGO_EXPORT int dlgo_swiglu_blocks(const void* in, void* out, int dtype, int T, int F, int block, cudaStream_t stream) {
-  return launch_swiglu(in, out, dtype, T, F, block, stream);
+  return launch_swiglu(in, out, dtype, T, F, block, GluForm{0.f, 1.f, 0.f}, stream);
+}
+
+// the clamped form (limit > 0)
+DLGO_EXPORT int dlgo_clamped_glu(const void* in, void* out, int dtype, int T, int F, int block, float limit, float alpha,
+                                 float offset, cudaStream_t stream) {
+  if (!(limit > 0.f)) return DLGO_ERR_SIZE;
+  return launch_swiglu(in, out, dtype, T, F, block, GluForm{limit, alpha, offset}, stream);
 }
 
 // x[*, d] f32 (updated in place), parts[S][*, d] f32 (slice stride part_stride floats), w[d] f32 or null,

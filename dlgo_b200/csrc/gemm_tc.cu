@@ -78,6 +78,7 @@ struct TcParams {
   int static_operand; // 0: none; 1: A, 2: B holds weights no earlier kernel writes (loaded before pdl_wait)
   const float* bias;  // TC_BIAS_ACT: one number per weight row (feature), or null
   int act;            // TC_BIAS_ACT: TC_ACT_*
+  GluForm glu;        // TC_SWIGLU: silu(gate) * up, or the clamped form
 };
 
 template <int BN> struct TcConfig {
@@ -100,6 +101,18 @@ __device__ __forceinline__ float silu_mul(float g, float u) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-g * 1.4426950408889634f));
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
   return g * u * r;
+}
+
+// the clamped form of a gated feed-forward (GluForm), with the same instructions
+__device__ __forceinline__ float clamped_mul(float g, float u, const GluForm& f) {
+  glu_clamp(f, g, u);
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-g * (f.alpha * 1.4426950408889634f)));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+  return g * u * r;
+}
+__device__ __forceinline__ float glu_mul(float g, float u, const GluForm& f) {
+  return f.limit > 0.f ? clamped_mul(g, u, f) : silu_mul(g, u);
 }
 
 template <int ACT> __device__ __forceinline__ float act_value(float z) {
@@ -161,7 +174,7 @@ __device__ __forceinline__ void epilogue_store_as(const TcParams& p, const float
         for (int j = 0; j < 16; ++j) {
           if (col0 + 16 + j < p.Rb) {
             const float g = v[j], u = v[16 + j];
-            o[j] = __float2bfloat16_rn(silu_mul(g, u));
+            o[j] = __float2bfloat16_rn(glu_mul(g, u, p.glu));
           }
         }
       }
@@ -174,7 +187,7 @@ __device__ __forceinline__ void epilogue_store_as(const TcParams& p, const float
         if (lane < 16 && row + 16 < p.Ra && col < p.Rb) {
           const float g = v[j];
           const int feature = (row >> 5) * 16 + (row & 15);
-          ((__nv_bfloat16*)p.out)[(size_t)col * p.ldo + feature] = __float2bfloat16_rn(silu_mul(g, other));
+          ((__nv_bfloat16*)p.out)[(size_t)col * p.ldo + feature] = __float2bfloat16_rn(glu_mul(g, other, p.glu));
         }
       }
     }
@@ -425,7 +438,7 @@ __device__ __forceinline__ void gemm_tc_body(const CUtensorMap& map_a, const CUt
 #pragma unroll
           for (int j = 0; j < NV; ++j) {
             const float other = __shfl_xor_sync(0xffffffffu, v[j], 16);
-            if (lane < 16) stage[(c0 + j) * 64 + quarter * 16 + lane] = __float2bfloat16_rn(silu_mul(v[j], other));
+            if (lane < 16) stage[(c0 + j) * 64 + quarter * 16 + lane] = __float2bfloat16_rn(glu_mul(v[j], other, p.glu));
           }
         }
       }
@@ -752,7 +765,7 @@ __device__ __forceinline__ void staged_epilogue(const TcParams& p, const CUtenso
 #pragma unroll
         for (int q = 0; q < 8; ++q) {
           const float g0 = v[2 * q], g1 = v[2 * q + 1], u0 = v[16 + 2 * q], u1 = v[16 + 2 * q + 1];
-          b2[q] = __floats2bfloat162_rn(silu_mul(g0, u0), silu_mul(g1, u1));
+          b2[q] = __floats2bfloat162_rn(glu_mul(g0, u0, p.glu), glu_mul(g1, u1, p.glu));
         }
         *reinterpret_cast<uint4*>(row + (((2 * h) ^ (r & 7)) << 4)) = *reinterpret_cast<uint4*>(&b2[0]);
         *reinterpret_cast<uint4*>(row + (((2 * h + 1) ^ (r & 7)) << 4)) = *reinterpret_cast<uint4*>(&b2[4]);
@@ -1292,14 +1305,24 @@ DLGO_EXPORT int dlgo_gemm_tc_tiles(int Ra, int Rb, int bn) {
 // tokens only: not transposed, one K-slice; bn is then ignored).
 static int gemm_tc_impl(const void* A, int Ra, int lda, const void* B, int Rb, int ldb, int K, void* out, int ldo,
                         int transposed, int epilogue, int bn, int splits, float* workspace, int* counters,
-                        int static_operand, int pair_tile, const float* bias, int act, cudaStream_t stream);
+                        int static_operand, int pair_tile, const float* bias, int act, GluForm glu, cudaStream_t stream);
 
 DLGO_EXPORT int dlgo_gemm_tc(const void* A, int Ra, int lda, const void* B, int Rb, int ldb, int K, void* out,
                              int ldo, int transposed, int epilogue, int bn, int splits, float* workspace,
                              int* counters, int static_operand, int pair_tile, cudaStream_t stream) {
   if (epilogue < 0 || epilogue > 5) return DLGO_ERR_SIZE;
   return gemm_tc_impl(A, Ra, lda, B, Rb, ldb, K, out, ldo, transposed, epilogue, bn, splits, workspace, counters,
-                      static_operand, pair_tile, nullptr, 0, stream);
+                      static_operand, pair_tile, nullptr, 0, GluForm{0.f, 1.f, 0.f}, stream);
+}
+
+// The same product with epilogue 3 in its clamped form (limit > 0; see GluForm).
+DLGO_EXPORT int dlgo_gemm_tc_clamped_glu(const void* A, int Ra, int lda, const void* B, int Rb, int ldb, int K, void* out,
+                                         int ldo, int transposed, int bn, int splits, float* workspace, int* counters,
+                                         int static_operand, int pair_tile, float limit, float alpha, float offset,
+                                         cudaStream_t stream) {
+  if (!(limit > 0.f)) return DLGO_ERR_SIZE;
+  return gemm_tc_impl(A, Ra, lda, B, Rb, ldb, K, out, ldo, transposed, TC_SWIGLU, bn, splits, workspace, counters,
+                      static_operand, pair_tile, nullptr, 0, GluForm{limit, alpha, offset}, stream);
 }
 
 // The same product with epilogue 7: out (bf16) = act(acc + bias[feature]) with bias (fp32, one per weight row, or
@@ -1310,12 +1333,12 @@ DLGO_EXPORT int dlgo_gemm_tc_bias_act(const void* A, int Ra, int lda, const void
                                       cudaStream_t stream) {
   if (act < TC_ACT_NONE || act > TC_ACT_GELU_TANH) return DLGO_ERR_SIZE;
   return gemm_tc_impl(A, Ra, lda, B, Rb, ldb, K, out, ldo, transposed, TC_BIAS_ACT, bn, splits, workspace, counters,
-                      static_operand, pair_tile, bias, act, stream);
+                      static_operand, pair_tile, bias, act, GluForm{0.f, 1.f, 0.f}, stream);
 }
 
 static int gemm_tc_impl(const void* A, int Ra, int lda, const void* B, int Rb, int ldb, int K, void* out, int ldo,
                         int transposed, int epilogue, int bn, int splits, float* workspace, int* counters,
-                        int static_operand, int pair_tile, const float* bias, int act, cudaStream_t stream) {
+                        int static_operand, int pair_tile, const float* bias, int act, GluForm glu, cudaStream_t stream) {
   if (Ra <= 0 || Rb <= 0) return DLGO_OK;
   if (K <= 0 || K % 8 || lda < K || ldb < K || splits < 1) return DLGO_ERR_SIZE;
   if (splits > (K + TILE_K - 1) / TILE_K) return DLGO_ERR_SIZE;
@@ -1338,6 +1361,7 @@ static int gemm_tc_impl(const void* A, int Ra, int lda, const void* B, int Rb, i
   p.static_operand = (static_operand == 1 || static_operand == 2) ? static_operand : 0;
   p.bias = bias;
   p.act = act;
+  p.glu = glu;
   if (!transposed && splits == 1 && pair_tile != 0) {
     // many tokens, CTA pairs: A's box is 128 rows, B's box is half the tile's width
     if (pair_tile != 128 && pair_tile != 256) return DLGO_ERR_SIZE;

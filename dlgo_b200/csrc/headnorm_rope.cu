@@ -2,9 +2,11 @@
 // append of this step's keys and values to the paged cache, in one pass over the fp32 result of the
 // q|k (or q|k|v) projection.
 //
-// proj[T, ld] (fp32): Hq query heads, then Hkv key heads, then (unless `v_from_k`) Hkv value heads, hd
-// numbers each; `bias` (fp32, one number per column, may be null) is added first.  With `v_from_k` the
-// value of a position is its key as projected (with the bias, before norm and rotation).
+// proj[T, ld] (fp32): Hq query heads, then Hkv key heads of `dk` numbers each, then (unless `v_from_k`) Hkv value
+// heads of `dv`; in the cache and in q_out every head is `hd` numbers wide (hd >= dk, dv) with zeros behind its own,
+// so that keys and values share one page shape.  `bias` (fp32, one number per column, may be null) is added first.
+// With `v_from_k` the value of a position is its key as projected (with the bias, before norm and rotation); value
+// heads of their own are kept times `v_scale`.
 //
 //   head norm (w_q / w_k not null):  u <- u / sqrt(mean(u^2) + eps) * w      (plain weight, per head; the mean runs
 //   over the first `norm_dim` numbers of a head: a head may be laid out with trailing zeros)
@@ -26,13 +28,14 @@ constexpr int HR_WARPS = 4;
 
 template <typename T>
 __global__ void __launch_bounds__(HR_WARPS * 32)
-headnorm_rope_append_kernel(float* __restrict__ proj, int ld, const float* __restrict__ bias,
+headnorm_rope_append_kernel(float* proj, int ld, const float* __restrict__ bias,
                             const float* __restrict__ w_q, const float* __restrict__ w_k, float eps,
                             const float* __restrict__ freq, int rot, const int* __restrict__ token_pos,
                             const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
-                            const int* __restrict__ page_table, int max_pages, T* __restrict__ kpages,
-                            T* __restrict__ vpages, T* __restrict__ q_out, int T_tokens, int Hq, int Hkv, int hd,
-                            int page_size, int v_from_k, int write_cache, int clear, int norm_dim) {
+                            const int* __restrict__ page_table, int max_pages, T* kpages,
+                            T* vpages, T* q_out, int T_tokens, int Hq, int Hkv, int dk,
+                            int dv, int hd, int page_size, int v_from_k, int write_cache, int clear, int norm_dim,
+                            float v_scale) {
   extern __shared__ float hr_smem[];
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -60,20 +63,25 @@ headnorm_rope_append_kernel(float* __restrict__ proj, int ld, const float* __res
   }
   const float* w = is_q ? w_q : (is_k ? w_k : nullptr);
   pdl_wait();
-  float* src = proj + (size_t)t * ld + (size_t)head * hd;
+  const bool is_v = !is_q && !is_k;
+  const int n = is_v ? dv : dk;                  // this head's own numbers
+  const size_t col = is_v ? (size_t)(Hq + Hkv) * dk + (size_t)(head - Hq - Hkv) * dv : (size_t)head * dk;
+  float* src = proj + (size_t)t * ld + col;
   float ss = 0.f;
-  for (int i = lane; i < hd; i += 32) {
+  for (int i = lane; i < n; i += 32) {
     float x = src[i];
-    if (bias != nullptr) x += bias[(size_t)head * hd + i];
+    if (bias != nullptr) x += bias[col + i];
     u[i] = x;
     ss += x * x;
     if (is_k && v_from_k && vdst != nullptr) vdst[i] = from_float<T>(x);
   }
+  if (is_k && v_from_k && vdst != nullptr)
+    for (int i = n + lane; i < hd; i += 32) vdst[i] = from_float<T>(0.f);
   if (clear)                     // (after every load of the row has been issued: a store right behind a load holds the loads up)
-    for (int i = lane; i < hd; i += 32) src[i] = 0.f;
-  if (!is_q && !is_k) {          // a value head of its own: stored as projected
+    for (int i = lane; i < n; i += 32) src[i] = 0.f;
+  if (is_v) {                    // a value head of its own: stored as projected
     if (vdst != nullptr)
-      for (int i = lane; i < hd; i += 32) vdst[i] = from_float<T>(u[i]);
+      for (int i = lane; i < hd; i += 32) vdst[i] = from_float<T>(i < n ? u[i] * v_scale : 0.f);
     return;
   }
   ss = warp_sum(ss);
@@ -92,8 +100,11 @@ headnorm_rope_append_kernel(float* __restrict__ proj, int ld, const float* __res
     dst[i + rh] = from_float<T>(b * cs + a * sn);
   }
   for (int i = rot + lane; i < hd; i += 32) {
-    float a = u[i] * r;
-    if (w != nullptr) a *= w[i];
+    float a = 0.f;
+    if (i < n) {
+      a = u[i] * r;
+      if (w != nullptr) a *= w[i];
+    }
     dst[i] = from_float<T>(a);
   }
 }
@@ -102,8 +113,8 @@ template <typename T>
 int launch_headnorm_rope(float* proj, int ld, const float* bias, const float* w_q, const float* w_k, float eps,
                          const float* freq, int rot, const int* token_pos, const int* token_seq, const int* seq_slot,
                          const int* page_table, int max_pages, void* kpages, void* vpages, void* q_out, int T_tokens,
-                         int Hq, int Hkv, int hd, int page_size, int v_from_k, int write_cache, int clear, int norm_dim,
-                         cudaStream_t stream) {
+                         int Hq, int Hkv, int dk, int dv, int hd, int page_size, int v_from_k, int write_cache, int clear,
+                         int norm_dim, float v_scale, cudaStream_t stream) {
   const int heads = Hq + Hkv + (v_from_k ? 0 : Hkv);
   const long long items = (long long)T_tokens * heads;
   const long long blocks = (items + HR_WARPS - 1) / HR_WARPS;
@@ -112,7 +123,7 @@ int launch_headnorm_rope(float* proj, int ld, const float* bias, const float* w_
   if (smem > 48 * 1024) return DLGO_ERR_SIZE;
   launch_kernel(headnorm_rope_append_kernel<T>, dim3((unsigned)blocks), dim3(HR_WARPS * 32), smem, stream, proj, ld,
                 bias, w_q, w_k, eps, freq, rot, token_pos, token_seq, seq_slot, page_table, max_pages, (T*)kpages,
-                (T*)vpages, (T*)q_out, T_tokens, Hq, Hkv, hd, page_size, v_from_k, write_cache, clear, norm_dim);
+                (T*)vpages, (T*)q_out, T_tokens, Hq, Hkv, dk, dv, hd, page_size, v_from_k, write_cache, clear, norm_dim, v_scale);
   return launch_status();
 }
 
@@ -122,21 +133,23 @@ DLGO_EXPORT int dlgo_headnorm_rope_append(float* proj, int ld, const float* bias
                                           float eps, const float* freq, int rot, const int* token_pos,
                                           const int* token_seq, const int* seq_slot, const int* page_table,
                                           int max_pages, void* kpages, void* vpages, void* q_out, int dtype, int T,
-                                          int Hq, int Hkv, int hd, int page_size, int v_from_k, int write_cache,
-                                          int clear, int norm_dim, cudaStream_t stream) {
+                                          int Hq, int Hkv, int dk, int dv, int hd, int page_size, int v_from_k,
+                                          int write_cache, int clear, int norm_dim, float v_scale, cudaStream_t stream) {
   if (T <= 0) return DLGO_OK;
-  if (Hq <= 0 || Hkv <= 0 || hd <= 0 || rot < 0 || rot > hd || rot % 2) return DLGO_ERR_SIZE;
+  if (Hq <= 0 || Hkv <= 0 || dk <= 0 || dv <= 0 || hd < dk || hd < dv || rot < 0 || rot > dk || rot % 2)
+    return DLGO_ERR_SIZE;
+  if (v_from_k && dv != dk) return DLGO_ERR_SIZE;
   if (rot > 0 && freq == nullptr) return DLGO_ERR_SIZE;
-  if (norm_dim <= 0 || norm_dim > hd) return DLGO_ERR_SIZE;
-  if (ld < (Hq + Hkv + (v_from_k ? 0 : Hkv)) * hd) return DLGO_ERR_SIZE;
+  if (norm_dim <= 0 || norm_dim > dk) return DLGO_ERR_SIZE;
+  if (ld < (Hq + Hkv) * dk + (v_from_k ? 0 : Hkv * dv)) return DLGO_ERR_SIZE;
   if (dtype == DLGO_F32)
     return dlgo::launch_headnorm_rope<float>(proj, ld, bias, w_q, w_k, eps, freq, rot, token_pos, token_seq, seq_slot,
-                                             page_table, max_pages, kpages, vpages, q_out, T, Hq, Hkv, hd, page_size,
-                                             v_from_k, write_cache, clear, norm_dim, stream);
+                                             page_table, max_pages, kpages, vpages, q_out, T, Hq, Hkv, dk, dv, hd,
+                                             page_size, v_from_k, write_cache, clear, norm_dim, v_scale, stream);
   if (dtype == DLGO_BF16)
     return dlgo::launch_headnorm_rope<__nv_bfloat16>(proj, ld, bias, w_q, w_k, eps, freq, rot, token_pos, token_seq,
                                                      seq_slot, page_table, max_pages, kpages, vpages, q_out, T, Hq,
-                                                     Hkv, hd, page_size, v_from_k, write_cache, clear, norm_dim, stream);
+                                                     Hkv, dk, dv, hd, page_size, v_from_k, write_cache, clear, norm_dim, v_scale, stream);
   return DLGO_ERR_DTYPE;
 }
 

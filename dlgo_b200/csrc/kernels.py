@@ -3,7 +3,8 @@ current stream.  Nothing here computes; a missing or failing library raises."""
 from __future__ import annotations
 
 import ctypes
-from typing import Sequence, List, Optional
+import functools
+from typing import List, NamedTuple, Optional, Sequence
 
 import torch
 
@@ -158,16 +159,40 @@ def add_rmsnorm(x: torch.Tensor, parts: torch.Tensor, w: Optional[torch.Tensor],
     return out
 
 
-def swiglu(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, block: Optional[int] = None) -> torch.Tensor:
+class ClampedGlu(NamedTuple):
+    """The clamped form of a gated feed-forward's hidden number: with g' = min(g, limit) and u' = clamp(u, -limit,
+    limit), ``g' sigmoid(alpha g') (u' + offset)`` in the place of ``silu(g) u``."""
+
+    limit: float
+    alpha: float = 1.702
+    offset: float = 1.0
+
+
+def _glu_args(glu: Optional[ClampedGlu]) -> list:
+    if glu is None:
+        return [_f(0.0), _f(1.0), _f(0.0)]
+    if not glu.limit > 0:
+        raise KernelError("a clamped gated feed-forward needs a positive limit")
+    return [_f(glu.limit), _f(glu.alpha), _f(glu.offset)]
+
+
+def swiglu(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, block: Optional[int] = None,
+           glu: Optional[ClampedGlu] = None) -> torch.Tensor:
     """[T, 2F] (gate | up) -> [T, F].  ``block``: gate and up columns alternate in blocks of this many columns
-    (a divisor of F) instead of two halves."""
+    (a divisor of F) instead of two halves.  ``glu``: the clamped form."""
     _need(gate_up, None, "gate_up")
     T, F2 = gate_up.shape
     F = F2 // 2
     if out is None:
         out = torch.empty((T, F), dtype=gate_up.dtype, device=gate_up.device)
     _need(out, gate_up.dtype, "out")
-    if block is None or block == F:
+    if glu is not None:
+        block = block or F
+        if block <= 0 or F % block:
+            raise KernelError(f"swiglu: blocks of {block} columns do not divide {F}")
+        st = _lib("elementwise").dlgo_clamped_glu(_ptr(gate_up), _ptr(out), _i(dtype_code(gate_up.dtype)), _i(T), _i(F),
+                                                  _i(block), *_glu_args(glu), _stream())
+    elif block is None or block == F:
         st = _lib("elementwise").dlgo_swiglu(_ptr(gate_up), _ptr(out), _i(dtype_code(gate_up.dtype)), _i(T), _i(F),
                                              _stream())
     else:
@@ -180,7 +205,7 @@ def swiglu(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, block: Opt
 
 
 # ----------------------------------------------- residual streams and their norms
-NORM_NONE, NORM_RMS, NORM_DYT = 0, 1, 2
+NORM_NONE, NORM_RMS, NORM_DYT, NORM_LAYER = 0, 1, 2, 3
 ACT_NONE, ACT_RELU2, ACT_SILU, ACT_GELU_TANH = 0, 1, 2, 3
 ACT_TANH = 4           # (the elementwise bias_act only)
 MOE_ACT_SWIGLU = 4     # (moe_gemm_tc only: W's rows in blocks of MOE_SWIGLU_BLOCK gate rows and as many up rows)
@@ -200,7 +225,7 @@ def streams_step(X: torch.Tensor, *, y: Optional[torch.Tensor] = None, y_bias: O
     Write part (with ``y`` [T, d] fp32): ``X[t, q] = sum_r mix[r, q] X[t, r] + write[q] * (y[t] + y_bias)``,
     all streams at once from the old values; ``clear_y`` leaves zeros in ``y``.  Read part (with
     ``out_dtype``): ``u = sum_r read[r] X[t, r]`` (``read`` None: the plain sum) through the norm
-    (``NORM_DYT``: tanh(alpha u) w + b; ``NORM_RMS``; ``NORM_NONE``: u itself) into a new [R, d] tensor;
+    (``NORM_DYT``: tanh(alpha u) w + b; ``NORM_LAYER``: layer norm with w and b; ``NORM_RMS``; ``NORM_NONE``: u itself) into a new [R, d] tensor;
     ``rows`` picks the rows to read (read part only)."""
     _need(X, torch.float32, "X")
     if X.dim() != 3:
@@ -224,8 +249,9 @@ def streams_step(X: torch.Tensor, *, y: Optional[torch.Tensor] = None, y_bias: O
     R = T if rows is None else rows.numel()
     out = None
     if out_dtype is not None:
-        if norm_kind != NORM_NONE and (norm_w is None or norm_w.numel() != d):
-            raise KernelError("streams_step: the norm needs a weight of the hidden size")
+        if norm_kind != NORM_NONE and (norm_w is None or norm_w.numel() != d or
+                                       (norm_b is not None and norm_b.numel() != d)):
+            raise KernelError("streams_step: the norm needs a weight (and bias) of the hidden size")
         if norm_kind == NORM_DYT and norm_alpha is None:
             raise KernelError("streams_step: Dynamic Tanh needs alpha")
         out = torch.empty((R, d), dtype=out_dtype, device=X.device)
@@ -680,21 +706,22 @@ def ssd_scratch_floats(n_tiles: int, shape: SsdShape) -> int:
     return n_tiles * shape.heads * (shape.state * shape.v_dim + 1)
 
 
-def ssd_segments(xbc: torch.Tensor, steps: torch.Tensor, D: torch.Tensor, tiles: torch.Tensor, n_tiles: int, direct: bool,
+def ssd_segments(xbc: torch.Tensor, steps: torch.Tensor, D: Optional[torch.Tensor], tiles: torch.Tensor, n_tiles: int, direct: bool,
                  seq_slot: torch.Tensor, state: torch.Tensor, scratch: Optional[torch.Tensor],
                  shape: SsdShape) -> torch.Tensor:
     """The recurrence over the step's tokens from :func:`ssd_conv`'s results: S <- f S + d B x^T, y = S^T C + D x, every
-    sequence from (and back into) its state row.  ``tiles`` cut a sequence's tokens into consecutive segments that run
+    sequence from (and back into) its state row (``D`` None: no such term).  ``tiles`` cut a sequence's tokens into consecutive segments that run
     side by side; ``direct``: one segment per sequence; else ``scratch`` holds :func:`ssd_scratch_floats`.
     Returns fp32 [T, heads * v_dim]."""
     _ssd_check("ssd_segments", shape, None, state)
-    _need(D, torch.float32, "D")
+    if D is not None:
+        _need(D, torch.float32, "D")
     _need(xbc, torch.float32, "xbc")
     _need(steps, torch.float32, "steps")
     _need(tiles, torch.int32, "tiles")
     _need(seq_slot, torch.int32, "seq_slot")
     T = xbc.shape[0]
-    if D.numel() != shape.heads or xbc.shape[1] < shape.channels or tuple(steps.shape) != (T, shape.heads, 2):
+    if (D is not None and D.numel() != shape.heads) or xbc.shape[1] < shape.channels or tuple(steps.shape) != (T, shape.heads, 2):
         raise KernelError("ssd_segments: shapes do not fit")
     if not direct:
         need = ssd_scratch_floats(n_tiles, shape)
@@ -716,11 +743,13 @@ def ssd_chunks_takes(dtype: torch.dtype, state_rows: int, v_dim: int) -> bool:
 def ssd_chunks(xbc: torch.Tensor, x_col: int, b_col: int, c_col: int, steps: Optional[torch.Tensor],
                log_decay: Optional[torch.Tensor], D: Optional[torch.Tensor], tiles: torch.Tensor, n_tiles: int,
                direct: bool, seq_slot: torch.Tensor, state: torch.Tensor, scratch: Optional[torch.Tensor],
-               heads: int, groups: int, state_rows: int, v_dim: int) -> torch.Tensor:
+               heads: int, groups: int, state_rows: int, v_dim: int, norm_off: Optional[int] = None):
     """:func:`ssd_segments` for prompts in bfloat16, on the tensor cores: x, B and C are the bfloat16 columns ``x_col``
     (heads of v_dim), ``b_col`` and ``c_col`` (groups of state_rows) of ``xbc`` [T, ld].  ``steps`` [T, heads, 2] fp32
     holds d and the logarithm of f; without it d = 1 and ``log_decay`` [heads] is the logarithm.  A slot's state is the
-    first heads * state_rows * v_dim numbers of its row of ``state`` (fp32)."""
+    first heads * state_rows * v_dim numbers of its row of ``state`` (fp32).  ``norm_off``: the recurrence also runs on
+    x = 1, whose state [heads, state_rows] lies at that place of the row (``scratch`` then needs n_tiles * heads *
+    state_rows floats more); returns (outputs, n_t . C_t [T, heads] fp32) instead of the outputs alone."""
     if xbc.dtype != torch.bfloat16 or xbc.dim() != 2 or xbc.stride(1) != 1 or not xbc.is_cuda:
         raise KernelError("ssd_chunks: xbc must be 2-D bfloat16 on the GPU with unit inner stride")
     T, width = xbc.shape
@@ -739,16 +768,22 @@ def ssd_chunks(xbc: torch.Tensor, x_col: int, b_col: int, c_col: int, steps: Opt
             if t.numel() != k:
                 raise KernelError(f"ssd_chunks: {n} must have {k} numbers, has {t.numel()}")
     if not direct:
-        need = n_tiles * heads * (state_rows * v_dim + 1)
+        need = n_tiles * heads * (state_rows * v_dim + 1 + (state_rows if norm_off is not None else 0))
         if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
             raise KernelError(f"ssd_chunks: {n_tiles} segments need {need} floats of scratch")
     out = torch.empty((T, heads * v_dim), dtype=torch.float32, device=xbc.device)
+    norm = norm_state = None
+    if norm_off is not None:
+        if state.dim() != 2 or norm_off < floats or norm_off + heads * state_rows > state.shape[1]:
+            raise KernelError("ssd_chunks: the normalizer's state must lie behind the state in the same row")
+        norm = torch.empty((T, heads), dtype=torch.float32, device=xbc.device)
+        norm_state = state[:, norm_off:]
     st = _lib("ssd_tc").dlgo_ssd_chunks(
         _ptr(xbc), _i(xbc.stride(0)), _i(x_col), _i(b_col), _i(c_col), _ptr(steps), _ptr(log_decay), _ptr(D), _ptr(tiles),
         _i(n_tiles), _i(1 if direct else 0), _ptr(seq_slot), _ptr(state), _ll(state.stride(0)), _ptr(scratch), _ptr(out),
-        _i(out.stride(0)), _i(heads), _i(groups), _i(state_rows), _i(v_dim), _stream())
-    _check(st, "ssd_chunks", 1 if direct else 3)
-    return out
+        _i(out.stride(0)), _i(heads), _i(groups), _i(state_rows), _i(v_dim), _ptr(norm_state), _ptr(norm), _stream())
+    _check(st, "ssd_chunks", 1 if direct else (3 if norm is None else 4))
+    return out if norm is None else (out, norm)
 
 
 def ssd_step(proj: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
@@ -791,6 +826,227 @@ def ssd_gate_norm(y: torch.Tensor, proj: torch.Tensor, w: torch.Tensor, norm_gro
                                         _i(dtype_code(out_dtype)), _i(norm_groups), _f(eps), _ptr(seqs), _i(n_seqs),
                                         _i(T), _ptr(seq_slot), _ptr(state), _ll(state.stride(0)), *shape.args(), _stream())
     _check(st, "ssd_gate_norm")
+    return out
+
+
+# ---------------------------------------------------------------- matrix memory
+def mlstm_state_floats(heads: int, qk_dim: int, v_dim: int) -> int:
+    """Numbers of one sequence's state row: S, n, m (to whole 16 bytes)."""
+    n = heads * (qk_dim * v_dim + qk_dim + 1)
+    return n + -n % 4
+
+
+def _mlstm_check(what: str, state: torch.Tensor, heads: int, qk_dim: int, v_dim: int) -> None:
+    need = mlstm_state_floats(heads, qk_dim, v_dim)
+    if qk_dim > SSD_MAX_STATE:
+        raise KernelError(f"{what}: at most {SSD_MAX_STATE} numbers per key, got {qk_dim}")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < need or not state.is_cuda:
+        raise KernelError(f"{what}: state must be [slots, >= {need}] float32 on the GPU")
+
+
+def _f32_rows(what: str, **tensors: torch.Tensor) -> None:
+    for n, t in tensors.items():
+        if t.dtype != torch.float32 or t.dim() != 2 or t.stride(1) != 1 or not t.is_cuda:
+            raise KernelError(f"{what}: {n} must be 2-D float32 on the GPU with unit inner stride")
+
+
+def mlstm_gates(zi: torch.Tensor, zf: torch.Tensor, bi: torch.Tensor, bf: torch.Tensor, cap: float, seqs: torch.Tensor,
+                n_seqs: int, longest: int, seq_slot: torch.Tensor, state: torch.Tensor, heads: int, qk_dim: int, v_dim: int,
+                log_decay: bool) -> tuple:
+    """Gates of a matrix memory over the step's tokens: from the logits ``zi``, ``zf`` [T, heads] (fp32 views of one
+    projection) the running maximum m (continued from and stored into the state rows) and per token d = exp(i - m) and
+    f' = exp(f + m_before - m) (``log_decay``: its logarithm).  ``seqs`` [n_seqs, 3] lists every sequence of the step
+    (sequence, first packed token, count).  Returns ((d, f') [T, heads, 2], m [T, heads])."""
+    _mlstm_check("mlstm_gates", state, heads, qk_dim, v_dim)
+    _f32_rows("mlstm_gates", zi=zi, zf=zf)
+    for n, t in (("bi", bi), ("bf", bf)):
+        _need(t, torch.float32, n)
+    for n, t in (("seqs", seqs), ("seq_slot", seq_slot)):
+        _need(t, torch.int32, n)
+    T = zi.shape[0]
+    if tuple(zi.shape) != (T, heads) or tuple(zf.shape) != (T, heads) or zi.stride(0) != zf.stride(0) or \
+            bi.numel() != heads or bf.numel() != heads:
+        raise KernelError("mlstm_gates: two logits and two biases per head, the logits in one projection")
+    steps = torch.empty((T, heads, 2), dtype=torch.float32, device=zi.device)
+    m = torch.empty((T, heads), dtype=torch.float32, device=zi.device)
+    st = _lib("mlstm").dlgo_mlstm_gates(_ptr(zi), _ptr(zf), _i(zi.stride(0)), _ptr(bi), _ptr(bf), _f(cap), _ptr(seqs),
+                                        _i(n_seqs), _i(longest), _ptr(seq_slot), _ptr(state), _ll(state.stride(0)),
+                                        _ptr(steps), _ptr(m), _i(1 if log_decay else 0), _i(heads), _i(qk_dim), _i(v_dim),
+                                        _stream())
+    _check(st, "mlstm_gates")
+    return steps, m
+
+
+def mlstm_norm_scan(k: torch.Tensor, q: torch.Tensor, steps: torch.Tensor, seqs: torch.Tensor, n_seqs: int,
+                    seq_slot: torch.Tensor, state: torch.Tensor, heads: int, qk_dim: int, v_dim: int) -> torch.Tensor:
+    """n_t . q_t [T, heads] of a matrix memory, token by token; n continues from and is stored into the state rows.  ``k``
+    and ``q``: fp32 views [T, heads * qk_dim] of one projection; ``steps`` of :func:`mlstm_gates` without the logarithm."""
+    _mlstm_check("mlstm_norm_scan", state, heads, qk_dim, v_dim)
+    _f32_rows("mlstm_norm_scan", k=k, q=q)
+    _need(steps, torch.float32, "steps")
+    T = k.shape[0]
+    if k.shape[1] != heads * qk_dim or q.shape != k.shape or k.stride(0) != q.stride(0) or steps.numel() != T * heads * 2:
+        raise KernelError("mlstm_norm_scan: shapes do not fit")
+    nq = torch.empty((T, heads), dtype=torch.float32, device=k.device)
+    st = _lib("mlstm").dlgo_mlstm_norm_scan(_ptr(k), _ptr(q), _i(k.stride(0)), _ptr(steps), _ptr(seqs), _i(n_seqs),
+                                            _ptr(seq_slot), _ptr(state), _ll(state.stride(0)), _ptr(nq), _i(heads),
+                                            _i(qk_dim), _i(v_dim), _stream())
+    _check(st, "mlstm_norm_scan")
+    return nq
+
+
+def mlstm_step(proj: torch.Tensor, zi: torch.Tensor, zf: torch.Tensor, bi: torch.Tensor, bf: torch.Tensor, cap: float,
+               seq_slot: torch.Tensor, state: torch.Tensor, heads: int, qk_dim: int, v_dim: int) -> tuple:
+    """One token per sequence (row t of ``proj``, fp32 with columns v | k | q, belongs to sequence t) through a matrix
+    memory: S and n move on in the state rows, m is left to :func:`mlstm_gate_norm`.  Returns (S^T q [T, heads * v_dim],
+    n . q [T, heads], m [T, heads])."""
+    _mlstm_check("mlstm_step", state, heads, qk_dim, v_dim)
+    _f32_rows("mlstm_step", proj=proj, zi=zi, zf=zf)
+    for n, t in (("bi", bi), ("bf", bf)):
+        _need(t, torch.float32, n)
+    _need(seq_slot, torch.int32, "seq_slot")
+    T = proj.shape[0]
+    if proj.shape[1] < heads * (2 * qk_dim + v_dim) or zi.stride(0) != proj.stride(0) or zf.stride(0) != proj.stride(0) or \
+            tuple(zi.shape) != (T, heads) or tuple(zf.shape) != (T, heads):
+        raise KernelError("mlstm_step: the projection must hold v, k, q and two logits per head")
+    out = torch.empty((T, heads * v_dim), dtype=torch.float32, device=proj.device)
+    nq = torch.empty((T, heads), dtype=torch.float32, device=proj.device)
+    m = torch.empty((T, heads), dtype=torch.float32, device=proj.device)
+    st = _lib("mlstm").dlgo_mlstm_step(_ptr(proj), _ptr(zi), _ptr(zf), _i(proj.stride(0)), _ptr(bi), _ptr(bf), _f(cap),
+                                       _ptr(seq_slot), _ptr(state), _ll(state.stride(0)), _ptr(out), _i(out.stride(0)),
+                                       _ptr(nq), _ptr(m), _i(T), _i(heads), _i(qk_dim), _i(v_dim), _stream())
+    _check(st, "mlstm_step")
+    return out, nq, m
+
+
+def mlstm_gate_norm(o: torch.Tensor, nq: torch.Tensor, m: torch.Tensor, qk_scale: float, gate: torch.Tensor, w: torch.Tensor,
+                    eps: float, out_scale: float, out_dtype: torch.dtype, seq_slot: torch.Tensor, state: torch.Tensor,
+                    store_m: bool, heads: int, qk_dim: int, v_dim: int) -> torch.Tensor:
+    """``rms(o c / (max(|nq c|, exp(-m)) + 1e-6)) * w * sigmoid(gate) * out_scale`` with c = ``qk_scale`` and the root mean
+    square per head, [T, heads * v_dim] in ``out_dtype``; ``store_m`` (one token per sequence): m goes into the state."""
+    _mlstm_check("mlstm_gate_norm", state, heads, qk_dim, v_dim)
+    _f32_rows("mlstm_gate_norm", o=o, gate=gate)
+    for n, t in (("nq", nq), ("m", m), ("w", w)):
+        _need(t, torch.float32, n)
+    T, n = o.shape
+    if n != heads * v_dim or tuple(gate.shape) != (T, n) or nq.numel() != T * heads or m.numel() != T * heads or w.numel() != n:
+        raise KernelError("mlstm_gate_norm: shapes do not fit")
+    out = torch.empty((T, n), dtype=out_dtype, device=o.device)
+    st = _lib("mlstm").dlgo_mlstm_gate_norm(_ptr(o), _i(o.stride(0)), _ptr(nq), _ptr(m), _f(qk_scale), _ptr(gate),
+                                            _i(gate.stride(0)), _ptr(w), _f(eps), _f(out_scale), _ptr(out),
+                                            _i(dtype_code(out_dtype)), _i(T), _ptr(seq_slot), _ptr(state),
+                                            _ll(state.stride(0)), _i(1 if store_m else 0), _i(heads), _i(qk_dim), _i(v_dim),
+                                            _stream())
+    _check(st, "mlstm_gate_norm")
+    return out
+
+
+# --------------------------------------------- real-gated linear recurrent unit
+class RglruShape:
+    """Sizes of a real-gated linear recurrent unit: channels, equal parts whose gates read their own part only, taps of
+    the convolution over time, and the constant factor of the decay's logarithm."""
+
+    __slots__ = ("width", "parts", "taps", "rate")
+
+    def __init__(self, width: int, parts: int, taps: int, rate: float):
+        self.width, self.parts, self.taps, self.rate = width, parts, taps, rate
+
+    def state_floats(self) -> int:
+        """Numbers of one sequence's state row: S, then as many inputs of the convolution as there are taps."""
+        n = self.width * (1 + self.taps)
+        return n + -n % 4
+
+
+def _rglru_check(what: str, s: RglruShape, state: torch.Tensor, **weights: torch.Tensor) -> None:
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < s.state_floats() or \
+            not state.is_cuda:
+        raise KernelError(f"{what}: state must be [slots, >= {s.state_floats()}] float32 on the GPU")
+    for n, t in weights.items():
+        _need(t, torch.float32, n)
+        if t.numel() != s.width * (s.taps if n == "taps" else 1):
+            raise KernelError(f"{what}: {n} has {t.numel()} numbers")
+
+
+def rglru_conv(x: torch.Tensor, bx: torch.Tensor, taps: torch.Tensor, bc: torch.Tensor, tiles: torch.Tensor, n_tiles: int,
+               token_seq: torch.Tensor, token_pos: torch.Tensor, seq_slot: torch.Tensor, state: torch.Tensor, shape: RglruShape,
+               rows_dtype: Optional[torch.dtype], by_part: bool) -> tuple:
+    """The causal convolution over time of ``x`` + bx (fp32 view [T, width]), reaching back into the state rows: u [T, width]
+    fp32, and with ``rows_dtype`` u as rows of a part in that type: [parts * T, width / parts] sorted by part
+    (``by_part``), else [T * parts, width / parts]."""
+    _rglru_check("rglru_conv", shape, state, bx=bx, taps=taps, bc=bc)
+    _f32_rows("rglru_conv", x=x)
+    for n, t in (("tiles", tiles), ("token_seq", token_seq), ("token_pos", token_pos), ("seq_slot", seq_slot)):
+        _need(t, torch.int32, n)
+    T = x.shape[0]
+    if x.shape[1] != shape.width:
+        raise KernelError("rglru_conv: x must have a column per channel")
+    u = torch.empty((T, shape.width), dtype=torch.float32, device=x.device)
+    rows = None
+    if rows_dtype is not None:
+        rows = torch.empty((T * shape.parts, shape.width // shape.parts), dtype=rows_dtype, device=x.device)
+    st = _lib("rglru").dlgo_rglru_conv(_ptr(x), _i(x.stride(0)), _ptr(bx), _ptr(taps), _ptr(bc), _ptr(tiles), _i(n_tiles),
+                                       _ptr(token_seq), _ptr(token_pos), _ptr(seq_slot), _ptr(state), _ll(state.stride(0)),
+                                       _ptr(u), _ptr(rows), _i(dtype_code(rows_dtype or torch.float32)),
+                                       _i(1 if by_part else 0), _i(T), _i(shape.width), _i(shape.parts), _i(shape.taps),
+                                       _stream())
+    _check(st, "rglru_conv")
+    return u, rows
+
+
+def rglru_scan(z: torch.Tensor, u: torch.Tensor, br: torch.Tensor, bi: torch.Tensor, lam: torch.Tensor, y: torch.Tensor,
+               by: Optional[torch.Tensor], x: torch.Tensor, bx: torch.Tensor, tiles: torch.Tensor, n_tiles: int, direct: bool,
+               token_seq: torch.Tensor, token_pos: torch.Tensor, seq_slot: torch.Tensor, state: torch.Tensor,
+               scratch: Optional[torch.Tensor], shape: RglruShape, out_dtype: torch.dtype) -> torch.Tensor:
+    """The recurrence over the step's tokens and its product with the other branch.  ``z`` [T * parts, 2 * width / parts]
+    fp32: the gates' logits without biases (overwritten); ``y``: the other branch, fp32 without bias and gelu (``by``) or
+    finished bfloat16 (``by`` None).  ``tiles`` cut a sequence's tokens into segments that run side by side; ``direct``:
+    one segment per sequence, else ``scratch`` holds n_tiles * 3 * width floats.  S and the newest inputs go into the
+    state rows.  Returns [T, width] in ``out_dtype``."""
+    _rglru_check("rglru_scan", shape, state, br=br, bi=bi, lam=lam, bx=bx)
+    _f32_rows("rglru_scan", z=z, u=u, x=x)
+    for n, t in (("tiles", tiles), ("token_seq", token_seq), ("token_pos", token_pos), ("seq_slot", seq_slot)):
+        _need(t, torch.int32, n)
+    T, w = u.shape
+    _need(z, None, "z")
+    if w != shape.width or z.numel() != T * 2 * w or x.shape[1] != w or y.shape != (T, w) or y.stride(1) != 1:
+        raise KernelError("rglru_scan: shapes do not fit")
+    if y.dtype != (torch.float32 if by is not None else torch.bfloat16):
+        raise KernelError("rglru_scan: y is float32 with a bias, or finished bfloat16")
+    if by is not None:
+        _need(by, torch.float32, "by")
+    if not direct and (scratch is None or scratch.dtype != torch.float32 or scratch.numel() < n_tiles * 3 * w):
+        raise KernelError(f"rglru_scan: {n_tiles} segments need {n_tiles * 3 * w} floats of scratch")
+    out = torch.empty((T, w), dtype=out_dtype, device=u.device)
+    st = _lib("rglru").dlgo_rglru_scan(
+        _ptr(z), _ptr(u), _ptr(br), _ptr(bi), _ptr(lam), _ptr(y), _i(dtype_code(y.dtype)), _i(y.stride(0)), _ptr(by), _ptr(x),
+        _i(x.stride(0)), _ptr(bx), _ptr(tiles), _i(n_tiles), _ptr(token_seq), _ptr(token_pos), _ptr(seq_slot), _ptr(state),
+        _ll(state.stride(0)), _ptr(scratch), _i(1 if direct else 0), _ptr(out), _i(dtype_code(out_dtype)), _i(w),
+        _i(shape.parts), _i(shape.taps), _f(shape.rate), _stream())
+    _check(st, "rglru_scan", 1 if direct else 2)
+    return out
+
+
+def rglru_step(proj: torch.Tensor, x_col: int, by: torch.Tensor, bx: torch.Tensor, taps: torch.Tensor, bc: torch.Tensor,
+               w_gates: torch.Tensor, br: torch.Tensor, bi: torch.Tensor, lam: torch.Tensor, token_pos: torch.Tensor,
+               seq_slot: torch.Tensor, state: torch.Tensor, shape: RglruShape) -> torch.Tensor:
+    """One token per sequence through the unit in one launch: ``proj`` [T, ld] fp32 holds y in its first ``width`` columns and
+    x from ``x_col`` on (without biases); ``w_gates`` [parts, 2 * width / parts, width / parts] (rows of r, then of i) in
+    the run's type, which is the result's [T, width]."""
+    _rglru_check("rglru_step", shape, state, by=by, bx=bx, taps=taps, bc=bc, br=br, bi=bi, lam=lam)
+    _f32_rows("rglru_step", proj=proj)
+    _need(w_gates, None, "w_gates")
+    _need(token_pos, torch.int32, "token_pos")
+    _need(seq_slot, torch.int32, "seq_slot")
+    b = shape.width // shape.parts
+    if tuple(w_gates.shape) != (shape.parts, 2 * b, b) or proj.shape[1] < x_col + shape.width or x_col < shape.width:
+        raise KernelError("rglru_step: shapes do not fit")
+    T = proj.shape[0]
+    out = torch.empty((T, shape.width), dtype=w_gates.dtype, device=proj.device)
+    st = _lib("rglru").dlgo_rglru_step(
+        _ptr(proj), _i(proj.stride(0)), _i(x_col), _ptr(by), _ptr(bx), _ptr(taps), _ptr(bc), _ptr(w_gates), _ptr(br), _ptr(bi),
+        _ptr(lam), _ptr(token_pos), _ptr(seq_slot), _ptr(state), _ll(state.stride(0)), _ptr(out),
+        _i(dtype_code(w_gates.dtype)), _i(T), _i(shape.width), _i(shape.parts), _i(shape.taps), _f(shape.rate), _stream())
+    _check(st, "rglru_step")
     return out
 
 
@@ -1152,14 +1408,18 @@ def headnorm_rope_append(proj: torch.Tensor, bias: Optional[torch.Tensor], w_q: 
                          token_pos: torch.Tensor, token_seq: torch.Tensor, seq_slot: torch.Tensor,
                          page_table: torch.Tensor, kpages: torch.Tensor, vpages: torch.Tensor, num_heads: int,
                          num_kv_heads: int, head_dim: int, values_from_keys: bool, write_cache: bool = True,
-                         clear: bool = False, norm_dim: Optional[int] = None) -> torch.Tensor:
+                         clear: bool = False, norm_dim: Optional[int] = None, qk_dim: Optional[int] = None,
+                         v_dim: Optional[int] = None, v_scale: float = 1.0) -> torch.Tensor:
     """From the fp32 projection ``proj`` [T, ld] (query heads, key heads and, unless ``values_from_keys``, value
     heads; ``bias`` fp32 per column added first): per-head RMS norm of queries and keys with the weights ``w_q`` /
     ``w_k`` (None: no norm), rotation of the first ``rotary_dim`` numbers of each head (pairs (i, i + rotary_dim/2))
     by the fp32 angle ``float(position) * freq[i]``, keys and values stored at their positions' pages (with
     ``values_from_keys`` a value is its key as projected, before norm and rotation).  Returns the queries
     [T, heads * head_dim] in the cache's type.  ``clear`` leaves zeros in ``proj``.  ``norm_dim``: the number of
-    entries the head norm's mean runs over (heads laid out with trailing zeros; default ``head_dim``)."""
+    entries the head norm's mean runs over (heads laid out with trailing zeros; default ``qk_dim``).  ``qk_dim`` and
+    ``v_dim`` (default ``head_dim``): a projected head's own numbers; in the cache and in the result every head is
+    ``head_dim`` wide with zeros behind them.  Value heads are kept times ``v_scale``."""
+    qk_dim, v_dim = qk_dim or head_dim, v_dim or qk_dim or head_dim
     if proj.dtype != torch.float32 or proj.dim() != 2 or proj.stride(1) != 1:
         raise KernelError("headnorm_rope_append: proj must be 2-D float32 with unit inner stride")
     for n, t in (("bias", bias), ("w_q", w_q), ("w_k", w_k), ("freq", freq)):
@@ -1170,12 +1430,12 @@ def headnorm_rope_append(proj: torch.Tensor, bias: Optional[torch.Tensor], w_q: 
     _need(kpages, None, "kpages")
     _need(vpages, kpages.dtype, "vpages")
     T = proj.shape[0]
-    cols = (num_heads + (1 if values_from_keys else 2) * num_kv_heads) * head_dim
+    cols = (num_heads + num_kv_heads) * qk_dim + (0 if values_from_keys else num_kv_heads * v_dim)
     if proj.shape[1] < cols or (bias is not None and bias.numel() != cols):
         raise KernelError(f"headnorm_rope_append: the projection (and its bias) must have {cols} columns")
     for n, t in (("w_q", w_q), ("w_k", w_k)):
-        if t is not None and t.numel() != head_dim:
-            raise KernelError(f"headnorm_rope_append: {n} must have head_dim elements")
+        if t is not None and t.numel() != qk_dim:
+            raise KernelError(f"headnorm_rope_append: {n} must have qk_dim elements")
     if rotary_dim and (freq is None or freq.numel() != rotary_dim // 2):
         raise KernelError("headnorm_rope_append: one frequency per rotated pair")
     if kpages.shape[-1] != head_dim or kpages.shape[-3] != num_kv_heads:
@@ -1184,9 +1444,9 @@ def headnorm_rope_append(proj: torch.Tensor, bias: Optional[torch.Tensor], w_q: 
     st = _lib("headnorm_rope").dlgo_headnorm_rope_append(
         _ptr(proj), _i(proj.stride(0)), _ptr(bias), _ptr(w_q), _ptr(w_k), _f(eps), _ptr(freq), _i(rotary_dim),
         _ptr(token_pos), _ptr(token_seq), _ptr(seq_slot), _ptr(page_table), _i(page_table.shape[1]), _ptr(kpages),
-        _ptr(vpages), _ptr(q), _i(dtype_code(kpages.dtype)), _i(T), _i(num_heads), _i(num_kv_heads), _i(head_dim),
-        _i(kpages.shape[-2]), _i(1 if values_from_keys else 0), _i(1 if write_cache else 0), _i(1 if clear else 0),
-        _i(norm_dim or head_dim), _stream())
+        _ptr(vpages), _ptr(q), _i(dtype_code(kpages.dtype)), _i(T), _i(num_heads), _i(num_kv_heads), _i(qk_dim),
+        _i(v_dim), _i(head_dim), _i(kpages.shape[-2]), _i(1 if values_from_keys else 0), _i(1 if write_cache else 0),
+        _i(1 if clear else 0), _i(norm_dim or qk_dim), _f(v_scale), _stream())
     _check(st, "headnorm_rope_append")
     return q
 
@@ -1223,11 +1483,12 @@ MOE_FEW_ROWS, MOE_TILE_ROWS, MOE_TC_ROWS, MOE_TC_PAIR_ROWS = 8, 64, 128, 256    
 def moe_router(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], n_outputs: int,
                has_gate: bool, top: int, groups: int, keep: int, sigmoid_scores: bool = False,
                renormalize: bool = False, plan: Optional[tuple] = None, logit_bias: Optional[torch.Tensor] = None,
-               weight_scale: float = 1.0):
+               weight_scale: float = 1.0, group_top: int = 1):
     """Router of a mixture of experts for ``h`` [T, d]: returns (chosen outputs [T, top] int32, their weights
     [T, top] fp32, times ``weight_scale``; gate [T] fp32 or None, plan).  ``w_router`` is fp32 [n_outputs (+ 1 gate row), d].
     ``plan`` = (experts that hold tensors, rows per tile): the :class:`MoEPlan` of :func:`moe_plan` is made as well,
-    in the choice's own launch where the step has few tokens, else by a launch of its own; without it None."""
+    in the choice's own launch where the step has few tokens, else by a launch of its own; without it None.
+    ``group_top``: a group's score is the sum of its one or two largest choice scores."""
     _need(w_router, torch.float32, "w_router")
     if h.dim() != 2 or h.stride(1) != 1:
         raise KernelError("moe_router: h must be 2-D with unit inner stride")
@@ -1252,7 +1513,7 @@ def moe_router(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[tor
     st = _lib("moe").dlgo_moe_router(
         _ptr(h), _i(dtype_code(h.dtype)), _i(h.stride(0)), _ptr(w_router), _ptr(correction), _ptr(logit_bias), _ptr(z), _ptr(idx),
         _ptr(wt), _ptr(gate), _i(T), _i(d), _i(n_outputs), _i(1 if has_gate else 0), _i(top), _i(groups), _i(keep),
-        _i(1 if sigmoid_scores else 0), _i(1 if renormalize else 0), _f(weight_scale), _i(plan[0] if p is not None else 0),
+        _i(group_top), _i(1 if sigmoid_scores else 0), _i(1 if renormalize else 0), _f(weight_scale), _i(plan[0] if p is not None else 0),
         _i(plan[1] if p is not None else 0), _ptr(p.offsets if p is not None else None),
         _ptr(p.sorted_pair if p is not None else None), _ptr(p.tile_expert if p is not None else None),
         _ptr(p.tile_row0 if p is not None else None), _ptr(p.n_tiles if p is not None else None),
@@ -1293,6 +1554,22 @@ def moe_plan(idx: torch.Tensor, n_experts: int, tile_rows: int, into: Optional[M
                                    _ptr(p.sorted_pair), _ptr(p.tile_expert), _ptr(p.tile_row0), _ptr(p.n_tiles),
                                    _i(p.max_tiles), _stream())
     _check(st, "moe_plan")
+    return p
+
+
+@functools.lru_cache(maxsize=32)
+def part_plan(parts: int, rows: int, tile_rows: int, device: torch.device) -> MoEPlan:
+    """The plan of a grouped contraction whose groups are ``parts`` equal parts of every one of ``rows`` rows (part p's
+    rows in order: sorted row p * rows + t is pair t * parts + p)."""
+    p = MoEPlan()
+    per = -(-rows // tile_rows)
+    p.pairs, p.tile_rows, p.max_tiles = parts * rows, tile_rows, parts * per
+    ar = torch.arange(parts, dtype=torch.int32)
+    p.offsets = (torch.arange(parts + 1, dtype=torch.int32) * rows).to(device)
+    p.sorted_pair = (ar[:, None] + torch.arange(rows, dtype=torch.int32)[None, :] * parts).reshape(-1).to(device)
+    p.tile_expert = ar[:, None].expand(parts, per).reshape(-1).contiguous().to(device)
+    p.tile_row0 = (ar[:, None] * rows + torch.arange(per, dtype=torch.int32)[None, :] * tile_rows).reshape(-1).to(device)
+    p.n_tiles = torch.tensor([p.max_tiles], dtype=torch.int32).to(device)
     return p
 
 
@@ -1346,7 +1623,8 @@ def moe_gather_rows(plan: MoEPlan, src: torch.Tensor, div: int, scale: Optional[
     return dst
 
 
-def moe_gemm_tc(plan: MoEPlan, a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scatter: bool, act: int) -> torch.Tensor:
+def moe_gemm_tc(plan: MoEPlan, a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scatter: bool, act: int,
+                glu: Optional[ClampedGlu] = None) -> torch.Tensor:
     """The grouped contraction on the tensor cores (bfloat16, a plan with tiles of 128 rows): ``a`` holds the rows
     in sorted order, ``w`` is [experts, N, K]; ``out`` (bfloat16 or fp32) receives row r, or with ``scatter`` row
     pair(r)."""
@@ -1365,7 +1643,7 @@ def moe_gemm_tc(plan: MoEPlan, a: torch.Tensor, w: torch.Tensor, out: torch.Tens
         _ptr(a), _ll(a.shape[0]), _ll(a.stride(0)), _ptr(w), _i(E), _ptr(out), _ll(out.stride(0)),
         _ptr(plan.sorted_pair if scatter else None), _ptr(plan.offsets), _ptr(plan.tile_expert), _ptr(plan.tile_row0),
         _ptr(plan.n_tiles), _i(plan.max_tiles), _i(plan.tile_rows), _i(N), _i(Kd), _i(act),
-        _i(1 if out.dtype == torch.float32 else 0), _stream())
+        _i(1 if out.dtype == torch.float32 else 0), *_glu_args(glu), _stream())
     _check(st, "moe_gemm_tc")
     return out
 
@@ -1434,12 +1712,21 @@ def attention_scratch_floats(T: int, num_heads: int, head_dim: int, n_splits: in
     return 0 if n_splits <= 1 else T * num_heads * n_splits * (head_dim + 2)
 
 
+def _check_sink(sink: Optional[torch.Tensor], num_heads: int) -> None:
+    if sink is not None:
+        _need(sink, torch.float32, "sink")
+        if sink.numel() != num_heads:
+            raise KernelError("a sink is one number per query head")
+
+
 def attention(q: torch.Tensor, ldq: int, T: int, kpages: torch.Tensor, vpages: torch.Tensor,
               page_table: torch.Tensor, tiles: torch.Tensor, tile_tokens_max: int, seq_slot: torch.Tensor,
               token_pos: torch.Tensor, out: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int,
               scale: float, window: int = 0, n_splits: int = 1, gchunk: int = 1,
-              scratch: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Causal grouped-query attention of T packed tokens over the paged cache."""
+              scratch: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal grouped-query attention of T packed tokens over the paged cache.  ``sink`` [heads] fp32: its exponential
+    joins the softmax's denominator."""
+    _check_sink(sink, num_heads)
     _need(out, q.dtype, "out")
     _need(kpages, q.dtype, "kpages")
     _need(vpages, q.dtype, "vpages")
@@ -1453,7 +1740,7 @@ def attention(q: torch.Tensor, ldq: int, T: int, kpages: torch.Tensor, vpages: t
         _ptr(q), _i(dtype_code(q.dtype)), _i(T), _i(ldq), _ptr(kpages), _ptr(vpages), _ptr(page_table),
         _i(page_table.shape[1]), _ptr(tiles), _i(tiles.shape[0]), _i(tile_tokens_max), _ptr(seq_slot),
         _ptr(token_pos), _ptr(out), _i(out.stride(0)), _ptr(scratch), _i(num_heads), _i(num_kv_heads), _i(head_dim),
-        _i(kpages.shape[-2]), _i(n_splits), _i(gchunk), _i(window), _f(scale), _stream())
+        _i(kpages.shape[-2]), _i(n_splits), _i(gchunk), _i(window), _f(scale), _ptr(sink), _stream())
     _check(st, "attention", 2 if n_splits > 1 else 1)
     return out
 
@@ -1598,7 +1885,8 @@ def gemm_tc_workspace_floats(ra: int, rb: int, bn: int, splits: int) -> int:
 
 def gemm_tc(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, transposed: bool, epilogue: int, bn: int,
             splits: int = 1, workspace: Optional[torch.Tensor] = None,
-            counters: Optional[torch.Tensor] = None, static_operand: int = 0, pair_tile: int = 0) -> torch.Tensor:
+            counters: Optional[torch.Tensor] = None, static_operand: int = 0, pair_tile: int = 0,
+            glu: Optional[ClampedGlu] = None) -> torch.Tensor:
     """D[Ra, Rb] = a[Ra, K] . b[Rb, K]^T on the tensor cores (bf16 in, fp32 accumulate).
 
     ``out`` receives D (``transposed``: D^T) through ``epilogue``; with ``splits`` > 1 the K range is
@@ -1608,7 +1896,7 @@ def gemm_tc(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, transposed: boo
     ``TC_PARTIAL`` (transposed only): every K-slice leaves its fp32 tile in ``out`` [splits, Rb, Ra] for the
     reader to add in order.  ``TC_RED_F32`` (transposed only): every K-slice adds itself into the fp32
     ``out`` with reductions at the memory; no workspace, and the order of the adds (the sum's last bits) is
-    not fixed.
+    not fixed.  ``glu`` (with ``TC_SWIGLU``): the clamped form.
     """
     if epilogue == TC_RED_F32 and not transposed:
         raise KernelError("gemm_tc: the atomic add is for transposed products")
@@ -1642,6 +1930,15 @@ def gemm_tc(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, transposed: boo
         if out.dtype != want_dtype:
             raise KernelError(f"gemm_tc: out must be {want_dtype}")
         ldo = out.stride(0)
+    if glu is not None:
+        if epilogue != TC_SWIGLU:
+            raise KernelError("gemm_tc: the clamped form goes with the gated epilogue")
+        st = _lib("gemm_tc").dlgo_gemm_tc_clamped_glu(
+            _ptr(a), _i(ra), _i(a.stride(0)), _ptr(b), _i(rb), _i(b.stride(0)), _i(k), _ptr(out), _i(ldo),
+            _i(1 if transposed else 0), _i(bn), _i(splits), _ptr(workspace), _ptr(counters), _i(static_operand),
+            _i(pair_tile), *_glu_args(glu), _stream())
+        _check(st, "gemm_tc")
+        return out
     st = _lib("gemm_tc").dlgo_gemm_tc(_ptr(a), _i(ra), _i(a.stride(0)), _ptr(b), _i(rb), _i(b.stride(0)), _i(k),
                                       _ptr(out), _i(ldo), _i(1 if transposed else 0), _i(epilogue), _i(bn),
                                       _i(splits), _ptr(workspace), _ptr(counters), _i(static_operand), _i(pair_tile),
@@ -1778,12 +2075,15 @@ def attention_decode_mma(q: Optional[torch.Tensor], ldq: int, B: int, kpages: to
                          window: int = 0, n_splits: int = 1, keys_per_tile: int = 16,
                          scratch: Optional[torch.Tensor] = None, parts: Optional[torch.Tensor] = None,
                          cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None,
-                         write_cache: bool = True, clear_parts: bool = False) -> torch.Tensor:
+                         write_cache: bool = True, clear_parts: bool = False, sink: Optional[torch.Tensor] = None,
+                         split: bool = False) -> torch.Tensor:
     """Attention of one new token per sequence over its cached keys and values, bfloat16, on the
     tensor cores (mma.sync); 2..8 slices combine inside a thread-block cluster, more go through
     ``scratch`` (``attention_scratch_floats`` floats) and a second kernel.  With ``parts`` (the q|k|v
     projection as fp32 [slices, sequences, columns], unrotated) the kernel sums the slices, rotates q and k
-    and appends k and v itself; ``clear_parts`` (one slice, at most 8 page slices): the sum is left zero."""
+    and appends k and v itself; ``clear_parts`` (one slice, at most 8 page slices): the sum is left zero.  ``sink``
+    [heads] joins the denominator; ``split``: probabilities meet the values as two bfloat16 terms."""
+    _check_sink(sink, num_heads)
     for n, t in (("out", out), ("kpages", kpages), ("vpages", vpages)):
         _need(t, torch.bfloat16, n)
     for n, t in (("page_table", page_table), ("seq_slot", seq_slot), ("token_pos", token_pos)):
@@ -1823,7 +2123,7 @@ def attention_decode_mma(q: Optional[torch.Tensor], ldq: int, B: int, kpages: to
         _ptr(seq_slot), _ptr(token_pos), _ptr(out), _i(out.stride(0)), _i(num_heads), _i(num_kv_heads), _i(head_dim),
         _i(page_size), _i(n_splits), _i(window), _f(scale), _i(keys_per_tile),
         _ptr(scratch if n_splits > 8 else None), _ptr(parts), _i(S), _ll(part_stride), _ptr(cos), _ptr(sin),
-        _i(1 if write_cache else 0), _i(1 if clear_parts else 0), _stream())
+        _i(1 if write_cache else 0), _i(1 if clear_parts else 0), _ptr(sink), _i(1 if split else 0), _stream())
     _check(st, "attention_decode_mma", 2 if n_splits > 8 else 1)
     return out
 
@@ -1836,11 +2136,13 @@ def attention_decode(q: torch.Tensor, ldq: int, B: int, kpages: torch.Tensor, vp
                      page_table: torch.Tensor, seq_slot: torch.Tensor, token_pos: torch.Tensor, out: torch.Tensor,
                      num_heads: int, num_kv_heads: int, head_dim: int, scale: float, window: int = 0,
                      n_splits: int = 1, scratch: Optional[torch.Tensor] = None,
-                     counters: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     counters: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of one new token per sequence over its cached keys and values.
 
     ``counters`` (int32, zero, at least ``B * num_kv_heads * ceil(group / 4)``): with them the slice that
-    finishes last combines the partial results; without them a second kernel does."""
+    finishes last combines the partial results; without them a second kernel does.  ``sink`` [heads] fp32 joins the
+    denominator."""
+    _check_sink(sink, num_heads)
     _need(out, q.dtype, "out")
     _need(kpages, q.dtype, "kpages")
     _need(vpages, q.dtype, "vpages")
@@ -1858,7 +2160,7 @@ def attention_decode(q: torch.Tensor, ldq: int, B: int, kpages: torch.Tensor, vp
         _ptr(q), _i(dtype_code(q.dtype)), _i(B), _i(ldq), _ptr(kpages), _ptr(vpages), _ptr(page_table),
         _i(page_table.shape[1]), _ptr(seq_slot), _ptr(token_pos), _ptr(out), _i(out.stride(0)), _ptr(scratch),
         _ptr(counters), _i(num_heads), _i(num_kv_heads), _i(head_dim), _i(kpages.shape[-2]), _i(n_splits), _i(window),
-        _f(scale), _stream())
+        _f(scale), _ptr(sink), _stream())
     _check(st, "attention_decode", 2 if (n_splits > 1 and counters is None and scratch is not None) else 1)
     return out
 
@@ -1874,8 +2176,11 @@ def attention_prefill_tc_takes(dtype: torch.dtype, head_dim: int, page_size: int
 def attention_prefill_tc(q: torch.Tensor, ldq: int, T: int, kpages: torch.Tensor, vpages: torch.Tensor,
                          page_table: torch.Tensor, tiles: torch.Tensor, seq_slot: torch.Tensor,
                          token_pos: torch.Tensor, out: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int,
-                         scale: float, window: int = 0) -> torch.Tensor:
-    """Causal attention of packed prompt tokens on the tensor cores; tiles hold at most 128 tokens each."""
+                         scale: float, window: int = 0, sink: Optional[torch.Tensor] = None,
+                         split: bool = False) -> torch.Tensor:
+    """Causal attention of packed prompt tokens on the tensor cores; tiles hold at most 128 tokens each.  ``sink``
+    [heads] joins the denominator; ``split``: probabilities enter P V as two bfloat16 terms."""
+    _check_sink(sink, num_heads)
     _need(out, torch.bfloat16, "out")
     _need(kpages, torch.bfloat16, "kpages")
     _need(vpages, torch.bfloat16, "vpages")
@@ -1886,7 +2191,8 @@ def attention_prefill_tc(q: torch.Tensor, ldq: int, T: int, kpages: torch.Tensor
     st = _lib("attention_prefill_tc").dlgo_attention_prefill_tc(
         _ptr(q), _i(T), _i(ldq), _ptr(kpages), _ptr(vpages), _i(kpages.shape[0]), _ptr(page_table),
         _i(page_table.shape[1]), _ptr(tiles), _i(tiles.shape[0]), _ptr(seq_slot), _ptr(token_pos), _ptr(out),
-        _i(out.stride(0)), _i(num_heads), _i(num_kv_heads), _i(head_dim), _i(window), _f(scale), _stream())
+        _i(out.stride(0)), _i(num_heads), _i(num_kv_heads), _i(head_dim), _i(window), _f(scale), _ptr(sink),
+        _i(1 if split else 0), _stream())
     _check(st, "attention_prefill_tc")
     return out
 

@@ -2,8 +2,8 @@
 //
 // 1. moe_router:   z = Wr h in fp32 (Wr is kept in fp32), scores s = softmax(z) (or sigmoid(z)) over all
 //                  router outputs, choice scores c = s + correction, group-limited choice of `top` outputs
-//                  (outputs form `groups` equal groups of neighbours; a group's score is its largest choice
-//                  score; only outputs of the `keep` best groups can be chosen, the others count as minus
+//                  (outputs form `groups` equal groups of neighbours; a group's score is the sum of its `group_top`
+//                  largest choice scores, one or two; only outputs of the `keep` best groups can be chosen, the others count as minus
 //                  infinity), weights = the chosen outputs' s (optionally renormalised) times a constant.  A bias on the logits
 //                  (`zbias`, one number per output) is part of z: it moves scores and weights alike.  A further row of Wr
 //                  (`has_gate`) gives a per-token gate sigmoid(w_g . h) for a shared expert.
@@ -150,8 +150,8 @@ constexpr int RC_WARPS = 4;
 __device__ __forceinline__ void choose_token(const float* zg, const float* __restrict__ corr,
                                              const float* __restrict__ zbias, int* idx, float* wt, float* gate,
                                              int t, int n, int has_gate, int top, int groups, int keep,
-                                             int sigmoid_scores, int renormalize, float wscale, float* zt, float* ct, float* gt,
-                                             int lane) {
+                                             int group_top, int sigmoid_scores, int renormalize, float wscale, float* zt,
+                                             float* ct, float* gt, int lane) {
   const int rows = n + (has_gate ? 1 : 0);
   for (int j = lane; j < rows; j += 32) zt[j] = zg[(size_t)t * rows + j] + (zbias != nullptr && j < n ? zbias[j] : 0.f);
   __syncwarp();
@@ -176,9 +176,13 @@ __device__ __forceinline__ void choose_token(const float* zg, const float* __res
   if (keep < groups) {
     const int gsz = n / groups;
     for (int g = lane; g < groups; g += 32) {
-      float m = -CUDART_INF_F;
-      for (int j = 0; j < gsz; ++j) m = fmaxf(m, ct[g * gsz + j]);
-      gt[g] = m;
+      float m = -CUDART_INF_F, second = -CUDART_INF_F;
+      for (int j = 0; j < gsz; ++j) {
+        const float c = ct[g * gsz + j];
+        second = fmaxf(second, fminf(m, c));
+        m = fmaxf(m, c);
+      }
+      gt[g] = group_top == 2 && gsz > 1 ? m + second : m;
     }
     __syncwarp();
     // a group that is found leaves the next rounds with a score of minus infinity (choice scores are finite);
@@ -214,14 +218,14 @@ __device__ __forceinline__ void choose_token(const float* zg, const float* __res
     __syncwarp();
   }
   if (renormalize)
-    for (int r = lane; r < top; r += 32) wt[(size_t)t * top + r] /= wsum;
+    for (int r = lane; r < top; r += 32) wt[(size_t)t * top + r] /= wsum + 1e-20f;
 }
 
 __global__ void __launch_bounds__(RC_WARPS * 32)
 moe_choose_kernel(const float* zg, const float* __restrict__ corr, const float* __restrict__ zbias,
                   int* idx,
                   float* wt, float* gate, int tokens, int n, int has_gate, int top, int groups,
-                  int keep, int sigmoid_scores, int renormalize, float wscale) {
+                  int keep, int group_top, int sigmoid_scores, int renormalize, float wscale) {
   extern __shared__ float rt_smem[];
   pdl_launch_dependents();
   const int rows = n + (has_gate ? 1 : 0);
@@ -230,7 +234,7 @@ moe_choose_kernel(const float* zg, const float* __restrict__ corr, const float* 
   const int t = blockIdx.x * RC_WARPS + warp;
   pdl_wait();
   if (t >= tokens) return;
-  choose_token(zg, corr, zbias, idx, wt, gate, t, n, has_gate, top, groups, keep, sigmoid_scores, renormalize, wscale, zt, zt + rows,
+  choose_token(zg, corr, zbias, idx, wt, gate, t, n, has_gate, top, groups, keep, group_top, sigmoid_scores, renormalize, wscale, zt, zt + rows,
                zt + rows + n, lane);
 }
 
@@ -291,7 +295,7 @@ __global__ void __launch_bounds__(PLAN_THREADS)
 moe_choose_plan_kernel(const float* zg, const float* __restrict__ corr,
                        const float* __restrict__ zbias, int* idx,
                        float* wt, float* gate, int tokens, int n, int has_gate, int top,
-                       int groups, int keep, int sigmoid_scores, int renormalize, float wscale, int n_experts, int tile_rows,
+                       int groups, int keep, int group_top, int sigmoid_scores, int renormalize, float wscale, int n_experts, int tile_rows,
                        int* offsets, int* sorted_pair, int* tile_expert,
                        int* tile_row0, int* n_tiles, int max_tiles) {
   extern __shared__ float rt_smem[];
@@ -304,7 +308,7 @@ moe_choose_plan_kernel(const float* zg, const float* __restrict__ corr,
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) count[e] = 0;
   pdl_wait();
   for (int t = warp; t < tokens; t += n_warps) {
-    choose_token(zg, corr, zbias, idx, wt, gate, t, n, has_gate, top, groups, keep, sigmoid_scores, renormalize, wscale, zt, zt + rows,
+    choose_token(zg, corr, zbias, idx, wt, gate, t, n, has_gate, top, groups, keep, group_top, sigmoid_scores, renormalize, wscale, zt, zt + rows,
                  zt + rows + n, lane);
     __syncwarp();
   }
@@ -597,12 +601,13 @@ static void launch_logits(const void* h, int ldh, const float* Wr, float* z, int
 DLGO_EXPORT int dlgo_moe_router(const void* h, int dtype, int ldh, const float* Wr, const float* corr,
                                 const float* zbias, float* z, int* idx,
                                 float* wt, float* gate, int tokens, int d, int n, int has_gate, int top, int groups,
-                                int keep, int sigmoid_scores, int renormalize, float wscale, int plan_experts, int tile_rows,
+                                int keep, int group_top, int sigmoid_scores, int renormalize, float wscale, int plan_experts, int tile_rows,
                                 int* offsets, int* sorted_pair, int* tile_expert, int* tile_row0, int* n_tiles,
                                 int max_tiles, int* fused, cudaStream_t stream) {
   if (fused != nullptr) *fused = 0;
   if (tokens <= 0) return DLGO_OK;
-  if (n <= 0 || top <= 0 || top > n || groups <= 0 || n % groups || keep <= 0 || keep > groups || d <= 0)
+  if (n <= 0 || top <= 0 || top > n || groups <= 0 || n % groups || keep <= 0 || keep > groups || d <= 0 ||
+      group_top < 1 || group_top > 2)
     return DLGO_ERR_SIZE;
   const int rows = n + (has_gate ? 1 : 0);
   const size_t smem = sizeof(float) * RC_WARPS * ((size_t)rows + n + groups);
@@ -618,15 +623,15 @@ DLGO_EXPORT int dlgo_moe_router(const void* h, int dtype, int ldh, const float* 
     const int pairs = tokens * top;
     if (both <= 48 * 1024 && tile_rows > 0 && max_tiles >= (pairs + tile_rows - 1) / tile_rows + plan_experts) {
       launch_kernel(moe_choose_plan_kernel, dim3(1), dim3(warps * 32), both, stream, (const float*)z, corr, zbias, idx, wt, gate,
-                    tokens, n, has_gate, top, groups, keep, sigmoid_scores, renormalize, wscale, plan_experts, tile_rows, offsets,
+                    tokens, n, has_gate, top, groups, keep, group_top, sigmoid_scores, renormalize, wscale, plan_experts, tile_rows, offsets,
                     sorted_pair, tile_expert, tile_row0, n_tiles, max_tiles);
       *fused = 1;
       return launch_status();
     }
   }
   launch_kernel(moe_choose_kernel, dim3((tokens + RC_WARPS - 1) / RC_WARPS), dim3(RC_WARPS * 32), smem, stream,
-                (const float*)z, corr, zbias, idx, wt, gate, tokens, n, has_gate, top, groups, keep, sigmoid_scores, renormalize,
-                wscale);
+                (const float*)z, corr, zbias, idx, wt, gate, tokens, n, has_gate, top, groups, keep, group_top, sigmoid_scores,
+                renormalize, wscale);
   return launch_status();
 }
 

@@ -26,7 +26,7 @@ using namespace sm100;
 constexpr int GT_M = 128, GT_K = 64, GT_UMMA_K = 16, GT_THREADS = 192;
 enum { GT_ACT_NONE = 0, GT_ACT_RELU2 = 1, GT_ACT_SILU = 2, GT_ACT_GELU_TANH = 3,
        // W's rows come in blocks of 16 gate rows followed by their 16 up rows: 32 columns of the accumulator give 16
-       // columns silu(gate) * up of an output that is N / 2 wide (N a multiple of 32; single-CTA tiles only)
+       // columns silu(gate) * up (or the clamped form, GluForm) of an output that is N / 2 wide (N a multiple of 32; single-CTA tiles only)
        GT_ACT_SWIGLU16 = 4 };
 
 __device__ int g_moe_tc_error = 0;
@@ -41,6 +41,7 @@ struct GroupedTcParams {
   long long ldo;
   int out_f32, act, N, K, stages;
   int nacc;                 // accumulators per CTA in tensor memory (1 or 2; the persistent single-CTA kernel)
+  GluForm glu;              // GT_ACT_SWIGLU16: which form
 };
 
 __device__ __forceinline__ float gt_act(float v, int act) {
@@ -184,8 +185,16 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
         if (!mine) continue;
         if (p.act == GT_ACT_SWIGLU16) {              // (N is a multiple of 32: no ragged edge)
           const int col = (n0 + c0) >> 1;
+          if (p.glu.limit > 0.f) {
 #pragma unroll
-          for (int q = 0; q < 16; ++q) v[q] = v[q] / (1.f + __expf(-v[q])) * v[q + 16];
+            for (int q = 0; q < 16; ++q) {
+              glu_clamp(p.glu, v[q], v[q + 16]);
+              v[q] = v[q] / (1.f + __expf(-p.glu.alpha * v[q])) * v[q + 16];
+            }
+          } else {
+#pragma unroll
+            for (int q = 0; q < 16; ++q) v[q] = v[q] / (1.f + __expf(-v[q])) * v[q + 16];
+          }
           if (p.out_f32) {
             float* dst = (float*)p.out + dst_row + col;
 #pragma unroll
@@ -592,7 +601,8 @@ DLGO_EXPORT int dlgo_moe_gemm_tc_takes(int N, int K) { return (N > 0 && K > 0 &&
 DLGO_EXPORT int dlgo_moe_gemm_tc(const void* A, long long a_rows, long long lda, const void* W, int experts, void* out,
                                  long long ldo, const int* o_scatter, const int* offsets, const int* tile_expert,
                                  const int* tile_row0, const int* n_tiles, int max_tiles, int tile_rows, int N, int K,
-                                 int act, int out_f32, cudaStream_t stream) {
+                                 int act, int out_f32, float glu_limit, float glu_alpha, float glu_offset,
+                                 cudaStream_t stream) {
   if (max_tiles <= 0 || max_tiles > 65535 || a_rows <= 0 || experts <= 0) return DLGO_ERR_SIZE;
   if (!dlgo_moe_gemm_tc_takes(N, K)) return DLGO_ERR_SIZE;
   if (act == GT_ACT_SWIGLU16 && (N % 32 != 0 || tile_rows != GT_M)) return DLGO_ERR_SIZE;
@@ -603,7 +613,7 @@ DLGO_EXPORT int dlgo_moe_gemm_tc(const void* A, long long a_rows, long long lda,
     if (st != DLGO_OK) return st;
     st = make_map(&mb, W, (long long)experts * N, K, K, 128);
     if (st != DLGO_OK) return st;
-    GroupedTcParams p{offsets, tile_expert, tile_row0, n_tiles, o_scatter, out, ldo, out_f32, act, N, K, 0, 1};
+    GroupedTcParams p{offsets, tile_expert, tile_row0, n_tiles, o_scatter, out, ldo, out_f32, act, N, K, 0, 1, GluForm{glu_limit, glu_alpha, glu_offset}};
     return launch_grouped_pair(ma, mb, p, max_tiles, stream);
   }
   if (tile_rows != GT_M) return DLGO_ERR_SIZE;
@@ -613,7 +623,7 @@ DLGO_EXPORT int dlgo_moe_gemm_tc(const void* A, long long a_rows, long long lda,
   if (st != DLGO_OK) return st;
   st = make_map(&mb, W, (long long)experts * N, K, K, bn);
   if (st != DLGO_OK) return st;
-  GroupedTcParams p{offsets, tile_expert, tile_row0, n_tiles, o_scatter, out, ldo, out_f32, act, N, K, 0, 1};
+  GroupedTcParams p{offsets, tile_expert, tile_row0, n_tiles, o_scatter, out, ldo, out_f32, act, N, K, 0, 1, GluForm{glu_limit, glu_alpha, glu_offset}};
   if (bn == 256) return launch_grouped<256>(ma, mb, p, max_tiles, 100, stream);
   if (bn == 64) return launch_grouped<64>(ma, mb, p, max_tiles, 75, stream);
   return launch_grouped<128>(ma, mb, p, max_tiles, 66, stream);

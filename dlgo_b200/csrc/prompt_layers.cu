@@ -28,7 +28,7 @@ typedef int (*RopeAppendFn)(void* qkv, int dtype, int T, int ld, const float* co
                             long long part_stride, int clear_parts, cudaStream_t stream);
 typedef int (*AttentionFn)(const void* q, int T, int ldq, const void* kpages, const void* vpages, int n_pages,
                            const int* page_table, int max_pages, const int* tiles, int n_tiles, const int* seq_slot,
-                           const int* token_pos, void* out, int ldo, int Hq, int Hkv, int hd, int window, float scale,
+                           const int* token_pos, void* out, int ldo, int Hq, int Hkv, int hd, int window, float scale, const float* sink, int split,
                            cudaStream_t stream);
 
 // as in gemm_tc.cu
@@ -148,7 +148,7 @@ DLGO_EXPORT int dlgo_prompt_layers(const DlgoPromptEntryPoints* fn, const DlgoPr
     }
     DLGO_STEP(fn->attention(p->qkv, T, n_cols, L.kpages, L.vpages, L.n_pages, p->page_table, p->max_pages, p->tiles,
                             p->n_tiles, p->seq_slot, p->token_pos, p->attn_out, q_dim, s->heads, s->kv_heads,
-                            s->head_dim, s->window, s->scale, stream));
+                            s->head_dim, s->window, s->scale, nullptr, 0, stream));
     DLGO_STEP(fn->gemm_tc(p->attn_out, T, q_dim, L.w_o, d, q_dim, q_dim, p->residual, d, 0, TC_ADD_F32, p->bn[1], 1,
                           nullptr, nullptr, 2, p->pair[1], stream));
     DLGO_STEP(fn->rmsnorm(p->residual, L.norm2_w, p->x, DLGO_BF16, nullptr, T, d, L.eps2, stream));

@@ -15,6 +15,10 @@
 // state's product, whose register layout is that of the second operand of C S.  Products are warp-level
 // (mma.sync m16n8k16): each is a few thousand multiplications between element-wise passes over the accumulators, which
 // stay in registers.
+//
+// With a normalizer (matrix memory) the recurrence also runs on x = 1: n_t = f_t n_(t-1) + d_t B_t, and n_t . C_t leaves
+// per token and head.  Its chunk form needs the row sums of the masked products, which pass through registers anyway;
+// the blocks of a head's first 64 columns carry it.
 #include "ssd.cuh"
 
 namespace dlgo {
@@ -68,6 +72,9 @@ struct SsdChunkArgs {
   float* out;                     // [T, ldo]
   int ldo, direct;
   SsdShape s;
+  float* norm_state;              // [slots at state_ld][H, N]: the normalizer's state, or null: none
+  float* norm_seg;                // [n_tiles, H, N]
+  float* norm_out;                // [T, H]: n_t . C_t
 };
 
 enum { CHUNK_LOCAL = 0, CHUNK_FULL = 1 };
@@ -75,7 +82,7 @@ enum { CHUNK_LOCAL = 0, CHUNK_FULL = 1 };
 template <int NT> struct SsdChunk {
   static constexpr int N = 16 * NT, LDN = N + TC_PAD, LDX = TC_COLS + TC_PAD, LDM = TC_TOKENS + TC_PAD;
   static constexpr int HALVES = 2 * TC_TOKENS * LDN + TC_TOKENS * LDX + 2 * TC_TOKENS * LDM;    // C, B, x, M (two terms)
-  static constexpr size_t BYTES = sizeof(__nv_bfloat16) * HALVES + sizeof(float) * 3 * TC_TOKENS;
+  static constexpr size_t BYTES = sizeof(__nv_bfloat16) * HALVES + sizeof(float) * (4 * TC_TOKENS + N);
 };
 
 template <int NT, int MODE>
@@ -93,6 +100,8 @@ ssd_chunks_kernel(SsdChunkArgs a) {
   float* ls = reinterpret_cast<float*>(Ml + TC_TOKENS * LDM);      // [64] running sums of the logarithms
   float* ds = ls + TC_TOKENS;                                      // [64] d
   float* ws = ds + TC_TOKENS;                                      // [64] exp(l_last - l_j) d_j
+  float* rsum = ws + TC_TOKENS;                                    // [64] row sums of the masked products (normalizer)
+  float* ns = rsum + TC_TOKENS;                                    // [N] the normalizer
   const SsdShape& s = a.s;
   const int tile = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * TC_COLS;
   const int seq = a.tiles[tile * 3 + 0], t0 = a.tiles[tile * 3 + 1], count = a.tiles[tile * 3 + 2];
@@ -124,6 +133,12 @@ ssd_chunks_kernel(SsdChunkArgs a) {
         S[t][q] = (MODE == CHUNK_FULL && n < N && p < P) ? src[(size_t)n * P + p] : 0.f;
       }
   }
+  const bool norm = a.norm_out != nullptr && blockIdx.z == 0;
+  float* nst = norm ? a.norm_state + (size_t)a.seq_slot[seq] * a.state_ld + (size_t)h * N : nullptr;
+  float* nsg = norm && a.norm_seg != nullptr ? a.norm_seg + ((size_t)tile * s.H + h) * N : nullptr;
+  if (norm)
+    for (int n = tid; n < SC::N; n += blockDim.x)
+      ns[n] = (MODE == CHUNK_FULL && n < N) ? (a.direct ? nst : nsg)[n] : 0.f;
   float total_log = 0.f;
   for (int b = 0; b < count; b += TC_TOKENS) {
     const int nt = min(TC_TOKENS, count - b), tok0 = t0 + b;
@@ -187,6 +202,7 @@ ssd_chunks_kernel(SsdChunkArgs a) {
         for (int kt = 0; kt < NT; ++kt) ldsm4(ca[kt], Cs + (mt * 16 + mrow) * LDN + kt * 16 + mcol);
         const int i0 = mt * 16 + r;
         const float li0 = ls[i0], li1 = ls[i0 + 8];
+        float sum0 = 0.f, sum1 = 0.f;                              // of rows i0 and i0 + 8
         for (int jt = 0; jt <= mt; ++jt) {
           float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}}, odd[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
@@ -215,10 +231,42 @@ ssd_chunks_kernel(SsdChunkArgs a) {
             split2(m10, m11, hi, lo);
             *reinterpret_cast<unsigned*>(Mh + (i0 + 8) * LDM + j) = hi;
             *reinterpret_cast<unsigned*>(Ml + (i0 + 8) * LDM + j) = lo;
+            sum0 += m00 + m01;
+            sum1 += m10 + m11;
+          }
+        }
+        if (norm) {
+#pragma unroll
+          for (int o = 1; o < 4; o <<= 1) {
+            sum0 += __shfl_xor_sync(0xffffffffu, sum0, o);
+            sum1 += __shfl_xor_sync(0xffffffffu, sum1, o);
+          }
+          if ((lane & 3) == 0) {
+            rsum[i0] = sum0;
+            rsum[i0 + 8] = sum1;
           }
         }
       }
       __syncthreads();
+      if (norm) {
+        // two lanes per token: the start's normalizer against the token's C, and the chunk's own tokens
+        for (int i = tid >> 1; i < TC_TOKENS; i += blockDim.x >> 1) {
+          const __nv_bfloat16* crow = Cs + i * LDN;
+          float dot = 0.f;
+          for (int n = (tid & 1) * 8; n < SC::N; n += 16) {
+            const uint4 v = *reinterpret_cast<const uint4*>(crow + n);
+            const unsigned w4[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+              const float2 c = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w4[q]));
+              dot = fmaf(c.x, ns[n + 2 * q], fmaf(c.y, ns[n + 2 * q + 1], dot));
+            }
+          }
+          dot += __shfl_xor_sync(0xffffffffu, dot, 1);
+          if ((tid & 1) == 0 && i < nt) a.norm_out[(size_t)(tok0 + i) * s.H + h] = fmaf(expf(ls[i]), dot, rsum[i]);
+        }
+        __syncthreads();                                           // every token has read the normalizer
+      }
       // y: what the chunk's start brings ...
       float y[4][2][4];
 #pragma unroll
@@ -292,6 +340,14 @@ ssd_chunks_kernel(SsdChunkArgs a) {
     if (MODE == CHUNK_FULL && !last && b + TC_TOKENS >= count) break;    // (nobody reads it)
     total_log += l_last;
     const float fl = expf(l_last);
+    if (norm) {
+      for (int n = tid; n < SC::N; n += blockDim.x) {
+        float v = fl * ns[n];
+#pragma unroll 8
+        for (int j = 0; j < TC_TOKENS; ++j) v = fmaf(ws[j], __bfloat162float(Bs[j * LDN + n]), v);   // (zeros beyond the chunk)
+        ns[n] = v;
+      }
+    }
 #pragma unroll
     for (int t = 0; t < 2 * NT; ++t)
 #pragma unroll
@@ -336,6 +392,8 @@ ssd_chunks_kernel(SsdChunkArgs a) {
         const int n = 8 * t + c2 + (q & 1), p = p0 + (q >> 1) * 8;
         if (n < N && p < P) dst[(size_t)n * P + p] = S[t][q];
       }
+    if (norm)
+      for (int n = tid; n < N; n += blockDim.x) (MODE == CHUNK_LOCAL ? nsg : nst)[n] = ns[n];      // (the thread's own)
   }
   if (MODE == CHUNK_LOCAL && tid == 0 && blockIdx.z == 0) a.seg_decay[(size_t)tile * s.H + h] = expf(total_log);
 }
@@ -355,6 +413,11 @@ static int launch_ssd_chunks(const SsdChunkArgs& a, cudaStream_t stream) {
     if (st != DLGO_OK) return st;
     st = launch_ssd_carry(a.tiles, a.n_tiles, a.seq_slot, a.state, a.state_ld, a.seg, a.seg_decay, a.s, stream);
     if (st != DLGO_OK) return st;
+    if (a.norm_out != nullptr) {                                   // the normalizer as a state of one column
+      st = launch_ssd_carry(a.tiles, a.n_tiles, a.seq_slot, a.norm_state, a.state_ld, a.norm_seg, a.seg_decay,
+                            SsdShape{a.s.H, a.s.G, a.s.N, 1, 1}, stream);
+      if (st != DLGO_OK) return st;
+    }
   }
   launch_kernel(ssd_chunks_kernel<NT, CHUNK_FULL>, grid, block, smem, stream, a);
   return launch_status();
@@ -370,18 +433,21 @@ DLGO_EXPORT int dlgo_ssd_chunks_takes(int N, int P) { return N > 0 && N <= 128 &
 // xbc [T, ld] bfloat16; columns x0 (H heads of P), b0 and c0 (G groups of N); steps [T, H, 2] fp32 (d, logarithm of f), or
 // null: d = 1 and log_decay [H]; D [H] fp32 or null; tiles [n_tiles, 3], a sequence's segments side by side in token
 // order; out [T, ldo >= H P] fp32.  `direct`: one segment per sequence; else scratch holds n_tiles * H * (N P + 1) floats.
+// norm_out [T, H] fp32 or null: n_t . C_t of the recurrence on x = 1, whose state [H, N] lies at norm_state + slot *
+// state_ld; scratch then holds n_tiles * H * N floats more.
 DLGO_EXPORT int dlgo_ssd_chunks(const void* xbc, int ld, int x0, int b0, int c0, const float* steps, const float* log_decay,
                                 const float* D, const int* tiles, int n_tiles, int direct, const int* seq_slot, float* state,
                                 long long state_ld, float* scratch, float* out, int ldo, int H, int G, int N, int P,
-                                cudaStream_t stream) {
+                                float* norm_state, float* norm_out, cudaStream_t stream) {
   if (n_tiles <= 0) return DLGO_OK;
   if (H <= 0 || H > 65535 || G <= 0 || H % G || n_tiles > 65535 || !dlgo_ssd_chunks_takes(N, P) || (steps == nullptr) == (log_decay == nullptr) ||
-      (!direct && scratch == nullptr))
+      (!direct && scratch == nullptr) || (norm_out != nullptr && norm_state == nullptr))
     return DLGO_ERR_SIZE;
   if (((ld | x0 | b0 | c0) & 7) || ((uintptr_t)xbc & 15) || (ldo & 1) || ((uintptr_t)out & 7)) return DLGO_ERR_ALIGN;
   SsdChunkArgs a{(const __nv_bfloat16*)xbc, ld, x0, b0, c0, steps, log_decay, D, tiles, n_tiles, seq_slot, state, state_ld,
                  direct ? nullptr : scratch, direct ? nullptr : scratch + (size_t)n_tiles * H * N * P, out, ldo, direct,
-                 SsdShape{H, G, N, P, 1}};
+                 SsdShape{H, G, N, P, 1}, norm_state,
+                 direct || norm_out == nullptr ? nullptr : scratch + (size_t)n_tiles * H * (N * P + 1), norm_out};
   if (N <= 16) return launch_ssd_chunks<1>(a, stream);
   if (N <= 32) return launch_ssd_chunks<2>(a, stream);
   if (N <= 64) return launch_ssd_chunks<4>(a, stream);

@@ -4,7 +4,8 @@
 //   streams  X[t, r, :] for r < s, fp32.  A sublayer reads u = sum_r a[r] X[t, r, :], runs on norm(u), and its
 //            result y goes back into every stream at once, from the old values:
 //            X'[t, q, :] = sum_r M[r, q] X[t, r, :] + b[q] * y[t, :]            (M indexed [from, to])
-//   norms    Dynamic Tanh: tanh(alpha * u) * w + beta (no statistics); RMS: u / sqrt(mean(u^2) + eps) * w
+//   norms    Dynamic Tanh: tanh(alpha * u) * w + beta (no statistics); RMS: u / sqrt(mean(u^2) + eps) * w;
+//            layer norm: (u - mean(u)) / sqrt(mean((u - mean(u))^2) + eps) * w + beta (beta may be absent)
 //   bias_act act(z + bias): none, relu(z)^2, silu, tanh-form gelu, tanh
 //   gated    rms(o) * w * gate(g) * c, the mean over the whole row or over each group of neighbours (a head);
 //            gate is sigmoid or silu, w may be absent
@@ -16,7 +17,7 @@
 namespace dlgo {
 
 constexpr int MAX_STREAMS = 8;
-enum { NORM_NONE = 0, NORM_RMS = 1, NORM_DYT = 2 };
+enum { NORM_NONE = 0, NORM_RMS = 1, NORM_DYT = 2, NORM_LAYER = 3 };
 enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SILU = 2, ACT_GELU_TANH = 3, ACT_TANH = 4 };
 enum { GATE_SIGMOID = 0, GATE_SILU = 1 };
 
@@ -33,7 +34,7 @@ struct StreamsStep {
   const float* coeff;   // [s], or null for the plain sum of the streams
   int norm_kind;
   const float* nw;      // [d]
-  const float* nb;      // [d] (Dynamic Tanh) or null
+  const float* nb;      // [d] (Dynamic Tanh, layer norm) or null
   const float* nalpha;  // [1] (Dynamic Tanh)
   float eps;
   void* out;            // [R, d]
@@ -137,6 +138,8 @@ __global__ void __launch_bounds__(256) streams_step_kernel(StreamsStep p) {
       }
       if (p.norm_kind == NORM_RMS) {
         for (int c = 0; c < W; ++c) ss = fmaf(u[c], u[c], ss);
+      } else if (p.norm_kind == NORM_LAYER) {
+        for (int c = 0; c < W; ++c) ss += u[c];
       } else {
         float r4[4];
 #pragma unroll
@@ -160,6 +163,124 @@ __global__ void __launch_bounds__(256) streams_step_kernel(StreamsStep p) {
       o[i] = from_float<TO>(u * sc * p.nw[i]);
     }
   }
+  if (o && p.norm_kind == NORM_LAYER) {
+    const float mean = block_sum(ss, scratch) / (float)d;    // (its barriers: every column written above is in place)
+    float dev = 0.f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+      float u = 0.f;
+      for (int a = 0; a < s; ++a) u = fmaf(s_coeff[a], xr[(size_t)a * d + i], u);
+      dev = fmaf(u - mean, u - mean, dev);
+    }
+    const float sc = 1.0f / sqrtf(block_sum(dev, scratch) / (float)d + p.eps);
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+      float u = 0.f;
+      for (int a = 0; a < s; ++a) u = fmaf(s_coeff[a], xr[(size_t)a * d + i], u);
+      o[i] = from_float<TO>(fmaf((u - mean) * sc, p.nw[i], p.nb ? p.nb[i] : 0.f));
+    }
+  }
+}
+
+// The same step for a layer norm over rows of a multiple of four numbers that fit a block's registers (NV float4 a
+// thread): one pass over the streams, the statistics from registers, mean first and then the squared deviations.
+template <typename TO, int THREADS, int NV>
+__global__ void __launch_bounds__(THREADS) streams_layernorm_kernel(StreamsStep p) {
+  pdl_launch_dependents();
+  __shared__ float s_mix[MAX_STREAMS * MAX_STREAMS], s_wout[MAX_STREAMS], s_coeff[MAX_STREAMS];
+  __shared__ float red[32];
+  const int s = p.s, d = p.d, tid = threadIdx.x;
+  if (tid < s * s && p.y) s_mix[tid] = p.mix[tid];
+  if (tid < s) {
+    if (p.y) s_wout[tid] = p.wout[tid];
+    s_coeff[tid] = p.coeff ? p.coeff[tid] : 1.0f;
+  }
+  const int r = blockIdx.x;
+  const int row = p.rows ? p.rows[r] : r;
+  float4 wv[NV], bv[NV], u[NV];
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {                   // weights: nothing of the step writes them
+    const int i = (v * THREADS + tid) * 4;
+    wv[v] = bv[v] = u[v] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < d) {
+      wv[v] = *reinterpret_cast<const float4*>(p.nw + i);
+      if (p.nb) bv[v] = *reinterpret_cast<const float4*>(p.nb + i);
+    }
+  }
+  __syncthreads();
+  pdl_wait();
+  float* xr = p.X + (size_t)row * s * d;
+  float* yr = p.y ? p.y + (size_t)row * d : nullptr;
+  float sum = 0.f;
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (v * THREADS + tid) * 4;
+    if (i >= d) continue;
+    float4 x[MAX_STREAMS];
+#pragma unroll
+    for (int a = 0; a < MAX_STREAMS; ++a)
+      if (a < s) x[a] = *reinterpret_cast<const float4*>(xr + (size_t)a * d + i);
+    if (yr) {
+      float4 y = *reinterpret_cast<const float4*>(yr + i);
+      if (p.y_bias) {
+        const float4 b = *reinterpret_cast<const float4*>(p.y_bias + i);
+        y.x += b.x; y.y += b.y; y.z += b.z; y.w += b.w;
+      }
+      if (p.clear_y) *reinterpret_cast<float4*>(yr + i) = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int q = 0; q < MAX_STREAMS; ++q) {
+        if (q < s) {
+          float4 n = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+          for (int a = 0; a < MAX_STREAMS; ++a) {
+            if (a < s) {
+              const float m = s_mix[a * s + q];
+              n.x = fmaf(m, x[a].x, n.x); n.y = fmaf(m, x[a].y, n.y);
+              n.z = fmaf(m, x[a].z, n.z); n.w = fmaf(m, x[a].w, n.w);
+            }
+          }
+          const float w = s_wout[q], c = s_coeff[q];
+          n.x = fmaf(w, y.x, n.x); n.y = fmaf(w, y.y, n.y); n.z = fmaf(w, y.z, n.z); n.w = fmaf(w, y.w, n.w);
+          *reinterpret_cast<float4*>(xr + (size_t)q * d + i) = n;
+          u[v].x = fmaf(c, n.x, u[v].x); u[v].y = fmaf(c, n.y, u[v].y);
+          u[v].z = fmaf(c, n.z, u[v].z); u[v].w = fmaf(c, n.w, u[v].w);
+        }
+      }
+    } else {
+#pragma unroll
+      for (int a = 0; a < MAX_STREAMS; ++a) {
+        if (a < s) {
+          const float c = s_coeff[a];
+          u[v].x = fmaf(c, x[a].x, u[v].x); u[v].y = fmaf(c, x[a].y, u[v].y);
+          u[v].z = fmaf(c, x[a].z, u[v].z); u[v].w = fmaf(c, x[a].w, u[v].w);
+        }
+      }
+    }
+    sum += (u[v].x + u[v].y) + (u[v].z + u[v].w);
+  }
+  const float mean = block_sum(sum, red) / (float)d;
+  float dev = 0.f;
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    if ((v * THREADS + tid) * 4 >= d) continue;
+    u[v].x -= mean; u[v].y -= mean; u[v].z -= mean; u[v].w -= mean;
+    dev += (u[v].x * u[v].x + u[v].y * u[v].y) + (u[v].z * u[v].z + u[v].w * u[v].w);
+  }
+  const float sc = 1.0f / sqrtf(block_sum(dev, red) / (float)d + p.eps);
+  TO* o = reinterpret_cast<TO*>(p.out) + (size_t)r * d;
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (v * THREADS + tid) * 4;
+    if (i < d)
+      store4<TO>(o + i, fmaf(u[v].x * sc, wv[v].x, bv[v].x), fmaf(u[v].y * sc, wv[v].y, bv[v].y),
+                 fmaf(u[v].z * sc, wv[v].z, bv[v].z), fmaf(u[v].w * sc, wv[v].w, bv[v].w));
+  }
+}
+
+template <typename TO>
+static void launch_streams_layernorm(const StreamsStep& p, int n_rows, cudaStream_t stream) {
+  if (p.d <= 512) launch_kernel(streams_layernorm_kernel<TO, 128, 1>, dim3(n_rows), dim3(128), 0, stream, p);
+  else if (p.d <= 1024) launch_kernel(streams_layernorm_kernel<TO, 256, 1>, dim3(n_rows), dim3(256), 0, stream, p);
+  else if (p.d <= 2048) launch_kernel(streams_layernorm_kernel<TO, 256, 2>, dim3(n_rows), dim3(256), 0, stream, p);
+  else launch_kernel(streams_layernorm_kernel<TO, 512, 2>, dim3(n_rows), dim3(512), 0, stream, p);
 }
 
 __device__ __forceinline__ float activate(float z, int act) {
@@ -311,8 +432,15 @@ DLGO_EXPORT int dlgo_streams_step(float* X, int T, int s, int d, float* y, const
   const int n_rows = y ? T : R;
   if (n_rows <= 0) return DLGO_OK;
   if (out && out_dtype != DLGO_F32 && out_dtype != DLGO_BF16) return DLGO_ERR_DTYPE;
+  if (norm_kind < NORM_NONE || norm_kind > NORM_LAYER) return DLGO_ERR_SIZE;
   if (out && norm_kind != NORM_NONE && !nw) return DLGO_ERR_SIZE;
   StreamsStep p{X, s, d, y, y_bias, mix, wout, clear_y, coeff, norm_kind, nw, nb, nalpha, eps, out, rows};
+  if (out && norm_kind == NORM_LAYER && d % 4 == 0 && d <= 4096 &&
+      (((uintptr_t)X | (uintptr_t)y | (uintptr_t)y_bias | (uintptr_t)nw | (uintptr_t)nb | (uintptr_t)out) & 15) == 0) {
+    if (out_dtype == DLGO_BF16) launch_streams_layernorm<__nv_bfloat16>(p, n_rows, stream);
+    else launch_streams_layernorm<float>(p, n_rows, stream);
+    return launch_status();
+  }
   const int threads = d >= 1024 ? 256 : 128;      // (four columns per thread and trip)
   if (out && out_dtype == DLGO_BF16)
     launch_kernel(streams_step_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, stream, p);

@@ -37,6 +37,10 @@ _FUSE_ROPE_MAX_HEAD = 64
 _PROMPT_ROPE = int(os.environ.get("DLGO_PROMPT_ROPE", 1))
 
 
+# head sizes of the tensor-core kernels, and how much a head may be stretched with zeros to reach one
+_TC_HEAD_SIZES = (64, 128)
+_TC_HEAD_STRETCH = float(os.environ.get("DLGO_ATTN_HEAD_STRETCH", 1.5))
+
 _DECODE_BLOCKS = int(os.environ.get("DLGO_ATTN_BLOCKS", 0))   # blocks wanted in flight for decode attention (0: as many as are resident)
 
 
@@ -68,6 +72,8 @@ class GQAAttention(Mixer):
         self.position_encoding = position_encoding
         self.cache_group = cache_group
         self.chunk: Optional[int] = None      # a subclass may cut the sequence into chunks instead of a window
+        self.sink: Optional[torch.Tensor] = None     # ... or give the softmax a sink per head (fp32)
+        self.split_weights = False                   # ... or keep 16 bits of the softmax's weights on the tensor cores
         self.q_dim = self.num_heads * self.head_dim
         self.kv_dim = self.num_kv_heads * self.head_dim
         self.wqkv: Optional[Linear] = None
@@ -154,17 +160,17 @@ class GQAAttention(Mixer):
         if mma:
             K.attention_decode_mma(qkv, qkv.stride(0), T, cache.keys, cache.values, cache.page_table, ctx.seq_slot,
                                    ctx.token_pos, out, self.num_heads, self.num_kv_heads, self.head_dim, self.scale,
-                                   self.span(), n_splits, _MMA_KEYS, scratch)
+                                   self.span(), n_splits, _MMA_KEYS, scratch, sink=self.sink, split=self.split_weights)
         elif decode_kernel:
             K.attention_decode(qkv, qkv.stride(0), T, cache.keys, cache.values, cache.page_table, ctx.seq_slot,
                                ctx.token_pos, out, self.num_heads, self.num_kv_heads, self.head_dim, self.scale,
-                               self.span(), n_splits, scratch, counters)
+                               self.span(), n_splits, scratch, counters, sink=self.sink)
         elif not ctx.decode and K.attention_prefill_tc_takes(qkv.dtype, self.head_dim, cache.page_size):
             # prompts: 128 query rows per CTA on the tensor cores
             tiles, n_tiles, _ = ctx.tiles(K.PREFILL_TC_TILE, heaviest_first=True)
             K.attention_prefill_tc(qkv, qkv.stride(0), T, cache.keys, cache.values, cache.page_table, tiles,
                                    ctx.seq_slot, ctx.token_pos, out, self.num_heads, self.num_kv_heads,
-                                   self.head_dim, self.scale, self.span())
+                                   self.head_dim, self.scale, self.span(), sink=self.sink, split=self.split_weights)
         else:
             qt, gchunk = K.attention_tile_shape(self.head_dim, group, ctx.decode)
             tiles, n_tiles, tile_max = ctx.tiles(qt)
@@ -178,7 +184,7 @@ class GQAAttention(Mixer):
                                       K.attention_scratch_floats(T, self.num_heads, self.head_dim, n_splits))
             K.attention(qkv, qkv.stride(0), T, cache.keys, cache.values, cache.page_table, tiles, tile_max,
                         ctx.seq_slot, ctx.token_pos, out, self.num_heads, self.num_kv_heads, self.head_dim,
-                        self.scale, self.span(), n_splits, gchunk, scratch)
+                        self.scale, self.span(), n_splits, gchunk, scratch, sink=self.sink)
 
     def _project_out(self, out: torch.Tensor, residual: torch.Tensor, ctx: Any) -> None:
         parts = self.wo.partials(out, for_residual=True) if hasattr(ctx, "defer") else None
@@ -446,6 +452,102 @@ class WholeNormAttention(GQAAttention):
         self._project_out(out, residual, ctx)
 
 
+class HeadNormAttention(GQAAttention):
+    """Grouped-query softmax attention whose queries and keys are normed head by head before the rotation, whose keys and
+    values may differ in size, and whose softmax has a sink:
+
+        q = Wq h,  k = Wk h,  v = Wv h                        (H x qk_dim, G x qk_dim, G x v_dim numbers)
+        q, k <- u / sqrt(mean(u^2) + eps) * w                 per head; one weight of qk_dim numbers for all heads
+        q, k: the rotation named by ``position_encoding``     (pairs (i, i + rot/2) of the first numbers of each head)
+        out_h = sum_j exp(s_j) v_j / (sum_j exp(s_j) + exp(sink_h)),  s_j = q_h . k_j * scale      (``sink``; else a softmax)
+        visible: j <= i and, with ``window`` w, i - j < w
+        result = Wo [out_1 .. out_H] * out_scale
+
+    Heads are laid out ``head_dim`` wide with zeros behind their own numbers, so that keys and values share the page shape
+    and the kernels of :class:`GQAAttention` run unchanged: max(qk_dim, v_dim) rounded up to a multiple of 8, or in
+    bfloat16 to the next size of the tensor-core kernels where there is one.  The projection's result stays fp32 until norm
+    and rotation are done (one kernel, which also appends to the cache, values times ``out_scale``: a factor of the result
+    that costs no rounding); on the tensor cores the softmax's weights meet the
+    values as two bfloat16 terms.  ``names``: tensor names below the part's prefix."""
+
+    head_multiple = 8
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, qk_dim: int, v_dim: int, scale: float,
+                 eps: float = 1e-6, window: Optional[int] = None, position_encoding: Optional[str] = None, sink: bool = False,
+                 cache_group: str = "full", out_scale: float = 1.0, names: Optional[Mapping[str, str]] = None):
+        self.qk_dim, self.v_dim = int(qk_dim), int(v_dim)
+        if self.qk_dim <= 0 or self.v_dim <= 0:
+            raise ValueError("qk_dim and v_dim must be positive")
+        padded = -(-max(self.qk_dim, self.v_dim) // self.head_multiple) * self.head_multiple
+        padded = next((s for s in _TC_HEAD_SIZES if padded <= s <= _TC_HEAD_STRETCH * padded), padded)
+        super().__init__(hidden_size, num_heads, num_kv_heads, padded, scale, window, position_encoding, cache_group)
+        self.params = dict(hidden_size=hidden_size, num_heads=num_heads, num_kv_heads=num_kv_heads, qk_dim=qk_dim,
+                           v_dim=v_dim, scale=scale, eps=eps, window=window, position_encoding=position_encoding, sink=sink,
+                           cache_group=cache_group, out_scale=out_scale, names=names)
+        self.eps, self.out_scale, self.has_sink = float(eps), float(out_scale), bool(sink)
+        self.split_weights = True
+        self.names = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "q_norm": "q_norm.weight",
+                      "k_norm": "k_norm.weight", "sink": "sink", "out": "o_proj.weight"}
+        self.names.update(names or {})
+        self.w_in: Optional[Linear] = None        # rows q | k | v
+        self.w_qnorm: Optional[torch.Tensor] = None
+        self.w_knorm: Optional[torch.Tensor] = None
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        n, d = self.names, self.hidden_size
+        H, G, dk, dv = self.num_heads, self.num_kv_heads, self.qk_dim, self.v_dim
+        specs = {n["q"]: ParamSpec((H * dk, d)), n["k"]: ParamSpec((G * dk, d)), n["v"]: ParamSpec((G * dv, d)),
+                 n["q_norm"]: ParamSpec((dk,), "one_plus_normal"), n["k_norm"]: ParamSpec((dk,), "one_plus_normal"),
+                 n["out"]: ParamSpec((d, H * dv))}
+        if self.has_sink:
+            specs[n["sink"]] = ParamSpec((H,))
+        return specs
+
+    def load(self, get: Callable[[str], torch.Tensor], runtime: Any) -> None:
+        n = self.names
+        self.w_in = Linear(stack_rows(runtime.compute_copy(get(n[key])) for key in ("q", "k", "v")), runtime)
+        wo = runtime.compute_copy(get(n["out"]))
+        hd, dv, H = self.head_dim, self.v_dim, self.num_heads
+        if dv != hd:        # zero columns where the heads' layout has zeros
+            wide = torch.zeros((wo.shape[0], H, hd), dtype=wo.dtype, device=wo.device)
+            wide[:, :, :dv] = wo.view(wo.shape[0], H, dv)
+            wo = wide.view(wo.shape[0], H * hd)
+        self.wo = Linear(wo.contiguous(), runtime)
+        # norms and sinks are 32-bit in every precision
+        self.w_qnorm = get(n["q_norm"]).to(torch.float32).contiguous()
+        self.w_knorm = get(n["k_norm"]).to(torch.float32).contiguous()
+        self.sink = get(n["sink"]).to(torch.float32).reshape(-1).contiguous() if self.has_sink else None
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: Any, cache: Any,
+                state: Optional[torch.Tensor], positions: Mapping[str, PositionEncoding]) -> None:
+        T = ctx.n_tokens
+        freq, rot = None, 0
+        if self.position_encoding is not None:
+            pe = positions[self.position_encoding]
+            if getattr(pe, "interleaved", False) or getattr(pe, "amplitude", 1.0) != 1.0:
+                raise ValueError("this mixer's kernel rotates pairs (i, i + rot/2) with plain cosine and sine")
+            freq, rot = pe.frequencies, pe.rotary_dim
+        act = self.w_in.weight.dtype
+        n_cols = self.w_in.out_features
+        decode_kernel, mma, n_splits, scratch, counters, pages = self._decode_plan(ctx, cache, act)
+        if _QKV_SUM and self.w_in.sums_slices_at_memory(T):
+            # few tokens: the projection's K-slices add themselves into one fp32 sum that is zero between steps; the
+            # norm-and-rotation kernel reads it once and leaves zeros behind
+            proj = ctx.zeros(f"qkv_norm_sum{n_cols}", T * n_cols, torch.float32)[:T * n_cols].view(T, n_cols)
+            self.w_in(x, ADD_F32, proj)
+            clear = True
+        else:
+            proj = self.w_in(x, STORE_F32)
+            clear = False
+        q = K.headnorm_rope_append(proj, None, self.w_qnorm, self.w_knorm, self.eps, freq, rot, ctx.token_pos,
+                                   ctx.token_seq, ctx.seq_slot, cache.page_table, cache.keys, cache.values,
+                                   self.num_heads, self.num_kv_heads, self.head_dim, False, cache.writes, clear,
+                                   qk_dim=self.qk_dim, v_dim=self.v_dim, v_scale=self.out_scale)
+        out = torch.empty((T, self.q_dim), dtype=act, device=x.device)
+        self._attend(q, ctx, cache, out, decode_kernel, mma, n_splits, scratch, counters, pages)
+        self._project_out(out, residual, ctx)
+
+
 _WHOLE_SEQUENCE = 1 << 30
 
 
@@ -583,5 +685,6 @@ class ShortConvAttention(GQAAttention):
 
 MIXERS.register("gqa_attention", GQAAttention)
 MIXERS.register("short_conv_attention", ShortConvAttention)
+MIXERS.register("headnorm_attention", HeadNormAttention)
 MIXERS.register("wholenorm_attention", WholeNormAttention)
 MIXERS.register("keys_as_values_attention", KeysAsValuesAttention)

@@ -71,11 +71,13 @@ class ParallelPreNormBlock(Block):
 class HyperConnection(Part):
     """How one sublayer sits on ``streams`` residual streams x_1 .. x_s: it reads ``u = sum_r read[r] x_r`` and
     its result y returns as ``x_q <- sum_r mix[r, q] x_r + write[q] * y`` for every q at once (``mix`` is
-    indexed [from, to]).  With one stream, read = write = mix = 1 this is the plain residual sum.
+    indexed [from, to]).  With one stream, read = write = mix = 1 this is the plain residual sum.  ``result_scale``: a
+    constant factor on y (joined with ``write`` in fp32 when the weights are loaded).
     ``names``: tensor names of the three below the part's prefix."""
 
-    def __init__(self, streams: int, names: Optional[Mapping[str, str]] = None):
-        super().__init__(streams=streams, names=names)
+    def __init__(self, streams: int, names: Optional[Mapping[str, str]] = None, result_scale: float = 1.0):
+        super().__init__(streams=streams, names=names, result_scale=result_scale)
+        self.result_scale = float(result_scale)
         if not 1 <= int(streams) <= K.MAX_STREAMS:
             raise ValueError(f"streams must be 1 to {K.MAX_STREAMS}, got {streams}")
         self.streams = int(streams)
@@ -94,7 +96,7 @@ class HyperConnection(Part):
     def load(self, get: Any, runtime: Any) -> None:
         # coefficients of the residual sum: fp32 in every precision
         self.read = get(self.names["read"]).to(torch.float32).contiguous()
-        self.write = get(self.names["write"]).to(torch.float32).contiguous()
+        self.write = (get(self.names["write"]).to(torch.float32) * self.result_scale).contiguous()
         self.mix = get(self.names["mix"]).to(torch.float32).contiguous()
 
 

@@ -4,12 +4,14 @@
                                      bias that is part of the logits, unlike ``correction``)
     s = softmax(z)  (or sigmoid(z))  over ALL router outputs
     c = s + correction               choice scores (``correction``: a stored per-output bias used for choosing only)
-    outputs form ``group_count`` equal groups of neighbours; a group's score is its largest c; only outputs of
-    the ``group_keep`` best groups can be chosen (the others count as minus infinity); the ``top`` largest c win
+    outputs form ``group_count`` equal groups of neighbours; a group's score is its largest c (``group_top`` 2: the sum
+    of its two largest); only outputs of the ``group_keep`` best groups can be chosen (the others count as minus infinity); the ``top`` largest c win
     y = sum over the chosen e of s_e * expert_e(h)            (``renormalize``: s_e / sum of the chosen s;
                                                               ``weight_scale``: s_e times a constant)
     expert_e(h) = Wdown_e act(Wup_e h)                        for e < num_experts
-                  (``gated``: Wdown_e (silu(Wgate_e h) * (Wup_e h)), a third matrix per expert)
+                  (``gated``: Wdown_e (silu(Wgate_e h) * (Wup_e h)), a third matrix per expert; ``clamp`` and
+                  ``shared_clamp``, each (limit, alpha, offset): the clamped form g sigmoid(alpha g) (u + offset) with
+                  g = min(Wgate h, limit), u = clamp(Wup h, -limit, limit), of the experts and of the shared one)
     expert_e(h) = h                                           for the ``identity_experts`` outputs after them
     y += gate * shared(h),  gate = sigmoid(w_g . h) per token (``shared_size``, ``shared_gate``; without the gate 1);
                                                               the shared expert has the experts' form (``gated`` or not)
@@ -26,7 +28,7 @@ depend on the rest of the batch.
 from __future__ import annotations
 
 import os
-from typing import Any, Callable, Dict, Mapping, Optional
+from typing import Any, Callable, Dict, Mapping, Optional, Sequence
 
 import torch
 
@@ -56,12 +58,20 @@ class RoutedExperts(FeedForward):
                  renormalize: bool = False, correction: bool = False, activation: str = "relu2",
                  shared_size: Optional[int] = None, shared_gate: bool = False,
                  names: Optional[Mapping[str, str]] = None, logit_bias: bool = False, gated: bool = False,
-                 weight_on: str = "output", weight_scale: float = 1.0):
+                 weight_on: str = "output", weight_scale: float = 1.0, group_top: int = 1,
+                 clamp: Optional[Sequence[float]] = None, shared_clamp: Optional[Sequence[float]] = None):
         super().__init__(hidden_size=hidden_size, intermediate_size=intermediate_size, num_experts=num_experts, top=top,
                          identity_experts=identity_experts, group_count=group_count, group_keep=group_keep,
                          score=score, renormalize=renormalize, correction=correction, activation=activation,
                          shared_size=shared_size, shared_gate=shared_gate, names=names, logit_bias=logit_bias,
-                         gated=gated, weight_on=weight_on, weight_scale=weight_scale)
+                         gated=gated, weight_on=weight_on, weight_scale=weight_scale, group_top=group_top, clamp=clamp,
+                         shared_clamp=shared_clamp)
+        if group_top not in (1, 2):
+            raise ValueError(f"group_top must be 1 or 2, got {group_top}")
+        if (clamp is not None or shared_clamp is not None) and not gated:
+            raise ValueError("the clamped form is one of gated experts")
+        self.group_top = int(group_top)
+        self.clamp = None if clamp is None else K.ClampedGlu(*(float(c) for c in clamp))
         if weight_on not in ("output", "input"):
             raise ValueError(f"weight_on must be 'output' or 'input', got {weight_on!r}")
         if weight_on == "input" and identity_experts:
@@ -109,7 +119,8 @@ class RoutedExperts(FeedForward):
         self.shared: Optional[SwiGLU] = None
         if self.gated and self.shared_size is not None:
             self.shared = SwiGLU(self.hidden_size, self.shared_size, names={
-                "gate": self.names["shared_gate_proj"], "up": self.names["shared_up"], "down": self.names["shared_down"]})
+                "gate": self.names["shared_gate_proj"], "up": self.names["shared_up"], "down": self.names["shared_down"]},
+                clamp=shared_clamp)
         self.on_tensor_cores = False
 
     def param_specs(self) -> Dict[str, ParamSpec]:
@@ -182,7 +193,7 @@ class RoutedExperts(FeedForward):
         idx, wt, gate, plan = K.moe_router(x, self.w_router, self.b_choice, self.n_outputs, self.shared_gate, self.top,
                                            self.group_count, self.group_keep, self.sigmoid_scores, self.renormalize,
                                            plan=(self.num_experts, tile_rows), logit_bias=self.b_logit,
-                                           weight_scale=self.weight_scale)
+                                           weight_scale=self.weight_scale, group_top=self.group_top)
         pair_out = None
         src, div, scale = x, self.top, None
         if self.weight_on_input:
@@ -205,14 +216,15 @@ class RoutedExperts(FeedForward):
             if on_tc:
                 # bfloat16: the tokens' rows copied into sorted order, then both contractions on tcgen05
                 rows = K.moe_gather_rows(plan, src, div, scale)
-                K.moe_gemm_tc(plan, rows, self.w_up, hidden, False, K.MOE_ACT_SWIGLU if fused else act)
+                K.moe_gemm_tc(plan, rows, self.w_up, hidden, False, K.MOE_ACT_SWIGLU if fused else act,
+                              glu=self.clamp if fused else None)
                 if self.gated and not fused:
-                    hidden = K.swiglu(hidden, block=self.gate_block)
+                    hidden = K.swiglu(hidden, block=self.gate_block, glu=self.clamp)
                 K.moe_gemm_tc(plan, hidden, self.w_down, pair_out, True, K.ACT_NONE)
             else:
                 K.moe_gemm(plan, src, self.w_up, hidden, div, False, act)                  # rows gathered by token (or pair)
                 if self.gated:
-                    hidden = K.swiglu(hidden, block=self.gate_block)
+                    hidden = K.swiglu(hidden, block=self.gate_block, glu=self.clamp)
                 K.moe_gemm(plan, hidden, self.w_down, pair_out, None, True, K.ACT_NONE)    # rows scattered by pair
         shared = None
         if self.shared is not None:

@@ -8,7 +8,7 @@ experts, no routing.
 from __future__ import annotations
 
 import os
-from typing import Any, Callable, Dict, Mapping, Optional
+from typing import Any, Callable, Dict, Mapping, Optional, Sequence
 
 import torch
 
@@ -19,10 +19,13 @@ from .registry import FEED_FORWARDS
 
 
 class SwiGLU(FeedForward):
-    """``names``: tensor names of gate, up and down below the part's prefix."""
+    """``names``: tensor names of gate, up and down below the part's prefix.  ``clamp``: the clamped form of the gated
+    product (:class:`kernels.ClampedGlu`, or its constants (limit, alpha, offset)) in the place of silu(gate) * up."""
 
-    def __init__(self, hidden_size: int, intermediate_size: int, names: Optional[Mapping[str, str]] = None):
-        super().__init__(hidden_size=hidden_size, intermediate_size=intermediate_size, names=names)
+    def __init__(self, hidden_size: int, intermediate_size: int, names: Optional[Mapping[str, str]] = None,
+                 clamp: Optional[Sequence[float]] = None):
+        super().__init__(hidden_size=hidden_size, intermediate_size=intermediate_size, names=names, clamp=clamp)
+        self.clamp = None if clamp is None else K.ClampedGlu(*(float(c) for c in clamp))
         self.hidden_size = int(hidden_size)
         self.intermediate_size = int(intermediate_size)
         self.names = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
@@ -47,7 +50,7 @@ class SwiGLU(FeedForward):
             # blocks of 16 gate rows followed by their 16 up rows: the contraction's epilogue then
             # holds a gate value and its up value side by side and writes silu(g) * u directly
             inter = torch.stack([gate.view(f // 16, 16, d), up.view(f // 16, 16, d)], dim=1).reshape(2 * f, d)
-            self.w_gate_up = Linear(inter.contiguous(), runtime, fused_swiglu=True)
+            self.w_gate_up = Linear(inter.contiguous(), runtime, fused_swiglu=True, clamp=self.clamp)
             self.fused = True
         else:
             self.w_gate_up = Linear(torch.cat([gate, up], dim=0), runtime)
@@ -55,7 +58,7 @@ class SwiGLU(FeedForward):
 
     def hidden(self, x: Any) -> torch.Tensor:
         """``silu(Wg . x) * (Wu . x)``: what the down projection reads."""
-        return self.w_gate_up(x) if self.fused else K.swiglu(self.w_gate_up(x, STORE))
+        return self.w_gate_up(x) if self.fused else K.swiglu(self.w_gate_up(x, STORE), glu=self.clamp)
 
     def forward(self, x: Any, residual: torch.Tensor, ctx: Any) -> None:
         h = self.hidden(x)
@@ -69,17 +72,23 @@ class SwiGLU(FeedForward):
 _FUSED_BIAS_ACT = os.environ.get("DLGO_FUSED_BIAS_ACT", "1") != "0"
 
 
-class ReluSquaredMLP(FeedForward):
-    """Dense two-matrix feed-forward with the square of relu between: ``y = Wd . relu(Wu . x + bu)^2 + bd``
-    (``bias`` False: no bu, bd).  ``names``: tensor names below the part's prefix.  Bias and activation run in
+class TwoMatrixMLP(FeedForward):
+    """Dense two-matrix feed-forward: ``y = Wd . act(Wu . x + bu) + bd`` (``bias`` False: no bu, bd); ``activation``:
+    ``relu2`` (the square of relu), ``silu`` or ``gelu_tanh`` (the tanh form).  ``names``: tensor names below the part's prefix.  Bias and activation run in
     fp32 on the contraction's accumulator (its epilogue on the tensor cores), or, with ``DLGO_FUSED_BIAS_ACT=0``,
     in a launch of their own on its fp32 result."""
 
     can_defer_bias = True
 
+    ACTIVATIONS = {"relu2": K.ACT_RELU2, "silu": K.ACT_SILU, "gelu_tanh": K.ACT_GELU_TANH}
+
     def __init__(self, hidden_size: int, intermediate_size: int, bias: bool = False,
-                 names: Optional[Mapping[str, str]] = None):
-        super().__init__(hidden_size=hidden_size, intermediate_size=intermediate_size, bias=bias, names=names)
+                 names: Optional[Mapping[str, str]] = None, activation: str = "relu2"):
+        super().__init__(hidden_size=hidden_size, intermediate_size=intermediate_size, bias=bias, names=names,
+                         activation=activation)
+        if activation not in self.ACTIVATIONS:
+            raise ValueError(f"activation must be one of {sorted(self.ACTIVATIONS)}, got {activation!r}")
+        self.act = self.ACTIVATIONS[activation]
         self.hidden_size = int(hidden_size)
         self.intermediate_size = int(intermediate_size)
         self.bias = bool(bias)
@@ -110,13 +119,14 @@ class ReluSquaredMLP(FeedForward):
     def forward(self, x: Any, residual: torch.Tensor, ctx: Any, defer_bias: bool = False) -> None:
         """``defer_bias``: the caller adds :attr:`output_bias` itself (fused into its next pass over the result)."""
         if _FUSED_BIAS_ACT:
-            h = self.w_up.bias_act(x, self.b_up, K.ACT_RELU2)      # bias and relu squared in the contraction's epilogue
+            h = self.w_up.bias_act(x, self.b_up, self.act)      # bias and activation in the contraction's epilogue
         else:
-            h = K.bias_act(self.w_up(x, STORE_F32), self.b_up, K.ACT_RELU2, self.w_down.weight.dtype)
+            h = K.bias_act(self.w_up(x, STORE_F32), self.b_up, self.act, self.w_down.weight.dtype)
         if self.output_bias is not None and not defer_bias:
             K.bias_act(residual, self.output_bias, K.ACT_NONE, torch.float32, in_place=True)
         self.w_down(h, ADD_F32, residual)
 
 
 FEED_FORWARDS.register("swiglu", SwiGLU)
-FEED_FORWARDS.register("relu2_mlp", ReluSquaredMLP)
+FEED_FORWARDS.register("relu2_mlp", TwoMatrixMLP)
+FEED_FORWARDS.register("two_matrix_mlp", TwoMatrixMLP)

@@ -30,16 +30,16 @@ def stack_rows(weights, multiple: int = 8) -> torch.Tensor:
 class Linear:
     """``fused_swiglu``: the weight holds gate and up rows in blocks of 16 + 16 and the contraction's
     epilogue writes ``silu(gate) * up`` ([T, out/2]); only the tensor-core kernel offers it
-    (:attr:`fuses_swiglu` says whether this weight got it)."""
+    (:attr:`fuses_swiglu` says whether this weight got it).  ``clamp`` (with it): the clamped form instead."""
 
-    def __init__(self, weight: torch.Tensor, runtime: Any, fused_swiglu: bool = False):
+    def __init__(self, weight: torch.Tensor, runtime: Any, fused_swiglu: bool = False, clamp: Optional[K.ClampedGlu] = None):
         self.weight = runtime.compute_copy(weight).contiguous()
         self.out_features, self.in_features = self.weight.shape
         self.runtime = runtime
         self._tc = None
         if self.weight.dtype == torch.bfloat16:
             from . import tensor_core
-            self._tc = tensor_core.plan_for(self.weight, swiglu=fused_swiglu)
+            self._tc = tensor_core.plan_for(self.weight, swiglu=fused_swiglu, clamp=clamp)
         self.fuses_swiglu = fused_swiglu and self._tc is not None
         if fused_swiglu and not self.fuses_swiglu:
             raise ValueError("this weight cannot take the fused SwiGLU epilogue")

@@ -47,26 +47,41 @@ RMSNorm.normed_kind = K.NORMED_RMS       # for arrangements that norm a sublayer
 
 class LayerNorm(Norm):
     """``out = (x - mean(x)) / sqrt(var(x) + eps) * w`` with the variance as the mean of the squared deviations;
-    a weight, no bias.  ``name``: the tensor's name below the part's prefix."""
+    a weight, no bias.  ``name``: the tensor's name below the part's prefix.  With ``bias_name`` a bias of that name is
+    added (such a norm runs in the pass over residual streams, also on one)."""
 
     normed_kind = K.NORMED_LAYER
 
-    def __init__(self, size: int, eps: float, name: str = "weight"):
-        super().__init__(size=size, eps=eps, name=name)
+    def __init__(self, size: int, eps: float, name: str = "weight", bias_name: Optional[str] = None):
+        super().__init__(size=size, eps=eps, name=name, bias_name=bias_name)
         self.size = int(size)
         self.eps = float(eps)
-        self.name = name
+        self.name, self.bias_name = name, bias_name
         self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
         self.out_dtype: Optional[torch.dtype] = None
+        if bias_name is not None:
+            self.normed_kind = None               # (the passes that norm a single stream's rows have no bias)
 
     def param_specs(self) -> Dict[str, ParamSpec]:
-        return {self.name: ParamSpec((self.size,), "one_plus_normal")}
+        specs = {self.name: ParamSpec((self.size,), "one_plus_normal")}
+        if self.bias_name is not None:
+            specs[self.bias_name] = ParamSpec((self.size,))
+        return specs
 
     def load(self, get: Callable[[str], torch.Tensor], runtime: Any) -> None:
         self.weight = get(self.name).to(torch.float32).contiguous()
+        if self.bias_name is not None:
+            self.bias = get(self.bias_name).to(torch.float32).contiguous()
         self.out_dtype = runtime.dtype
 
+    def step_args(self) -> Dict[str, Any]:
+        """This norm as arguments of :func:`kernels.streams_step` (for a caller that fuses it with a write)."""
+        return dict(norm_kind=K.NORM_LAYER, norm_w=self.weight, norm_b=self.bias, eps=self.eps, out_dtype=self.out_dtype)
+
     def forward(self, residual: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if self.bias is not None:
+            return self.forward_streams(residual.view(residual.shape[0], 1, -1), None, rows)
         return K.layernorm_rows(residual, self.weight, self.eps, self.out_dtype, rows, self.normed_kind)
 
     def forward_in_place(self, x: torch.Tensor) -> torch.Tensor:
@@ -118,8 +133,8 @@ class DynamicTanh(Norm):
                     out_dtype=self.out_dtype)
 
 
-def _rms_forward_streams(self, streams: torch.Tensor, read: Optional[torch.Tensor] = None,
-                         rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+def _forward_streams(self, streams: torch.Tensor, read: Optional[torch.Tensor] = None,
+                     rows: Optional[torch.Tensor] = None) -> torch.Tensor:
     return K.streams_step(streams, read=read, rows=rows, **self.step_args())
 
 
@@ -127,7 +142,8 @@ def _rms_step_args(self) -> Dict[str, Any]:
     return dict(norm_kind=K.NORM_RMS, norm_w=self.weight, eps=self.eps, out_dtype=self.out_dtype)
 
 
-RMSNorm.forward_streams = _rms_forward_streams
+RMSNorm.forward_streams = _forward_streams
+LayerNorm.forward_streams = _forward_streams
 RMSNorm.step_args = _rms_step_args
 
 NORMS.register("rmsnorm", RMSNorm)

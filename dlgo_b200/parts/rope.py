@@ -13,6 +13,8 @@ scaling at all); it follows the published Llama 3.1 rule: with wavelength
 ``lam > orig/low`` are divided by ``factor``, and those between are blended by
 ``s = (orig/lam - low) / (high - low)``: ``f <- (1-s) * f/factor + s * f``.
 
+Linear scaling (``rope_type`` "linear": ``factor``) divides every frequency: ``f_i <- f_i / factor``.
+
 YaRN scaling (``rope_type`` "yarn": ``factor``, ``original_max_position_embeddings``, ``beta_fast``,
 ``beta_slow``) blends by the pair's index instead.  With ``where(t) = rot * ln(orig / (2 pi t)) / (2 ln base)`` (the
 index whose pair makes t turns over the original context), ``lo = max(floor(where(beta_fast)), 0)``,
@@ -50,6 +52,8 @@ def rotary_frequencies(rotary_dim: int, theta: float, scaling: Optional[Dict[str
             r = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
             out.append(f / factor * r + f * (1.0 - r))
         return out
+    if kind == "linear":
+        return [f / float(scaling["factor"]) for f in freqs]
     if kind != "llama3":
         raise ValueError(f"rotary scaling {kind!r} is not supported")
     factor = float(scaling["factor"])

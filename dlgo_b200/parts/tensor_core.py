@@ -100,7 +100,8 @@ def skinny_shape(tokens: int, n: int, k: int, device: Optional[torch.device] = N
 
 
 class TensorCorePlan:
-    def __init__(self, weight: torch.Tensor, swiglu: bool = False):
+    def __init__(self, weight: torch.Tensor, swiglu: bool = False, clamp: Optional[K.ClampedGlu] = None):
+        self.clamp = clamp          # of the gated product (swiglu)
         self.weight = weight
         self.n, self.k = weight.shape
         self.swiglu = swiglu
@@ -126,9 +127,9 @@ class TensorCorePlan:
             if splits > 1:
                 ws = _workspace(x.device, K.gemm_tc_workspace_floats(self.n, t, bn, splits))
                 cnt = _counter_buffer(x.device)
-            return K.gemm_tc(self.weight, x, out, True, epi, bn, splits, ws, cnt, static_operand=1)
+            return K.gemm_tc(self.weight, x, out, True, epi, bn, splits, ws, cnt, static_operand=1, glu=self.clamp)
         bn, pair = self.many_token_shape(t)
-        return K.gemm_tc(x, self.weight, out, False, epi, bn, static_operand=2, pair_tile=pair)
+        return K.gemm_tc(x, self.weight, out, False, epi, bn, static_operand=2, pair_tile=pair, glu=self.clamp)
 
     def bias_act(self, x, bias: Optional[torch.Tensor], act: int) -> torch.Tensor:
         """``act(x . W^T + bias)`` as bfloat16 [tokens, out], bias and activation in the contraction's epilogue
@@ -186,7 +187,7 @@ class TensorCorePlan:
         return out
 
 
-def plan_for(weight: torch.Tensor, swiglu: bool = False) -> Optional[Callable]:
+def plan_for(weight: torch.Tensor, swiglu: bool = False, clamp: Optional[K.ClampedGlu] = None) -> Optional[Callable]:
     n, k = weight.shape
     if weight.dtype != torch.bfloat16 or k % 8 or weight.stride(1) != 1 or weight.stride(0) % 8:
         return None
@@ -194,4 +195,4 @@ def plan_for(weight: torch.Tensor, swiglu: bool = False) -> Optional[Callable]:
         return None
     if swiglu and n % 32:
         return None
-    return TensorCorePlan(weight, swiglu)
+    return TensorCorePlan(weight, swiglu, clamp)
