@@ -43,7 +43,7 @@ mlstm_gates_kernel(const float* zi, const float* zf, int ld, const float* __rest
                    long long state_ld, float* steps, float* m_out, int log_decay, MlstmShape s) {
   pdl_launch_dependents();
   __shared__ float w_sum[8], w_max[8], carry;
-  const int h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+  const int h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t0 = seqs[blockIdx.x * 3 + 1], count = seqs[blockIdx.x * 3 + 2];
   float* kept = state + (size_t)seq_slot[seqs[blockIdx.x * 3]] * state_ld + s.max_off() + h;
   const float b_i = bi[h], b_f = bf[h];
@@ -103,12 +103,13 @@ mlstm_gates_kernel(const float* zi, const float* zf, int ld, const float* __rest
         m = now;
       }
     }
-    if (threadIdx.x == blockDim.x - 1) carry = m;   // (threads beyond the end hand on what they got)
+    // the newest token's m, as it is (the state's scale), from the thread that holds that token
+    const int end = min(count - base, (int)blockDim.x * MG_PER) - 1;
+    if ((int)threadIdx.x == end / MG_PER) carry = m;
     __syncthreads();
     m0 = carry;
   }
   if (threadIdx.x == 0) *kept = m0;                 // (nobody else of this launch reads it)
-  (void)n_warps;
 }
 
 // ------------------------------------------------------------------------------- n . q, token by token

@@ -82,13 +82,13 @@ CONFIGS: Dict[str, dict] = {
         layer(rec(50, 5, 6), moe(18, 6, 4, 5.0, 1.0, (3, 2))),
         layer(par(att(5, 1, 8, 8, 0.5, window=70), mem(2, 33, 12, 30.0), 0.4, 1.6), dense(51))], streams=1, mult=1.0, eps=1e-6),
     # sizes that the tensor-core kernels take in bfloat16: heads of 64 and 128 (also stretched to them), memories of 32, 64
-    # and 128, parts of 64 and 32 channels, experts of 64 and 96; the whole list runs twice
+    # and 128, parts of 64 and 32 channels, experts of 64 and 96
     "R": model(260, 128, [
         layer(att(4, 2, 64, 48, 0.125, 64, 250000.0, window=64), moe(64, 8, 2, 2.0, 2.5, (4, 3), (96, 1.0))),
         layer(par(att(3, 1, 48, 64, 0.15, 32, 1e5, 8.0), mem(2, 64, 64, 15.0), 1.2, 0.9), dense(192)),
         layer(rec(256, 4, 3), dense(96)),
         layer(par(att(2, 2, 96, 128, 0.1, 96, 1e4, window=129), mem(3, 32, 72, 4.0), 0.8, 0.5), moe(96, 12, 4, 1.0, 1.0, (3, 2))),
-        layer(rec(96, 3, 2))], streams=4, mult=0.5, loop=(0, 5, 2), eps=1e-6),
+        layer(rec(96, 3, 2))], streams=4, mult=0.5, loop=(2, 4, 2), eps=1e-6),
 }
 SEEDS = {"P": 61, "Q": 62, "R": 63}
 

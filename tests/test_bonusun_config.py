@@ -36,8 +36,10 @@ def test_registry_and_round_trip():
 def test_run_order_repeats_the_span():
     assert [e.layer for e in spec_of(CONFIGS["P"]).order] == [0, 1, 2, 1, 2, 3]
     assert [e.layer for e in spec_of(CONFIGS["Q"]).order] == [0, 1, 2, 3, 4]
-    assert [e.layer for e in spec_of(CONFIGS["R"]).order] == list(range(5)) * 2
+    assert [e.layer for e in spec_of(CONFIGS["R"]).order] == [0, 1, 2, 3, 2, 3, 4]
     assert all(e.cache_of is None for e in spec_of(CONFIGS["R"]).order)
+    cfg = dict(CONFIGS["P"], loop={"start": 0, "stop": 4, "times": 3})
+    assert [e.layer for e in spec_of(cfg).order] == [0, 1, 2, 3] * 3
     cfg = dict(CONFIGS["P"], loop={"start": 3, "stop": 4, "times": 1})
     assert [e.layer for e in spec_of(cfg).order] == [0, 1, 2, 3]
 
@@ -86,7 +88,7 @@ def test_cache_and_state_needs():
     n = 3 * (16 * 20 + 16 + 1)
     assert states[1].shape == states[3].shape == (n + -n % 4,)                    # S, n and m per head, whole 16 bytes
     # every pass of the loop has a place of its own
-    assert len(CausalLM(spec_of(CONFIGS["R"])).cache_needs()[2]) == 8
+    assert len(CausalLM(spec_of(CONFIGS["R"])).cache_needs()[2]) == 6
 
 
 @pytest.mark.parametrize("path, value, word", [

@@ -685,7 +685,7 @@ def test_sinks_count_once_and_unscaled(dtype):
     tokens = random_tokens(120, cfg["vocab"], 2)
     gone = dict(w)
     gone["l0.mix.sink"] = torch.full((4,), -1e4).to(torch.bfloat16)
-    assert float(row_error(plain_of(cfg, gone, tokens), plain_of(cfg, w, tokens)).min()) > 0.05
+    assert float(row_error(plain_of(cfg, gone, tokens), plain_of(cfg, w, tokens)).median()) > 0.05
     check_model(cfg, w, dtype, "sinks", n=120, start=3)
 
 
@@ -698,9 +698,10 @@ def test_a_token_far_back_in_the_state(which, dtype):
                     par(att(1, 1, 8, 8, 0.3), mem(2, 64 if "tensor" in which else 20, 24, 12.0), 0.02, 1.5))
     w = make_weights(cfg, 78)
     if which == "unit":
-        w["l0.mix.lam"] = torch.full_like(w["l0.mix.lam"], -8.0)
-        w["l0.mix.ri"] *= 6                                          # (an input gate that is nearly shut or open)
-        w["l0.mix.ri.b"] = torch.full_like(w["l0.mix.ri.b"], -2.0)
+        # (a gate that is nearly shut, keeping the state as it is, or open, replacing most of it)
+        w["l0.mix.lam"] = torch.full_like(w["l0.mix.lam"], -2.0)
+        w["l0.mix.ra"] *= 5
+        w["l0.mix.ra.b"] = torch.full_like(w["l0.mix.ra.b"], -5.0)
     else:
         w["l0.mix.right.f.b"] = torch.full_like(w["l0.mix.right.f.b"], 9.0)
         w["l0.mix.right.f"] *= 0.2
@@ -885,7 +886,7 @@ def test_greedy_generation_through_the_entry_point(dirs):
                 lg = P.forward(cfg, w, p + want[:k])[-1]
                 assert float(lg[want[k]] - lg[g[k]]) < 1e-4 * float(lg.abs().max()), (name, g, want)
         info = llm.model_info()
-        assert info.architecture == "Bonusun" and info.layers == len(cfg["layers"]) and info.vocab_size == cfg["vocab"]
+        assert info.architecture == "Bonusun" and info.layers == len(P.run_order(cfg)) and info.vocab_size == cfg["vocab"]
         out = llm.generate(prompts[:2], max_tokens=5, temperature=0.8, top_k=20, seed=3, ignore_eos=True)
         assert all(len(o) == 5 and all(0 <= t < cfg["vocab"] for t in o) for o in out)
 
