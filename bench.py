@@ -496,6 +496,45 @@ def zetavik_set(size):
     return [("zetavik", zet), ("bazurax", baz), ("ragilorn", ragilorn_pair(size)[0]), ("llama", llama)]
 
 
+# --only bonusun: the Bonusun design beside its closest relatives and Llama at equal layer sizes (random weights)
+BONUSUN_SIZES = {
+    # width; heads, kv heads, head size and window of the attention layers; heads, key and value sizes of the matrix memory;
+    # width and parts of the recurrent unit; dense feed-forward; experts, groups, kept, chosen, expert and shared widths
+    "small": dict(width=1024, heads=16, kv=4, dim=64, window=512, mheads=16, mdim=64, mv=64, rwidth=1280, blocks=10,
+                  ff=4224, experts=16, groups=4, keep=2, top=2, eff=896, shared=1024, vocab=32000),
+    "1b": dict(width=2048, heads=16, kv=4, dim=128, window=1024, mheads=16, mdim=128, mv=128, rwidth=2560, blocks=10,
+               ff=8448, experts=32, groups=8, keep=4, top=4, eff=1024, shared=1536, vocab=32000),
+    "3b": dict(width=3072, heads=24, kv=8, dim=128, window=1024, mheads=24, mdim=128, mv=128, rwidth=3840, blocks=15,
+               ff=12288, experts=32, groups=8, keep=4, top=4, eff=1536, shared=2048, vocab=32000),
+}
+
+
+def bonusun_set(size):
+    """[(name, config.json)]: Bonusun with four layers on three streams (attention beside a matrix memory and a dense
+    feed-forward; the recurrent unit and experts; window attention and experts; the recurrent unit and a dense
+    feed-forward; a token's chosen and shared experts spend the dense one's FLOPs), and the models closest to it at the
+    same width and feed-forward FLOPs: Zetavik (recurrences, experts in groups, a shared expert), Dedutar (streams, sinks;
+    its four layers run twice) and Llama."""
+    z = BONUSUN_SIZES[size]
+    hd = z["dim"]
+    att = {"heads": z["heads"], "kv_heads": z["kv"], "dim": hd, "vdim": hd, "scale": hd ** -0.5, "rot": {"base": 500000.0, "dims": hd}}
+    full = dict(att, rot=dict(att["rot"], scaling={"factor": 8.0}))
+    par = {"left": full, "right": {"heads": z["mheads"], "dim": z["mdim"], "vdim": z["mv"], "gate_cap": 15.0},
+           "left_scale": 1.0, "right_scale": 1.0}
+    unit = {"width": z["rwidth"], "blocks": z["blocks"], "conv": 4}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["eff"], "limit": 7.0}, "shared": {"ff": z["shared"], "limit": 7.0},
+           "router": {"experts": z["experts"], "top": z["top"], "scale": 2.5, "groups": {"count": z["groups"], "keep": z["keep"]}}}
+    bon = {"architecture": "Bonusun", "vocab": z["vocab"], "width": z["width"], "streams": 3, "residual_mult": 0.7,
+           "norm": {"eps": 1e-6}, "loop": {"start": 0, "stop": 0, "times": 1},
+           "layers": [{"type": "parallel", "mixer": par, "mlp": dense}, {"type": "rglru", "mixer": unit, "mlp": moe},
+                      {"type": "attention", "mixer": dict(att, mask={"size": z["window"]}), "mlp": moe},
+                      {"type": "rglru", "mixer": unit, "mlp": dense}]}
+    ded, _ = dedutar_pair(size)
+    near = dict(zetavik_set(size))
+    return [("bonusun", bon), ("zetavik", near["zetavik"]), ("dedutar", ded), ("llama", near["llama"])]
+
+
 def dedutar_compare(size, batch, steps, warmup, prefill_tokens, profile, design="dedutar", only_models=()):
     """Prefill and decode throughput of the models (``only_models``: of these), and (with `profile`) the time per kernel entry point of
     one prompt step and of decode steps launched one by one."""
@@ -506,8 +545,8 @@ def dedutar_compare(size, batch, steps, warmup, prefill_tokens, profile, design=
     from dlgo_b200.weights import write_random_model
     out = {"only": design, "size": size, "batch": batch, "prefill_tokens": prefill_tokens, "dtype": "bf16",
            "data": "synthetic", "models": {}}
-    if design == "zetavik":
-        models = zetavik_set(size)
+    if design in ("zetavik", "bonusun"):
+        models = {"zetavik": zetavik_set, "bonusun": bonusun_set}[design](size)
     else:
         pair = {"monolix": monolix_pair, "dedutar": dedutar_pair, "bazurax": bazurax_pair, "ragilorn": ragilorn_pair}[design]
         models = list(zip((design, "llama"), pair(size)))
@@ -609,13 +648,14 @@ def main() -> int:
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="--only prefill: tokens of the prompt")
     ap.add_argument("--prefill-batch", type=int, default=0,
                     help="--only prefill: a packed batch of that many prompts with lengths from --prompt-range")
-    ap.add_argument("--only", choices=["decode", "prefill", "phases", "sampled", "dedutar", "monolix", "bazurax", "ragilorn", "zetavik"],
+    ap.add_argument("--only", choices=["decode", "prefill", "phases", "sampled", "dedutar", "monolix", "bazurax", "ragilorn", "zetavik", "bonusun"],
                     help="run one small workload (for profiling) and stop; phases: see phase_stamps(); dedutar, "
                          "monolix, bazurax, ragilorn, zetavik: prefill and decode of that design beside Llama (zetavik: and its "
                          "closest relatives) at equal layer sizes")
     ap.add_argument("--bazurax-size", default="1b", choices=sorted(BAZURAX_SIZES), help="--only bazurax: layer sizes")
     ap.add_argument("--zetavik-size", default="1b", choices=sorted(ZETAVIK_SIZES), help="--only zetavik: layer sizes")
-    ap.add_argument("--models", default="", help="--only zetavik: names of the models to run (default: all of the set)")
+    ap.add_argument("--bonusun-size", default="1b", choices=sorted(BONUSUN_SIZES), help="--only bonusun: layer sizes")
+    ap.add_argument("--models", default="", help="--only zetavik, bonusun: names of the models to run (default: all of the set)")
     ap.add_argument("--ragilorn-size", default="1b", choices=sorted(RAGILORN_SIZES), help="--only ragilorn: layer sizes")
     ap.add_argument("--monolix-size", default="1b", choices=sorted(MONOLIX_SIZES), help="--only monolix: layer sizes")
     ap.add_argument("--dedutar-size", default="1b", choices=sorted(DEDUTAR_SIZES), help="--only dedutar: layer sizes")
@@ -646,6 +686,10 @@ def main() -> int:
     if a.only == "ragilorn":
         print(json.dumps(dedutar_compare(a.ragilorn_size, a.batch, a.steps, warmup, a.prefill_tokens, a.kernels,
                                          design="ragilorn")))
+        return 0
+    if a.only == "bonusun":
+        print(json.dumps(dedutar_compare(a.bonusun_size, a.batch, a.steps, warmup, a.prefill_tokens, a.kernels,
+                                         design="bonusun", only_models=tuple(n for n in a.models.split(",") if n))))
         return 0
     if a.only == "zetavik":
         print(json.dumps(dedutar_compare(a.zetavik_size, a.batch, a.steps, warmup, a.prefill_tokens, a.kernels,

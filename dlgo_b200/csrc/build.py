@@ -55,6 +55,7 @@ LIBRARIES: Dict[str, List[str]] = {
     "ssd_tc": ["ssd_tc.cu"],
     "mlstm": ["mlstm.cu"],
     "rglru": ["rglru.cu"],
+    "rglru_tc": ["rglru_tc.cu"],
 }
 _HEADERS = ["common.cuh", "attention_noalloc.h", "attention_combine.cuh", "attention_decode_tiles.cuh", "tcgen05.cuh",
             "async_copy.cuh", "ssd.cuh", "ssd_state.cuh"]

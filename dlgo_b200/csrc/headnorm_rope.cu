@@ -109,6 +109,103 @@ headnorm_rope_append_kernel(float* proj, int ld, const float* __restrict__ bias,
   }
 }
 
+// The same with a block per token (q|k|v with norms and no bias, heads of a multiple of four numbers up to 128 NV): the
+// angles' cosines and sines once per token, rows in 16-byte pieces, several heads of a warp in flight together.
+constexpr int HT_WARPS = 8, HT_HEADS = 3;
+
+template <typename T, int NV>
+__global__ void __launch_bounds__(HT_WARPS * 32)
+headnorm_rope_token_kernel(float* proj, int ld, const float* __restrict__ w_q, const float* __restrict__ w_k, float eps,
+                           const float* __restrict__ freq, int rot, const int* __restrict__ token_pos,
+                           const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
+                           const int* __restrict__ page_table, int max_pages, T* kpages, T* vpages, T* q_out, int Hq,
+                           int Hkv, int dk, int dv, int hd, int page_size, int write_cache, int clear, float v_scale) {
+  extern __shared__ __align__(16) float ht_smem[];
+  pdl_launch_dependents();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, rh = rot / 2;
+  float* cs = ht_smem;                                             // [rh] cosines, [rh] sines
+  float* u_s = ht_smem + ((2 * rh + 3) & ~3) + warp * (128 * NV);  // a head, normed
+  const int pos = token_pos[t];
+  long long row_base = -1;
+  if (write_cache) {
+    const int page = page_table[(size_t)seq_slot[token_seq[t]] * max_pages + pos / page_size];
+    if (page < 0) {
+      if (threadIdx.x == 0) atomicExch(&g_headnorm_rope_error, 1);
+    } else {
+      row_base = ((long long)page * Hkv * page_size + pos % page_size) * hd;
+    }
+  }
+  for (int i = threadIdx.x; i < rh; i += HT_WARPS * 32) sincosf((float)pos * freq[i], &cs[rh + i], &cs[i]);
+  __syncthreads();
+  pdl_wait();
+  const int heads = Hq + 2 * Hkv;
+  float* row = proj + (size_t)t * ld;
+  for (int g = warp; g < heads; g += HT_WARPS * HT_HEADS) {
+    float4 x[HT_HEADS][NV];
+#pragma unroll
+    for (int k = 0; k < HT_HEADS; ++k) {
+      const int head = g + k * HT_WARPS;
+      const bool is_v = head >= Hq + Hkv;
+      const int n = is_v ? dv : dk;
+      float* src = row + (is_v ? (size_t)(Hq + Hkv) * dk + (size_t)(head - Hq - Hkv) * dv : (size_t)head * dk);
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        const int i = (v * 32 + lane) * 4;
+        x[k][v] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (head < heads && i < n) x[k][v] = *reinterpret_cast<const float4*>(src + i);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < HT_HEADS; ++k) {
+      const int head = g + k * HT_WARPS;
+      if (head >= heads) break;
+      const bool is_q = head < Hq, is_v = head >= Hq + Hkv;
+      const int n = is_v ? dv : dk;
+      if (clear) {
+        float* src = row + (is_v ? (size_t)(Hq + Hkv) * dk + (size_t)(head - Hq - Hkv) * dv : (size_t)head * dk);
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+          const int i = (v * 32 + lane) * 4;
+          if (i < n) *reinterpret_cast<float4*>(src + i) = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+      }
+      T* dst = is_q ? q_out + ((size_t)t * Hq + head) * hd
+                    : (row_base < 0 ? nullptr
+                                    : (is_v ? vpages : kpages) + row_base + (size_t)(head - Hq - (is_v ? Hkv : 0)) * page_size * hd);
+      float r = v_scale;
+      const float* w = nullptr;
+      if (!is_v) {
+        float ss = 0.f;
+#pragma unroll
+        for (int v = 0; v < NV; ++v)
+          ss += (x[k][v].x * x[k][v].x + x[k][v].y * x[k][v].y) + (x[k][v].z * x[k][v].z + x[k][v].w * x[k][v].w);
+        r = 1.0f / sqrtf(warp_sum(ss) / (float)dk + eps);
+        w = is_q ? w_q : w_k;
+      }
+      __syncwarp();                                                // the head before has been read
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        const int i = (v * 32 + lane) * 4;
+        float4 o = make_float4(x[k][v].x * r, x[k][v].y * r, x[k][v].z * r, x[k][v].w * r);
+        if (w != nullptr && i < n) {
+          const float4 m = *reinterpret_cast<const float4*>(w + i);
+          o.x *= m.x; o.y *= m.y; o.z *= m.z; o.w *= m.w;
+        }
+        *reinterpret_cast<float4*>(u_s + i) = o;                   // (zeros behind the head's own numbers)
+      }
+      __syncwarp();
+      if (dst == nullptr) continue;
+      const int turned = is_v ? 0 : rot;
+      for (int i = lane; i < (turned >> 1); i += 32) {
+        const float a = u_s[i], b = u_s[i + rh];
+        dst[i] = from_float<T>(a * cs[i] - b * cs[rh + i]);
+        dst[i + rh] = from_float<T>(b * cs[i] + a * cs[rh + i]);
+      }
+      for (int i = turned + lane; i < hd; i += 32) dst[i] = from_float<T>(u_s[i]);
+    }
+  }
+}
+
 template <typename T>
 int launch_headnorm_rope(float* proj, int ld, const float* bias, const float* w_q, const float* w_k, float eps,
                          const float* freq, int rot, const int* token_pos, const int* token_seq, const int* seq_slot,
@@ -119,6 +216,18 @@ int launch_headnorm_rope(float* proj, int ld, const float* bias, const float* w_
   const long long items = (long long)T_tokens * heads;
   const long long blocks = (items + HR_WARPS - 1) / HR_WARPS;
   if (blocks > 0x7fffffffLL) return DLGO_ERR_SIZE;
+  const int wide = dk > dv ? dk : dv;
+  if (!v_from_k && bias == nullptr && w_q != nullptr && w_k != nullptr && norm_dim == dk && ((dk | dv | ld) & 3) == 0 && hd <= 256 &&
+      (((uintptr_t)proj | (uintptr_t)w_q | (uintptr_t)w_k) & 15) == 0) {
+    const int nv = (hd > wide ? hd : wide) <= 128 ? 1 : 2;
+    const size_t ht = sizeof(float) * (((size_t)rot + 3) / 4 * 4 + HT_WARPS * 128 * nv);
+#define HT_ARGS dim3(T_tokens), dim3(HT_WARPS * 32), ht, stream, proj, ld, w_q, w_k, eps, freq, rot, token_pos, token_seq, seq_slot, \
+                page_table, max_pages, (T*)kpages, (T*)vpages, (T*)q_out, Hq, Hkv, dk, dv, hd, page_size, write_cache, clear, v_scale
+    if (nv == 1) launch_kernel(headnorm_rope_token_kernel<T, 1>, HT_ARGS);
+    else launch_kernel(headnorm_rope_token_kernel<T, 2>, HT_ARGS);
+#undef HT_ARGS
+    return launch_status();
+  }
   const size_t smem = (size_t)HR_WARPS * hd * sizeof(float);
   if (smem > 48 * 1024) return DLGO_ERR_SIZE;
   launch_kernel(headnorm_rope_append_kernel<T>, dim3((unsigned)blocks), dim3(HR_WARPS * 32), smem, stream, proj, ld,

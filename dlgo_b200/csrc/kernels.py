@@ -993,15 +993,50 @@ def rglru_conv(x: torch.Tensor, bx: torch.Tensor, taps: torch.Tensor, bc: torch.
     return u, rows
 
 
+def rglru_gates_tc_takes(dtype: torch.dtype, part: int) -> bool:
+    """Whether the tensor-core gates take parts of this many channels (bfloat16 runs)."""
+    return dtype == torch.bfloat16 and bool(_lib("rglru_tc").dlgo_rglru_gates_tc_takes(_i(part)))
+
+
+RGLRU_TC_SEGMENT = 32          # most tokens of a segment of rglru_gates_tc
+
+
+def rglru_gates_tc(rows: torch.Tensor, w_gates: torch.Tensor, br: torch.Tensor, bi: torch.Tensor, lam: torch.Tensor,
+                   tiles: torch.Tensor, n_tiles: int, T: int, scratch: torch.Tensor, shape: RglruShape) -> torch.Tensor:
+    """Both gates of every token on the tensor cores and, in the same launch, a and the recurrence's input of every token and
+    every segment's end from zero.  ``rows`` [parts * T, width / parts] bfloat16 sorted by part, ``w_gates`` [parts,
+    2 * width / parts, width / parts] bfloat16; ``tiles``: segments of at most :data:`RGLRU_TC_SEGMENT` tokens; ``scratch``:
+    n_tiles * 3 * width floats.  Returns z [T * parts, 2 * width / parts] fp32 for :func:`rglru_scan` (``prepared``)."""
+    b = shape.width // shape.parts
+    _need(rows, torch.bfloat16, "rows")
+    _need(w_gates, torch.bfloat16, "w_gates")
+    _need(tiles, torch.int32, "tiles")
+    for n, t in (("br", br), ("bi", bi), ("lam", lam)):
+        _need(t, torch.float32, n)
+        if t.numel() != shape.width:
+            raise KernelError(f"rglru_gates_tc: {n} must have a number per channel")
+    if tuple(rows.shape) != (shape.parts * T, b) or tuple(w_gates.shape) != (shape.parts, 2 * b, b) or tiles.numel() < 3 * n_tiles:
+        raise KernelError("rglru_gates_tc: shapes do not fit")
+    if scratch.dtype != torch.float32 or scratch.numel() < n_tiles * 3 * shape.width:
+        raise KernelError(f"rglru_gates_tc: {n_tiles} segments need {n_tiles * 3 * shape.width} floats of scratch")
+    z = torch.empty((T * shape.parts, 2 * b), dtype=torch.float32, device=rows.device)
+    st = _lib("rglru_tc").dlgo_rglru_gates_tc(_ptr(rows), _ptr(w_gates), _ptr(br), _ptr(bi), _ptr(lam), _ptr(tiles), _i(n_tiles),
+                                              _i(T), _i(shape.parts), _i(b), _f(shape.rate), _ptr(z), _ptr(scratch), _stream())
+    _check(st, "rglru_gates_tc")
+    return z
+
+
 def rglru_scan(z: torch.Tensor, u: torch.Tensor, br: torch.Tensor, bi: torch.Tensor, lam: torch.Tensor, y: torch.Tensor,
                by: Optional[torch.Tensor], x: torch.Tensor, bx: torch.Tensor, tiles: torch.Tensor, n_tiles: int, direct: bool,
                token_seq: torch.Tensor, token_pos: torch.Tensor, seq_slot: torch.Tensor, state: torch.Tensor,
-               scratch: Optional[torch.Tensor], shape: RglruShape, out_dtype: torch.dtype) -> torch.Tensor:
+               scratch: Optional[torch.Tensor], shape: RglruShape, out_dtype: torch.dtype,
+               prepared: bool = False) -> torch.Tensor:
     """The recurrence over the step's tokens and its product with the other branch.  ``z`` [T * parts, 2 * width / parts]
     fp32: the gates' logits without biases (overwritten); ``y``: the other branch, fp32 without bias and gelu (``by``) or
     finished bfloat16 (``by`` None).  ``tiles`` cut a sequence's tokens into segments that run side by side; ``direct``:
     one segment per sequence, else ``scratch`` holds n_tiles * 3 * width floats.  S and the newest inputs go into the
-    state rows.  Returns [T, width] in ``out_dtype``."""
+    state rows.  ``prepared``: ``z`` and ``scratch`` are :func:`rglru_gates_tc`'s (over the same tiles).  Returns [T, width]
+    in ``out_dtype``."""
     _rglru_check("rglru_scan", shape, state, br=br, bi=bi, lam=lam, bx=bx)
     _f32_rows("rglru_scan", z=z, u=u, x=x)
     for n, t in (("tiles", tiles), ("token_seq", token_seq), ("token_pos", token_pos), ("seq_slot", seq_slot)):
@@ -1020,9 +1055,10 @@ def rglru_scan(z: torch.Tensor, u: torch.Tensor, br: torch.Tensor, bi: torch.Ten
     st = _lib("rglru").dlgo_rglru_scan(
         _ptr(z), _ptr(u), _ptr(br), _ptr(bi), _ptr(lam), _ptr(y), _i(dtype_code(y.dtype)), _i(y.stride(0)), _ptr(by), _ptr(x),
         _i(x.stride(0)), _ptr(bx), _ptr(tiles), _i(n_tiles), _ptr(token_seq), _ptr(token_pos), _ptr(seq_slot), _ptr(state),
-        _ll(state.stride(0)), _ptr(scratch), _i(1 if direct else 0), _ptr(out), _i(dtype_code(out_dtype)), _i(w),
+        _ll(state.stride(0)), _ptr(scratch), _i(1 if direct else 0), _i(1 if prepared else 0), _ptr(out),
+        _i(dtype_code(out_dtype)), _i(w),
         _i(shape.parts), _i(shape.taps), _f(shape.rate), _stream())
-    _check(st, "rglru_scan", 1 if direct else 2)
+    _check(st, "rglru_scan", 1 if direct else (2 if prepared else 3))
     return out
 
 
@@ -2035,7 +2071,7 @@ def gemm_tc_rope(x: torch.Tensor, w: torch.Tensor, qkv: torch.Tensor, pair_tile:
 def check_device_errors() -> None:
     """Raise if a kernel gave up a bounded wait on the device since the last check (synchronises)."""
     for lib, fn in (("gemm_tc", "dlgo_gemm_tc_error"), ("attention_prefill_tc", "dlgo_attention_tc_error"),
-                    ("moe_tc", "dlgo_moe_tc_error")):
+                    ("moe_tc", "dlgo_moe_tc_error"), ("rglru_tc", "dlgo_rglru_gates_tc_error")):
         if lib in build._loaded:
             v = getattr(build._loaded[lib], fn)()
             if v != 0:

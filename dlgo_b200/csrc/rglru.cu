@@ -14,11 +14,12 @@
 // rglru_conv   prompts: u for all tokens (fp32, and the operand of the gates' contraction in the run's type, in rows of a
 //              part: [parts, T, B], sorted by part, or [T, parts, B])
 // rglru_scan   prompts: a sequence's tokens are cut into segments that run side by side
-//                LOCAL   a and the input's factor of every token take the places of the gates' logits; every segment's
-//                        end (a sequence's first from the stored state, which it also copies aside; the others from
-//                        zero) and the product of its a (as the sum of logarithms)
-//                FULL    every segment forms its start from the ends before it and walks its tokens again; the last one
-//                        of a sequence stores the state and the inputs that the next step reads back
+//                LOCAL   a and the input of every token take the places of the gates' logits; every segment's end from
+//                        zero and the product of its a (as the sum of logarithms).  In bfloat16 the gates' contraction
+//                        does this in its epilogue (rglru_tc.cu).
+//                carry   the start of every segment from the stored state and the ends before it
+//                FULL    every segment walks its tokens again from its start; the last one of a sequence stores the state
+//                        and the inputs that the next step reads back
 //              with one segment per sequence DIRECT runs alone from the logits
 // rglru_step   decoding: convolution, gates, recurrence and output of one token per sequence in one launch
 // Everything is fp32 but the gates' operand and weights, and y where the contraction before has finished it in bfloat16.
@@ -156,6 +157,38 @@ rglru_conv_kernel(const float* x, int ldx, const float* __restrict__ bx, const f
 }
 
 // ------------------------------------------------------------------------------- recurrence (prompts)
+// The start of every segment: a thread per channel of a sequence, the ends of several segments in flight together.
+constexpr int CY_THREADS = 64, CY_FLY = 16;
+__global__ void __launch_bounds__(CY_THREADS)
+rglru_carry_kernel(const int* __restrict__ tiles, int n_tiles, const int* __restrict__ seq_slot, const float* state,
+                   long long state_ld, float* seg, int W) {
+  pdl_launch_dependents();
+  const int j0 = blockIdx.y, seq = tiles[j0 * 3];
+  if (j0 > 0 && tiles[(j0 - 1) * 3] == seq) return;                // a block row per first segment of a sequence
+  const int c = blockIdx.x * CY_THREADS + threadIdx.x;
+  if (c >= W) return;
+  int end = j0 + 1;
+  while (end < n_tiles && tiles[end * 3] == seq) ++end;
+  pdl_wait();
+  float S = state[(size_t)seq_slot[seq] * state_ld + c];
+  for (int j = j0; j < end; j += CY_FLY) {
+    float e[CY_FLY], l[CY_FLY];
+#pragma unroll
+    for (int q = 0; q < CY_FLY; ++q) {
+      const float* sg = seg + (size_t)min(j + q, end - 1) * 3 * W + c;
+      e[q] = sg[0];
+      l[q] = sg[W];
+    }
+#pragma unroll
+    for (int q = 0; q < CY_FLY; ++q) {
+      if (j + q < end) {
+        seg[((size_t)(j + q) * 3 + 2) * W + c] = S;
+        S = fmaf(expf(l[q]), S, e[q]);
+      }
+    }
+  }
+}
+
 enum { RG_LOCAL = 0, RG_FULL = 1, RG_DIRECT = 2 };
 constexpr int RS_THREADS = 128, RS_FLY = 8;
 
@@ -179,7 +212,7 @@ struct RglruScan {
   const int* seq_slot;
   float* state;
   long long state_ld;
-  float* seg;                     // [n_tiles, 3, W]: end, sum of the logarithms, start (a sequence's first segment)
+  float* seg;                     // [n_tiles, 3, W]: end from zero, sum of the logarithms, start
   RglruShape s;
 };
 
@@ -201,34 +234,8 @@ rglru_scan_kernel(RglruScan a, TO* out) {
   const size_t ldz = (size_t)2 * s.W;
   pdl_wait();
   float S = 0.f;
-  if (MODE == RG_DIRECT) {
-    S = row[c];
-  } else if (MODE == RG_LOCAL) {
-    if (tile == 0 || a.tiles[(tile - 1) * 3] != seq) {
-      S = row[c];
-      a.seg[((size_t)tile * 3 + 2) * s.W + c] = S;
-    }
-  } else {
-    // (not from the stored state: the sequence's last segment replaces it in this launch)
-    int j0 = tile;                                 // the sequence's first segment
-    while (j0 > 0 && a.tiles[(j0 - 1) * 3] == seq) --j0;
-    if (j0 == tile) {
-      S = a.seg[((size_t)tile * 3 + 2) * s.W + c];
-    } else {
-      for (int j = j0; j < tile; j += RS_FLY) {
-        float e[RS_FLY], l[RS_FLY];
-#pragma unroll
-        for (int q = 0; q < RS_FLY; ++q) {
-          const float* sg = a.seg + (size_t)min(j + q, tile - 1) * 3 * s.W + c;
-          e[q] = sg[0];
-          l[q] = sg[s.W];
-        }
-#pragma unroll
-        for (int q = 0; q < RS_FLY; ++q)
-          if (j + q < tile) S = fmaf(expf(l[q]), S, e[q]);
-      }
-    }
-  }
+  if (MODE == RG_DIRECT) S = row[c];
+  if (MODE == RG_FULL) S = a.seg[((size_t)tile * 3 + 2) * s.W + c];    // (the stored state is replaced in this launch)
   float total = 0.f;
   for (int tb = 0; tb < count; tb += RS_FLY) {
     float f0[RS_FLY], f1[RS_FLY], uu[RS_FLY], yy[RS_FLY];
@@ -287,6 +294,7 @@ rglru_scan_kernel(RglruScan a, TO* out) {
 // A block owns CH neighbouring channels of one part for up to TOK tokens: their part of u in shared memory, a warp per
 // output channel at a time over the rows of both matrices, then the recurrence.
 constexpr int ST_THREADS = 256, ST_CH = 16, ST_TOK = 8;
+static_assert(ST_CH * ST_TOK <= ST_THREADS, "the last pass has a thread per channel and token");
 
 template <typename TW> struct Pair;
 template <> struct Pair<float> {
@@ -299,7 +307,7 @@ template <> struct Pair<__nv_bfloat16> {
 };
 
 template <typename TW, typename TO, bool PAIRS>
-__global__ void __launch_bounds__(ST_THREADS)
+__global__ void __launch_bounds__(ST_THREADS, 2)
 rglru_step_kernel(const float* proj, int ld, int x0, const float* __restrict__ by, const float* __restrict__ bx,
                   const float* __restrict__ w_taps, const float* __restrict__ bc, const TW* __restrict__ w_gates,
                   const float* __restrict__ br, const float* __restrict__ bi, const float* __restrict__ lam,
@@ -308,6 +316,7 @@ rglru_step_kernel(const float* proj, int ld, int x0, const float* __restrict__ b
   pdl_launch_dependents();
   extern __shared__ __align__(16) float u_s[];                     // [tok][B]
   __shared__ float z_s[2][ST_CH][ST_TOK];
+  __shared__ int pos_s[ST_TOK], slot_s[ST_TOK];
   const int B = s.B(), n = s.taps, per_part = (B + ST_CH - 1) / ST_CH;
   const int part = blockIdx.x / per_part, o0 = (blockIdx.x - part * per_part) * ST_CH, no = min(ST_CH, B - o0);
   const int t0 = blockIdx.y * tok, nt = min(tok, T - t0);
@@ -317,16 +326,46 @@ rglru_step_kernel(const float* proj, int ld, int x0, const float* __restrict__ b
     const char* p = (const char*)(w_gates + ((size_t)part * 2 * B + (o & 1) * B + o0 + (o >> 1)) * B);
     for (int b = lane * 128; b < B * (int)sizeof(TW); b += 32 * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(p + b));
   }
+  if (threadIdx.x < nt) {                                          // the step's own inputs
+    pos_s[threadIdx.x] = token_pos[t0 + threadIdx.x];
+    slot_s[threadIdx.x] = seq_slot[t0 + threadIdx.x];
+  }
+  __syncthreads();
   pdl_wait();
-  for (int i = threadIdx.x; i < nt * B; i += ST_THREADS) {
-    const int q = i / B, c = part * B + (i - q * B), t = t0 + q, pos = token_pos[t];
-    const float* ring = state + (size_t)seq_slot[t] * state_ld + s.W + c;
-    float a = fmaf(w_taps[(size_t)c * n + n - 1], proj[(size_t)t * ld + x0 + c] + bx[c], bc[c]);
+  // what the last pass needs of this block's own channels: requested now
+  float S_old = 0.f, y_now = 0.f, x_now = 0.f;
+  const int fq = threadIdx.x / ST_CH, fo = threadIdx.x - fq * ST_CH, fc = part * B + o0 + fo;
+  const bool fin = fq < nt && fo < no;                             // (ST_TOK * ST_CH items, no more than threads)
+  if (fin) {
+    const float* pr = proj + (size_t)(t0 + fq) * ld;
+    S_old = state[(size_t)slot_s[fq] * state_ld + fc];
+    y_now = pr[fc];
+    x_now = pr[x0 + fc];
+  }
+  // u of the part: a thread per channel, every token's inputs in flight together
+  for (int i = threadIdx.x; i < B; i += ST_THREADS) {
+    const int c = part * B + i;
+    const float b_x = bx[c], b_c = bc[c];
+    float a[ST_TOK];
+#pragma unroll
+    for (int q = 0; q < ST_TOK; ++q) a[q] = q < nt ? proj[(size_t)(t0 + q) * ld + x0 + c] : 0.f;
+    const float w_now = w_taps[(size_t)c * n + n - 1];
+#pragma unroll
+    for (int q = 0; q < ST_TOK; ++q) a[q] = fmaf(w_now, a[q] + b_x, b_c);
+#pragma unroll 3
     for (int j = 0; j < n - 1; ++j) {
-      const int p = pos - (n - 1) + j;
-      if (p >= 0) a = fmaf(w_taps[(size_t)c * n + j], ring[(size_t)(p % n) * s.W], a);
+      const float w = w_taps[(size_t)c * n + j];
+#pragma unroll
+      for (int q = 0; q < ST_TOK; ++q) {
+        if (q < nt) {
+          const int p = pos_s[q] - (n - 1) + j;
+          if (p >= 0) a[q] = fmaf(w, state[(size_t)slot_s[q] * state_ld + s.W + (size_t)(p % n) * s.W + c], a[q]);
+        }
+      }
     }
-    u_s[q * B + (i - q * B)] = a;
+#pragma unroll
+    for (int q = 0; q < ST_TOK; ++q)
+      if (q < nt) u_s[q * B + i] = a[q];
   }
   __syncthreads();
   for (int o = warp; o < no; o += ST_THREADS / 32) {
@@ -372,18 +411,15 @@ rglru_step_kernel(const float* proj, int ld, int x0, const float* __restrict__ b
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < nt * ST_CH; i += ST_THREADS) {
-    const int q = i / ST_CH, o = i - q * ST_CH;
-    if (o >= no) continue;
-    const int t = t0 + q, c = part * B + o0 + o;
-    float* row = state + (size_t)seq_slot[t] * state_ld;
+  if (fin) {
+    float* row = state + (size_t)slot_s[fq] * state_ld;
     float log_a, g;
-    rg_factors(z_s[0][o][q] + br[c], z_s[1][o][q] + bi[c], s.rate * rg_softplus(lam[c]), log_a, g);
-    const float S = fmaf(expf(log_a), row[c], g * u_s[q * B + o0 + o]);
-    row[c] = S;
+    rg_factors(z_s[0][fo][fq] + br[fc], z_s[1][fo][fq] + bi[fc], s.rate * rg_softplus(lam[fc]), log_a, g);
+    const float S = fmaf(expf(log_a), S_old, g * u_s[fq * B + o0 + fo]);
+    row[fc] = S;
     // (the entry of this position: no block of this launch reads it)
-    row[s.W + (size_t)(token_pos[t] % n) * s.W + c] = proj[(size_t)t * ld + x0 + c] + bx[c];
-    out[(size_t)t * s.W + c] = from_float<TO>(S * rg_gelu(proj[(size_t)t * ld + c] + by[c]));
+    row[s.W + (size_t)(pos_s[fq] % n) * s.W + fc] = x_now + bx[fc];
+    out[(size_t)(t0 + fq) * s.W + fc] = from_float<TO>(S * rg_gelu(y_now + by[fc]));
   }
 }
 
@@ -410,14 +446,21 @@ static int launch_rglru_conv(const float* x, int ldx, const float* bx, const flo
 }
 
 template <typename TO>
-static int launch_rglru_scan(const RglruScan& a, TO* out, int direct, cudaStream_t stream) {
+static int launch_rglru_scan(const RglruScan& a, TO* out, int direct, int prepared, cudaStream_t stream) {
   const dim3 grid(a.n_tiles, (a.s.W + RS_THREADS - 1) / RS_THREADS), block(RS_THREADS);
   if (direct) {
     launch_kernel(rglru_scan_kernel<TO, RG_DIRECT>, grid, block, 0, stream, a, out);
     return launch_status();
   }
-  launch_kernel(rglru_scan_kernel<TO, RG_LOCAL>, grid, block, 0, stream, a, out);
-  const int st = launch_status();
+  int st = DLGO_OK;
+  if (!prepared) {
+    launch_kernel(rglru_scan_kernel<TO, RG_LOCAL>, grid, block, 0, stream, a, out);
+    st = launch_status();
+    if (st != DLGO_OK) return st;
+  }
+  launch_kernel(rglru_carry_kernel, dim3((a.s.W + CY_THREADS - 1) / CY_THREADS, a.n_tiles), dim3(CY_THREADS), 0, stream, a.tiles,
+                a.n_tiles, a.seq_slot, (const float*)a.state, a.state_ld, a.seg, a.s.W);
+  st = launch_status();
   if (st != DLGO_OK) return st;
   launch_kernel(rglru_scan_kernel<TO, RG_FULL>, grid, block, 0, stream, a, out);
   return launch_status();
@@ -473,21 +516,21 @@ DLGO_EXPORT int dlgo_rglru_conv(const float* x, int ldx, const float* bx, const 
 // z [T, parts, 2 B] fp32: the gates' logits without biases (r, then i); u of dlgo_rglru_conv; y: fp32 without bias and
 // gelu (y_dtype 0, by [W]) or finished bfloat16 (y_dtype 1), row stride ldy; x, bx as in dlgo_rglru_conv; tiles: a
 // sequence's segments side by side in token order; seg: n_tiles * 3 * W floats of scratch (unused when `direct`: one
-// segment per sequence); out [T, W] in out_dtype.
+// segment per sequence); out [T, W] in out_dtype.  `prepared` (not direct): z and seg hold what LOCAL leaves.
 DLGO_EXPORT int dlgo_rglru_scan(float* z, const float* u, const float* br, const float* bi, const float* lam, const void* y,
                                 int y_dtype, int ldy, const float* by, const float* x, int ldx, const float* bx,
                                 const int* tiles, int n_tiles, const int* token_seq, const int* token_pos,
-                                const int* seq_slot, float* state, long long state_ld, float* seg, int direct, void* out,
-                                int out_dtype, int W, int parts, int taps, float rate, cudaStream_t stream) {
+                                const int* seq_slot, float* state, long long state_ld, float* seg, int direct, int prepared,
+                                void* out, int out_dtype, int W, int parts, int taps, float rate, cudaStream_t stream) {
   if (n_tiles <= 0) return DLGO_OK;
   const RglruShape s{W, parts, taps, rate};
-  if (!rglru_ok(s) || (!direct && seg == nullptr) || (y_dtype == DLGO_F32 && by == nullptr)) return DLGO_ERR_SIZE;
+  if (!rglru_ok(s) || (!direct && seg == nullptr) || (direct && prepared) || n_tiles > 65535 || (y_dtype == DLGO_F32 && by == nullptr)) return DLGO_ERR_SIZE;
   if (y_dtype != DLGO_F32 && y_dtype != DLGO_BF16) return DLGO_ERR_DTYPE;
   RglruScan a{z, u, br, bi, lam, y_dtype == DLGO_F32 ? (const float*)y : nullptr, by,
               y_dtype == DLGO_BF16 ? (const __nv_bfloat16*)y : nullptr, ldy, x, ldx, bx, tiles, n_tiles, token_seq,
               token_pos, seq_slot, state, state_ld, seg, s};
-  if (out_dtype == DLGO_F32) return launch_rglru_scan<float>(a, (float*)out, direct, stream);
-  if (out_dtype == DLGO_BF16) return launch_rglru_scan<__nv_bfloat16>(a, (__nv_bfloat16*)out, direct, stream);
+  if (out_dtype == DLGO_F32) return launch_rglru_scan<float>(a, (float*)out, direct, prepared, stream);
+  if (out_dtype == DLGO_BF16) return launch_rglru_scan<__nv_bfloat16>(a, (__nv_bfloat16*)out, direct, prepared, stream);
   return DLGO_ERR_DTYPE;
 }
 

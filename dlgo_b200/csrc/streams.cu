@@ -181,13 +181,14 @@ __global__ void __launch_bounds__(256) streams_step_kernel(StreamsStep p) {
 }
 
 // The same step for a layer norm over rows of a multiple of four numbers that fit a block's registers (NV float4 a
-// thread): one pass over the streams, the statistics from registers, mean first and then the squared deviations.
-template <typename TO, int THREADS, int NV>
+// thread): one pass over the streams, the statistics from registers, mean first and then the squared deviations.  S is
+// the number of streams, or MAX_STREAMS for any.
+template <typename TO, int THREADS, int NV, int S>
 __global__ void __launch_bounds__(THREADS) streams_layernorm_kernel(StreamsStep p) {
   pdl_launch_dependents();
   __shared__ float s_mix[MAX_STREAMS * MAX_STREAMS], s_wout[MAX_STREAMS], s_coeff[MAX_STREAMS];
   __shared__ float red[32];
-  const int s = p.s, d = p.d, tid = threadIdx.x;
+  const int s = S < MAX_STREAMS ? S : p.s, d = p.d, tid = threadIdx.x;
   if (tid < s * s && p.y) s_mix[tid] = p.mix[tid];
   if (tid < s) {
     if (p.y) s_wout[tid] = p.wout[tid];
@@ -214,9 +215,9 @@ __global__ void __launch_bounds__(THREADS) streams_layernorm_kernel(StreamsStep 
   for (int v = 0; v < NV; ++v) {
     const int i = (v * THREADS + tid) * 4;
     if (i >= d) continue;
-    float4 x[MAX_STREAMS];
+    float4 x[S];
 #pragma unroll
-    for (int a = 0; a < MAX_STREAMS; ++a)
+    for (int a = 0; a < S; ++a)
       if (a < s) x[a] = *reinterpret_cast<const float4*>(xr + (size_t)a * d + i);
     if (yr) {
       float4 y = *reinterpret_cast<const float4*>(yr + i);
@@ -226,11 +227,11 @@ __global__ void __launch_bounds__(THREADS) streams_layernorm_kernel(StreamsStep 
       }
       if (p.clear_y) *reinterpret_cast<float4*>(yr + i) = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int q = 0; q < MAX_STREAMS; ++q) {
+      for (int q = 0; q < S; ++q) {
         if (q < s) {
           float4 n = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-          for (int a = 0; a < MAX_STREAMS; ++a) {
+          for (int a = 0; a < S; ++a) {
             if (a < s) {
               const float m = s_mix[a * s + q];
               n.x = fmaf(m, x[a].x, n.x); n.y = fmaf(m, x[a].y, n.y);
@@ -246,7 +247,7 @@ __global__ void __launch_bounds__(THREADS) streams_layernorm_kernel(StreamsStep 
       }
     } else {
 #pragma unroll
-      for (int a = 0; a < MAX_STREAMS; ++a) {
+      for (int a = 0; a < S; ++a) {
         if (a < s) {
           const float c = s_coeff[a];
           u[v].x = fmaf(c, x[a].x, u[v].x); u[v].y = fmaf(c, x[a].y, u[v].y);
@@ -275,12 +276,22 @@ __global__ void __launch_bounds__(THREADS) streams_layernorm_kernel(StreamsStep 
   }
 }
 
+template <typename TO, int S>
+static void launch_streams_layernorm_of(const StreamsStep& p, int n_rows, cudaStream_t stream) {
+  if (p.d <= 512) launch_kernel(streams_layernorm_kernel<TO, 128, 1, S>, dim3(n_rows), dim3(128), 0, stream, p);
+  else if (p.d <= 1024) launch_kernel(streams_layernorm_kernel<TO, 256, 1, S>, dim3(n_rows), dim3(256), 0, stream, p);
+  else if (p.d <= 2048) launch_kernel(streams_layernorm_kernel<TO, 512, 1, S>, dim3(n_rows), dim3(512), 0, stream, p);
+  else launch_kernel(streams_layernorm_kernel<TO, 512, 2, S>, dim3(n_rows), dim3(512), 0, stream, p);
+}
 template <typename TO>
 static void launch_streams_layernorm(const StreamsStep& p, int n_rows, cudaStream_t stream) {
-  if (p.d <= 512) launch_kernel(streams_layernorm_kernel<TO, 128, 1>, dim3(n_rows), dim3(128), 0, stream, p);
-  else if (p.d <= 1024) launch_kernel(streams_layernorm_kernel<TO, 256, 1>, dim3(n_rows), dim3(256), 0, stream, p);
-  else if (p.d <= 2048) launch_kernel(streams_layernorm_kernel<TO, 256, 2>, dim3(n_rows), dim3(256), 0, stream, p);
-  else launch_kernel(streams_layernorm_kernel<TO, 512, 2>, dim3(n_rows), dim3(512), 0, stream, p);
+  switch (p.s) {
+    case 1: launch_streams_layernorm_of<TO, 1>(p, n_rows, stream); break;
+    case 2: launch_streams_layernorm_of<TO, 2>(p, n_rows, stream); break;
+    case 3: launch_streams_layernorm_of<TO, 3>(p, n_rows, stream); break;
+    case 4: launch_streams_layernorm_of<TO, 4>(p, n_rows, stream); break;
+    default: launch_streams_layernorm_of<TO, MAX_STREAMS>(p, n_rows, stream); break;
+  }
 }
 
 __device__ __forceinline__ float activate(float z, int act) {

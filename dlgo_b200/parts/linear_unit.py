@@ -95,17 +95,14 @@ class RealGatedLinearUnit(Mixer):
             get(n[k]).to(torch.float32).reshape(-1).contiguous() for k in
             ("y_bias", "x_bias", "conv", "conv_bias", "r_bias", "i_bias", "decay"))
 
-    def _gate_logits(self, u: torch.Tensor, rows: Optional[torch.Tensor], by_part: bool) -> torch.Tensor:
+    def _gate_logits(self, u: torch.Tensor, rows: Optional[torch.Tensor]) -> torch.Tensor:
         """[T * parts, 2 B] fp32: a part's rows of both matrices times its part of u (a grouped contraction whose groups
         are the parts, every one with all tokens)."""
         T, B = u.shape[0], self.width // self.parts
         z = torch.empty((T * self.parts, 2 * B), dtype=torch.float32, device=u.device)
-        if by_part:
-            K.moe_gemm_tc(K.part_plan(self.parts, T, K.MOE_TC_ROWS, u.device), rows, self.w_gates, z, True, K.ACT_NONE)
-        else:
-            tile_rows = K.MOE_FEW_ROWS if T <= 64 else K.MOE_TILE_ROWS
-            a = rows if rows is not None else u.view(T * self.parts, B)
-            K.moe_gemm(K.part_plan(self.parts, T, tile_rows, u.device), a, self.w_gates, z, 1, True, K.ACT_NONE)
+        a = rows if rows is not None else u.view(T * self.parts, B)
+        K.moe_gemm(K.part_plan(self.parts, T, K.MOE_FEW_ROWS if T <= 64 else K.MOE_TILE_ROWS, u.device), a, self.w_gates, z,
+                   1, True, K.ACT_NONE)
         return z
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: Any, cache: Any,
@@ -120,8 +117,9 @@ class RealGatedLinearUnit(Mixer):
                              self.b_r, self.b_i, self.lam, ctx.token_pos, ctx.seq_slot, st, s)
             self.wo(a, ADD_F32, residual)
             return
-        on_tc = T >= TC_MIN_TOKENS and K.moe_gemm_tc_takes(act, 2 * w // self.parts, w // self.parts)
-        if on_tc:
+        # bfloat16 prompts: the gates, and a segment's walk from zero behind them, in one launch on the tensor cores
+        on_tc = T >= TC_MIN_TOKENS and K.rglru_gates_tc_takes(act, w // self.parts)
+        if act == torch.bfloat16 and T >= TC_MIN_TOKENS:
             y, by = self.w_y.bias_act(x, self.b_y, K.ACT_GELU_TANH), None
             xs = self.w_x(x, STORE_F32)
         else:
@@ -130,12 +128,15 @@ class RealGatedLinearUnit(Mixer):
         tiles, n_tiles, _ = ctx.tiles(CONV_TILE)
         u, rows = K.rglru_conv(xs, self.b_x, self.taps, self.b_conv, tiles, n_tiles, ctx.token_seq, ctx.token_pos,
                                ctx.seq_slot, st, s, None if act == torch.float32 else act, on_tc)
-        z = self._gate_logits(u, rows, on_tc)
-        tiles, n_tiles, _ = ctx.tiles(segment(T, w))
-        direct = n_tiles == ctx.n_seqs
+        tiles, n_tiles, _ = ctx.tiles(K.RGLRU_TC_SEGMENT if on_tc else segment(T, w))
+        direct = not on_tc and n_tiles == ctx.n_seqs
         scratch = None if direct else ctx.scratch("rglru_segments", n_tiles * 3 * w)
+        if on_tc:
+            z = K.rglru_gates_tc(rows, self.w_gates, self.b_r, self.b_i, self.lam, tiles, n_tiles, T, scratch, s)
+        else:
+            z = self._gate_logits(u, rows)
         a = K.rglru_scan(z, u, self.b_r, self.b_i, self.lam, y, by, xs, self.b_x, tiles, n_tiles, direct, ctx.token_seq,
-                         ctx.token_pos, ctx.seq_slot, st, scratch, s, act)
+                         ctx.token_pos, ctx.seq_slot, st, scratch, s, act, prepared=on_tc)
         self.wo(a, ADD_F32, residual)
 
 
