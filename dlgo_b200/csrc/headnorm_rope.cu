@@ -113,6 +113,11 @@ headnorm_rope_append_kernel(float* proj, int ld, const float* __restrict__ bias,
 // angles' cosines and sines once per token, rows in 16-byte pieces, several heads of a warp in flight together.
 constexpr int HT_WARPS = 8, HT_HEADS = 3;
 
+__device__ __forceinline__ void ht_store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void ht_store2(__nv_bfloat16* p, float a, float b) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+}
+
 template <typename T, int NV>
 __global__ void __launch_bounds__(HT_WARPS * 32)
 headnorm_rope_token_kernel(float* proj, int ld, const float* __restrict__ w_q, const float* __restrict__ w_k, float eps,
@@ -135,12 +140,11 @@ headnorm_rope_token_kernel(float* proj, int ld, const float* __restrict__ w_q, c
       row_base = ((long long)page * Hkv * page_size + pos % page_size) * hd;
     }
   }
-  for (int i = threadIdx.x; i < rh; i += HT_WARPS * 32) sincosf((float)pos * freq[i], &cs[rh + i], &cs[i]);
-  __syncthreads();
+  bool angles = false;
   pdl_wait();
   const int heads = Hq + 2 * Hkv;
   float* row = proj + (size_t)t * ld;
-  for (int g = warp; g < heads; g += HT_WARPS * HT_HEADS) {
+  for (int g = warp; g - warp < heads; g += HT_WARPS * HT_HEADS) {      // (every warp takes part in the first round)
     float4 x[HT_HEADS][NV];
 #pragma unroll
     for (int k = 0; k < HT_HEADS; ++k) {
@@ -154,6 +158,11 @@ headnorm_rope_token_kernel(float* proj, int ld, const float* __restrict__ w_q, c
         x[k][v] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (head < heads && i < n) x[k][v] = *reinterpret_cast<const float4*>(src + i);
       }
+    }
+    if (!angles) {                                                 // (while the first rows are on their way)
+      for (int i = threadIdx.x; i < rh; i += HT_WARPS * 32) sincosf((float)pos * freq[i], &cs[rh + i], &cs[i]);
+      __syncthreads();
+      angles = true;
     }
 #pragma unroll
     for (int k = 0; k < HT_HEADS; ++k) {
@@ -196,12 +205,22 @@ headnorm_rope_token_kernel(float* proj, int ld, const float* __restrict__ w_q, c
       __syncwarp();
       if (dst == nullptr) continue;
       const int turned = is_v ? 0 : rot;
-      for (int i = lane; i < (turned >> 1); i += 32) {
-        const float a = u_s[i], b = u_s[i + rh];
-        dst[i] = from_float<T>(a * cs[i] - b * cs[rh + i]);
-        dst[i + rh] = from_float<T>(b * cs[i] + a * cs[rh + i]);
+      if ((rh & 1) == 0) {                                         // (then rot is a multiple of four: whole pieces)
+        for (int i = 2 * lane; i < (turned >> 1); i += 64) {
+          const float2 a = *reinterpret_cast<const float2*>(u_s + i), b = *reinterpret_cast<const float2*>(u_s + i + rh);
+          const float2 c = *reinterpret_cast<const float2*>(cs + i), sn = *reinterpret_cast<const float2*>(cs + rh + i);
+          ht_store2(dst + i, a.x * c.x - b.x * sn.x, a.y * c.y - b.y * sn.y);
+          ht_store2(dst + i + rh, b.x * c.x + a.x * sn.x, b.y * c.y + a.y * sn.y);
+        }
+        for (int i = turned + 2 * lane; i < hd; i += 64) ht_store2(dst + i, u_s[i], u_s[i + 1]);
+      } else {
+        for (int i = lane; i < (turned >> 1); i += 32) {
+          const float a = u_s[i], b = u_s[i + rh];
+          dst[i] = from_float<T>(a * cs[i] - b * cs[rh + i]);
+          dst[i + rh] = from_float<T>(b * cs[i] + a * cs[rh + i]);
+        }
+        for (int i = turned + lane; i < hd; i += 32) dst[i] = from_float<T>(u_s[i]);
       }
-      for (int i = turned + lane; i < hd; i += 32) dst[i] = from_float<T>(u_s[i]);
     }
   }
 }
@@ -217,7 +236,7 @@ int launch_headnorm_rope(float* proj, int ld, const float* bias, const float* w_
   const long long blocks = (items + HR_WARPS - 1) / HR_WARPS;
   if (blocks > 0x7fffffffLL) return DLGO_ERR_SIZE;
   const int wide = dk > dv ? dk : dv;
-  if (!v_from_k && bias == nullptr && w_q != nullptr && w_k != nullptr && norm_dim == dk && ((dk | dv | ld) & 3) == 0 && hd <= 256 &&
+  if (!v_from_k && bias == nullptr && w_q != nullptr && w_k != nullptr && norm_dim == dk && ((dk | dv | ld) & 3) == 0 && hd % 2 == 0 && hd <= 256 &&
       (((uintptr_t)proj | (uintptr_t)w_q | (uintptr_t)w_k) & 15) == 0) {
     const int nv = (hd > wide ? hd : wide) <= 128 ? 1 : 2;
     const size_t ht = sizeof(float) * (((size_t)rot + 3) / 4 * 4 + HT_WARPS * 128 * nv);

@@ -214,19 +214,27 @@ GATE_SIGMOID, GATE_SILU = 0, 1
 MAX_STREAMS = 8
 
 
+def streams_step_passes(norm_kind: int, d: int) -> bool:
+    """Whether a write can be read on without storing the streams (``keep`` False) through this norm: rows are not read
+    twice."""
+    return norm_kind in (NORM_NONE, NORM_DYT) or (norm_kind == NORM_LAYER and d % 4 == 0 and d <= 4096)
+
+
 def streams_step(X: torch.Tensor, *, y: Optional[torch.Tensor] = None, y_bias: Optional[torch.Tensor] = None,
                  mix: Optional[torch.Tensor] = None, write: Optional[torch.Tensor] = None, clear_y: bool = False,
                  read: Optional[torch.Tensor] = None, norm_kind: int = NORM_NONE,
                  norm_w: Optional[torch.Tensor] = None, norm_b: Optional[torch.Tensor] = None,
                  norm_alpha: Optional[torch.Tensor] = None, eps: float = 0.0,
-                 out_dtype: Optional[torch.dtype] = None, rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                 out_dtype: Optional[torch.dtype] = None, rows: Optional[torch.Tensor] = None,
+                 keep: bool = True) -> Optional[torch.Tensor]:
     """One hand-over on residual streams ``X`` [T, s, d] (fp32, in place).
 
     Write part (with ``y`` [T, d] fp32): ``X[t, q] = sum_r mix[r, q] X[t, r] + write[q] * (y[t] + y_bias)``,
     all streams at once from the old values; ``clear_y`` leaves zeros in ``y``.  Read part (with
     ``out_dtype``): ``u = sum_r read[r] X[t, r]`` (``read`` None: the plain sum) through the norm
     (``NORM_DYT``: tanh(alpha u) w + b; ``NORM_LAYER``: layer norm with w and b; ``NORM_RMS``; ``NORM_NONE``: u itself) into a new [R, d] tensor;
-    ``rows`` picks the rows to read (read part only)."""
+    ``rows`` picks the rows to read (read part only).  ``keep`` False: the new streams are only read on, not stored
+    (:func:`streams_step_passes`; ``rows`` may then pick rows of a write as well, and ``y`` is left as it is)."""
     _need(X, torch.float32, "X")
     if X.dim() != 3:
         raise KernelError("streams_step: X must be [tokens, streams, hidden]")
@@ -235,7 +243,7 @@ def streams_step(X: torch.Tensor, *, y: Optional[torch.Tensor] = None, y_bias: O
         raise KernelError(f"streams_step: at most {MAX_STREAMS} streams, got {s}")
     if y is not None:
         _need(y, torch.float32, "y")
-        if tuple(y.shape) != (T, d) or mix is None or write is None or rows is not None:
+        if tuple(y.shape) != (T, d) or mix is None or write is None or (rows is not None and keep):
             raise KernelError("streams_step: the write part needs y [T, d], mix, write, and no row selection")
         _need(mix, torch.float32, "mix")
         _need(write, torch.float32, "write")
@@ -258,9 +266,9 @@ def streams_step(X: torch.Tensor, *, y: Optional[torch.Tensor] = None, y_bias: O
     elif y is None:
         return None
     st = _lib("streams").dlgo_streams_step(
-        _ptr(X), _i(T), _i(s), _i(d), _ptr(y), _ptr(y_bias), _ptr(mix), _ptr(write), _i(1 if clear_y else 0),
+        _ptr(X), _i(T), _i(s), _i(d), _ptr(y), _ptr(y_bias), _ptr(mix), _ptr(write), _i(1 if clear_y and keep else 0),
         _ptr(read), _i(norm_kind), _ptr(norm_w), _ptr(norm_b), _ptr(norm_alpha), _f(eps), _ptr(out),
-        _i(dtype_code(out_dtype) if out_dtype is not None else F32), _ptr(rows), _i(R), _stream())
+        _i(dtype_code(out_dtype) if out_dtype is not None else F32), _ptr(rows), _i(R), _i(1 if keep else 0), _stream())
     _check(st, "streams_step")
     return out
 
@@ -969,9 +977,9 @@ def _rglru_check(what: str, s: RglruShape, state: torch.Tensor, **weights: torch
 
 def rglru_conv(x: torch.Tensor, bx: torch.Tensor, taps: torch.Tensor, bc: torch.Tensor, tiles: torch.Tensor, n_tiles: int,
                token_seq: torch.Tensor, token_pos: torch.Tensor, seq_slot: torch.Tensor, state: torch.Tensor, shape: RglruShape,
-               rows_dtype: Optional[torch.dtype], by_part: bool) -> tuple:
+               rows_dtype: Optional[torch.dtype], by_part: bool, f32: bool = True) -> tuple:
     """The causal convolution over time of ``x`` + bx (fp32 view [T, width]), reaching back into the state rows: u [T, width]
-    fp32, and with ``rows_dtype`` u as rows of a part in that type: [parts * T, width / parts] sorted by part
+    fp32 (``f32`` False: None), and with ``rows_dtype`` u as rows of a part in that type: [parts * T, width / parts] sorted by part
     (``by_part``), else [T * parts, width / parts]."""
     _rglru_check("rglru_conv", shape, state, bx=bx, taps=taps, bc=bc)
     _f32_rows("rglru_conv", x=x)
@@ -980,7 +988,7 @@ def rglru_conv(x: torch.Tensor, bx: torch.Tensor, taps: torch.Tensor, bc: torch.
     T = x.shape[0]
     if x.shape[1] != shape.width:
         raise KernelError("rglru_conv: x must have a column per channel")
-    u = torch.empty((T, shape.width), dtype=torch.float32, device=x.device)
+    u = torch.empty((T, shape.width), dtype=torch.float32, device=x.device) if f32 else None
     rows = None
     if rows_dtype is not None:
         rows = torch.empty((T * shape.parts, shape.width // shape.parts), dtype=rows_dtype, device=x.device)
@@ -1026,7 +1034,7 @@ def rglru_gates_tc(rows: torch.Tensor, w_gates: torch.Tensor, br: torch.Tensor, 
     return z
 
 
-def rglru_scan(z: torch.Tensor, u: torch.Tensor, br: torch.Tensor, bi: torch.Tensor, lam: torch.Tensor, y: torch.Tensor,
+def rglru_scan(z: torch.Tensor, u: Optional[torch.Tensor], br: torch.Tensor, bi: torch.Tensor, lam: torch.Tensor, y: torch.Tensor,
                by: Optional[torch.Tensor], x: torch.Tensor, bx: torch.Tensor, tiles: torch.Tensor, n_tiles: int, direct: bool,
                token_seq: torch.Tensor, token_pos: torch.Tensor, seq_slot: torch.Tensor, state: torch.Tensor,
                scratch: Optional[torch.Tensor], shape: RglruShape, out_dtype: torch.dtype,
@@ -1038,12 +1046,16 @@ def rglru_scan(z: torch.Tensor, u: torch.Tensor, br: torch.Tensor, bi: torch.Ten
     state rows.  ``prepared``: ``z`` and ``scratch`` are :func:`rglru_gates_tc`'s (over the same tiles).  Returns [T, width]
     in ``out_dtype``."""
     _rglru_check("rglru_scan", shape, state, br=br, bi=bi, lam=lam, bx=bx)
-    _f32_rows("rglru_scan", z=z, u=u, x=x)
+    _f32_rows("rglru_scan", z=z, x=x)
+    if u is not None:
+        _f32_rows("rglru_scan", u=u)
+    elif not prepared:
+        raise KernelError("rglru_scan: u is needed unless the gates' launch has been there")
     for n, t in (("tiles", tiles), ("token_seq", token_seq), ("token_pos", token_pos), ("seq_slot", seq_slot)):
         _need(t, torch.int32, n)
-    T, w = u.shape
+    T, w = x.shape
     _need(z, None, "z")
-    if w != shape.width or z.numel() != T * 2 * w or x.shape[1] != w or y.shape != (T, w) or y.stride(1) != 1:
+    if w != shape.width or (u is not None and u.shape != x.shape) or z.numel() != T * 2 * w or y.shape != (T, w) or y.stride(1) != 1:
         raise KernelError("rglru_scan: shapes do not fit")
     if y.dtype != (torch.float32 if by is not None else torch.bfloat16):
         raise KernelError("rglru_scan: y is float32 with a bias, or finished bfloat16")
@@ -1051,7 +1063,7 @@ def rglru_scan(z: torch.Tensor, u: torch.Tensor, br: torch.Tensor, bi: torch.Ten
         _need(by, torch.float32, "by")
     if not direct and (scratch is None or scratch.dtype != torch.float32 or scratch.numel() < n_tiles * 3 * w):
         raise KernelError(f"rglru_scan: {n_tiles} segments need {n_tiles * 3 * w} floats of scratch")
-    out = torch.empty((T, w), dtype=out_dtype, device=u.device)
+    out = torch.empty((T, w), dtype=out_dtype, device=x.device)
     st = _lib("rglru").dlgo_rglru_scan(
         _ptr(z), _ptr(u), _ptr(br), _ptr(bi), _ptr(lam), _ptr(y), _i(dtype_code(y.dtype)), _i(y.stride(0)), _ptr(by), _ptr(x),
         _i(x.stride(0)), _ptr(bx), _ptr(tiles), _i(n_tiles), _ptr(token_seq), _ptr(token_pos), _ptr(seq_slot), _ptr(state),

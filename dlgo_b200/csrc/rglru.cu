@@ -81,11 +81,11 @@ rglru_conv_kernel(const float* x, int ldx, const float* __restrict__ bx, const f
     }
   };
   auto emit = [&](int t, const float (&y)[W4]) {
-    float* dst = u_out + (size_t)t * s.W + c;
+    float* dst = u_out == nullptr ? nullptr : u_out + (size_t)t * s.W + c;
     TO* row = rows == nullptr ? nullptr
                               : rows + (by_part ? ((size_t)part * T + t) * B + (c - part * B) : (size_t)t * s.W + c);
     if (W4 == 4) {
-      *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1 % W4], y[2 % W4], y[3 % W4]);
+      if (dst != nullptr) *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1 % W4], y[2 % W4], y[3 % W4]);
       if (row != nullptr) {
         if (sizeof(TO) == 2) {
           __nv_bfloat162 h[2] = {__floats2bfloat162_rn(y[0], y[1 % W4]), __floats2bfloat162_rn(y[2 % W4], y[3 % W4])};
@@ -95,7 +95,7 @@ rglru_conv_kernel(const float* x, int ldx, const float* __restrict__ bx, const f
         }
       }
     } else {
-      dst[0] = y[0];
+      if (dst != nullptr) dst[0] = y[0];
       if (row != nullptr) row[0] = from_float<TO>(y[0]);
     }
   };
@@ -157,35 +157,56 @@ rglru_conv_kernel(const float* x, int ldx, const float* __restrict__ bx, const f
 }
 
 // ------------------------------------------------------------------------------- recurrence (prompts)
-// The start of every segment: a thread per channel of a sequence, the ends of several segments in flight together.
-constexpr int CY_THREADS = 64, CY_FLY = 16;
-__global__ void __launch_bounds__(CY_THREADS)
+// The start of every segment.  A block takes 32 channels of a sequence and CY_WAYS * CY_FLY segments at a time: a warp
+// composes CY_FLY neighbouring segments (each a map S -> f S + e) of its lanes' channels, the warps' maps meet in shared
+// memory, and every warp walks its segments again from its start.
+constexpr int CY_WAYS = 8, CY_FLY = 8;
+__global__ void __launch_bounds__(CY_WAYS * 32)
 rglru_carry_kernel(const int* __restrict__ tiles, int n_tiles, const int* __restrict__ seq_slot, const float* state,
                    long long state_ld, float* seg, int W) {
   pdl_launch_dependents();
-  const int j0 = blockIdx.y, seq = tiles[j0 * 3];
+  __shared__ float f_s[CY_WAYS][32], e_s[CY_WAYS][32];
+  const int j0 = blockIdx.y, seq = tiles[j0 * 3], lane = threadIdx.x & 31, way = threadIdx.x >> 5;
   if (j0 > 0 && tiles[(j0 - 1) * 3] == seq) return;                // a block row per first segment of a sequence
-  const int c = blockIdx.x * CY_THREADS + threadIdx.x;
-  if (c >= W) return;
+  const int c = min(blockIdx.x * 32 + lane, W - 1);                // (lanes beyond the channels repeat the last one)
   int end = j0 + 1;
   while (end < n_tiles && tiles[end * 3] == seq) ++end;
   pdl_wait();
   float S = state[(size_t)seq_slot[seq] * state_ld + c];
-  for (int j = j0; j < end; j += CY_FLY) {
-    float e[CY_FLY], l[CY_FLY];
+  for (int base = j0; base < end; base += CY_WAYS * CY_FLY) {
+    const int j = base + way * CY_FLY;
+    float e[CY_FLY], f[CY_FLY];
 #pragma unroll
     for (int q = 0; q < CY_FLY; ++q) {
       const float* sg = seg + (size_t)min(j + q, end - 1) * 3 * W + c;
       e[q] = sg[0];
-      l[q] = sg[W];
+      f[q] = sg[W];
+    }
+    float F = 1.f, E = 0.f;
+#pragma unroll
+    for (int q = 0; q < CY_FLY; ++q) {
+      f[q] = expf(f[q]);
+      if (j + q < end) {
+        F *= f[q];
+        E = fmaf(f[q], E, e[q]);
+      }
+    }
+    f_s[way][lane] = F;
+    e_s[way][lane] = E;
+    __syncthreads();
+    float mine = S;
+    for (int w = 0; w < CY_WAYS; ++w) {
+      if (w == way) mine = S;
+      S = fmaf(f_s[w][lane], S, e_s[w][lane]);
     }
 #pragma unroll
     for (int q = 0; q < CY_FLY; ++q) {
       if (j + q < end) {
-        seg[((size_t)(j + q) * 3 + 2) * W + c] = S;
-        S = fmaf(expf(l[q]), S, e[q]);
+        seg[((size_t)(j + q) * 3 + 2) * W + c] = mine;
+        mine = fmaf(f[q], mine, e[q]);
       }
     }
+    __syncthreads();                                               // the maps have been read
   }
 }
 
@@ -291,22 +312,47 @@ rglru_scan_kernel(RglruScan a, TO* out) {
 }
 
 // ------------------------------------------------------------------------------- one token per sequence
-// A block owns CH neighbouring channels of one part for up to TOK tokens: their part of u in shared memory, a warp per
-// output channel at a time over the rows of both matrices, then the recurrence.
-constexpr int ST_THREADS = 256, ST_CH = 16, ST_TOK = 8;
+// A block owns CH neighbouring channels of one part for up to TOK tokens: their part of u in shared memory (a thread per
+// channel, all inputs of all tokens in flight together), a warp per output channel at a time over the rows of both
+// matrices, then the recurrence.
+constexpr int ST_THREADS = 256, ST_CH = 16, ST_TOK = 8, ST_TAPS = 4;
 static_assert(ST_CH * ST_TOK <= ST_THREADS, "the last pass has a thread per channel and token");
 
-template <typename TW> struct Pair;
-template <> struct Pair<float> {
-  static __device__ __forceinline__ float2 load(const float* p) { return *reinterpret_cast<const float2*>(p); }
+template <typename TW, int VEC> struct WRow;
+template <typename TW> struct WRow<TW, 1> {
+  static __device__ __forceinline__ void load(const TW* p, float (&o)[1]) { o[0] = to_float(p[0]); }
 };
-template <> struct Pair<__nv_bfloat16> {
-  static __device__ __forceinline__ float2 load(const __nv_bfloat16* p) {
-    return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+template <> struct WRow<float, 4> {
+  static __device__ __forceinline__ void load(const float* p, float (&o)[4]) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
+  }
+};
+template <> struct WRow<__nv_bfloat16, 4> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&o)[4]) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y;
   }
 };
 
-template <typename TW, typename TO, bool PAIRS>
+// v[k] summed over the warp for k < 16: lane l ends with the sum of entry l >> 1 (halves of the entries are traded at
+// distances 16, 8, 4, 2, then neighbours add up)
+__device__ __forceinline__ float warp_sum16(float (&v)[16], int lane) {
+#pragma unroll
+  for (int o = 16, n = 8; n > 0; o >>= 1, n >>= 1) {
+    const bool hi = (lane & o) != 0;
+#pragma unroll
+    for (int k = 0; k < n; ++k) {
+      const float give = hi ? v[k] : v[k + n], keep = hi ? v[k + n] : v[k];
+      v[k] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+    }
+  }
+  return v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
+}
+
+template <typename TW, typename TO, int VEC>
 __global__ void __launch_bounds__(ST_THREADS, 2)
 rglru_step_kernel(const float* proj, int ld, int x0, const float* __restrict__ by, const float* __restrict__ bx,
                   const float* __restrict__ w_taps, const float* __restrict__ bc, const TW* __restrict__ w_gates,
@@ -315,8 +361,9 @@ rglru_step_kernel(const float* proj, int ld, int x0, const float* __restrict__ b
                   TO* out, int T, int tok, RglruShape s) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float u_s[];                     // [tok][B]
-  __shared__ float z_s[2][ST_CH][ST_TOK];
-  __shared__ int pos_s[ST_TOK], slot_s[ST_TOK];
+  __shared__ float z_s[2][ST_TOK][ST_CH];
+  __shared__ int pos_s[ST_TOK], entry_s[ST_TAPS - 1][ST_TOK];
+  __shared__ long long row_s[ST_TOK];
   const int B = s.B(), n = s.taps, per_part = (B + ST_CH - 1) / ST_CH;
   const int part = blockIdx.x / per_part, o0 = (blockIdx.x - part * per_part) * ST_CH, no = min(ST_CH, B - o0);
   const int t0 = blockIdx.y * tok, nt = min(tok, T - t0);
@@ -326,100 +373,103 @@ rglru_step_kernel(const float* proj, int ld, int x0, const float* __restrict__ b
     const char* p = (const char*)(w_gates + ((size_t)part * 2 * B + (o & 1) * B + o0 + (o >> 1)) * B);
     for (int b = lane * 128; b < B * (int)sizeof(TW); b += 32 * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(p + b));
   }
-  if (threadIdx.x < nt) {                                          // the step's own inputs
-    pos_s[threadIdx.x] = token_pos[t0 + threadIdx.x];
-    slot_s[threadIdx.x] = seq_slot[t0 + threadIdx.x];
+  if (threadIdx.x < ST_TOK) {                                      // the step's own inputs (tokens beyond the last repeat it)
+    const int t = t0 + min((int)threadIdx.x, nt - 1), pos = token_pos[t];
+    pos_s[threadIdx.x] = pos;
+    row_s[threadIdx.x] = (long long)seq_slot[t] * state_ld;
+#pragma unroll
+    for (int j = 0; j < ST_TAPS - 1; ++j) {                        // the entry of the input j + 1 tokens before, or none
+      const int p = pos - 1 - j;
+      entry_s[j][threadIdx.x] = (j < n - 1 && p >= 0) ? p % n : -1;
+    }
   }
   __syncthreads();
+  const int fq = threadIdx.x / ST_CH, fo = threadIdx.x - fq * ST_CH, fc = part * B + o0 + min(fo, no - 1);
+  const bool fin = fq < nt && fo < no;
+  float f_br = 0.f, f_bi = 0.f, f_rate = 0.f, f_by = 0.f, f_bx = 0.f;
+  if (fin) {                                                       // weights
+    f_br = br[fc];
+    f_bi = bi[fc];
+    f_rate = s.rate * rg_softplus(lam[fc]);
+    f_by = by[fc];
+    f_bx = bx[fc];
+  }
   pdl_wait();
   // what the last pass needs of this block's own channels: requested now
   float S_old = 0.f, y_now = 0.f, x_now = 0.f;
-  const int fq = threadIdx.x / ST_CH, fo = threadIdx.x - fq * ST_CH, fc = part * B + o0 + fo;
-  const bool fin = fq < nt && fo < no;                             // (ST_TOK * ST_CH items, no more than threads)
   if (fin) {
     const float* pr = proj + (size_t)(t0 + fq) * ld;
-    S_old = state[(size_t)slot_s[fq] * state_ld + fc];
+    S_old = state[row_s[fq] + fc];
     y_now = pr[fc];
     x_now = pr[x0 + fc];
   }
-  // u of the part: a thread per channel, every token's inputs in flight together
   for (int i = threadIdx.x; i < B; i += ST_THREADS) {
     const int c = part * B + i;
-    const float b_x = bx[c], b_c = bc[c];
-    float a[ST_TOK];
+    float now[ST_TOK], old[ST_TAPS - 1][ST_TOK], w[ST_TAPS - 1];
 #pragma unroll
-    for (int q = 0; q < ST_TOK; ++q) a[q] = q < nt ? proj[(size_t)(t0 + q) * ld + x0 + c] : 0.f;
-    const float w_now = w_taps[(size_t)c * n + n - 1];
+    for (int q = 0; q < ST_TOK; ++q) now[q] = proj[(size_t)(t0 + min(q, nt - 1)) * ld + x0 + c];
 #pragma unroll
-    for (int q = 0; q < ST_TOK; ++q) a[q] = fmaf(w_now, a[q] + b_x, b_c);
-#pragma unroll 3
-    for (int j = 0; j < n - 1; ++j) {
-      const float w = w_taps[(size_t)c * n + j];
+    for (int j = 0; j < ST_TAPS - 1; ++j) {
+      w[j] = j < n - 1 ? w_taps[(size_t)c * n + n - 2 - j] : 0.f;
 #pragma unroll
       for (int q = 0; q < ST_TOK; ++q) {
-        if (q < nt) {
-          const int p = pos_s[q] - (n - 1) + j;
-          if (p >= 0) a[q] = fmaf(w, state[(size_t)slot_s[q] * state_ld + s.W + (size_t)(p % n) * s.W + c], a[q]);
-        }
+        const int entry = entry_s[j][q];
+        old[j][q] = 0.f;
+        if (entry >= 0) old[j][q] = state[row_s[q] + s.W + (size_t)entry * s.W + c];
       }
     }
+    const float w_now = w_taps[(size_t)c * n + n - 1], b_x = bx[c], b_c = bc[c];
 #pragma unroll
-    for (int q = 0; q < ST_TOK; ++q)
-      if (q < nt) u_s[q * B + i] = a[q];
+    for (int q = 0; q < ST_TOK; ++q) {
+      float a = b_c;
+      for (int j = n - 2; j >= ST_TAPS - 1; --j) {                 // taps beyond those in registers, oldest first
+        const int p = pos_s[q] - 1 - j;
+        if (p >= 0) a = fmaf(w_taps[(size_t)c * n + n - 2 - j], state[row_s[q] + s.W + (size_t)(p % n) * s.W + c], a);
+      }
+#pragma unroll
+      for (int j = ST_TAPS - 2; j >= 0; --j) a = fmaf(w[j], old[j][q], a);
+      a = fmaf(w_now, now[q] + b_x, a);
+      if (q < nt) u_s[q * B + i] = a;
+    }
   }
   __syncthreads();
   for (int o = warp; o < no; o += ST_THREADS / 32) {
     const TW* wr = w_gates + ((size_t)part * 2 * B + o0 + o) * B;
     const TW* wi = wr + (size_t)B * B;
-    float ar[ST_TOK], ai[ST_TOK];
+    float acc[2 * ST_TOK];                                         // r of every token, then i
 #pragma unroll
-    for (int q = 0; q < ST_TOK; ++q) ar[q] = ai[q] = 0.f;
-    if (PAIRS) {
+    for (int q = 0; q < 2 * ST_TOK; ++q) acc[q] = 0.f;
 #pragma unroll 2
-      for (int k = lane * 2; k < B; k += 64) {
-        const float2 r = Pair<TW>::load(wr + k), i = Pair<TW>::load(wi + k);
+    for (int k = lane * VEC; k < B; k += 32 * VEC) {
+      float r[VEC], i[VEC];
+      WRow<TW, VEC>::load(wr + k, r);
+      WRow<TW, VEC>::load(wi + k, i);
 #pragma unroll
-        for (int q = 0; q < ST_TOK; ++q) {
-          if (q < nt) {
-            const float2 u = *reinterpret_cast<const float2*>(u_s + q * B + k);
-            ar[q] = fmaf(r.x, u.x, fmaf(r.y, u.y, ar[q]));
-            ai[q] = fmaf(i.x, u.x, fmaf(i.y, u.y, ai[q]));
-          }
-        }
-      }
-    } else {
-      for (int k = lane; k < B; k += 32) {
-        const float r = to_float(wr[k]), i = to_float(wi[k]);
+      for (int q = 0; q < ST_TOK; ++q) {
+        if (q < nt) {
+          float u[VEC];
+          WRow<float, VEC>::load(u_s + q * B + k, u);
 #pragma unroll
-        for (int q = 0; q < ST_TOK; ++q) {
-          if (q < nt) {
-            ar[q] = fmaf(r, u_s[q * B + k], ar[q]);
-            ai[q] = fmaf(i, u_s[q * B + k], ai[q]);
+          for (int e = 0; e < VEC; ++e) {
+            acc[q] = fmaf(r[e], u[e], acc[q]);
+            acc[ST_TOK + q] = fmaf(i[e], u[e], acc[ST_TOK + q]);
           }
         }
       }
     }
-#pragma unroll
-    for (int q = 0; q < ST_TOK; ++q) {
-      if (q < nt) {                                                // (uniform over the block)
-        const float r = warp_sum(ar[q]), i = warp_sum(ai[q]);
-        if (lane == 0) {
-          z_s[0][o][q] = r;
-          z_s[1][o][q] = i;
-        }
-      }
-    }
+    const float sum = warp_sum16(acc, lane);
+    if ((lane & 1) == 0) z_s[lane >> 4][(lane >> 1) & (ST_TOK - 1)][o] = sum;
   }
   __syncthreads();
   if (fin) {
-    float* row = state + (size_t)slot_s[fq] * state_ld;
+    float* row = state + row_s[fq];
     float log_a, g;
-    rg_factors(z_s[0][fo][fq] + br[fc], z_s[1][fo][fq] + bi[fc], s.rate * rg_softplus(lam[fc]), log_a, g);
+    rg_factors(z_s[0][fq][fo] + f_br, z_s[1][fq][fo] + f_bi, f_rate, log_a, g);
     const float S = fmaf(expf(log_a), S_old, g * u_s[fq * B + o0 + fo]);
     row[fc] = S;
     // (the entry of this position: no block of this launch reads it)
-    row[s.W + (size_t)(pos_s[fq] % n) * s.W + fc] = x_now + bx[fc];
-    out[(size_t)(t0 + fq) * s.W + fc] = from_float<TO>(S * rg_gelu(y_now + by[fc]));
+    row[s.W + (size_t)(pos_s[fq] % n) * s.W + fc] = x_now + f_bx;
+    out[(size_t)(t0 + fq) * s.W + fc] = from_float<TO>(S * rg_gelu(y_now + f_by));
   }
 }
 
@@ -458,7 +508,7 @@ static int launch_rglru_scan(const RglruScan& a, TO* out, int direct, int prepar
     st = launch_status();
     if (st != DLGO_OK) return st;
   }
-  launch_kernel(rglru_carry_kernel, dim3((a.s.W + CY_THREADS - 1) / CY_THREADS, a.n_tiles), dim3(CY_THREADS), 0, stream, a.tiles,
+  launch_kernel(rglru_carry_kernel, dim3((a.s.W + 31) / 32, a.n_tiles), dim3(CY_WAYS * 32), 0, stream, a.tiles,
                 a.n_tiles, a.seq_slot, (const float*)a.state, a.state_ld, a.seg, a.s.W);
   st = launch_status();
   if (st != DLGO_OK) return st;
@@ -478,15 +528,15 @@ static int launch_rglru_step(const float* proj, int ld, int x0, const float* by,
   if (smem > 200 * 1024) return DLGO_ERR_SIZE;
   const long long gx = (long long)s.parts * ((B + ST_CH - 1) / ST_CH);
   const dim3 grid((unsigned)gx, (T + tok - 1) / tok), block(ST_THREADS);
-  const bool pairs = B % 2 == 0 && ((uintptr_t)w_gates & 7) == 0;
+  const bool four = B % 4 == 0 && ((uintptr_t)w_gates & 15) == 0;
 #define ST_ARGS grid, block, smem, stream, proj, ld, x0, by, bx, w_taps, bc, w_gates, br, bi, lam, token_pos, seq_slot, state, \
                 state_ld, out, T, tok, s
-  if (pairs) {
-    if (smem > 40 * 1024) cudaFuncSetAttribute(rglru_step_kernel<TW, TO, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_kernel(rglru_step_kernel<TW, TO, true>, ST_ARGS);
+  if (four) {
+    if (smem > 40 * 1024) cudaFuncSetAttribute(rglru_step_kernel<TW, TO, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_kernel(rglru_step_kernel<TW, TO, 4>, ST_ARGS);
   } else {
-    if (smem > 40 * 1024) cudaFuncSetAttribute(rglru_step_kernel<TW, TO, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_kernel(rglru_step_kernel<TW, TO, false>, ST_ARGS);
+    if (smem > 40 * 1024) cudaFuncSetAttribute(rglru_step_kernel<TW, TO, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_kernel(rglru_step_kernel<TW, TO, 1>, ST_ARGS);
   }
 #undef ST_ARGS
   return launch_status();
@@ -497,7 +547,7 @@ static int launch_rglru_step(const float* proj, int ld, int x0, const float* by,
 using namespace dlgo;
 
 // x [T, ldx] fp32 (W columns), bx, bc [W], w_taps [W, taps] fp32; tiles [n_tiles, 3] (sequence, first packed token,
-// count); u [T, W] fp32; rows in `rows_dtype` or null: u as rows of a part, [parts, T, B] (by_part) or [T, W].
+// count); u [T, W] fp32 or null; rows in `rows_dtype` or null: u as rows of a part, [parts, T, B] (by_part) or [T, W].
 DLGO_EXPORT int dlgo_rglru_conv(const float* x, int ldx, const float* bx, const float* w_taps, const float* bc,
                                 const int* tiles, int n_tiles, const int* token_seq, const int* token_pos,
                                 const int* seq_slot, const float* state, long long state_ld, float* u, void* rows,

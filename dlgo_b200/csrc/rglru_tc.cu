@@ -9,9 +9,9 @@
 //   z[t, part, 0 .. B) = a_t,  z[t, part, B .. 2 B) = sqrt(1 - a_t^2) i_t u_t;  per segment: its end, sum of log a_t
 //
 // A CTA keeps its 128 rows of both matrices in shared memory for good and walks segments (a few CTAs per block of
-// channels); the segments' rows of u arrive by TMA (128-byte swizzle, no multicast) in two stages; two accumulator pairs
-// in tensor memory, each with four epilogue warps of its own, so that one segment's elementwise work runs beside the
-// other's products.  Warp 0 loads, warp 1 issues MMAs, warps 2-5 and 6-9 are the two epilogues.  Every wait is bounded
+// channels); the segments' rows of u arrive by TMA (128-byte swizzle, no multicast) in four stages; four accumulator
+// pairs in tensor memory, each with four epilogue warps of its own, so that segments' elementwise work runs beside one
+// another's and the next products.  Warp 0 loads, warp 1 issues MMAs, the others are the epilogues.  Every wait is bounded
 // and sets an error word.
 #include "common.cuh"
 #include "tcgen05.cuh"
@@ -20,9 +20,9 @@ namespace dlgo {
 
 using namespace sm100;
 
-constexpr int GU_TOK = 32, GU_M = 128, GU_K = 64, GU_THREADS = 320;
+constexpr int GU_TOK = 32, GU_M = 128, GU_K = 64, GU_GROUPS = 4, GU_THREADS = 64 + GU_GROUPS * 128;
 constexpr int GU_W_BYTES = GU_M * GU_K * 2, GU_U_BYTES = GU_TOK * GU_K * 2;      // of one k-block
-constexpr int GU_TMEM = 128;                  // two pairs of 32 columns
+constexpr int GU_TMEM = GU_GROUPS * 2 * GU_TOK;      // columns: a pair of 32 per group
 
 __device__ int g_rglru_tc_error = 0;
 
@@ -67,20 +67,20 @@ rglru_gates_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
   uint8_t* smem = (uint8_t*)(((uintptr_t)gu_smem_raw + 1023) & ~(uintptr_t)1023);
   const int nk = (p.B + GU_K - 1) / GU_K;
   uint8_t* w_s = smem;                                   // [nk][r: 128 rows | i: 128 rows]
-  uint8_t* u_s = w_s + nk * 2 * GU_W_BYTES;              // [2][nk][32 rows]
-  uint64_t* w_full = (uint64_t*)(u_s + 2 * nk * GU_U_BYTES);
-  uint64_t* u_full = w_full + 1;                         // [2]
-  uint64_t* u_empty = u_full + 2;                        // [2]
-  uint64_t* acc_full = u_empty + 2;                      // [2]
-  uint64_t* acc_empty = acc_full + 2;                    // [2]
-  uint32_t* tmem_slot = (uint32_t*)(acc_empty + 2);
+  uint8_t* u_s = w_s + nk * 2 * GU_W_BYTES;              // [groups][nk][32 rows]
+  uint64_t* w_full = (uint64_t*)(u_s + GU_GROUPS * nk * GU_U_BYTES);
+  uint64_t* u_full = w_full + 1;                         // [groups], like the next three
+  uint64_t* u_empty = u_full + GU_GROUPS;
+  uint64_t* acc_full = u_empty + GU_GROUPS;
+  uint64_t* acc_empty = acc_full + GU_GROUPS;
+  uint32_t* tmem_slot = (uint32_t*)(acc_empty + GU_GROUPS);
   volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int part = blockIdx.y / p.chunks, c0 = (blockIdx.y - part * p.chunks) * GU_M;
   if (threadIdx.x == 0) {
     mbar_init(w_full, 1);
-    for (int b = 0; b < 2; ++b) {
+    for (int b = 0; b < GU_GROUPS; ++b) {
       mbar_init(&u_full[b], 1);
       mbar_init(&u_empty[b], 1);
       mbar_init(&acc_full[b], 1);
@@ -115,8 +115,8 @@ rglru_gates_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
     if (elect_one()) {
       int it = 0;
       for (int tile = blockIdx.x; tile < p.n_tiles; tile += gridDim.x, ++it) {
-        const int s = it & 1;
-        if (it >= 2 && !mbar_wait(&u_empty[s], ((it >> 1) - 1) & 1, abort_flag)) break;
+        const int s = it % GU_GROUPS;
+        if (it >= GU_GROUPS && !mbar_wait(&u_empty[s], (it / GU_GROUPS - 1) & 1, abort_flag)) break;
         mbar_expect_tx(&u_full[s], nk * GU_U_BYTES);
         const int row = part * p.T + p.tiles[3 * tile + 1];
         for (int kb = 0; kb < nk; ++kb)
@@ -129,9 +129,9 @@ rglru_gates_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
       bool ok = mbar_wait(w_full, 0, abort_flag);
       int it = 0;
       for (int tile = blockIdx.x; ok && tile < p.n_tiles; tile += gridDim.x, ++it) {
-        const int s = it & 1;
-        if (it >= 2) ok = mbar_wait(&acc_empty[s], ((it >> 1) - 1) & 1, abort_flag);
-        if (ok) ok = mbar_wait(&u_full[s], (it >> 1) & 1, abort_flag);
+        const int s = it % GU_GROUPS;
+        if (it >= GU_GROUPS) ok = mbar_wait(&acc_empty[s], (it / GU_GROUPS - 1) & 1, abort_flag);
+        if (ok) ok = mbar_wait(&u_full[s], (it / GU_GROUPS) & 1, abort_flag);
         if (!ok) break;
         tc_fence_after_sync();
         const uint32_t w_addr = smem_u32(w_s), u_addr = smem_u32(u_s + s * nk * GU_U_BYTES);
@@ -160,35 +160,42 @@ rglru_gates_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
     const size_t ldz = (size_t)2 * p.W;
     float* zc = p.z + (size_t)part * 2 * p.B + (mine ? cb : 0);
     int it = group;
-    for (int tile = blockIdx.x + group * gridDim.x; tile < p.n_tiles; tile += 2 * gridDim.x, it += 2) {
+    for (int tile = blockIdx.x + group * gridDim.x; tile < p.n_tiles; tile += GU_GROUPS * gridDim.x, it += GU_GROUPS) {
       const int t0 = p.tiles[3 * tile + 1], n = p.tiles[3 * tile + 2];
       __nv_bfloat16 uu[GU_TOK];
       const __nv_bfloat16* ur = p.u + ((size_t)part * p.T + t0) * p.B + (mine ? cb : 0);
 #pragma unroll
       for (int q = 0; q < GU_TOK; ++q) uu[q] = ur[(size_t)min(q, n - 1) * p.B];      // on its way during the products
-      if (!mbar_wait(&acc_full[group], (it >> 1) & 1, abort_flag)) break;
+      if (!mbar_wait(&acc_full[group], (it / GU_GROUPS) & 1, abort_flag)) break;
       __syncwarp();                                              // (tensor-memory reads are the whole warp's)
       tc_fence_after_sync();
-      float r[GU_TOK], i[GU_TOK];
-      const uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(group * 2 * GU_TOK);
-      tmem_ld_32x32(taddr, r);
-      tmem_ld_32x32(taddr + GU_TOK, i);
-      tmem_ld_wait();
-      tc_fence_before_sync();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&acc_empty[group]);
       float S = 0.f, total = 0.f;
       float* zt = zc + (size_t)t0 * ldz;
+      const uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(group * 2 * GU_TOK);
 #pragma unroll
-      for (int q = 0; q < GU_TOK; ++q) {
-        if (mine && q < n) {
-          const float log_a = -rate_sp * gu_sigmoid(r[q] + b_r), a = expf(log_a);
-          const float in = gu_input_factor(log_a, a) * gu_sigmoid(i[q] + b_i) * __bfloat162float(uu[q]);
-          zt[(size_t)q * ldz] = a;
-          zt[(size_t)q * ldz + p.B] = in;
-          total += log_a;
-          S = fmaf(a, S, in);
+      for (int half = 0; half < 2; ++half) {
+        float r[GU_TOK / 2], i[GU_TOK / 2];
+        tmem_ld_32x16(taddr + half * (GU_TOK / 2), r);
+        tmem_ld_32x16(taddr + GU_TOK + half * (GU_TOK / 2), i);
+        tmem_ld_wait();
+        if (half == 1) {
+          tc_fence_before_sync();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&acc_empty[group]);
         }
+#pragma unroll
+        for (int k = 0; k < GU_TOK / 2; ++k) {
+          const int q = half * (GU_TOK / 2) + k;
+          if (mine && q < n) {
+            const float log_a = -rate_sp * gu_sigmoid(r[k] + b_r), a = __expf(log_a);
+            const float in = gu_input_factor(log_a, a) * gu_sigmoid(i[k] + b_i) * __bfloat162float(uu[q]);
+            zt[(size_t)q * ldz] = a;
+            zt[(size_t)q * ldz + p.B] = in;
+            total += log_a;
+            S = fmaf(a, S, in);
+          }
+        }
+        __syncwarp();
       }
       if (mine) {
         float* sg = p.seg + (size_t)tile * 3 * p.W + c;
@@ -247,7 +254,7 @@ int make_map(CUtensorMap* m, const void* base, long long rows, int K, int box_ro
 
 int smem_bytes(int B) {
   const int nk = (B + GU_K - 1) / GU_K;
-  return nk * (2 * GU_W_BYTES + 2 * GU_U_BYTES) + 1024 + 256;
+  return nk * (2 * GU_W_BYTES + GU_GROUPS * GU_U_BYTES) + 1024 + 256;
 }
 
 }  // namespace
@@ -255,7 +262,7 @@ int smem_bytes(int B) {
 
 using namespace dlgo;
 
-// 1 if the kernel takes parts of B channels: rows in whole 16-byte pieces, both matrices' rows and two stages of u in
+// 1 if the kernel takes parts of B channels: rows in whole 16-byte pieces, both matrices' rows and four stages of u in
 // shared memory
 DLGO_EXPORT int dlgo_rglru_gates_tc_takes(int B) { return B > 0 && B % 8 == 0 && smem_bytes(B) <= 227 * 1024; }
 DLGO_EXPORT int dlgo_rglru_gates_tc_tokens() { return GU_TOK; }
@@ -281,11 +288,8 @@ DLGO_EXPORT int dlgo_rglru_gates_tc(const void* u, const void* w, const float* b
     if (e != cudaSuccess) { sms = 0; return (int)e; }
   }
   const int chunks = (B + GU_M - 1) / GU_M, smem = smem_bytes(B);
-  int per_sm = (227 * 1024) / (smem + 1024);
-  if (per_sm < 1) per_sm = 1;
-  if (per_sm > 3) per_sm = 3;                            // (threads' registers)
-  int per_chunk = sms * per_sm / (parts * chunks);
-  if (per_chunk > (n_tiles + 1) / 2) per_chunk = (n_tiles + 1) / 2;
+  int per_chunk = sms / (parts * chunks);                // (one CTA per SM: its threads' registers)
+  if (per_chunk > (n_tiles + GU_GROUPS - 1) / GU_GROUPS) per_chunk = (n_tiles + GU_GROUPS - 1) / GU_GROUPS;
   if (per_chunk < 1) per_chunk = 1;
   if ((long long)parts * chunks > 65535) return DLGO_ERR_SIZE;
   GuParams p{(const __nv_bfloat16*)u, br, bi, lam, tiles, n_tiles, T, parts * B, B, parts, chunks, rate, z, seg};

@@ -38,7 +38,8 @@ struct StreamsStep {
   const float* nalpha;  // [1] (Dynamic Tanh)
   float eps;
   void* out;            // [R, d]
-  const int* rows;      // [R] rows of X to read (read part only), or null
+  const int* rows;      // [R] rows of X to read (read part only, or keep == 0), or null
+  int keep;             // write part: the new streams are stored (0: only read on, for a step's last reader)
 };
 
 template <typename TO> __device__ __forceinline__ void store4(TO* o, float a, float b, float c, float d);
@@ -114,6 +115,7 @@ __global__ void __launch_bounds__(256) streams_step_kernel(StreamsStep p) {
               if (a < s) acc = fmaf(s_mix[a * s + q], x[a][c], acc);
             nx[q][c] = fmaf(s_wout[q], yv[c], acc);
           }
+          if (!p.keep) continue;
           if (W == 4)
             *reinterpret_cast<float4*>(xr + (size_t)q * d + i0) = make_float4(nx[q][0], nx[q][1], nx[q][2], nx[q][3]);
           else
@@ -210,21 +212,31 @@ __global__ void __launch_bounds__(THREADS) streams_layernorm_kernel(StreamsStep 
   pdl_wait();
   float* xr = p.X + (size_t)row * s * d;
   float* yr = p.y ? p.y + (size_t)row * d : nullptr;
+  // every fetch of the row before its first store (the compiler may not move one ahead of the other)
+  float4 x[NV][S], y[NV];
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (v * THREADS + tid) * 4;
+#pragma unroll
+    for (int a = 0; a < S; ++a) {
+      x[v][a] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (a < s && i < d) x[v][a] = *reinterpret_cast<const float4*>(xr + (size_t)a * d + i);
+    }
+    y[v] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (yr && i < d) {
+      y[v] = *reinterpret_cast<const float4*>(yr + i);
+      if (p.y_bias) {
+        const float4 b = *reinterpret_cast<const float4*>(p.y_bias + i);
+        y[v].x += b.x; y[v].y += b.y; y[v].z += b.z; y[v].w += b.w;
+      }
+    }
+  }
   float sum = 0.f;
 #pragma unroll
   for (int v = 0; v < NV; ++v) {
     const int i = (v * THREADS + tid) * 4;
     if (i >= d) continue;
-    float4 x[S];
-#pragma unroll
-    for (int a = 0; a < S; ++a)
-      if (a < s) x[a] = *reinterpret_cast<const float4*>(xr + (size_t)a * d + i);
     if (yr) {
-      float4 y = *reinterpret_cast<const float4*>(yr + i);
-      if (p.y_bias) {
-        const float4 b = *reinterpret_cast<const float4*>(p.y_bias + i);
-        y.x += b.x; y.y += b.y; y.z += b.z; y.w += b.w;
-      }
       if (p.clear_y) *reinterpret_cast<float4*>(yr + i) = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
       for (int q = 0; q < S; ++q) {
@@ -234,13 +246,13 @@ __global__ void __launch_bounds__(THREADS) streams_layernorm_kernel(StreamsStep 
           for (int a = 0; a < S; ++a) {
             if (a < s) {
               const float m = s_mix[a * s + q];
-              n.x = fmaf(m, x[a].x, n.x); n.y = fmaf(m, x[a].y, n.y);
-              n.z = fmaf(m, x[a].z, n.z); n.w = fmaf(m, x[a].w, n.w);
+              n.x = fmaf(m, x[v][a].x, n.x); n.y = fmaf(m, x[v][a].y, n.y);
+              n.z = fmaf(m, x[v][a].z, n.z); n.w = fmaf(m, x[v][a].w, n.w);
             }
           }
           const float w = s_wout[q], c = s_coeff[q];
-          n.x = fmaf(w, y.x, n.x); n.y = fmaf(w, y.y, n.y); n.z = fmaf(w, y.z, n.z); n.w = fmaf(w, y.w, n.w);
-          *reinterpret_cast<float4*>(xr + (size_t)q * d + i) = n;
+          n.x = fmaf(w, y[v].x, n.x); n.y = fmaf(w, y[v].y, n.y); n.z = fmaf(w, y[v].z, n.z); n.w = fmaf(w, y[v].w, n.w);
+          if (p.keep) *reinterpret_cast<float4*>(xr + (size_t)q * d + i) = n;
           u[v].x = fmaf(c, n.x, u[v].x); u[v].y = fmaf(c, n.y, u[v].y);
           u[v].z = fmaf(c, n.z, u[v].z); u[v].w = fmaf(c, n.w, u[v].w);
         }
@@ -250,8 +262,8 @@ __global__ void __launch_bounds__(THREADS) streams_layernorm_kernel(StreamsStep 
       for (int a = 0; a < S; ++a) {
         if (a < s) {
           const float c = s_coeff[a];
-          u[v].x = fmaf(c, x[a].x, u[v].x); u[v].y = fmaf(c, x[a].y, u[v].y);
-          u[v].z = fmaf(c, x[a].z, u[v].z); u[v].w = fmaf(c, x[a].w, u[v].w);
+          u[v].x = fmaf(c, x[v][a].x, u[v].x); u[v].y = fmaf(c, x[v][a].y, u[v].y);
+          u[v].z = fmaf(c, x[v][a].z, u[v].z); u[v].w = fmaf(c, x[v][a].w, u[v].w);
         }
       }
     }
@@ -278,6 +290,10 @@ __global__ void __launch_bounds__(THREADS) streams_layernorm_kernel(StreamsStep 
 
 template <typename TO, int S>
 static void launch_streams_layernorm_of(const StreamsStep& p, int n_rows, cudaStream_t stream) {
+  if (n_rows >= 512 && p.d > 1024 && p.d <= 2048) {       // many rows: smaller blocks, one's barriers beside others' fetches
+    launch_kernel(streams_layernorm_kernel<TO, 256, 2, S>, dim3(n_rows), dim3(256), 0, stream, p);
+    return;
+  }
   if (p.d <= 512) launch_kernel(streams_layernorm_kernel<TO, 128, 1, S>, dim3(n_rows), dim3(128), 0, stream, p);
   else if (p.d <= 1024) launch_kernel(streams_layernorm_kernel<TO, 256, 1, S>, dim3(n_rows), dim3(256), 0, stream, p);
   else if (p.d <= 2048) launch_kernel(streams_layernorm_kernel<TO, 512, 1, S>, dim3(n_rows), dim3(512), 0, stream, p);
@@ -437,21 +453,22 @@ using namespace dlgo;
 DLGO_EXPORT int dlgo_streams_step(float* X, int T, int s, int d, float* y, const float* y_bias, const float* mix,
                                   const float* wout, int clear_y, const float* coeff, int norm_kind, const float* nw,
                                   const float* nb, const float* nalpha, float eps, void* out, int out_dtype,
-                                  const int* rows, int R, cudaStream_t stream) {
+                                  const int* rows, int R, int keep, cudaStream_t stream) {
   if (s < 1 || s > MAX_STREAMS || d <= 0) return DLGO_ERR_SIZE;
-  if (y && rows) return DLGO_ERR_SIZE;      // the write part runs on every row
-  const int n_rows = y ? T : R;
+  if (y && rows && (keep || clear_y)) return DLGO_ERR_SIZE;      // the write part runs on every row
+  const int n_rows = y && !rows ? T : R;
   if (n_rows <= 0) return DLGO_OK;
   if (out && out_dtype != DLGO_F32 && out_dtype != DLGO_BF16) return DLGO_ERR_DTYPE;
   if (norm_kind < NORM_NONE || norm_kind > NORM_LAYER) return DLGO_ERR_SIZE;
   if (out && norm_kind != NORM_NONE && !nw) return DLGO_ERR_SIZE;
-  StreamsStep p{X, s, d, y, y_bias, mix, wout, clear_y, coeff, norm_kind, nw, nb, nalpha, eps, out, rows};
+  StreamsStep p{X, s, d, y, y_bias, mix, wout, clear_y, coeff, norm_kind, nw, nb, nalpha, eps, out, rows, keep || !y};
   if (out && norm_kind == NORM_LAYER && d % 4 == 0 && d <= 4096 &&
       (((uintptr_t)X | (uintptr_t)y | (uintptr_t)y_bias | (uintptr_t)nw | (uintptr_t)nb | (uintptr_t)out) & 15) == 0) {
     if (out_dtype == DLGO_BF16) launch_streams_layernorm<__nv_bfloat16>(p, n_rows, stream);
     else launch_streams_layernorm<float>(p, n_rows, stream);
     return launch_status();
   }
+  if (y && !keep && norm_kind != NORM_NONE && norm_kind != NORM_DYT) return DLGO_ERR_SIZE;    // (these read the row again)
   const int threads = d >= 1024 ? 256 : 128;      // (four columns per thread and trip)
   if (out && out_dtype == DLGO_BF16)
     launch_kernel(streams_step_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, stream, p);

@@ -138,6 +138,13 @@ class CausalLM:
             blk.forward(residual, ctx, cache.view(i), cache.state.view(i), self.positions)
             i += 1
         if streams is not None:
+            through = getattr(self.final_norm, "forward_write", None)
+            if want_rows is not None and want_rows.numel() > 0 and ctx.owed is not None and through is not None:
+                # the last sublayer's write, of the wanted rows only and straight through the final norm
+                x = through(residual, ctx.owed, None if ctx.want_identity else want_rows)
+                if x is not None:
+                    ctx.take_owed_write()
+                    return self.head.forward(x)
             ctx.settle_streams(residual)       # the last sublayer's write
             if want_rows is None or want_rows.numel() == 0:
                 return None

@@ -127,7 +127,7 @@ class RealGatedLinearUnit(Mixer):
             y, by, xs = proj[:, :w], self.b_y, proj[:, self.x_col:self.x_col + w]
         tiles, n_tiles, _ = ctx.tiles(CONV_TILE)
         u, rows = K.rglru_conv(xs, self.b_x, self.taps, self.b_conv, tiles, n_tiles, ctx.token_seq, ctx.token_pos,
-                               ctx.seq_slot, st, s, None if act == torch.float32 else act, on_tc)
+                               ctx.seq_slot, st, s, None if act == torch.float32 else act, on_tc, f32=not on_tc)
         tiles, n_tiles, _ = ctx.tiles(K.RGLRU_TC_SEGMENT if on_tc else segment(T, w))
         direct = not on_tc and n_tiles == ctx.n_seqs
         scratch = None if direct else ctx.scratch("rglru_segments", n_tiles * 3 * w)

@@ -142,7 +142,20 @@ def _rms_step_args(self) -> Dict[str, Any]:
     return dict(norm_kind=K.NORM_RMS, norm_w=self.weight, eps=self.eps, out_dtype=self.out_dtype)
 
 
+def _forward_write(self, streams: torch.Tensor, write: Dict[str, Any], rows: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
+    """The norm of the plain sum of the streams as ``write`` (arguments of :func:`kernels.streams_step`) leaves them, for the
+    rows wanted (``rows`` None: all, in order), when nobody reads the streams afterwards; None where this norm cannot.  A
+    buffer that is to be zero again is cleared where every row is read."""
+    args = self.step_args()
+    if rows is None:
+        return K.streams_step(streams, **write, **args)
+    if not K.streams_step_passes(args["norm_kind"], streams.shape[-1]):
+        return None
+    return K.streams_step(streams, **write, **args, rows=rows, keep=False)
+
+
 RMSNorm.forward_streams = _forward_streams
+RMSNorm.forward_write = LayerNorm.forward_write = DynamicTanh.forward_write = _forward_write
 LayerNorm.forward_streams = _forward_streams
 RMSNorm.step_args = _rms_step_args
 

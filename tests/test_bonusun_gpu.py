@@ -110,9 +110,29 @@ def test_layer_norm_over_streams(d, s, act_dtype):
     assert worst(K.streams_step(dev[0], rows=i32(rows), **args), n) < tol
     n = P.layer_norm(X.double().sum(1), w.double(), torch.zeros(d).double(), eps)
     assert worst(K.streams_step(dev[0], **dict(args, norm_b=None)), n) < tol
+    if K.streams_step_passes(K.NORM_LAYER, d):       # read on without being stored, rows in any order and twice
+        out = K.streams_step(dev[0], y=dev[1], mix=dev[6], write=dev[5], clear_y=True, rows=i32(rows), keep=False, **args)
+        assert worst(out, P.layer_norm(new.double().sum(1)[rows], w.double(), b.double(), eps)) < tol
+        assert torch.equal(dev[0].cpu(), X) and torch.equal(dev[1].cpu(), y)
     out = K.streams_step(dev[0], y=dev[1], mix=dev[6], write=dev[5], clear_y=True, read=dev[4], **args)
     assert worst(out, P.layer_norm(torch.einsum("q,tqd->td", read.double(), new.double()), w.double(), b.double(), eps)) < tol
     assert worst(dev[0], new) < 1e-6 and not dev[1].any()
+
+
+@pytest.mark.parametrize("d, s", [(72, 2), (600, 3), (1000, 1), (2048, 3), (3072, 4), (1536, 6)])
+def test_layer_norm_over_streams_of_many_tokens(d, s):
+    from dlgo_b200.csrc import kernels as K
+    g = torch.Generator().manual_seed(d)
+    T, eps = 700, 1e-5
+    X, y = torch.randn(T, s, d, generator=g), torch.randn(T, d, generator=g)
+    w, b = 1 + 0.3 * torch.randn(d, generator=g), torch.randn(d, generator=g)
+    read, write, mix = torch.randn(s, generator=g), torch.randn(s, generator=g), torch.randn(s, s, generator=g)
+    new = torch.einsum("rq,trd->tqd", mix, X) + write[None, :, None] * y[:, None]
+    dev = [t.to(DEV) for t in (X, y, w, b, read, write, mix)]
+    out = K.streams_step(dev[0], y=dev[1], mix=dev[6], write=dev[5], clear_y=True, read=dev[4], norm_kind=K.NORM_LAYER, norm_w=dev[2],
+                         norm_b=dev[3], eps=eps, out_dtype=torch.float32)
+    want = P.layer_norm(torch.einsum("q,tqd->td", read.double(), new.double()), w.double(), b.double(), eps)
+    assert worst(out, want) < 1e-4 and worst(dev[0], new) < 1e-6 and not dev[1].any()
 
 
 @pytest.mark.parametrize("act_dtype", [torch.float32, torch.bfloat16])
