@@ -449,7 +449,7 @@ def test_running_maximum_of_long_sequences(T):
         assert torch.equal(state[1, off:off + H].cpu(), mm[-1])
 
 
-UNITS = [(64, 4, 3), (60, 3, 4), (33, 1, 1), (50, 5, 6), (256, 2, 4), (7, 7, 2), (640, 1, 4), (24, 3, 9), (128, 4, 2)]
+UNITS = [(512, 2, 4), (400, 2, 4), (64, 4, 3), (60, 3, 4), (33, 1, 1), (50, 5, 6), (256, 2, 4), (7, 7, 2), (640, 1, 4), (24, 3, 9), (128, 4, 2)]
 
 
 @pytest.mark.parametrize("act_dtype", [torch.float32, torch.bfloat16])
