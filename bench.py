@@ -650,7 +650,7 @@ def main() -> int:
                     help="--only prefill: a packed batch of that many prompts with lengths from --prompt-range")
     ap.add_argument("--only", choices=["decode", "prefill", "phases", "sampled", "dedutar", "monolix", "bazurax", "ragilorn", "zetavik", "bonusun"],
                     help="run one small workload (for profiling) and stop; phases: see phase_stamps(); dedutar, "
-                         "monolix, bazurax, ragilorn, zetavik: prefill and decode of that design beside Llama (zetavik: and its "
+                         "monolix, bazurax, ragilorn, zetavik, bonusun: prefill and decode of that design beside Llama (zetavik, bonusun: and its "
                          "closest relatives) at equal layer sizes")
     ap.add_argument("--bazurax-size", default="1b", choices=sorted(BAZURAX_SIZES), help="--only bazurax: layer sizes")
     ap.add_argument("--zetavik-size", default="1b", choices=sorted(ZETAVIK_SIZES), help="--only zetavik: layer sizes")
@@ -659,7 +659,7 @@ def main() -> int:
     ap.add_argument("--ragilorn-size", default="1b", choices=sorted(RAGILORN_SIZES), help="--only ragilorn: layer sizes")
     ap.add_argument("--monolix-size", default="1b", choices=sorted(MONOLIX_SIZES), help="--only monolix: layer sizes")
     ap.add_argument("--dedutar-size", default="1b", choices=sorted(DEDUTAR_SIZES), help="--only dedutar: layer sizes")
-    ap.add_argument("--kernels", action="store_true", help="--only dedutar / monolix / bazurax: also the time per kernel entry point")
+    ap.add_argument("--kernels", action="store_true", help="with these designs: also the time per kernel entry point")
     ap.add_argument("--no-graphs", action="store_true", help="launch decode kernels one by one (for profiling)")
     a = ap.parse_args()
     if a.impl == "reference":

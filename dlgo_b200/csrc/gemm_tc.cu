@@ -118,7 +118,12 @@ __device__ __forceinline__ float glu_mul(float g, float u, const GluForm& f) {
 template <int ACT> __device__ __forceinline__ float act_value(float z) {
   if (ACT == TC_ACT_RELU2) { const float r = fmaxf(z, 0.f); return r * r; }
   if (ACT == TC_ACT_SILU) return silu_mul(z, 1.0f);      // (results here are rounded to bfloat16 too)
-  if (ACT == TC_ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  if (ACT == TC_ACT_GELU_TANH) {      // 0.5 (1 + tanh(u)) is the logistic function at 2 u: the same two instructions
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(z * fmaf(z * z, -0.044715f, -1.0f) * (2.0f * 0.7978845608028654f * 1.4426950408889634f)));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+    return z * r;
+  }
   return z;
 }
 // n accumulator values + bias (b: per value, or one number when `same`) through the activation, in place;
